@@ -67,6 +67,16 @@ class CacheGroup:
     window: int = 0          # 0: every token; W: the last W tokens
     layers: tuple = ()       # indices of the layers whose caches live in this group
     keep_first: int = 0      # with a window: the first tokens of a request stay too
+    chunk: int = 0           # without a window: only the run of ``chunk`` positions at hand
+
+    def first_needed(self, length: int) -> int:
+        """The first position a query at ``length`` or later can see (kept first tokens
+        aside): what lies before it is never read again."""
+        if self.window > 0:
+            return length - self.window + 1
+        if self.chunk > 0:
+            return length // self.chunk * self.chunk
+        return 0
 
 
 @dataclass
@@ -202,11 +212,12 @@ class CacheManager:
                 f"{self.capacity(rid)}")
         r.length = new_len
         for g, grp in enumerate(self.groups):
-            if grp.window <= 0:
+            # the next query sits at position >= new_len and sees keys from here on (the
+            # window before it, or the start of its run): a page whose last position is
+            # below that is dead
+            first_needed = grp.first_needed(new_len)
+            if first_needed <= 0:
                 continue
-            # the next query sits at position >= new_len and sees keys from
-            # new_len - window + 1 on: a page whose last position is below that is dead
-            first_needed = new_len - grp.window + 1
             table = r.tables[g]
             i = r.first_live[g]
             # (a page that holds one of the first tokens a windowed layer keeps visible
@@ -252,9 +263,9 @@ def groups_for(cache_needs_per_layer) -> List[CacheGroup]:
     """Group layers by the span of tokens their paged needs keep.
 
     ``cache_needs_per_layer[i]`` is the list of needs of layer ``i``'s mixer.  The span
-    alone decides the group (the window, and how many first tokens stay beside it): a page
-    is a span of tokens, so layers whose records differ in shape or number of entries can
-    share page numbers and block tables."""
+    alone decides the group (the window, how many first tokens stay beside it, or the length
+    of the runs): a page is a span of tokens, so layers whose records differ in shape or
+    number of entries can share page numbers and block tables."""
     by_span: Dict[tuple, List[int]] = {}
     for i, needs in enumerate(cache_needs_per_layer):
         for need in needs:
@@ -262,12 +273,14 @@ def groups_for(cache_needs_per_layer) -> List[CacheGroup]:
                 key = span_key(need)
                 if i not in by_span.setdefault(key, []):
                     by_span[key].append(i)
-    return [CacheGroup(window=w, layers=tuple(ls), keep_first=k)
-            for (w, k), ls in sorted(by_span.items())]
+    return [CacheGroup(window=w, layers=tuple(ls), keep_first=k, chunk=c)
+            for (w, k, c), ls in sorted(by_span.items())]
 
 
 def span_key(need) -> tuple:
-    """(window, first tokens kept beside it) of a paged need; without a window every token
-    stays and the second number says nothing."""
+    """(window, first tokens kept beside it, run length) of a paged need, or of a group;
+    without a window the second number says nothing, with one the third."""
     window = int(need.window)
-    return (window, int(getattr(need, "keep_first", 0)) if window > 0 else 0)
+    if window > 0:
+        return (window, int(getattr(need, "keep_first", 0)), 0)
+    return (0, 0, int(getattr(need, "chunk", 0)))

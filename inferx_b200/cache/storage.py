@@ -25,8 +25,7 @@ class CacheStorage:
         self.paged: Dict[int, Dict[str, torch.Tensor]] = {}
         self.group_of_layer: Dict[int, int] = {}
         self.state: Dict[int, Dict[str, torch.Tensor]] = {}
-        span_to_group = {(g.window, getattr(g, "keep_first", 0)): i
-                         for i, g in enumerate(manager.groups)}
+        span_to_group = {span_key(g): i for i, g in enumerate(manager.groups)}
         for layer, needs in enumerate(cache_needs_per_layer):
             for need in needs:
                 if is_paged_need(need):

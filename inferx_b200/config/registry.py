@@ -72,6 +72,10 @@ def _register_builtin():
     from .fudulix_config import FudulixConfig
     register_architecture(FudulixConfig.ARCHITECTURE, FudulixConfig.from_json,
                           fudulix.build_spec, replace=True)
+    from ..models import dominex
+    from .dominex_config import DominexConfig
+    register_architecture(DominexConfig.ARCHITECTURE, DominexConfig.from_json,
+                          dominex.build_spec, replace=True)
 
 
 _register_builtin()

@@ -18,7 +18,7 @@ from typing import Any, Dict, Hashable, Iterator, List, Mapping, Optional, Seque
 
 import torch
 
-from ..cache.manager import is_paged_need, groups_for
+from ..cache.manager import groups_for, is_paged_need, span_key
 from ..sampling.params import SamplingParams
 from ..sampling.sampler import Sampler
 from ..weights.loader import RandomSource
@@ -66,7 +66,7 @@ def cache_bytes_per_page(model, page_size: int) -> List[int]:
         b = 0
         for layer in g.layers:
             for need in needs[layer]:
-                if is_paged_need(need) and int(need.window) == g.window:
+                if is_paged_need(need) and span_key(need) == span_key(g):
                     b += need.bytes_per_token(model.ctx.dtype) * page_size
         out.append(b)
     return out

@@ -316,7 +316,7 @@ class Executor:
             groups.append(GroupView(
                 block_table=seg(_FIXED_SEGS + 2 * g + 1).view(lay.S, lay.widths[g]),
                 slots=seg(_FIXED_SEGS + 2 * g), page_size=mgr.page_size, window=grp.window,
-                keep_first=getattr(grp, "keep_first", 0),
+                keep_first=getattr(grp, "keep_first", 0), chunk=getattr(grp, "chunk", 0),
                 first_live=None if static else list(lay.first_live[g])))
         max_kv = max(lay.kv_lens)
         if static:   # a captured graph must hold for every length its table width allows

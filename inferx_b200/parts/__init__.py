@@ -1,5 +1,5 @@
 # importing a module registers the kinds it defines
-from . import (attention, embedding, feed_forward, latent_attention,  # noqa: F401
+from . import (attention, embedding, feed_forward, gated_pair, latent_attention,  # noqa: F401
                linear_recurrence, norm, position, state_space, token_shift)
 from .base import (BuildContext, GroupView, LayerCache, PagedKvNeed, StateNeed,  # noqa: F401
                    StepContext)

@@ -318,3 +318,87 @@ class PreparedAttentionMixer:
 
 
 register_part("mixer", "attention_prepared", PreparedAttentionMixer)
+
+
+class DistanceAttentionMixer:
+    """Grouped-query attention without a rotation: every score is multiplied by its head's
+    temperature and loses r1 ln(1 + r2 distance), and a query may be confined to its own run
+    of ``chunk`` positions.  The cache manager then keeps the run at hand and takes the pages
+    before it back.  Scores, the penalty and the weights are fp32 in every element type.
+
+    The mixer comes in two halves that a pair of mixers can join with another mixer's: the
+    matrices that read the mixer's input (``front_matrices``), and ``mix_front``, which takes
+    their product and writes the heads' outputs, times a factor, into columns of a row of
+    the caller's; ``out_matrix`` is what those columns are multiplied with."""
+
+    def __init__(self, spec, ctx, prefix: str):
+        self.spec, self.ctx, self.prefix = spec, ctx, prefix
+        s = spec
+        if s.heads % s.kv_heads:
+            raise ValueError(f"{prefix}: {s.heads} heads do not split over {s.kv_heads} "
+                             "key/value heads")
+        self.dq, self.dk = s.heads * s.head_dim, s.kv_heads * s.head_dim
+        self.dv = s.kv_heads * s.value_dim
+        self.front_width = self.dq + self.dk + self.dv
+        self.inner = s.heads * s.value_dim
+        self.names = dict(s.names)
+        self.temp = self.r1 = self.r2 = self.front_w = self.o_w = None
+
+    def check_limits(self):
+        check = getattr(self.ctx.ops, "check_attention_limits", None)
+        if check is not None:
+            s = self.spec
+            check(s.heads, s.kv_heads, s.head_dim, self.ctx.dtype, self.prefix, allow_odd=True)
+            check(s.heads, s.kv_heads, s.value_dim, self.ctx.dtype, self.prefix, allow_odd=True)
+
+    def _n(self, key):
+        return f"{self.prefix}.{self.names[key]}"
+
+    def tensors(self):
+        s = self.spec
+        decls = [TensorDecl(self._n("q"), (self.dq, s.hidden)),
+                 TensorDecl(self._n("k"), (self.dk, s.hidden)),
+                 TensorDecl(self._n("v"), (self.dv, s.hidden)),
+                 TensorDecl(self._n("o"), (s.hidden, self.inner))]
+        return decls + [TensorDecl(self._n(k), (s.heads,), keep="float32", init="gain")
+                        for k in ("temp", "r1", "r2")]
+
+    def front_matrices(self, w):
+        return [w[self._n("q")], w[self._n("k")], w[self._n("v")]]
+
+    def out_matrix(self, w):
+        return w[self._n("o")]
+
+    def bind_vectors(self, w):
+        self.temp, self.r1, self.r2 = (w[self._n(k)].contiguous() for k in ("temp", "r1", "r2"))
+
+    def bind(self, w):
+        self.bind_vectors(w)
+        self.front_w = torch.cat(self.front_matrices(w), dim=0).contiguous()
+        self.o_w = self.out_matrix(w)
+
+    def cache_needs(self):
+        s = self.spec
+        return [PagedKvNeed(s.kv_heads, s.head_dim, 0, entry_dims=(s.head_dim, s.value_dim),
+                            chunk=s.chunk)]
+
+    def mix_front(self, front, step, cache, out, out_scale):
+        """``front`` [T, q | k | v] (a view of columns); ``out`` [T, heads * value_dim], a view
+        too, receives the heads' outputs times ``out_scale``."""
+        s, ops = self.spec, self.ctx.ops
+        group = step.groups[cache.group]
+        if cache.writes:
+            ops.append_kv_rows(front[:, self.dq:self.dq + self.dk],
+                               front[:, self.dq + self.dk:self.front_width], cache.k, cache.v,
+                               group.slots)
+        ops.distance_attention(front[:, :self.dq], cache.k, cache.v, group.block_table, step,
+                               s.scale, self.temp, self.r1, self.r2, s.chunk, out, out_scale)
+
+    def forward(self, x, step, cache):
+        front = self.ctx.ops.linear(x, self.front_w)
+        out = torch.empty((x.shape[0], self.inner), dtype=x.dtype, device=x.device)
+        self.mix_front(front, step, cache, out, 1.0)
+        return self.ctx.ops.linear(out, self.o_w)
+
+
+register_part("mixer", "attention_distance", DistanceAttentionMixer)

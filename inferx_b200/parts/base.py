@@ -60,6 +60,9 @@ class PagedKvNeed:
     entry_dims: Optional[Tuple[int, ...]] = None
     # with a window: the first ``keep_first`` tokens of a request stay as well
     keep_first: int = 0
+    # without a window: tokens are kept in runs of ``chunk`` positions counted from 0; pages
+    # wholly before the run the next token falls into may be given back
+    chunk: int = 0
 
     def dim_of(self, index: int) -> int:
         return self.head_dim if self.entry_dims is None else int(self.entry_dims[index])
@@ -90,6 +93,7 @@ class GroupView:
     # were given back as the window passed them); None in a step recorded for replay
     first_live: Optional[List[int]] = None
     keep_first: int = 0         # tokens at the start of a request that a windowed group keeps
+    chunk: int = 0              # a group that keeps runs of this many positions (0: no runs)
 
 
 @dataclass

@@ -340,7 +340,10 @@ class DecoderModel:
         n = self.final_norm.forward(resid, pending, rows=logit_rows)
         logits = ops.linear(n, self.head, out_dtype=torch.float32)
         scale = float(getattr(self.spec, "logit_scale", 1.0))
-        return logits if scale == 1.0 else ops.scale_rows(logits, scale)
+        if scale != 1.0:
+            logits = ops.scale_rows(logits, scale)
+        cap = float(getattr(self.spec, "logit_softcap", 0.0))
+        return ops.softcap_rows(logits, cap) if cap > 0 else logits
 
 
 Block = PreNormBlock

@@ -8,7 +8,9 @@ all experts -> top-k (ties to the lower index) -> optional renormalisation ->
 routed scale; stable dispatch by expert; per expert ``down(silu(gate(x)) *
 up(x))``; combine in slot order with fp32 weights; a shared expert over every
 token whose output is scaled by ``sigmoid(x . w_gate)`` when gated
-(moe_ffn.cc:308-355).  Expert weights are stacked per layer as
+(moe_ffn.cc:308-355).  A spec may ask for sigmoid scores in the softmax's place, and for the
+weight on the expert's input instead of its output: the gate and up products being linear,
+the weight then multiplies their accumulators ahead of the activation.  Expert weights are stacked per layer as
 ``[E, 2I, H]`` (gate rows then up rows per expert) and ``[E, H, I]``
 (src/model/deepseek_v2.cc:519-556).
 """
@@ -143,8 +145,15 @@ class MoeFeedForward:
         self.renorm_eps = float(getattr(spec, "renorm_eps", -1.0))
         self.correction_name = getattr(spec, "correction_name", None)
         self.correction = None
+        self.score = getattr(spec, "score", "softmax")
+        self.weight_input = bool(getattr(spec, "weight_input", False))
+        if self.score not in ("softmax", "sigmoid"):
+            raise ValueError(f"{prefix}: router score {self.score!r}")
+        if self.weight_input and self.identity:
+            raise ValueError(f"{prefix}: identity experts are not combined with weights on the "
+                             "experts' inputs")
         self.ruled = bool(self.identity or self.group_count or self.correction_name
-                          or self.renorm_eps >= 0)
+                          or self.renorm_eps >= 0 or self.score != "softmax")
         if spec.top_k > self.outputs:
             raise ValueError("top_k exceeds the number of experts")
         if self.group_count and (self.outputs % self.group_count
@@ -300,20 +309,30 @@ class MoeFeedForward:
                 x, self.router_w, s.top_k, s.renormalize, s.routed_scale,
                 extra_w=self.shared_gate_w, correction=self.correction,
                 group_count=self.group_count, group_keep=self.group_keep,
-                renorm_eps=self.renorm_eps)
+                renorm_eps=self.renorm_eps, **({} if self.score == "softmax"
+                                               else {"score": self.score}))
         else:
             topk_w, topk_idx, shared_logit = ops.router_topk(
                 x, self.router_w, s.top_k, s.renormalize, s.routed_scale,
                 extra_w=self.shared_gate_w)
         # identity experts are the router's last outputs: the stable dispatch puts their
         # rows behind every expert's, where no product writes
-        all_offsets, rows, dest = ops.moe_dispatch(topk_idx, self.outputs)
+        row_w = None
+        if self.weight_input:       # the weights travel with the rows into the experts
+            all_offsets, rows, dest, row_w = ops.moe_dispatch(topk_idx, self.outputs,
+                                                              topk_w=topk_w)
+        else:
+            all_offsets, rows, dest = ops.moe_dispatch(topk_idx, self.outputs)
         offsets = all_offsets[:s.num_experts + 1] if self.identity else all_offsets
         if ready is not None:
             side.wait_event(ready)
             with torch.cuda.stream(side):
                 shared = self.shared.forward(x, step)
-        act = ops.grouped_gate_up_swiglu(x, rows, offsets, self.expert_gate_up)
+        if row_w is None:
+            act = ops.grouped_gate_up_swiglu(x, rows, offsets, self.expert_gate_up)
+        else:
+            act = ops.grouped_gate_up_swiglu(x, rows, offsets, self.expert_gate_up,
+                                             row_scale=row_w)
         # `offsets` was written by the dispatch, two launches back: the down product may
         # start on its weights while the gate/up product drains
         y = ops.grouped_down(act, offsets, self.expert_down, offsets_settled=True)
@@ -325,6 +344,8 @@ class MoeFeedForward:
         elif self.shared is not None:
             shared = self.shared.forward(x, step)
         combine = getattr(ops, "moe_combine_pending", ops.moe_combine)
+        if self.weight_input:
+            return combine(y, dest, topk_w, shared, shared_logit, weighted=False)
         return combine(y, dest, topk_w, shared, shared_logit)
 
 

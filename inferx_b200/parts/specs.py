@@ -106,9 +106,20 @@ class LatentAttentionSpec:
     position: Any      # encoding of the rotated part, or None
     latent_eps: float
     output_gate: bool = True
+    # Queries through a latent of their own: q = W_uq norm(W_dq h), an RMS norm with a gain
+    # over ``q_rank`` entries and ``latent_eps``.  0: q = W_q h; -1: the size is the
+    # checkpoint's.
+    q_rank: int = 0
+    # False: the layer has no down-projection and reads the records another layer keeps
+    # (the schedule names it); sizes and rotation of the records are that layer's.
+    own_records: bool = True
+    # softmax weights keep 16 bits in their product with the latents in bfloat16 runs
+    fp32_weights: bool = False
+    out_float32: bool = True     # the output projection leaves in fp32
     # tensor names inside the mixer's prefix
     names: tuple = (("q", "q"), ("dkv", "dkv"), ("dkv_norm", "dkv.norm"), ("uk", "uk"),
-                    ("uv", "uv"), ("g", "g"), ("o", "o"))
+                    ("uv", "uv"), ("g", "g"), ("o", "o"), ("dq", "dq"), ("dq_norm", "dq.norm"),
+                    ("uq", "uq"))
     kind: str = "latent_attention"
 
 
@@ -277,6 +288,54 @@ class NormedPairSpec:
 
 
 @dataclass(frozen=True)
+class DistanceAttentionSpec:
+    """Grouped-query softmax attention without a rotation whose scores lose a logarithm of
+    the distance: (q . k) * scale * temp_h - r1_h ln(1 + r2_h (i - j)), with ``temp``,
+    ``r1`` and ``r2`` vectors of the checkpoint, one number per head.  ``chunk`` > 0: a
+    query sees only the keys of its own run of ``chunk`` positions, runs being counted from
+    position 0 of the sequence (0: every earlier key).  Scores, weights and their products
+    with the values are 32-bit arithmetic in every element type."""
+    hidden: int
+    heads: int
+    kv_heads: int
+    head_dim: int
+    value_dim: int
+    scale: float
+    chunk: int = 0
+    names: tuple = (("q", "q"), ("k", "k"), ("v", "v"), ("o", "o"), ("temp", "temp"),
+                    ("r1", "r1"), ("r2", "r2"))
+    kind: str = "attention_distance"
+
+
+@dataclass(frozen=True)
+class MinGruSpec:
+    """Gated recurrence whose gates read the current token alone: z = sigmoid(W_z h + b_z),
+    u = W_x h + b_x, candidate c = u + ``shift`` where u >= 0 and sigmoid(u) where u < 0;
+    entry by entry S_t = (1 - z) S_(t-1) + z c; output W_o (S_t * silu(W_g h)).  State per
+    request: S [width] fp32."""
+    hidden: int
+    width: int
+    shift: float = 0.5
+    names: tuple = (("z", "z"), ("z_bias", "z.b"), ("x", "x"), ("x_bias", "x.b"), ("g", "g"),
+                    ("o", "o"))
+    kind: str = "min_gru"
+
+
+@dataclass(frozen=True)
+class ScaledPairSpec:
+    """Two mixers side by side reading the same input; the result is
+    ``left_scale`` * left + ``right_scale`` * right."""
+    hidden: int
+    left: Any
+    right: Any
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+    left_name: str = "left"
+    right_name: str = "right"
+    kind: str = "scaled_pair"
+
+
+@dataclass(frozen=True)
 class ReluSquaredSpec:
     """down(relu(up h)^2), no biases."""
     hidden: int
@@ -427,6 +486,11 @@ class MoeSpec:
     group_count: int = 0
     group_keep: int = 0
     renorm_eps: float = -1.0
+    # What a router output becomes before the choice: its "softmax" over all outputs, or
+    # its own "sigmoid".
+    score: str = "softmax"
+    # The weight multiplies the expert's input instead of its output: expert(w h).
+    weight_input: bool = False
     kind: str = "moe"
 
 
@@ -506,5 +570,6 @@ class ModelSpec:
     head_name: str = "lm_head.weight"
     embed_scale: float = 1.0     # the residual stream starts as embed[token] * embed_scale
     logit_scale: float = 1.0     # the head's products are multiplied by this
+    logit_softcap: float = 0.0   # > 0: logits become softcap * tanh(logits / softcap)
     embed_position: Any = None   # a position spec whose vector is added to the embedding
     embedding: Any = None        # a spec of what forms the stream from the tokens (None: the table's rows)

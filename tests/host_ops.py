@@ -130,13 +130,15 @@ def paged_attention(q, k_cache, v_cache, block_table, step, window, scale, softc
 
 
 def router_topk(x, w, top_k, renormalize, scale, extra_w=None, correction=None, group_count=0,
-                group_keep=0, renorm_eps=-1.0):
+                group_keep=0, renorm_eps=-1.0, score="softmax"):
     logits = _f(x) @ w.T
-    p = torch.softmax(logits, dim=-1)
+    p = torch.sigmoid(logits) if score == "sigmoid" else torch.softmax(logits, dim=-1)
     T, E = p.shape
-    if correction is not None or group_count or renorm_eps >= 0:
+    if correction is not None or group_count or renorm_eps >= 0 or score != "softmax":
         # the choice is by score + correction, inside the best groups; weights are the scores
         pick = p + (correction if correction is not None else 0.0)
+        if score == "sigmoid" and correction is None:
+            pick = logits.clone()         # the same order, also where the sigmoid is flat
         if group_count:
             size = E // group_count
             best = pick.view(T, group_count, size).max(-1).values
@@ -181,7 +183,7 @@ def router_topk(x, w, top_k, renormalize, scale, extra_w=None, correction=None, 
     return tw * scale, ti, ex
 
 
-def moe_dispatch(topk_idx, num_experts):
+def moe_dispatch(topk_idx, num_experts, topk_w=None):
     T, k = topk_idx.shape
     flat = topk_idx.reshape(-1).long()
     order = torch.sort(flat, stable=True).indices
@@ -191,10 +193,12 @@ def moe_dispatch(topk_idx, num_experts):
     rows = (order // k).to(torch.int32)
     dest = torch.empty(T * k, dtype=torch.int32)
     dest[order] = torch.arange(T * k, dtype=torch.int32)
+    if topk_w is not None:
+        return offsets, rows, dest, topk_w.reshape(-1)[order].clone()
     return offsets, rows, dest
 
 
-def grouped_gate_up_swiglu(x, rows, offsets, w_gate_up):
+def grouped_gate_up_swiglu(x, rows, offsets, w_gate_up, row_scale=None):
     E, two_i, H = w_gate_up.shape
     i = two_i // 2
     out = torch.zeros(rows.numel(), i, dtype=torch.float32)
@@ -202,6 +206,8 @@ def grouped_gate_up_swiglu(x, rows, offsets, w_gate_up):
         lo, hi = int(offsets[e]), int(offsets[e + 1])
         if hi > lo:
             xe = _f(x[rows[lo:hi].long()])
+            if row_scale is not None:
+                xe = xe * row_scale[lo:hi, None]
             g = xe @ _f(w_gate_up[e, :i]).T
             u = xe @ _f(w_gate_up[e, i:]).T
             out[lo:hi] = g / (1.0 + torch.exp(-g)) * u
@@ -218,8 +224,10 @@ def grouped_down(act, offsets, w_down, offsets_settled=False):
     return out.to(act.dtype)
 
 
-def moe_combine(y, dest, topk_w, shared, shared_logit):
+def moe_combine(y, dest, topk_w, shared, shared_logit, weighted=True):
     T, k = topk_w.shape
+    if not weighted:
+        topk_w = torch.ones_like(topk_w)
     out = torch.zeros(T, y.shape[1], dtype=torch.float32)
     for s in range(k):
         out += topk_w[:, s:s + 1] * _f(y[dest.view(T, k)[:, s].long()])
@@ -364,8 +372,12 @@ def gate_up_glu_clamped(x, w_gate_up, limit, alpha, up_shift):
     return glu_clamped(linear(x, w_gate_up), limit, alpha, up_shift)
 
 
-def batched_linear(x, w):
-    return torch.bmm(_f(x), _f(w).transpose(1, 2)).to(x.dtype)
+def batched_linear(x, w, out=None):
+    y = torch.bmm(_f(x), _f(w).transpose(1, 2)).to(x.dtype)
+    if out is not None:
+        out.copy_(y)
+        return out
+    return y
 
 
 def _turn_pairs(v, positions, freq, mag, rot_dims):
@@ -397,7 +409,7 @@ def latent_prepare(proj, q_off, kv_off, positions, freq, mag, gain, eps, heads, 
     return q_rot, q[..., :dim].transpose(0, 1).contiguous().to(proj.dtype)
 
 
-def latent_attention(q_lat, q_rot, cache, block_table, step, window, scale):
+def latent_attention(q_lat, q_rot, cache, block_table, step, window, scale, fp32_weights=False):
     H, T, rank = q_lat.shape
     page = cache.shape[2]
     out = torch.zeros(H, T, rank, dtype=torch.float32)
@@ -749,3 +761,78 @@ def identity_rows(x, rows, offsets, first_identity, y):
     if hi > lo:
         y[lo:hi] = x[rows[lo:hi].long()].to(y.dtype)
     return y
+
+
+# ---------------------------------------------------------------------------------------
+# parts of decoders that pair chunked attention and a gated recurrence, and whose latent
+# queries have a latent of their own
+def append_kv_rows(k, v, k_cache, v_cache, slots):
+    T = k.shape[0]
+    _scatter(k_cache, k.reshape(T, k_cache.shape[1], k_cache.shape[3]), slots)
+    _scatter(v_cache, v.reshape(T, v_cache.shape[1], v_cache.shape[3]), slots)
+
+
+def distance_attention(q, k_cache, v_cache, block_table, step, scale, temp, r1, r2, chunk, out,
+                       out_scale=1.0):
+    P, kvh, page, hd = k_cache.shape
+    vd = v_cache.shape[3]
+    T, heads = q.shape[0], q.shape[1] // hd
+    rep = heads // kvh
+    for t in range(T):
+        s, pos = int(step.seq_of_token[t]), int(step.positions[t])
+        kp = torch.arange(pos // chunk * chunk if chunk > 0 else 0, pos + 1)
+        pages = block_table[s][(kp // page).long()].long()
+        assert (pages >= 0).all(), "attention reads a page that was given back"
+        offs = (kp % page).long()
+        d = (pos - kp).to(torch.float32)
+        for h in range(heads):
+            keys = _f(k_cache[pages, h // rep, offs, :])
+            sc = (keys @ _f(q[t, h * hd:(h + 1) * hd])) * scale * temp[h]
+            sc = sc - r1[h] * torch.log1p(r2[h] * d)
+            a = torch.softmax(sc, dim=0)
+            o = (a[:, None] * _f(v_cache[pages, h // rep, offs, :])).sum(0)
+            out[t, h * vd:(h + 1) * vd] = (o * out_scale).to(out.dtype)
+    return out
+
+
+def min_gru(front, z_bias, x_bias, shift, state, step, out, out_scale=1.0):
+    W = z_bias.numel()
+    z = torch.sigmoid(_f(front[:, :W]) + z_bias)
+    u = _f(front[:, W:2 * W]) + x_bias
+    g = _f(front[:, 2 * W:3 * W])
+    c = torch.where(u >= 0, u + shift, torch.sigmoid(u))
+    cu = [int(v) for v in step.cu_q]
+    for s in range(len(cu) - 1):
+        slot = int(step.state_slot[s])
+        S = state[slot].clone()
+        for t in range(cu[s], cu[s + 1]):
+            S = (1.0 - z[t]) * S + z[t] * c[t]
+            out[t] = (S * g[t] * torch.sigmoid(g[t]) * out_scale).to(out.dtype)
+        state[slot] = S
+    return out
+
+
+def latent_front(proj, q_rank, q_gain, eps, kv_off, positions, freq, mag, kv_gain, rank, rot_dim,
+                 rot_dims, cache, slots):
+    x = _f(proj)
+
+    def norm(v, gain):
+        return v * (1.0 / torch.sqrt((v * v).sum(-1, keepdim=True) / v.shape[-1] + eps)) * gain
+    if cache is not None:
+        c = norm(x[:, kv_off:kv_off + rank], kv_gain)
+        kr = _turn_pairs(x[:, kv_off + rank:kv_off + rank + rot_dim], positions, freq, mag,
+                         rot_dims)
+        _scatter(cache, torch.cat([c, kr], dim=-1)[:, None, :], slots)
+    return norm(x[:, :q_rank], q_gain).to(proj.dtype)
+
+
+def latent_queries(q, positions, freq, mag, heads, dim, rot_dim, rot_dims):
+    T = q.shape[0]
+    x = _f(q).reshape(T, heads, dim + rot_dim)
+    q_rot = _turn_pairs(x[..., dim:], positions, freq, mag, rot_dims).contiguous().to(q.dtype)
+    return q_rot, x[..., :dim].transpose(0, 1).contiguous().to(q.dtype)
+
+
+def softcap_rows(x, cap):
+    x.copy_(cap * torch.tanh(x / cap))
+    return x
