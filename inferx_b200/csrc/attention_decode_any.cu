@@ -18,8 +18,11 @@
 // one to the softmax's denominator (a key of score 0 without a value), where the result
 // is normalised: in this kernel when the sequence is not split, else in the merge.
 //
+// A third form (attention_distance.cuh) multiplies a score by its head's temperature, takes
+// r1 ln(1 + r2 distance) off and may confine the query to its own run of positions.
+//
 // Scratch: partial outputs [S, heads, splits, vd] and (max, sum) [S, heads, splits, 2], fp32.
-#include "common.cuh"
+#include "attention_distance.cuh"
 
 #define DA_THREADS 128
 #define DA_WARPS 4
@@ -33,7 +36,8 @@ attn_decode_any_kernel(const TA* __restrict__ q, const TA* __restrict__ kc,
                        const int* __restrict__ kv_len, float* __restrict__ part_o,
                        float* __restrict__ part_ml, TA* __restrict__ out, int heads, int kvh,
                        int hd, int vd, int page_size, int maxb, int window, float scale,
-                       float softcap, int splits, int keep_first, int sink) {
+                       float softcap, int splits, int keep_first, int sink, IxRows rows,
+                       IxDistance dist) {
   extern __shared__ float sm[];
   float* sm_acc = sm;                               // [G][DA_WARPS][vd]
   float* sm_m = sm_acc + (size_t)G * DA_WARPS * vd; // [G][DA_WARPS]
@@ -49,7 +53,7 @@ attn_decode_any_kernel(const TA* __restrict__ q, const TA* __restrict__ kc,
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
 
   const int len = kv_len[s];
-  const int start = window > 0 ? max(0, len - window) : 0;
+  const int start = ix_first_key(len - 1, window, dist.chunk);
   // the kept first keys stand, in the walk, directly before the window: walk index j means
   // key j - (start - kept) below `start` and key j from there on
   const int kept = min(keep_first, start);
@@ -62,15 +66,21 @@ attn_decode_any_kernel(const TA* __restrict__ q, const TA* __restrict__ kc,
   const int* bt = block_table + (size_t)s * maxb;
 
   float qr[G][D], acc[G][D], m[G], l[G];
+  const bool far = dist.temp != nullptr;
+  float temp[G], r1[G], r2[G];
 #pragma unroll
   for (int g = 0; g < G; ++g) {
+    const bool on = far && g < gcount;
+    temp[g] = on ? dist.temp[h0 + g] : 1.f;
+    r1[g] = on ? dist.r1[h0 + g] : 0.f;
+    r2[g] = on ? dist.r2[h0 + g] : 0.f;
     m[g] = -INFINITY;
     l[g] = 0.f;
 #pragma unroll
     for (int e = 0; e < D; ++e) {
       const int d = lane + 32 * e;
       acc[g][e] = 0.f;
-      qr[g][e] = (g < gcount && d < hd) ? to_f32(q[((size_t)s * heads + h0 + g) * hd + d]) : 0.f;
+      qr[g][e] = (g < gcount && d < hd) ? to_f32(q[(size_t)s * rows.q_ld + (size_t)(h0 + g) * hd + d]) : 0.f;
     }
   }
 
@@ -124,6 +134,7 @@ attn_decode_any_kernel(const TA* __restrict__ q, const TA* __restrict__ kc,
         for (int e = 0; e < D; ++e) dot = fmaf(qr[g][e], kf[u][e], dot);
         dot = warp_sum(dot);
         float sv = dot * scale;
+        if (far) sv = sv * temp[g] - r1[g] * log1pf(r2[g] * (float)max(0, len - 1 - (kb + u)));
         if (softcap > 0.f) sv = softcap * tanhf(sv / softcap);
         sc[u] = valid[u] ? sv : -INFINITY;
       }
@@ -189,7 +200,8 @@ attn_decode_any_kernel(const TA* __restrict__ q, const TA* __restrict__ kc,
         o *= c;
         L = L * c + expf(-top);
       }
-      out[hrow * vd + d] = from_f32<TA>(L > 0.f ? o / L : 0.f);
+      out[(size_t)s * rows.o_ld + (size_t)(h0 + g) * vd + d] =
+          from_f32<TA>(L > 0.f ? o / L * rows.o_scale : 0.f);
     } else {
       part_o[(hrow * splits + split) * vd + d] = o;
       if (d == 0) {
@@ -203,8 +215,8 @@ attn_decode_any_kernel(const TA* __restrict__ q, const TA* __restrict__ kc,
 template <typename TA>
 __global__ void attn_decode_any_merge_kernel(const float* __restrict__ part_o,
                                              const float* __restrict__ part_ml,
-                                             TA* __restrict__ out, int vd, int splits,
-                                             int sink) {
+                                             TA* __restrict__ out, int heads, int vd,
+                                             int splits, int sink, IxRows rows) {
   IX_PDL_WAIT();
   const size_t hrow = blockIdx.x;   // s * heads + h
   const float* ml = part_ml + hrow * splits * 2;
@@ -224,7 +236,8 @@ __global__ void attn_decode_any_merge_kernel(const float* __restrict__ part_o,
     for (int j = 0; j < splits; ++j)
       if (ml[2 * j] != -INFINITY)
         o = fmaf(part_o[(hrow * splits + j) * vd + d], expf(ml[2 * j] - M), o);
-    out[hrow * vd + d] = from_f32<TA>(L > 0.f ? o * c / L : 0.f);
+    out[hrow / heads * rows.o_ld + hrow % heads * vd + d] =
+        from_f32<TA>(L > 0.f ? o * c / L * rows.o_scale : 0.f);
   }
 }
 
@@ -255,12 +268,12 @@ IX_API int ix_attn_decode_any_splits(int S, int heads, int kvh, int hd, int vd, 
   return want < 1 ? 1 : (int)want;
 }
 
-IX_API int ix_paged_attention_decode_any(const void* q, const void* k_cache, const void* v_cache,
-                                         const int* block_table, const int* kv_len, float* part_o,
-                                         float* part_ml, void* out, int act_dtype, int S, int heads,
-                                         int kvh, int hd, int vd, int page_size, int max_blocks,
-                                         int window, float scale, float softcap, int splits,
-                                         int keep_first, int sink, cudaStream_t stream) {
+static int decode_any_checked(const void* q, const void* k_cache, const void* v_cache,
+                              const int* block_table, const int* kv_len, float* part_o,
+                              float* part_ml, void* out, int act_dtype, int S, int heads, int kvh,
+                              int hd, int vd, int page_size, int max_blocks, int window,
+                              float scale, float softcap, int splits, int keep_first, int sink,
+                              IxRows rows, IxDistance dist, cudaStream_t stream) {
   if (S <= 0) return IX_OK;
   if (heads <= 0 || kvh <= 0 || heads % kvh != 0 || page_size <= 0 || max_blocks <= 0)
     return IX_ERR_SIZE;
@@ -282,7 +295,8 @@ IX_API int ix_paged_attention_decode_any(const void* q, const void* k_cache, con
       cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);      \
     ix_launch(kern, grid, dim3(DA_THREADS), smem, stream, (const TA*)q, (const TA*)k_cache,    \
               (const TA*)v_cache, block_table, kv_len, part_o, part_ml, (TA*)out, heads, kvh,  \
-              hd, vd, page_size, max_blocks, window, scale, softcap, splits, keep_first, sink); \
+              hd, vd, page_size, max_blocks, window, scale, softcap, splits, keep_first, sink, \
+              rows, dist);                                                                     \
   })
 #define DA_D(DD)                                                                               \
   do {                                                                                         \
@@ -301,7 +315,35 @@ IX_API int ix_paged_attention_decode_any(const void* q, const void* k_cache, con
   if (rc != 0 || splits == 1) return rc;
   IX_DISPATCH_DTYPE(act_dtype, TA, {
     ix_launch(attn_decode_any_merge_kernel<TA>, dim3(S * heads), dim3(vd >= 128 ? 128 : 64), 0,
-              stream, (const float*)part_o, (const float*)part_ml, (TA*)out, vd, splits, sink);
+              stream, (const float*)part_o, (const float*)part_ml, (TA*)out, heads, vd, splits, sink,
+              rows);
   });
   return ix_launch_status();
+}
+
+IX_API int ix_paged_attention_decode_any(const void* q, const void* k_cache, const void* v_cache,
+                                         const int* block_table, const int* kv_len, float* part_o,
+                                         float* part_ml, void* out, int act_dtype, int S, int heads,
+                                         int kvh, int hd, int vd, int page_size, int max_blocks,
+                                         int window, float scale, float softcap, int splits,
+                                         int keep_first, int sink, cudaStream_t stream) {
+  return decode_any_checked(q, k_cache, v_cache, block_table, kv_len, part_o, part_ml, out,
+                            act_dtype, S, heads, kvh, hd, vd, page_size, max_blocks, window, scale,
+                            softcap, splits, keep_first, sink,
+                            IxRows{(long long)heads * hd, (long long)heads * vd, 1.f},
+                            ix_no_distance(), stream);
+}
+
+// With a temperature and a distance penalty per head (see attention_distance.cuh).
+IX_API int ix_distance_attention_decode_any(
+    const void* q, long long q_ld, const void* k_cache, const void* v_cache,
+    const int* block_table, const int* kv_len, float* part_o, float* part_ml, void* out,
+    long long o_ld, float o_scale, int act_dtype, int S, int heads, int kvh, int hd, int vd,
+    int page_size, int max_blocks, float scale, int splits, const float* temp, const float* r1,
+    const float* r2, int chunk, cudaStream_t stream) {
+  if (!temp || !r1 || !r2 || chunk < 0) return IX_ERR_SIZE;
+  return decode_any_checked(q, k_cache, v_cache, block_table, kv_len, part_o, part_ml, out,
+                            act_dtype, S, heads, kvh, hd, vd, page_size, max_blocks, 0, scale, 0.f,
+                            splits, 0, 0, IxRows{q_ld, o_ld, o_scale},
+                            IxDistance{temp, r1, r2, chunk}, stream);
 }

@@ -21,10 +21,12 @@
 //  * `keep_first`: the sequence's first keep_first keys stay visible beside the window;
 //    the walk goes over them and then over the window as one range that is split;
 //  * `sink`: one is added to the denominator where the result is normalised.
+//  * DIST: a score is multiplied by its head's temperature and loses r1 ln(1 + r2 distance),
+//    and the query may be confined to its own run of positions (attention_distance.cuh).
 //
 // Scratch: partial outputs [S, heads, splits, vd] and (max, sum) [S, heads, splits, 2],
 // fp32; maxima are in units of log2 (scores are pre-multiplied by log2 e).
-#include "common.cuh"
+#include "attention_distance.cuh"
 
 #define DX_THREADS 128
 #define DX_WARPS 4
@@ -68,14 +70,15 @@ __device__ __forceinline__ unsigned dx_pack(float lo, float hi) {
   return *reinterpret_cast<unsigned*>(&v);
 }
 
-template <int HD, int VD, bool FOLD>
+template <int HD, int VD, bool FOLD, bool DIST>
 __global__ void __launch_bounds__(DX_THREADS)
 attn_decode_exact_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc,
                          const bf16* __restrict__ vc, const int* __restrict__ block_table,
                          const int* __restrict__ kv_len, float* __restrict__ part_o,
                          float* __restrict__ part_ml, bf16* __restrict__ out, int heads, int kvh,
                          int page_size, int page_shift, int maxb, int window, float scale_log2e,
-                         int splits, int keep_first, int sink) {
+                         int splits, int keep_first, int sink, IxRows rows,
+                         IxDistance dist) {
   constexpr int CH = HD / 8, CHV = VD / 8, KS = HD / 16, DT = VD / 8;
   constexpr int K_TILE = DX_BN * HD * 2, V_TILE = DX_BN * VD * 2;
   extern __shared__ __align__(128) unsigned char dsm[];
@@ -97,7 +100,7 @@ attn_decode_exact_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc
   const int g = lane >> 2, t = lane & 3;
 
   const int len = kv_len[s];
-  const int start = window > 0 ? max(0, len - window) : 0;
+  const int start = ix_first_key(len - 1, window, DIST ? dist.chunk : 0);
   // the kept first keys stand, in the walk, directly before the window: walk index j means
   // key j - shift below `start` and key j from there on
   const int kept = min(keep_first, start);
@@ -113,7 +116,21 @@ attn_decode_exact_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc
   for (int idx = tid; idx < 16 * CH; idx += DX_THREADS) {
     const int r = idx / CH, c = idx - r * CH;
     const bool ok = r < rows_valid;
-    dx_cp16(Qs + dx_swz<CH>(r, c), q + ((size_t)s * heads + h0 + (ok ? r : 0)) * HD + c * 8, ok);
+    dx_cp16(Qs + dx_swz<CH>(r, c),
+            q + (size_t)s * rows.q_ld + (size_t)(h0 + (ok ? r : 0)) * HD + c * 8, ok);
+  }
+  // DIST: this thread's two rows' factor on a raw score and penalty (log2 units)
+  float hs[2] = {scale_log2e, scale_log2e}, r1[2] = {0.f, 0.f}, r2[2] = {0.f, 0.f};
+  if (DIST) {
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      if (g + 8 * r < rows_valid) {
+        const int h = h0 + g + 8 * r;
+        hs[r] = scale_log2e * dist.temp[h];
+        r1[r] = dist.r1[h];
+        r2[r] = dist.r2[h];
+      }
+    }
   }
   auto load_kv = [&](int it) {
     if (it < n_tiles) {
@@ -201,7 +218,12 @@ attn_decode_exact_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
           const int kp = kw + j * 8 + 2 * t + (c & 1);
-          const float v = kp < k1 ? sc[j][c] * scale_log2e : -INFINITY;
+          float v = sc[j][c] * hs[c >> 1];
+          if (DIST) {
+            const float d = (float)max(0, len - 1 - kp);
+            v -= r1[c >> 1] * ix_log2(fmaf(r2[c >> 1], d, 1.f));
+          }
+          if (kp >= k1) v = -INFINITY;
           sc[j][c] = v;
           mx[c >> 1] = fmaxf(mx[c >> 1], v);
         }
@@ -306,7 +328,8 @@ attn_decode_exact_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc
         ov *= c;
         L = L * c + dx_exp2(-top);
       }
-      out[hrow * VD + d] = __float2bfloat16_rn(L > 0.f ? ov / L : 0.f);
+      out[(size_t)s * rows.o_ld + (size_t)(h0 + r) * VD + d] =
+          __float2bfloat16_rn(L > 0.f ? ov / L * rows.o_scale : 0.f);
     } else {
       part_o[(hrow * splits + split) * VD + d] = ov;
       if (d == 0) {
@@ -319,8 +342,8 @@ attn_decode_exact_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc
 
 __global__ void attn_decode_exact_merge_kernel(const float* __restrict__ part_o,
                                                const float* __restrict__ part_ml,
-                                               bf16* __restrict__ out, int vd, int splits,
-                                               int sink) {
+                                               bf16* __restrict__ out, int heads, int vd,
+                                               int splits, int sink, IxRows rows) {
   IX_PDL_WAIT();
   const size_t hrow = blockIdx.x;   // s * heads + h
   const float* ml = part_ml + hrow * splits * 2;
@@ -340,7 +363,8 @@ __global__ void attn_decode_exact_merge_kernel(const float* __restrict__ part_o,
     for (int j = 0; j < splits; ++j)
       if (ml[2 * j] != -INFINITY)
         o += part_o[(hrow * splits + j) * vd + d] * dx_exp2(ml[2 * j] - M);
-    out[hrow * vd + d] = __float2bfloat16_rn(L > 0.f ? o * c / L : 0.f);
+    out[hrow / heads * rows.o_ld + hrow % heads * vd + d] =
+        __float2bfloat16_rn(L > 0.f ? o * c / L * rows.o_scale : 0.f);
   }
 }
 
@@ -348,8 +372,8 @@ template <int HD, int VD>
 static int launch_decode_exact(const void* q, const void* kc, const void* vc, const int* bt,
                                const int* kv_len, float* part_o, float* part_ml, void* out, int S,
                                int heads, int kvh, int page_size, int maxb, int window,
-                               float scale, int splits, int keep_first, int sink,
-                               cudaStream_t stream) {
+                               float scale, int splits, int keep_first, int sink, IxRows rows,
+                               IxDistance dist, cudaStream_t stream) {
   const int rep = heads / kvh;
   const float sl2 = scale * 1.4426950408889634f;
   const int smem = 16 * HD * 2 + DX_STAGES * DX_BN * (HD + VD) * 2;
@@ -357,23 +381,29 @@ static int launch_decode_exact(const void* q, const void* kc, const void* vc, co
   int page_shift = -1;
   if ((page_size & (page_size - 1)) == 0)
     for (page_shift = 0; (1 << page_shift) < page_size; ++page_shift) {}
-#define DX_LAUNCH(FOLD_)                                                                        \
+#define DX_LAUNCH(FOLD_, DIST_)                                                                    \
   do {                                                                                          \
-    auto kern = attn_decode_exact_kernel<HD, VD, FOLD_>;                                        \
+    auto kern = attn_decode_exact_kernel<HD, VD, FOLD_, DIST_>;                                  \
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize,     \
                                          smem);                                                 \
     if (e != cudaSuccess) return (int)e;                                                        \
     ix_launch(kern, grid, dim3(DX_THREADS), smem, stream, (const bf16*)q, (const bf16*)kc,      \
               (const bf16*)vc, bt, kv_len, part_o, part_ml, (bf16*)out, heads, kvh, page_size,  \
-              page_shift, maxb, window, sl2, splits, keep_first, sink);                         \
+              page_shift, maxb, window, sl2, splits, keep_first, sink, rows, dist);             \
   } while (0)
-  if (rep <= 8) DX_LAUNCH(true);
-  else DX_LAUNCH(false);
+  if (dist.temp) {
+    if (rep <= 8) DX_LAUNCH(true, true);
+    else DX_LAUNCH(false, true);
+  } else {
+    if (rep <= 8) DX_LAUNCH(true, false);
+    else DX_LAUNCH(false, false);
+  }
 #undef DX_LAUNCH
   int rc = ix_launch_status();
   if (rc != 0 || splits == 1) return rc;
   ix_launch(attn_decode_exact_merge_kernel, dim3(S * heads), dim3(VD >= 128 ? 128 : 64), 0,
-            stream, (const float*)part_o, (const float*)part_ml, (bf16*)out, VD, splits, sink);
+            stream, (const float*)part_o, (const float*)part_ml, (bf16*)out, heads, VD, splits, sink,
+            rows);
   return ix_launch_status();
 }
 
@@ -382,6 +412,34 @@ IX_API int ix_paged_attention_decode_exact_applies(int hd, int vd) {
 }
 
 // q [S, heads, hd], out [S, heads, vd], caches [pages, kvh, page_size, hd or vd], bfloat16.
+static int decode_exact_checked(const void* q, const void* k_cache, const void* v_cache,
+                                const int* block_table, const int* kv_len, float* part_o,
+                                float* part_ml, void* out, int S, int heads, int kvh, int hd,
+                                int vd, int page_size, int max_blocks, int window, float scale,
+                                int splits, int keep_first, int sink, IxRows rows,
+                                IxDistance dist, cudaStream_t stream) {
+  if (S <= 0) return IX_OK;
+  if (heads <= 0 || kvh <= 0 || heads % kvh != 0 || page_size <= 0 || max_blocks <= 0 ||
+      window < 0 || keep_first < 0 || splits < 1 || (!dist.temp && !(scale > 0.f)))
+    return IX_ERR_SIZE;
+  if (splits > 1 && (!part_o || !part_ml)) return IX_ERR_SIZE;
+  if ((long long)kvh * ((heads / kvh + 15) / 16) > 65535 || S > 65535) return IX_ERR_SIZE;
+  if (((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15) return IX_ERR_ALIGN;
+  if (rows.q_ld % 8) return IX_ERR_ALIGN;
+#define DX_GO(H_, V_)                                                                         \
+  if (hd == H_ && vd == V_)                                                                   \
+    return launch_decode_exact<H_, V_>(q, k_cache, v_cache, block_table, kv_len, part_o,      \
+                                       part_ml, out, S, heads, kvh, page_size, max_blocks,    \
+                                       window, scale, splits, keep_first, sink, rows, dist,   \
+                                       stream);
+  DX_GO(64, 64)
+  DX_GO(64, 128)
+  DX_GO(128, 64)
+  DX_GO(128, 128)
+#undef DX_GO
+  return IX_ERR_UNSUPPORTED;
+}
+
 IX_API int ix_paged_attention_decode_exact(const void* q, const void* k_cache,
                                            const void* v_cache, const int* block_table,
                                            const int* kv_len, float* part_o, float* part_ml,
@@ -389,22 +447,23 @@ IX_API int ix_paged_attention_decode_exact(const void* q, const void* k_cache,
                                            int page_size, int max_blocks, int window, float scale,
                                            int splits, int keep_first, int sink,
                                            cudaStream_t stream) {
-  if (S <= 0) return IX_OK;
-  if (heads <= 0 || kvh <= 0 || heads % kvh != 0 || page_size <= 0 || max_blocks <= 0 ||
-      window < 0 || keep_first < 0 || splits < 1 || !(scale > 0.f))
-    return IX_ERR_SIZE;
-  if (splits > 1 && (!part_o || !part_ml)) return IX_ERR_SIZE;
-  if ((long long)kvh * ((heads / kvh + 15) / 16) > 65535 || S > 65535) return IX_ERR_SIZE;
-  if (((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15) return IX_ERR_ALIGN;
-#define DX_GO(H_, V_)                                                                         \
-  if (hd == H_ && vd == V_)                                                                   \
-    return launch_decode_exact<H_, V_>(q, k_cache, v_cache, block_table, kv_len, part_o,      \
-                                       part_ml, out, S, heads, kvh, page_size, max_blocks,    \
-                                       window, scale, splits, keep_first, sink, stream);
-  DX_GO(64, 64)
-  DX_GO(64, 128)
-  DX_GO(128, 64)
-  DX_GO(128, 128)
-#undef DX_GO
-  return IX_ERR_UNSUPPORTED;
+  return decode_exact_checked(q, k_cache, v_cache, block_table, kv_len, part_o, part_ml, out, S,
+                              heads, kvh, hd, vd, page_size, max_blocks, window, scale, splits,
+                              keep_first, sink,
+                              IxRows{(long long)heads * hd, (long long)heads * vd, 1.f},
+                              ix_no_distance(), stream);
+}
+
+// With a temperature and a distance penalty per head (see attention_distance.cuh).
+IX_API int ix_distance_attention_decode_exact(
+    const void* q, long long q_ld, const void* k_cache, const void* v_cache,
+    const int* block_table, const int* kv_len, float* part_o, float* part_ml, void* out,
+    long long o_ld, float o_scale, int S, int heads, int kvh, int hd, int vd, int page_size,
+    int max_blocks, float scale, int splits, const float* temp, const float* r1, const float* r2,
+    int chunk, cudaStream_t stream) {
+  if (!temp || !r1 || !r2 || chunk < 0) return IX_ERR_SIZE;
+  return decode_exact_checked(q, k_cache, v_cache, block_table, kv_len, part_o, part_ml, out, S,
+                              heads, kvh, hd, vd, page_size, max_blocks, 0, scale, splits, 0, 0,
+                              IxRows{q_ld, o_ld, o_scale}, IxDistance{temp, r1, r2, chunk},
+                              stream);
 }

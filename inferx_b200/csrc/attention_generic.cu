@@ -19,7 +19,10 @@
 // keep_first keys visible beside the window (they are walked first, as if they stood
 // directly before the window), and `sink` adds one to the softmax's denominator (a key
 // of score 0 that has no value).
-#include "common.cuh"
+//
+// A third form (attention_distance.cuh) multiplies a score by its head's temperature, takes
+// r1 ln(1 + r2 distance) off and may confine a query to its own run of positions.
+#include "attention_distance.cuh"
 
 #define ATT_TILE 128
 #define ATT_THREADS 128
@@ -33,7 +36,7 @@ paged_attention_generic_kernel(const TA* __restrict__ q, const TA* __restrict__ 
                                const int* __restrict__ positions, TA* __restrict__ out, int heads,
                                int kvh, int hd, int vd, int page_size, int max_blocks,
                                int window, float scale, float softcap, int keep_first,
-                               int sink) {
+                               int sink, IxRows rows, IxDistance dist) {
   extern __shared__ float smem[];
   float* qs = smem;        // [hd]
   float* sc = smem + hd;   // [ATT_TILE]
@@ -46,7 +49,10 @@ paged_attention_generic_kernel(const TA* __restrict__ q, const TA* __restrict__ 
   const int nwarps = ATT_THREADS / 32;
   const int* bt = block_table + (size_t)s * max_blocks;
 
-  const TA* qrow = q + ((size_t)t * heads + h) * hd;
+  const TA* qrow = q + (size_t)t * rows.q_ld + (size_t)h * hd;
+  const bool far = dist.temp != nullptr;
+  const float temp = far ? dist.temp[h] : 1.f;
+  const float r1 = far ? dist.r1[h] : 0.f, r2 = far ? dist.r2[h] : 0.f;
   for (int d = threadIdx.x; d < hd; d += ATT_THREADS) qs[d] = to_f32(qrow[d]);
   __syncthreads();
 
@@ -55,7 +61,7 @@ paged_attention_generic_kernel(const TA* __restrict__ q, const TA* __restrict__ 
   for (int i = 0; i < ATT_MAX_DPT; ++i) acc[i] = 0.f;
   float m = -INFINITY, l = 0.f;
 
-  const int start = window > 0 ? max(0, pos - window + 1) : 0;
+  const int start = ix_first_key(pos, window, dist.chunk);
   // the kept first keys count as positions start - kept .. start - 1 of the walk
   const int kept = min(keep_first, start);
   for (int tile0 = start - kept; tile0 <= pos; tile0 += ATT_TILE) {
@@ -71,7 +77,8 @@ paged_attention_generic_kernel(const TA* __restrict__ q, const TA* __restrict__ 
       for (int d = lane; d < hd; d += 32) dot += qs[d] * to_f32(krow[d]);
       dot = warp_sum(dot);
       if (lane == 0) {
-        const float sv = dot * scale;
+        float sv = dot * scale;
+        if (far) sv = sv * temp - r1 * log1pf(r2 * (float)(pos - kp));
         sc[j] = softcap > 0.f ? softcap * tanhf(sv / softcap) : sv;   // squashed scores
       }
     }
@@ -104,7 +111,7 @@ paged_attention_generic_kernel(const TA* __restrict__ q, const TA* __restrict__ 
     }
     __syncthreads();
   }
-  TA* orow = out + ((size_t)t * heads + h) * vd;
+  TA* orow = out + (size_t)t * rows.o_ld + (size_t)h * vd;
   float inv_l = 1.0f / l;
   if (sink) {          // one more term, exp(0 - max), in the denominator
     const float top = fmaxf(m, 0.f);
@@ -114,7 +121,7 @@ paged_attention_generic_kernel(const TA* __restrict__ q, const TA* __restrict__ 
 #pragma unroll
   for (int i = 0; i < ATT_MAX_DPT; ++i) {
     const int d = threadIdx.x + i * ATT_THREADS;
-    if (d < vd) orow[d] = from_f32<TA>(acc[i] * inv_l);
+    if (d < vd) orow[d] = from_f32<TA>(acc[i] * inv_l * rows.o_scale);
   }
 }
 
@@ -122,12 +129,12 @@ paged_attention_generic_kernel(const TA* __restrict__ q, const TA* __restrict__ 
 // kernels take fewer); a model is checked against it when it is built.
 IX_API int ix_attention_max_head_dim() { return ATT_THREADS * ATT_MAX_DPT; }
 
-IX_API int ix_paged_attention_generic(const void* q, const void* k_cache, const void* v_cache,
-                                      const int* block_table, const int* seq_of_token,
-                                      const int* positions, void* out, int act_dtype, int T,
-                                      int heads, int kvh, int hd, int vd, int page_size,
-                                      int max_blocks, int window, float scale, float softcap,
-                                      int keep_first, int sink, cudaStream_t stream) {
+static int generic_checked(const void* q, const void* k_cache, const void* v_cache,
+                           const int* block_table, const int* seq_of_token, const int* positions,
+                           void* out, int act_dtype, int T, int heads, int kvh, int hd, int vd,
+                           int page_size, int max_blocks, int window, float scale, float softcap,
+                           int keep_first, int sink, IxRows rows, IxDistance dist,
+                           cudaStream_t stream) {
   if (T <= 0) return IX_OK;
   if (heads <= 0 || kvh <= 0 || heads % kvh != 0 || page_size <= 0 || max_blocks <= 0)
     return IX_ERR_SIZE;
@@ -141,6 +148,31 @@ IX_API int ix_paged_attention_generic(const void* q, const void* k_cache, const 
                     (paged_attention_generic_kernel<TA><<<grid, ATT_THREADS, smem, stream>>>(
                         (const TA*)q, (const TA*)k_cache, (const TA*)v_cache, block_table,
                         seq_of_token, positions, (TA*)out, heads, kvh, hd, vd, page_size,
-                        max_blocks, window, scale, softcap, keep_first, sink)));
+                        max_blocks, window, scale, softcap, keep_first, sink, rows, dist)));
   return ix_launch_status();
+}
+
+IX_API int ix_paged_attention_generic(const void* q, const void* k_cache, const void* v_cache,
+                                      const int* block_table, const int* seq_of_token,
+                                      const int* positions, void* out, int act_dtype, int T,
+                                      int heads, int kvh, int hd, int vd, int page_size,
+                                      int max_blocks, int window, float scale, float softcap,
+                                      int keep_first, int sink, cudaStream_t stream) {
+  return generic_checked(q, k_cache, v_cache, block_table, seq_of_token, positions, out, act_dtype,
+                         T, heads, kvh, hd, vd, page_size, max_blocks, window, scale, softcap,
+                         keep_first, sink, IxRows{(long long)heads * hd, (long long)heads * vd, 1.f},
+                         ix_no_distance(), stream);
+}
+
+// With a temperature and a distance penalty per head (see attention_distance.cuh).
+IX_API int ix_distance_attention_generic(
+    const void* q, long long q_ld, const void* k_cache, const void* v_cache,
+    const int* block_table, const int* seq_of_token, const int* positions, void* out,
+    long long o_ld, float o_scale, int act_dtype, int T, int heads, int kvh, int hd, int vd,
+    int page_size, int max_blocks, float scale, const float* temp, const float* r1,
+    const float* r2, int chunk, cudaStream_t stream) {
+  if (!temp || !r1 || !r2 || chunk < 0) return IX_ERR_SIZE;
+  return generic_checked(q, k_cache, v_cache, block_table, seq_of_token, positions, out, act_dtype,
+                         T, heads, kvh, hd, vd, page_size, max_blocks, 0, scale, 0.f, 0, 0,
+                         IxRows{q_ld, o_ld, o_scale}, IxDistance{temp, r1, r2, chunk}, stream);
 }

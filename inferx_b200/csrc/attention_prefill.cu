@@ -18,7 +18,7 @@
 //
 // Sizes: bf16, head_dim 64 or 128; everything else is refused with
 // IX_ERR_UNSUPPORTED and the caller uses the general kernel.
-#include "common.cuh"
+#include "attention_distance.cuh"
 
 #define PF_BM 64
 #define PF_BN 64
@@ -281,15 +281,17 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc,
 // window and one added to the softmax's denominator (`sink`).  For decoders that want their
 // attention weights in 32-bit arithmetic: the scores are exact products of bfloat16 numbers
 // summed in fp32, maxima, exponentials and sums are fp32, and the weights lose nothing a
-// bfloat16 value would not lose many times over.
-template <int HD, int VD>
+// bfloat16 value would not lose many times over.  DIST: a score is multiplied by its head's
+// temperature and loses r1 ln(1 + r2 distance), and a query may be confined to its own run
+// of positions (attention_distance.cuh).
+template <int HD, int VD, bool DIST>
 __global__ void __launch_bounds__(PF_THREADS)
 attn_prefill_exact_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc,
                     const bf16* __restrict__ vc, const int* __restrict__ block_table,
                     const int* __restrict__ cu_q, const int* __restrict__ q_pos0,
                     bf16* __restrict__ out, int S, int heads, int kvh, int page_size,
                     int page_shift, int maxb, int window, float scale_log2e,
-                          int keep_first, int sink) {
+                          int keep_first, int sink, IxRows rows, IxDistance dist) {
   constexpr int CH = HD / 8;            // 16-byte chunks per row
   constexpr int KS = HD / 16;           // k-steps of Q K^T
   constexpr int CHV = VD / 8;           // 16-byte chunks per value row
@@ -322,7 +324,10 @@ attn_prefill_exact_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k
   const int rows_valid = min(PF_BM, nq - q0);
   const int pos0 = q_pos0[s] + q0;               // position of the tile's first query
   const int pmax = pos0 + rows_valid - 1;
-  const int kv_lo = window > 0 ? max(0, pos0 - window + 1) : 0;
+  const int kv_lo = ix_first_key(pos0, window, DIST ? dist.chunk : 0);
+  const int lo_last = ix_first_key(pmax, window, DIST ? dist.chunk : 0);
+  const float hs = DIST ? scale_log2e * dist.temp[h] : scale_log2e;
+  const float r1 = DIST ? dist.r1[h] : 0.f, r2 = DIST ? dist.r2[h] : 0.f;
   const int kv_hi = pmax + 1;
   const int kt0 = (kv_lo / PF_BN) * PF_BN;
   // keys below `kept` stay visible although the window has passed them: their tiles (those
@@ -339,7 +344,7 @@ attn_prefill_exact_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k
   for (int idx = tid; idx < PF_BM * CH; idx += PF_THREADS) {
     const int r = idx / CH, c = idx - r * CH;
     const bool ok = r < rows_valid;
-    const bf16* src = q + ((size_t)(tok0 + q0 + (ok ? r : 0)) * heads + h) * HD + c * 8;
+    const bf16* src = q + (size_t)(tok0 + q0 + (ok ? r : 0)) * rows.q_ld + (size_t)h * HD + c * 8;
     cp_async16(Qs + swz<CH>(r, c), src, ok);
   }
   auto load_kv = [&](int it, int stage) {
@@ -389,6 +394,8 @@ attn_prefill_exact_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k
   unsigned qf[KS][4];
   const int row_a = warp * 16 + g, row_b = row_a + 8;     // this thread's two query rows
   const int pos_a = pos0 + row_a, pos_b = pos0 + row_b;
+  const int lo_a = ix_first_key(pos_a, window, DIST ? dist.chunk : 0);
+  const int lo_b = ix_first_key(pos_b, window, DIST ? dist.chunk : 0);
 
   for (int it = 0; it < n_tiles; ++it) {
     const int stage = it & 1;
@@ -426,19 +433,19 @@ attn_prefill_exact_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k
       }
     }
     // scale, mask by position, row max
-    const bool need_mask = (kbase + PF_BN - 1 > pos0) || (window > 0 && kbase < pmax - window + 1)
-                           || kbase < kv_lo || it < n_kept;
+    const bool need_mask = (kbase + PF_BN - 1 > pos0) || kbase < lo_last || kbase < kv_lo ||
+                           it < n_kept;
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int j = 0; j < PF_BN / 8; ++j) {
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
-        float v = sc[j][c] * scale_log2e;
+        const int kp = kbase + j * 8 + 2 * t + (c & 1);
+        const int pos = (c & 2) ? pos_b : pos_a;
+        float v = sc[j][c] * hs;
+        if (DIST) v -= r1 * ix_log2(fmaf(r2, (float)max(0, pos - kp), 1.f));
         if (need_mask) {
-          const int kp = kbase + j * 8 + 2 * t + (c & 1);
-          const int pos = (c & 2) ? pos_b : pos_a;
-          const bool vis = kp <= pos && (window <= 0 || kp >= pos - window + 1 ||
-                                         kp < keep_first);
+          const bool vis = kp <= pos && (kp >= ((c & 2) ? lo_b : lo_a) || kp < keep_first);
           if (!vis) v = -INFINITY;
         }
         sc[j][c] = v;
@@ -504,15 +511,15 @@ attn_prefill_exact_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k
     l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 1);
     l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
   }
-  float inv_a = l_run[0] > 0.f ? 1.0f / l_run[0] : 0.f;
-  float inv_b = l_run[1] > 0.f ? 1.0f / l_run[1] : 0.f;
+  float inv_a = l_run[0] > 0.f ? rows.o_scale / l_run[0] : 0.f;
+  float inv_b = l_run[1] > 0.f ? rows.o_scale / l_run[1] : 0.f;
   if (sink) {      // one more term in the denominator: 2^(0 - max), maxima being in log2 units
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
       if (!(l_run[r] > 0.f)) continue;
       const float top = fmaxf(m_run[r], 0.f);
       const float c = fast_exp2(m_run[r] - top);
-      const float inv = c / (l_run[r] * c + fast_exp2(-top));
+      const float inv = rows.o_scale * c / (l_run[r] * c + fast_exp2(-top));
       if (r == 0) inv_a = inv; else inv_b = inv;
     }
   }
@@ -520,11 +527,11 @@ attn_prefill_exact_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k
   for (int j = 0; j < DT; ++j) {
     const int d = j * 8 + 2 * t;
     if (row_a < rows_valid) {
-      bf16* dst = out + ((size_t)(tok0 + q0 + row_a) * heads + h) * VD + d;
+      bf16* dst = out + (size_t)(tok0 + q0 + row_a) * rows.o_ld + (size_t)h * VD + d;
       *reinterpret_cast<unsigned*>(dst) = pack_bf16(o[j][0] * inv_a, o[j][1] * inv_a);
     }
     if (row_b < rows_valid) {
-      bf16* dst = out + ((size_t)(tok0 + q0 + row_b) * heads + h) * VD + d;
+      bf16* dst = out + (size_t)(tok0 + q0 + row_b) * rows.o_ld + (size_t)h * VD + d;
       *reinterpret_cast<unsigned*>(dst) = pack_bf16(o[j][2] * inv_b, o[j][3] * inv_b);
     }
   }
@@ -576,13 +583,14 @@ IX_API int ix_paged_attention_prefill(const void* q, const void* k_cache, const 
   return IX_ERR_UNSUPPORTED;
 }
 
-template <int HD, int VD>
+template <int HD, int VD, bool DIST>
 static int launch_prefill_exact(const void* q, const void* kc, const void* vc, const int* bt,
                                 const int* cu_q, const int* q_pos0, void* out, int T, int S,
                                 int heads, int kvh, int page_size, int maxb, int window,
-                                float scale, int keep_first, int sink, cudaStream_t stream) {
+                                float scale, int keep_first, int sink, IxRows rows,
+                                IxDistance dist, cudaStream_t stream) {
   const size_t smem = (size_t)(PF_BM + 2 * PF_BN) * HD * 2 + (size_t)2 * PF_BN * VD * 2;
-  auto kern = attn_prefill_exact_kernel<HD, VD>;
+  auto kern = attn_prefill_exact_kernel<HD, VD, DIST>;
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          (int)smem);
@@ -597,7 +605,8 @@ static int launch_prefill_exact(const void* q, const void* kc, const void* vc, c
   kern<<<grid, PF_THREADS, smem, stream>>>((const bf16*)q, (const bf16*)kc, (const bf16*)vc, bt,
                                            cu_q, q_pos0, (bf16*)out, S, heads, kvh, page_size,
                                            page_shift, maxb, window,
-                                           scale * 1.4426950408889634f, keep_first, sink);
+                                           scale * 1.4426950408889634f, keep_first, sink, rows,
+                                           dist);
   return ix_launch_status();
 }
 
@@ -606,27 +615,60 @@ IX_API int ix_paged_attention_prefill_exact_applies(int hd, int vd) {
 }
 
 // q [T, heads, hd], out [T, heads, vd], caches [pages, kvh, page_size, hd or vd], bfloat16.
-IX_API int ix_paged_attention_prefill_exact(const void* q, const void* k_cache,
-                                            const void* v_cache, const int* block_table,
-                                            const int* cu_q, const int* q_pos0, void* out, int T,
-                                            int S, int heads, int kvh, int hd, int vd,
-                                            int page_size, int max_blocks, int window, float scale,
-                                            int keep_first, int sink, cudaStream_t stream) {
+static int prefill_exact_checked(const void* q, const void* k_cache, const void* v_cache,
+                                 const int* block_table, const int* cu_q, const int* q_pos0,
+                                 void* out, int T, int S, int heads, int kvh, int hd, int vd,
+                                 int page_size, int max_blocks, int window, float scale,
+                                 int keep_first, int sink, IxRows rows, IxDistance dist,
+                                 cudaStream_t stream) {
   if (T <= 0 || S <= 0) return IX_OK;
   if (heads <= 0 || kvh <= 0 || heads % kvh != 0 || page_size <= 0 || max_blocks <= 0 ||
-      window < 0 || keep_first < 0 || !(scale > 0.f))
+      window < 0 || keep_first < 0 || (!dist.temp && !(scale > 0.f)))
     return IX_ERR_SIZE;
   if (((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)out) & 15)
     return IX_ERR_ALIGN;
+  if (rows.q_ld % 8 || rows.o_ld % 2) return IX_ERR_ALIGN;
 #define PF_EXACT(H_, V_)                                                                       \
   if (hd == H_ && vd == V_)                                                                    \
-    return launch_prefill_exact<H_, V_>(q, k_cache, v_cache, block_table, cu_q, q_pos0, out, T, \
-                                        S, heads, kvh, page_size, max_blocks, window, scale,   \
-                                        keep_first, sink, stream);
+    return dist.temp                                                                           \
+               ? launch_prefill_exact<H_, V_, true>(q, k_cache, v_cache, block_table, cu_q,    \
+                                                    q_pos0, out, T, S, heads, kvh, page_size,  \
+                                                    max_blocks, window, scale, keep_first,     \
+                                                    sink, rows, dist, stream)                  \
+               : launch_prefill_exact<H_, V_, false>(q, k_cache, v_cache, block_table, cu_q,   \
+                                                     q_pos0, out, T, S, heads, kvh, page_size, \
+                                                     max_blocks, window, scale, keep_first,    \
+                                                     sink, rows, dist, stream);
   PF_EXACT(64, 64)
   PF_EXACT(64, 128)
   PF_EXACT(128, 64)
   PF_EXACT(128, 128)
 #undef PF_EXACT
   return IX_ERR_UNSUPPORTED;
+}
+
+IX_API int ix_paged_attention_prefill_exact(const void* q, const void* k_cache,
+                                            const void* v_cache, const int* block_table,
+                                            const int* cu_q, const int* q_pos0, void* out, int T,
+                                            int S, int heads, int kvh, int hd, int vd,
+                                            int page_size, int max_blocks, int window, float scale,
+                                            int keep_first, int sink, cudaStream_t stream) {
+  return prefill_exact_checked(q, k_cache, v_cache, block_table, cu_q, q_pos0, out, T, S, heads,
+                               kvh, hd, vd, page_size, max_blocks, window, scale, keep_first, sink,
+                               IxRows{(long long)heads * hd, (long long)heads * vd, 1.f},
+                               ix_no_distance(), stream);
+}
+
+// With a temperature and a distance penalty per head (see attention_distance.cuh).
+IX_API int ix_distance_attention_prefill_exact(
+    const void* q, long long q_ld, const void* k_cache, const void* v_cache,
+    const int* block_table, const int* cu_q, const int* q_pos0, void* out, long long o_ld,
+    float o_scale, int T, int S, int heads, int kvh, int hd, int vd, int page_size,
+    int max_blocks, float scale, const float* temp, const float* r1, const float* r2, int chunk,
+    cudaStream_t stream) {
+  if (!temp || !r1 || !r2 || chunk < 0) return IX_ERR_SIZE;
+  return prefill_exact_checked(q, k_cache, v_cache, block_table, cu_q, q_pos0, out, T, S, heads,
+                               kvh, hd, vd, page_size, max_blocks, 0, scale, 0, 0,
+                               IxRows{q_ld, o_ld, o_scale}, IxDistance{temp, r1, r2, chunk},
+                               stream);
 }

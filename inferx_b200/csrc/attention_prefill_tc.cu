@@ -34,7 +34,7 @@
 // meaningful).
 //
 // Requires bf16, head_dim 64 or 128, page_size a power of two from 8 to 64.
-#include "common.cuh"
+#include "attention_distance.cuh"
 #include "tma_common.cuh"
 #include "tcgen05_common.cuh"
 
@@ -51,6 +51,9 @@ struct FaBars {
   unsigned tmem_holder;
   int abort_flag;
 };
+
+// DIST: penalties of a softmax warp's 32 rows against a tile of 64 keys, by distance
+#define FA_BAND 96
 
 __device__ __forceinline__ float fa_exp2(float x) {
   float y;
@@ -94,7 +97,12 @@ __device__ __forceinline__ float fa_max3(float a, float b, float c) {
 // weight).  The sequence's first `keep_first` keys stay visible beside the window (their
 // tiles are walked first) and `sink` adds one to the softmax's denominator.  One run of
 // keys per query tile (nsplit 1).
-template <int HD, bool EXACT>
+// DIST (with EXACT): a score is multiplied by its head's temperature and loses r1 ln(1 + r2
+// distance), and a query may be confined to its own run of positions (attention_distance.cuh).
+// A softmax warp's rows and a tile's keys span 95 distances; the warp forms their penalties
+// once per tile, in shared memory, and a thread reads 64 of them (neighbouring rows read
+// neighbouring entries).
+template <int HD, bool EXACT, bool DIST>
 __global__ void __launch_bounds__(FA_THREADS, 2)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                        const __grid_constant__ CUtensorMap map_k,
@@ -104,7 +112,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                        int kvh, int page_size, int page_shift, int maxb, int window,
                        float scale_log2e, int* __restrict__ status, int nsplit,
                        float* __restrict__ part_o, float* __restrict__ part_ml, float cap_c1,
-                       float cap_over_scale, int keep_first, int sink) {
+                       float cap_over_scale, int keep_first, int sink, IxRows rows,
+                       IxDistance dist) {
   constexpr int HALVES = HD / 64;
   constexpr int Q_BYTES = FA_BM * HD * 2;
   constexpr int Q_HALF = FA_BM * 128;
@@ -125,6 +134,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
   unsigned char* Ks = Qs + Q_BYTES;             // [2][halves][64 keys][128 B]
   unsigned char* Vs = Ks + 2 * KV_TILE;
   FaBars* bars = reinterpret_cast<FaBars*>(Vs + 2 * KV_TILE);
+  float* bands = reinterpret_cast<float*>(bars + 1);     // [4][FA_BAND] with DIST
 
   // which sequence and which 128-query tile of it; heavy tiles first (see the
   // mma.sync kernel)
@@ -147,7 +157,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
   const int rows_valid = min(FA_BM, nq - q0);
   const int pos0 = q_pos0[s] + q0;               // position of the tile's first query
   const int pmax = pos0 + rows_valid - 1;
-  const int kv_lo = window > 0 ? max(0, pos0 - window + 1) : 0;
+  const int kv_lo = ix_first_key(pos0, window, DIST ? dist.chunk : 0);
+  const int lo_last = ix_first_key(pmax, window, DIST ? dist.chunk : 0);
   const int kv_hi = pmax + 1;
   // the tile's keys, cut into nsplit runs of whole 64-key tiles (blockIdx.z takes one)
   const int kt_first = kv_lo & ~(FA_BN - 1);
@@ -312,12 +323,26 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
     const int quarter = warp & 3;                  // TMEM lanes this warp may touch
     const int row = quarter * 32 + lane;
     const int pos = pos0 + row;
-    const int lo_r = window > 0 ? pos - window + 1 : 0;
+    const int lo_r = ix_first_key(pos, window, DIST ? dist.chunk : 0);
+    float* band = bands + quarter * FA_BAND;
+    const float head_scale = DIST ? scale_log2e * dist.temp[h] : 0.f;
+    const float r1 = DIST ? dist.r1[h] : 0.f, r2 = DIST ? dist.r2[h] : 0.f;
+    // what a score is still multiplied with when its exponent is taken
+    const float s_mul = DIST ? 1.f : scale_log2e;
     const unsigned lane_addr = tmem_base + ((unsigned)(quarter * 32) << 16);
     float m_ref = -INFINITY, l_run = 0.f;
     bool ok = true;
     for (int j = 0; j < n_tiles; ++j) {
       const int st = j & 1;
+      if (DIST) {
+        // entry x: the distance of row r and key k with x = r - k + 63
+        __syncwarp();
+        const int d0 = pos0 + quarter * 32 - tile_key0(j) - (FA_BN - 1);
+#pragma unroll
+        for (int x = 0; x < FA_BAND; x += 32)
+          band[x + lane] = r1 * log2f(fmaf(r2, (float)max(0, d0 + x + lane), 1.f));
+        __syncwarp();
+      }
       ok = __all_sync(0xffffffffu, mbar_wait(&bars->s_full[st], (j >> 1) & 1, abortp));
       if (!ok) break;
       tc_fence_after();
@@ -328,9 +353,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
 #pragma unroll
         for (int i = 0; i < FA_BN; ++i) sc[i] = ix_cap_raw_score(sc[i], cap_c1, cap_over_scale);
       }
+      if (DIST) {
+#pragma unroll
+        for (int i = 0; i < FA_BN; ++i)
+          sc[i] = fmaf(sc[i], head_scale, -band[lane - i + FA_BN - 1]);
+      }
       const int kbase = tile_key0(j);
-      const bool need_mask = (kbase + FA_BN - 1 > pos0) || kbase < kv_lo ||
-                             (window > 0 && kbase < pmax - window + 1) || j < n_kept;
+      const bool need_mask = (kbase + FA_BN - 1 > pos0) || kbase < kv_lo || kbase < lo_last ||
+                             j < n_kept;
       if (need_mask) {
 #pragma unroll
         for (int i = 0; i < FA_BN; ++i) {
@@ -347,7 +377,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
         mxb = fa_max3(mxb, sc[i + 2], sc[i + 3]);
       }
       const float mx = fmaxf(mxa, mxb);
-      const float m_new = fmaxf(m_ref, mx * scale_log2e);
+      const float m_new = fmaxf(m_ref, mx * s_mul);
       // rescale when this row's max has outgrown the reference by more than the step
       // (or when the row sees its first key); the decision is the warp's
       const bool grow = m_new > m_ref + FA_RESCALE_STEP || (m_ref == -INFINITY && m_new > m_ref);
@@ -365,8 +395,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
 #pragma unroll
       for (int i = 0; i < FA_BN; i += 4) {
         float a0, a1, a2, a3;
-        fa_fma2(a0, a1, sc[i], sc[i + 1], scale_log2e, nbase);   // -inf stays -inf
-        fa_fma2(a2, a3, sc[i + 2], sc[i + 3], scale_log2e, nbase);
+        fa_fma2(a0, a1, sc[i], sc[i + 1], s_mul, nbase);   // -inf stays -inf
+        fa_fma2(a2, a3, sc[i + 2], sc[i + 3], s_mul, nbase);
         const float p0 = fa_exp2(a0), p1 = fa_exp2(a1), p2 = fa_exp2(a2), p3 = fa_exp2(a3);
         fa_add2(sum0, sum1, p0, p1);
         fa_add2(sum2, sum3, p2, p3);
@@ -437,13 +467,13 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
       }
     } else if (n_tiles > 0) {
       tc_fence_after();
-      float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
+      float inv = l_run > 0.f ? rows.o_scale / l_run : 0.f;
       if (EXACT && sink && l_run > 0.f) {   // one more term, 2^(0 - reference), in the denominator
         const float top = fmaxf(m_ref, 0.f);
         const float c = fa_exp2(m_ref - top);
-        inv = c / (l_run * c + fa_exp2(-top));
+        inv = rows.o_scale * c / (l_run * c + fa_exp2(-top));
       }
-      bf16* dst = out + ((size_t)(tok0 + q0 + row) * heads + h) * HD;
+      bf16* dst = out + (size_t)(tok0 + q0 + row) * rows.o_ld + (size_t)h * HD;
 #pragma unroll
       for (int c0 = 0; c0 < HD; c0 += 32) {
         float o[32];
@@ -504,22 +534,25 @@ __global__ void attn_prefill_tc_merge_kernel(const float* __restrict__ part_o,
   }
 }
 
-template <int HD, bool EXACT = false>
+template <int HD, bool EXACT = false, bool DIST = false>
 static int launch_prefill_tc(const void* q, const void* kc, const void* vc, long long cache_rows,
                              const int* bt, const int* cu_q, const int* q_pos0, void* out, int T,
                              int S, int heads, int kvh, int page_size, int page_shift, int maxb,
                              int window, float scale, float softcap, int* status, int nsplit,
                              float* part_o, float* part_ml, cudaStream_t stream,
-                             int keep_first = 0, int sink = 0) {
+                             int keep_first = 0, int sink = 0, IxRows rows = {0, 0, 1.f},
+                             IxDistance dist = ix_no_distance()) {
   CUtensorMap map_q, map_k, map_v;
-  int rc = ix_tensor_map_bf16_2d(&map_q, q, T, (long long)heads * HD, 64, FA_BM);
+  if (rows.q_ld == 0) rows.q_ld = rows.o_ld = (long long)heads * HD;
+  int rc = ix_tensor_map_bf16_2d(&map_q, q, T, (long long)heads * HD, 64, FA_BM, rows.q_ld);
   if (rc != IX_OK) return rc;
   rc = ix_tensor_map_bf16_2d(&map_k, kc, cache_rows, HD, 64, page_size);
   if (rc != IX_OK) return rc;
   rc = ix_tensor_map_bf16_2d(&map_v, vc, cache_rows, HD, 64, page_size);
   if (rc != IX_OK) return rc;
-  const int smem = FA_BM * HD * 2 + 4 * FA_BN * HD * 2 + (int)sizeof(FaBars);
-  auto kern = attn_prefill_tc_kernel<HD, EXACT>;
+  const int smem = FA_BM * HD * 2 + 4 * FA_BN * HD * 2 + (int)sizeof(FaBars) +
+                   (DIST ? 4 * FA_BAND * (int)sizeof(float) : 0);
+  auto kern = attn_prefill_tc_kernel<HD, EXACT, DIST>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e != cudaSuccess) return (int)e;
   const int tiles = (T + FA_BM - 1) / FA_BM + S;   // every sequence can add one partial tile
@@ -531,7 +564,8 @@ static int launch_prefill_tc(const void* q, const void* kc, const void* vc, long
                                            part_ml,
                                            softcap > 0.f ? 2.f * scale * 1.4426950408889634f / softcap
                                                          : 0.f,
-                                           softcap > 0.f ? softcap / scale : 0.f, keep_first, sink);
+                                           softcap > 0.f ? softcap / scale : 0.f, keep_first, sink,
+                                           rows, dist);
   rc = ix_launch_status();
   if (rc != IX_OK || nsplit == 1) return rc;
   attn_prefill_tc_merge_kernel<<<T * heads, HD >= 128 ? 128 : 64, 0, stream>>>(
@@ -654,4 +688,38 @@ IX_API int ix_paged_attention_prefill_tc_exact(
                                      out, T, S, heads, kvh, page_size, page_shift, max_blocks,
                                      window, scale, 0.f, status, 1, nullptr, nullptr, stream,
                                      keep_first, sink);
+}
+
+// The EXACT form with a temperature and a distance penalty per head (attention_distance.cuh).
+// q: rows of pitch q_ld starting on 16-byte boundaries, heads beside each other; out likewise.
+IX_API int ix_distance_attention_prefill_tc(
+    const void* q, long long q_ld, const void* k_cache, const void* v_cache, int num_pages,
+    const int* block_table, const int* cu_q, const int* q_pos0, void* out, long long o_ld,
+    float o_scale, int T, int S, int heads, int kvh, int hd, int page_size, int max_blocks,
+    float scale, const float* temp, const float* r1, const float* r2, int chunk, int* status,
+    cudaStream_t stream) {
+  if (T <= 0 || S <= 0) return IX_OK;
+  if (heads <= 0 || kvh <= 0 || heads % kvh != 0 || max_blocks <= 0 || num_pages <= 0 ||
+      status == nullptr || heads > 65535 || !temp || !r1 || !r2 || chunk < 0 ||
+      q_ld < (long long)heads * hd || o_ld < (long long)heads * hd)
+    return IX_ERR_SIZE;
+  if (!ix_paged_attention_prefill_tc_exact_applies(hd, hd, page_size)) return IX_ERR_UNSUPPORTED;
+  if (((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)out) & 15)
+    return IX_ERR_ALIGN;
+  if (q_ld % 8 || o_ld % 8) return IX_ERR_ALIGN;
+  int page_shift = 0;
+  while ((1 << page_shift) < page_size) ++page_shift;
+  const long long cache_rows = (long long)num_pages * kvh * page_size;
+  if (cache_rows > 0x7fffffffLL) return IX_ERR_SIZE;
+  const IxRows rows = {q_ld, o_ld, o_scale};
+  const IxDistance dist = {temp, r1, r2, chunk};
+  if (hd == 128)
+    return launch_prefill_tc<128, true, true>(q, k_cache, v_cache, cache_rows, block_table, cu_q,
+                                              q_pos0, out, T, S, heads, kvh, page_size, page_shift,
+                                              max_blocks, 0, scale, 0.f, status, 1, nullptr,
+                                              nullptr, stream, 0, 0, rows, dist);
+  return launch_prefill_tc<64, true, true>(q, k_cache, v_cache, cache_rows, block_table, cu_q,
+                                           q_pos0, out, T, S, heads, kvh, page_size, page_shift,
+                                           max_blocks, 0, scale, 0.f, status, 1, nullptr, nullptr,
+                                           stream, 0, 0, rows, dist);
 }

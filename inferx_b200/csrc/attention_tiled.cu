@@ -16,8 +16,12 @@
 // window: their tiles (also at multiples of 64) are walked before the window's.  With
 // `sink` one is added to the softmax's denominator.
 //
+// A third form (attention_distance.cuh) multiplies a score by its head's temperature, takes
+// r1 ln(1 + r2 distance) off and may confine a query to its own run of positions; the
+// penalties of a tile, one per distance, are formed once in shared memory.
+//
 // Takes any element type, head sizes that are a multiple of 4 up to 256, any page size.
-#include "common.cuh"
+#include "attention_distance.cuh"
 
 #define TA_BQ 32
 #define TA_BK 64
@@ -55,8 +59,10 @@ paged_attention_tiled_kernel(const TA* __restrict__ q, const TA* __restrict__ kc
                              const int* __restrict__ cu_q, const int* __restrict__ q_pos0,
                              TA* __restrict__ out, int S, int heads, int kvh, int hd, int vd,
                              int page_size, int max_blocks, int window, float scale,
-                             float softcap, int keep_first, int sink) {
+                             float softcap, int keep_first, int sink, IxRows rows,
+                             IxDistance dist) {
   extern __shared__ __align__(16) float tsm[];
+  __shared__ float band[TA_BQ + TA_BK];          // penalty per distance, see below
   const int ld = hd + 4;                         // row pitch: 16-byte rows, no bank conflicts
   const int ldv = vd + 4;                        // the values' size may differ from the keys'
   float* Qs = tsm;                               // [TA_BQ][ld]
@@ -81,7 +87,10 @@ paged_attention_tiled_kernel(const TA* __restrict__ q, const TA* __restrict__ kc
   const int rows_valid = min(TA_BQ, cu_q[s + 1] - tok0);
   const int pos0 = q_pos0[s] + tile * TA_BQ;     // position of the tile's first query
   const int kv_hi = pos0 + rows_valid;           // one past the last visible key
-  const int kv_lo = window > 0 ? max(0, pos0 - window + 1) : 0;
+  const int kv_lo = ix_first_key(pos0, window, dist.chunk);
+  const bool far = dist.temp != nullptr;
+  const float temp = far ? dist.temp[h] : 1.f;
+  const float r1 = far ? dist.r1[h] : 0.f, r2 = far ? dist.r2[h] : 0.f;
   const int* bt = block_table + (size_t)s * max_blocks;
   const int tid = threadIdx.x;
   const int chunks = hd >> 2;
@@ -90,7 +99,7 @@ paged_attention_tiled_kernel(const TA* __restrict__ q, const TA* __restrict__ kc
   for (int idx = tid; idx < TA_BQ * chunks; idx += TA_THREADS) {
     const int r = idx / chunks, c = idx - r * chunks;
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (r < rows_valid) v = TaLoad4<TA>::load(q + ((size_t)(tok0 + r) * heads + h) * hd + 4 * c);
+    if (r < rows_valid) v = TaLoad4<TA>::load(q + (size_t)(tok0 + r) * rows.q_ld + (size_t)h * hd + 4 * c);
     *reinterpret_cast<float4*>(Qs + r * ld + 4 * c) = v;
   }
   if (tid < TA_BQ) {
@@ -143,6 +152,10 @@ paged_attention_tiled_kernel(const TA* __restrict__ q, const TA* __restrict__ kc
       }
       *reinterpret_cast<float4*>(Vs + r * ldv + 4 * c) = vv4;
     }
+    // entry x stands for the distance pos0 - kv0 - (TA_BK - 1) + x of query r and key k with
+    // x = r - k + TA_BK - 1
+    if (far && tid < TA_BQ + TA_BK - 1)
+      band[tid] = r1 * log1pf(r2 * (float)max(0, pos0 - kv0 - (TA_BK - 1) + tid));
     __syncthreads();
 
     float sc[2][4];
@@ -173,13 +186,14 @@ paged_attention_tiled_kernel(const TA* __restrict__ q, const TA* __restrict__ kc
     for (int i = 0; i < 2; ++i) {
       const int r = sq + 16 * i;
       const int qp = pos0 + r;
-      const int first = window > 0 ? max(0, qp - window + 1) : 0;
+      const int first = ix_first_key(qp, window, dist.chunk);
       float tm = -INFINITY;
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int kp = kv0 + sk + 16 * j;
         const bool seen = r < rows_valid && kp <= qp && (kp >= first || kp < keep_first);
         float sv = sc[i][j] * scale;
+        if (far) sv = sv * temp - band[r - (sk + 16 * j) + TA_BK - 1];
         if (softcap > 0.f) sv = softcap * tanhf(sv / softcap);   // squashed scores
         sc[i][j] = seen ? sv : -INFINITY;
         tm = fmaxf(tm, sc[i][j]);
@@ -241,17 +255,17 @@ paged_attention_tiled_kernel(const TA* __restrict__ q, const TA* __restrict__ kc
   for (int i = 0; i < 4; ++i) {
     const int r = 4 * ow + i;
     if (r >= rows_valid) continue;
-    float inv_l = 1.0f / l_run[r];
+    float inv_l = rows.o_scale / l_run[r];
     if (sink) {        // one more term, exp(0 - max), in the denominator
       const float top = fmaxf(m_run[r], 0.f);
       const float c = expf(m_run[r] - top);
-      inv_l = c / (l_run[r] * c + expf(-top));
+      inv_l = rows.o_scale * c / (l_run[r] * c + expf(-top));
     }
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
       const int d = 4 * ol + 128 * j;
       if (d < vd)
-        TaLoad4<TA>::store(out + ((size_t)(tok0 + r) * heads + h) * vd + d,
+        TaLoad4<TA>::store(out + (size_t)(tok0 + r) * rows.o_ld + (size_t)h * vd + d,
                            make_float4(acc[i][j][0] * inv_l, acc[i][j][1] * inv_l,
                                        acc[i][j][2] * inv_l, acc[i][j][3] * inv_l));
     }
@@ -263,12 +277,12 @@ IX_API int ix_paged_attention_tiled_applies(int hd) { return hd > 0 && hd % 4 ==
 // q: [T, heads, hd]; out: [T, heads, vd]; caches [pages, kvh, page_size, hd or vd];
 // block_table [S, max_blocks];
 // cu_q [S + 1]: token range of each sequence; q_pos0 [S]: position of its first token here.
-IX_API int ix_paged_attention_tiled(const void* q, const void* k_cache, const void* v_cache,
-                                    const int* block_table, const int* cu_q, const int* q_pos0,
-                                    void* out, int act_dtype, int T, int S, int heads, int kvh,
-                                    int hd, int vd, int page_size, int max_blocks, int window,
-                                    float scale, float softcap, int keep_first, int sink,
-                                    cudaStream_t stream) {
+static int tiled_checked(const void* q, const void* k_cache, const void* v_cache,
+                         const int* block_table, const int* cu_q, const int* q_pos0, void* out,
+                         int act_dtype, int T, int S, int heads, int kvh, int hd, int vd,
+                         int page_size, int max_blocks, int window, float scale, float softcap,
+                         int keep_first, int sink, IxRows rows, IxDistance dist,
+                         cudaStream_t stream) {
   if (T <= 0) return IX_OK;
   if (S <= 0 || heads <= 0 || kvh <= 0 || heads % kvh != 0 || page_size <= 0 || max_blocks <= 0 ||
       window < 0 || keep_first < 0)
@@ -279,6 +293,7 @@ IX_API int ix_paged_attention_tiled(const void* q, const void* k_cache, const vo
   const int esize = act_dtype == IX_F32 ? 4 : 2;
   if (((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)out) % (4 * esize))
     return IX_ERR_ALIGN;
+  if (rows.q_ld % 4 || rows.o_ld % 4) return IX_ERR_ALIGN;
   const int ld = hd + 4, ldv = vd + 4;
   const size_t smem = ((size_t)(TA_BQ + TA_BK) * ld + (size_t)TA_BK * ldv + TA_BQ * (TA_BK + 4) +
                        3 * TA_BQ) * 4;
@@ -293,7 +308,32 @@ IX_API int ix_paged_attention_tiled(const void* q, const void* k_cache, const vo
     kern<<<grid, TA_THREADS, smem, stream>>>((const TA*)q, (const TA*)k_cache, (const TA*)v_cache,
                                              block_table, cu_q, q_pos0, (TA*)out, S, heads, kvh,
                                              hd, vd, page_size, max_blocks, window, scale,
-                                             softcap, keep_first, sink);
+                                             softcap, keep_first, sink, rows, dist);
   });
   return ix_launch_status();
+}
+
+IX_API int ix_paged_attention_tiled(const void* q, const void* k_cache, const void* v_cache,
+                                    const int* block_table, const int* cu_q, const int* q_pos0,
+                                    void* out, int act_dtype, int T, int S, int heads, int kvh,
+                                    int hd, int vd, int page_size, int max_blocks, int window,
+                                    float scale, float softcap, int keep_first, int sink,
+                                    cudaStream_t stream) {
+  return tiled_checked(q, k_cache, v_cache, block_table, cu_q, q_pos0, out, act_dtype, T, S, heads,
+                       kvh, hd, vd, page_size, max_blocks, window, scale, softcap, keep_first, sink,
+                       IxRows{(long long)heads * hd, (long long)heads * vd, 1.f}, ix_no_distance(),
+                       stream);
+}
+
+// With a temperature and a distance penalty per head (see attention_distance.cuh).
+IX_API int ix_distance_attention_tiled(
+    const void* q, long long q_ld, const void* k_cache, const void* v_cache,
+    const int* block_table, const int* cu_q, const int* q_pos0, void* out, long long o_ld,
+    float o_scale, int act_dtype, int T, int S, int heads, int kvh, int hd, int vd, int page_size,
+    int max_blocks, float scale, const float* temp, const float* r1, const float* r2, int chunk,
+    cudaStream_t stream) {
+  if (!temp || !r1 || !r2 || chunk < 0) return IX_ERR_SIZE;
+  return tiled_checked(q, k_cache, v_cache, block_table, cu_q, q_pos0, out, act_dtype, T, S, heads,
+                       kvh, hd, vd, page_size, max_blocks, 0, scale, 0.f, 0, 0,
+                       IxRows{q_ld, o_ld, o_scale}, IxDistance{temp, r1, r2, chunk}, stream);
 }

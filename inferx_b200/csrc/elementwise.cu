@@ -269,7 +269,7 @@ __global__ void moe_combine_kernel(const TA* __restrict__ y, const int* __restri
     float acc = 0.f;
     for (int s = 0; s < k; ++s) {
       const int row = dest[t * k + s];
-      acc += w[t * k + s] * to_f32(y[(size_t)row * H + i]);
+      acc += (w ? w[t * k + s] : 1.0f) * to_f32(y[(size_t)row * H + i]);
     }
     if (shared) acc += sg * to_f32(shared[(size_t)t * H + i]);
     out[(size_t)t * H + i] = from_f32<TA>(acc);
@@ -291,7 +291,7 @@ __global__ void moe_combine_bf16_vec_kernel(const uint4* __restrict__ y, const i
     for (int j = 0; j < 8; ++j) acc[j] = 0.f;
     for (int s = 0; s < k; ++s) {
       const int row = dest[t * k + s];
-      const float ws = w[t * k + s];
+      const float ws = w ? w[t * k + s] : 1.0f;   // null: the plain sum
       float f[8];
       bf8_to_f32(y[(size_t)row * chunks + c], f);
 #pragma unroll
@@ -335,7 +335,7 @@ __global__ void combine_add_rmsnorm_bf16_vec_kernel(
       for (int j = 0; j < 8; ++j) acc[j] = 0.f;
       for (int s = 0; s < k; ++s) {
         const int row = dest[t * k + s];
-        const float ws = w[t * k + s];
+        const float ws = w ? w[t * k + s] : 1.0f;   // null: the plain sum
         float f[8];
         bf8_to_f32(y[(size_t)row * chunks + c], f);
 #pragma unroll

@@ -109,7 +109,8 @@ __global__ void __launch_bounds__(TC_THREADS, 1)
 grouped_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a,
                        const __grid_constant__ CUtensorMap map_w,
                        const int* __restrict__ offsets, bf16* __restrict__ out, int N, int K,
-                       int E, int w_rows_per_expert, int* __restrict__ status) {
+                       int E, int w_rows_per_expert, int* __restrict__ status,
+                       const float* __restrict__ row_scale) {
   constexpr bool DUAL = MODE != 0;      // two weight tiles and two accumulators an item
   constexpr bool SWIGLU = MODE == 1;
   constexpr int F_ITEM = MODE == 2 ? 2 * TC_BF : TC_BF;   // output features of an item
@@ -285,6 +286,16 @@ grouped_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a,
         // would serialise their latencies.  The fast reciprocal's error is far below a
         // bf16 ulp.
         bf16 r[32];
+        if (SWIGLU && row_scale) {
+          // the rows' inputs count times w: both products do, a lane fetching one row's w
+          const float w_lane = c0 + lane < it.n_valid ? row_scale[it.m0 + c0 + lane] : 0.f;
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            const float w_row = __shfl_sync(0xffffffffu, w_lane, i);
+            g[i] *= w_row;
+            u[DUAL ? i : 0] *= w_row;
+          }
+        }
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
           float a = g[i];
@@ -343,7 +354,8 @@ IX_API int ix_gather_rows(const void* src, const int* rows, void* dst, int n_row
 // ran out leaves a nonzero code there.
 template <int MODE, int BT>
 static int launch_tc(const void* a, const int* offsets, const void* w, void* out, int A_rows,
-                     int N, int K, int E, long long w_rows, int* status, cudaStream_t stream) {
+                     int N, int K, int E, long long w_rows, int* status,
+                     const float* row_scale, cudaStream_t stream) {
   CUtensorMap map_a, map_w;
   int rc = ix_tensor_map_bf16_2d(&map_a, a, A_rows, K, TC_BK, TC_BOX_T);
   if (rc != IX_OK) return rc;
@@ -367,13 +379,14 @@ static int launch_tc(const void* a, const int* offsets, const void* w, void* out
   cudaError_t e2 = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e2 != cudaSuccess) return (int)e2;
   kern<<<grid, TC_THREADS, smem, stream>>>(map_a, map_w, offsets, (bf16*)out, N, K, E,
-                                           (int)w_rows, status);
+                                           (int)w_rows, status, row_scale);
   return ix_launch_status();
 }
 
 IX_API int ix_grouped_gemm_tc(const void* a, const int* offsets, const void* w, void* out,
                               int dual, int A_rows, int N, int K, int E, int* status,
-                              cudaStream_t stream) {
+                              const float* row_scale, cudaStream_t stream) {
+  if (row_scale && !dual) return IX_ERR_UNSUPPORTED;
   if (A_rows <= 0) return IX_OK;
   if (N <= 0 || K <= 0 || E <= 0 || status == nullptr) return IX_ERR_SIZE;
   if (K % 8 != 0 || E > TC_MAX_EXPERTS) return IX_ERR_UNSUPPORTED;
@@ -393,10 +406,10 @@ IX_API int ix_grouped_gemm_tc(const void* a, const int* offsets, const void* w, 
   const int bt = per <= 128.0 ? 128 : per <= 160.0 ? 160 : per <= 192.0 ? 192 : 256;
 #define IX_TC(D)                                                                              \
   do {                                                                                        \
-    if (bt == 128) return launch_tc<D, 128>(a, offsets, w, out, A_rows, N, K, E, w_rows, status, stream); \
-    if (bt == 160) return launch_tc<D, 160>(a, offsets, w, out, A_rows, N, K, E, w_rows, status, stream); \
-    if (bt == 192) return launch_tc<D, 192>(a, offsets, w, out, A_rows, N, K, E, w_rows, status, stream); \
-    return launch_tc<D, 256>(a, offsets, w, out, A_rows, N, K, E, w_rows, status, stream);   \
+    if (bt == 128) return launch_tc<D, 128>(a, offsets, w, out, A_rows, N, K, E, w_rows, status, row_scale, stream); \
+    if (bt == 160) return launch_tc<D, 160>(a, offsets, w, out, A_rows, N, K, E, w_rows, status, row_scale, stream); \
+    if (bt == 192) return launch_tc<D, 192>(a, offsets, w, out, A_rows, N, K, E, w_rows, status, row_scale, stream); \
+    return launch_tc<D, 256>(a, offsets, w, out, A_rows, N, K, E, w_rows, status, row_scale, stream);   \
   } while (0)
   if (dual) IX_TC(1);
   // plain: two feature tiles an item when the features fill them (measured at 60 experts

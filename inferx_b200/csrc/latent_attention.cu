@@ -13,6 +13,9 @@
 //                        part (angles, cos and sin in fp32), record written into its
 //                        cache slot; the plain query parts laid out heads outermost
 //                        for the product with the folded key matrix
+//   ix_latent_front      the record likewise, from a product that makes the queries' latent
+//                        beside the down-projection: one pass also RMS-norms that latent
+//                        (ix_latent_prepare then splits and rotates what it is widened to)
 //   ix_latent_attention  general kernel: any sizes, fp32 arithmetic, either element
 //                        type; one warp per (token, head), keys in tiles of 32 that
 //                        start on multiples of 32 of the absolute position, so that a
@@ -107,6 +110,93 @@ IX_API int ix_latent_prepare(const void* proj, long long ld, int q_off, int kv_o
                               (const TA*)proj, ld, q_off, kv_off, positions, freq, mag, gain, eps,
                               slots, (TA*)cache, (TA*)q_rot, (TA*)q_plain, T, H, dn, dr, rot_dims,
                               rank));
+  return ix_launch_status();
+}
+
+// ---------------------------------------------------------------------------
+// front.  proj: [T, ld]; columns [0, q_rank) are the queries' latent, kv_off.. the
+// down-projection (rank, then dr; absent with cache == null).  blockIdx.y 0 norms the
+// queries' latent into c_q [T, q_rank], 1 makes the token's record.
+// ---------------------------------------------------------------------------
+#define LF_THREADS 128
+#define LF_KEEP 8     // row entries a thread keeps in registers between the two passes
+
+template <typename TA>
+__device__ __forceinline__ void norm_row(const TA* __restrict__ x, const float* __restrict__ gain,
+                                         TA* __restrict__ out, int n, float eps, float* scratch) {
+  float kept[LF_KEEP];
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < LF_KEEP; ++j) {
+    const int i = threadIdx.x + j * LF_THREADS;
+    kept[j] = i < n ? to_f32(x[i]) : 0.f;
+    ss += kept[j] * kept[j];
+  }
+  for (int i = threadIdx.x + LF_KEEP * LF_THREADS; i < n; i += LF_THREADS) {
+    const float v = to_f32(x[i]);
+    ss += v * v;
+  }
+  const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)n + eps);
+#pragma unroll
+  for (int j = 0; j < LF_KEEP; ++j) {
+    const int i = threadIdx.x + j * LF_THREADS;
+    if (i < n) out[i] = from_f32<TA>(kept[j] * inv * gain[i]);
+  }
+  for (int i = threadIdx.x + LF_KEEP * LF_THREADS; i < n; i += LF_THREADS)
+    out[i] = from_f32<TA>(to_f32(x[i]) * inv * gain[i]);
+}
+
+template <typename TA>
+__global__ void __launch_bounds__(LF_THREADS)
+latent_front_kernel(const TA* __restrict__ proj, long long ld, int q_rank,
+                    const float* __restrict__ q_gain, int kv_off,
+                    const int* __restrict__ positions, const float* __restrict__ freq, float mag,
+                    const float* __restrict__ kv_gain, float eps, const int* __restrict__ slots,
+                    TA* __restrict__ cache, TA* __restrict__ c_q, int dr, int rot_dims, int rank) {
+  __shared__ float scratch[32];
+  IX_PDL_WAIT();
+  const int t = blockIdx.x;
+  const TA* row = proj + (size_t)t * ld;
+  if (blockIdx.y == 0) {
+    norm_row<TA>(row, q_gain, c_q + (size_t)t * q_rank, q_rank, eps, scratch);
+    return;
+  }
+  const TA* kv = row + kv_off;
+  TA* rec = cache + (size_t)slots[t] * (rank + dr);
+  norm_row<TA>(kv, kv_gain, rec, rank, eps, scratch);
+  const float pos = (float)positions[t];
+  const int half = rot_dims >> 1;
+  for (int p = threadIdx.x; p < (dr + 1) / 2; p += blockDim.x) {
+    const float u = to_f32(kv[rank + 2 * p]);
+    const float v = 2 * p + 1 < dr ? to_f32(kv[rank + 2 * p + 1]) : 0.f;
+    float a = u, b = v;
+    if (p < half) {
+      const float ang = pos * freq[p];
+      const float c = cosf(ang) * mag, s = sinf(ang) * mag;
+      a = u * c - v * s;
+      b = v * c + u * s;
+    }
+    rec[rank + 2 * p] = from_f32<TA>(a);
+    if (2 * p + 1 < dr) rec[rank + 2 * p + 1] = from_f32<TA>(b);
+  }
+}
+
+IX_API int ix_latent_front(const void* proj, long long ld, int q_rank, const float* q_gain,
+                           int kv_off, const int* positions, const float* freq, float mag,
+                           const float* kv_gain, float eps, const int* slots, void* cache,
+                           void* c_q, int act_dtype, int T, int dr, int rot_dims, int rank,
+                           cudaStream_t stream) {
+  if (T <= 0) return IX_OK;
+  if (q_rank <= 0 || q_rank > ld || !q_gain || !c_q) return IX_ERR_SIZE;
+  if (cache != nullptr && (!slots || !kv_gain || rank <= 0 || dr < 0 || rot_dims < 0 ||
+                           rot_dims > dr || rot_dims % 2 || kv_off < 0 ||
+                           (long long)kv_off + rank + dr > ld))
+    return IX_ERR_SIZE;
+  IX_DISPATCH_DTYPE(act_dtype, TA,
+                    ix_launch(latent_front_kernel<TA>, dim3(T, cache != nullptr ? 2 : 1),
+                              dim3(LF_THREADS), 0, stream, (const TA*)proj, ld, q_rank, q_gain,
+                              kv_off, positions, freq, mag, kv_gain, eps, slots, (TA*)cache,
+                              (TA*)c_q, dr, rot_dims, rank));
   return ix_launch_status();
 }
 

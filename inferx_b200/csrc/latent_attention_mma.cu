@@ -21,6 +21,10 @@
 //      latents (the first `rank` entries of the same records, read transposed),
 //      CW = rank / NSPLIT <= 128 columns a warp, accumulators in registers.
 //
+// WIDE_W: for decoders that want their softmax weights in 32-bit arithmetic, a weight enters
+// its product with the latents as two bfloat16 terms, its rounding and the rounding of what
+// that left over, both into the same fp32 accumulators (16 bits of the weight).
+//
 // When few blocks would run over long runs of keys (single tokens late in long sequences),
 // the keys are cut into chunks of `chunk_tiles` tiles that start on multiples of the chunk
 // in absolute position; blockIdx.y picks the chunk, partial results (unnormalised output,
@@ -66,7 +70,7 @@ static inline int lm_ld(int dk) { return dk + (((dk / 8) % 2 == 0) ? 8 : 16); }
 
 #define LM_PLD 40   // bf16 per row of weights: 32 + 8 (80 bytes: an odd number of 16-byte units)
 
-template <int CW, int NSPLIT, int RG>
+template <int CW, int NSPLIT, int RG, bool WIDE_W>
 __global__ void __launch_bounds__(32 * RG * NSPLIT)
 latent_attention_mma_kernel(const bf16* __restrict__ q_lat, long long ql_sh, long long ql_st,
                             const bf16* __restrict__ q_rot, const bf16* __restrict__ cache,
@@ -90,7 +94,8 @@ latent_attention_mma_kernel(const bf16* __restrict__ q_lat, long long ql_sh, lon
   bf16* Ks = Qs + LM_ROWS * ld;                                      // [2][32][ld]
   float* Sp = reinterpret_cast<float*>(Ks + 2 * LM_KT * ld);         // [NSPLIT][64][LM_SLD]
   bf16* Ps = reinterpret_cast<bf16*>(Sp + NSPLIT * LM_ROWS * LM_SLD);  // [64][LM_PLD]
-  float* corr_s = reinterpret_cast<float*>(Ps + LM_ROWS * LM_PLD);   // [64]
+  bf16* Pr = Ps + (WIDE_W ? LM_ROWS * LM_PLD : 0);                   // [64][LM_PLD]: second terms
+  float* corr_s = reinterpret_cast<float*>(Pr + LM_ROWS * LM_PLD);   // [64]
   float* m_s = corr_s + LM_ROWS;                                     // [64] (at the end)
   float* l_s = m_s + LM_ROWS;                                        // [64] (at the end)
 
@@ -293,8 +298,15 @@ latent_attention_mma_kernel(const bf16* __restrict__ q_lat, long long ql_sh, lon
       m_run = m_new;
       bf16* pd = Ps + srow * LM_PLD + scol;
 #pragma unroll
-      for (int c = 0; c < CPL; c += 2)
-        *reinterpret_cast<unsigned*>(pd + c) = lm_pack(sv[c], sv[c + 1]);
+      for (int c = 0; c < CPL; c += 2) {
+        const __nv_bfloat162 hi = __floats2bfloat162_rn(sv[c], sv[c + 1]);
+        *reinterpret_cast<__nv_bfloat162*>(pd + c) = hi;
+        if (WIDE_W) {
+          const float2 f = __bfloat1622float2(hi);
+          *reinterpret_cast<unsigned*>(pd + LM_ROWS * LM_PLD + c) =
+              lm_pack(sv[c] - f.x, sv[c + 1] - f.y);
+        }
+      }
       if (lane % LPR == 0) corr_s[srow] = corr;
     }
     __syncthreads();
@@ -315,6 +327,12 @@ latent_attention_mma_kernel(const bf16* __restrict__ q_lat, long long ql_sh, lon
         unsigned pa[2][4];
         lm_ldsm4(pa[0][0], pa[0][1], pa[0][2], pa[0][3], pa_src);
         lm_ldsm4(pa[1][0], pa[1][1], pa[1][2], pa[1][3], pa_src + 16);
+        unsigned pb[WIDE_W ? 2 : 1][4];
+        if (WIDE_W) {
+          lm_ldsm4(pb[0][0], pb[0][1], pb[0][2], pb[0][3], pa_src + LM_ROWS * LM_PLD);
+          lm_ldsm4(pb[WIDE_W ? 1 : 0][0], pb[WIDE_W ? 1 : 0][1], pb[WIDE_W ? 1 : 0][2],
+                   pb[WIDE_W ? 1 : 0][3], pa_src + LM_ROWS * LM_PLD + 16);
+        }
         // 2 x CW / 16 steps, each one 16 keys x 16 columns; the next step's latents are
         // fetched before this step's products are issued
         constexpr int STEPS = 2 * (CW / 16);
@@ -330,6 +348,10 @@ latent_attention_mma_kernel(const bf16* __restrict__ q_lat, long long ql_sh, lon
           }
           lm_mma(o[2 * np], pa[ks2], vb0, vb1);
           lm_mma(o[2 * np + 1], pa[ks2], vb2, vb3);
+          if (WIDE_W) {
+            lm_mma(o[2 * np], pb[WIDE_W ? ks2 : 0], vb0, vb1);
+            lm_mma(o[2 * np + 1], pb[WIDE_W ? ks2 : 0], vb2, vb3);
+          }
           vb0 = n0; vb1 = n1; vb2 = n2; vb3 = n3;
         }
       } else {
@@ -337,12 +359,18 @@ latent_attention_mma_kernel(const bf16* __restrict__ q_lat, long long ql_sh, lon
         for (int ks2 = 0; ks2 < 2; ++ks2) {
           unsigned pa[4];
           lm_ldsm4(pa[0], pa[1], pa[2], pa[3], pa_src + ks2 * 16);
+          unsigned pb[4];
+          if (WIDE_W) lm_ldsm4(pb[0], pb[1], pb[2], pb[3], pa_src + LM_ROWS * LM_PLD + ks2 * 16);
 #pragma unroll
           for (int np = 0; np < CW / 16; ++np) {
             unsigned b0, b1, b2, b3;
             lm_ldsm4t(b0, b1, b2, b3, vb + ks2 * 16 * ld + np * 16);
             lm_mma(o[2 * np], pa, b0, b1);
             lm_mma(o[2 * np + 1], pa, b2, b3);
+            if (WIDE_W) {
+              lm_mma(o[2 * np], pb, b0, b1);
+              lm_mma(o[2 * np + 1], pb, b2, b3);
+            }
           }
         }
       }
@@ -447,7 +475,7 @@ IX_API int ix_latent_attention_mma_chunks(int blocks, int span, int* chunk_tiles
   return (tiles + ct - 1) / ct + 1;
 }
 
-template <int CW, int NSPLIT, int RG>
+template <int CW, int NSPLIT, int RG, bool WIDE_W>
 static int launch_lm(const void* q_lat, long long ql_sh, long long ql_st, const void* q_rot,
                      const void* cache, const int* block_table, int max_blocks, const int* cu_q,
                      const int* q_pos0, int S, void* out, long long o_sh, long long o_st, int H,
@@ -458,9 +486,9 @@ static int launch_lm(const void* q_lat, long long ql_sh, long long ql_st, const 
   const int ld = lm_ld(Dk);
   const size_t smem = (size_t)(LM_ROWS + 2 * LM_KT) * ld * sizeof(bf16) +
                       (size_t)NSPLIT * LM_ROWS * LM_SLD * sizeof(float) +
-                      (size_t)LM_ROWS * LM_PLD * sizeof(bf16) + 3 * LM_ROWS * sizeof(float);
+                      (size_t)LM_ROWS * LM_PLD * sizeof(bf16) * (WIDE_W ? 2 : 1) + 3 * LM_ROWS * sizeof(float);
   if (smem > 227 * 1024) return IX_ERR_SMEM;
-  auto kern = latent_attention_mma_kernel<CW, NSPLIT, RG>;
+  auto kern = latent_attention_mma_kernel<CW, NSPLIT, RG, WIDE_W>;
   static bool raised = false;     // per instantiation
   if (!raised) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -491,7 +519,8 @@ IX_API int ix_latent_attention_mma(const void* q_lat, long long ql_sh, long long
                                    void* out, long long o_sh, long long o_st, int T, int H,
                                    int rank, int dr, int page, int window, float scale,
                                    int num_tiles, int rows, int chunk_tiles, int nchunks,
-                                   float* part_o, float* part_ml, cudaStream_t stream) {
+                                   float* part_o, float* part_ml, int wide_weights,
+                                   cudaStream_t stream) {
   if (num_tiles <= 0 || S <= 0) return IX_OK;
   if (rows != 16 && rows != 64) return IX_ERR_SIZE;
   if (!ix_latent_attention_mma_applies(rank, dr) || H <= 0 || page <= 0 || max_blocks <= 0)
@@ -503,9 +532,9 @@ IX_API int ix_latent_attention_mma(const void* q_lat, long long ql_sh, long long
     return IX_ERR_ALIGN;
   int code;
 #define IX_LM1(CW, NS, RG)                                                                       \
-  code = launch_lm<CW, NS, RG>(q_lat, ql_sh, ql_st, q_rot, cache, block_table, max_blocks, cu_q, \
-                               q_pos0, S, out, o_sh, o_st, H, dr, page, window, scale,           \
-                               num_tiles, chunk_tiles, nchunks, part_o, part_ml, stream)
+  code = (wide_weights ? launch_lm<CW, NS, RG, true> : launch_lm<CW, NS, RG, false>)(            \
+      q_lat, ql_sh, ql_st, q_rot, cache, block_table, max_blocks, cu_q, q_pos0, S, out, o_sh,    \
+      o_st, H, dr, page, window, scale, num_tiles, chunk_tiles, nchunks, part_o, part_ml, stream)
 #define IX_LM(CW, NS)            \
   do {                           \
     if (rows == 16) {            \

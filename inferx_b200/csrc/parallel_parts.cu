@@ -83,7 +83,7 @@ __global__ void add_rmsnorm_sum_kernel(float* __restrict__ resid, const void* __
     bool any = false;
     if (cy) {     // a mixture's output that was never written: expert rows, weights, shared part
       for (int e = 0; e < ck; ++e)
-        add += cw[(size_t)tok * ck + e] * to_f32(cy[(size_t)cdest[(size_t)tok * ck + e] * W + i]);
+        add += (cw ? cw[(size_t)tok * ck + e] : 1.0f) * to_f32(cy[(size_t)cdest[(size_t)tok * ck + e] * W + i]);
       if (cshared) add += sg * to_f32(cshared[src + i]);
       any = true;
     }
@@ -151,7 +151,7 @@ __global__ void add_rmsnorm_sum_bf16_vec_kernel(
       for (int j = 0; j < 8; ++j) add[j] = 0.f;
       if (cy) {
         for (int e = 0; e < ck; ++e) {
-          const float ws = cw[(size_t)tok * ck + e];
+          const float ws = cw ? cw[(size_t)tok * ck + e] : 1.0f;
           bf8_to_f32(reinterpret_cast<const uint4*>(cy)[(size_t)cdest[(size_t)tok * ck + e] * chunks + c], f);
 #pragma unroll
           for (int j = 0; j < 8; ++j) add[j] += ws * f[j];
@@ -223,7 +223,7 @@ IX_API int ix_add_rmsnorm_sum(float* resid, const void* d0, int c0, const void* 
                               cudaStream_t stream) {
   if (R <= 0) return IX_OK;
   if (W <= 0 || !g0 || !out0 || (out1 && !g1)) return IX_ERR_SIZE;
-  if (cy && (!cdest || !cw || ck <= 0)) return IX_ERR_SIZE;
+  if (cy && (!cdest || ck <= 0)) return IX_ERR_SIZE;    // cw null: weights of one
   const uintptr_t all = (uintptr_t)resid | (uintptr_t)d0 | (uintptr_t)d1 | (uintptr_t)d2 |
                         (uintptr_t)vec | (uintptr_t)g0 | (uintptr_t)g1 | (uintptr_t)out0 |
                         (uintptr_t)out1 | (uintptr_t)cy | (uintptr_t)cshared;

@@ -80,6 +80,7 @@ struct RouteRule {
   int keep;
   float renorm_eps;
   int active;
+  int sigmoid;      // scores are sigmoid(logit), each on its own, instead of the softmax
 };
 
 #define ROUTER_MAX_GROUPS 32
@@ -102,18 +103,22 @@ __device__ __forceinline__ void warp_argmax(float& best, int& bi) {
 __device__ __forceinline__ void select_topk_ruled(float* p, int E, int k, int renorm, float scale,
                                                   const RouteRule& rule, float* __restrict__ out_w,
                                                   int* __restrict__ out_i, int lane) {
-  float mx = -INFINITY;
-  for (int e = lane; e < E; e += 32) mx = fmaxf(mx, p[e]);
-  mx = warp_max(mx);
-  float sum = 0.f;
-  for (int e = lane; e < E; e += 32) {
-    const float v = expf(p[e] - mx);
-    p[e] = v;
-    sum += v;
+  if (rule.sigmoid) {
+    for (int e = lane; e < E; e += 32) p[e] = 1.0f / (1.0f + expf(-p[e]));
+  } else {
+    float mx = -INFINITY;
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, p[e]);
+    mx = warp_max(mx);
+    float sum = 0.f;
+    for (int e = lane; e < E; e += 32) {
+      const float v = expf(p[e] - mx);
+      p[e] = v;
+      sum += v;
+    }
+    sum = warp_sum(sum);
+    __syncwarp();
+    for (int e = lane; e < E; e += 32) p[e] = p[e] / sum;       // the scores
   }
-  sum = warp_sum(sum);
-  __syncwarp();
-  for (int e = lane; e < E; e += 32) p[e] = p[e] / sum;       // the scores
   __syncwarp();
   // groups that may be chosen from, as a mask over at most 32 groups (lane g owns group g)
   unsigned allowed = 0xffffffffu;
@@ -161,10 +166,50 @@ __device__ __forceinline__ void select_topk_ruled(float* p, int E, int k, int re
   }
 }
 
+// Sigmoid scores without a correction or groups: the k largest logits (the same order as
+// their scores', also where fp32 scores are all one), each weighing its own score.
+__device__ __forceinline__ void select_topk_sigmoid(float* p, int E, int k, int renorm,
+                                                    float scale, float renorm_eps,
+                                                    float* __restrict__ out_w,
+                                                    int* __restrict__ out_i, int lane) {
+  float total = 0.f, my_w = 0.f;
+  int my_i = 0;
+  unsigned long long taken = 0ull;      // this lane's entries lane + 32 j, j < 64, by bit
+  for (int s = 0; s < k; ++s) {
+    float best = -INFINITY;
+    int bi = 0x7fffffff;
+    for (int e = lane, j = 0; e < E; e += 32, ++j) {
+      const float v = p[e];
+      const bool out = j < 64 ? ((taken >> j) & 1ull) != 0ull : v == -INFINITY;
+      if (!out && (bi == 0x7fffffff || v > best)) { best = v; bi = e; }
+    }
+    warp_argmax(best, bi);
+    const float score = 1.0f / (1.0f + expf(-best));
+    if (lane == s) { my_w = score; my_i = bi < E ? bi : 0; }
+    total += score;
+    if (bi < E && (bi & 31) == lane) {
+      const int j = bi >> 5;
+      if (j < 64) taken |= 1ull << j;
+      else p[bi] = -INFINITY;
+    }
+    __syncwarp();
+  }
+  if (lane < k) {
+    float wv = my_w;
+    if (renorm_eps >= 0.f) wv = wv / (total + renorm_eps);
+    else if (renorm && total > 0.f) wv = wv / total;
+    wv *= scale;
+    out_w[lane] = wv;
+    out_i[lane] = my_i;
+  }
+}
+
 __device__ __forceinline__ void select_by_rule(float* p, int E, int k, int renorm, float scale,
                                                const RouteRule& rule, float* __restrict__ out_w,
                                                int* __restrict__ out_i, int lane) {
-  if (rule.active) select_topk_ruled(p, E, k, renorm, scale, rule, out_w, out_i, lane);
+  if (rule.active && rule.sigmoid && !rule.correction && rule.groups == 0)
+    select_topk_sigmoid(p, E, k, renorm, scale, rule.renorm_eps, out_w, out_i, lane);
+  else if (rule.active) select_topk_ruled(p, E, k, renorm, scale, rule, out_w, out_i, lane);
   else select_topk(p, E, k, renorm, scale, out_w, out_i, lane);
 }
 
@@ -445,22 +490,23 @@ IX_API int ix_router_topk(const void* x, const float* w, const float* extra_w, i
                           int T, int H, int E, int k, int renorm, float scale, float* topk_w,
                           int* topk_idx, float* extra_out, float* logits_scratch,
                           cudaStream_t stream) {
-  RouteRule rule = {nullptr, 0, 0, -1.f, 0};
+  RouteRule rule = {nullptr, 0, 0, -1.f, 0, 0};
   return router_topk_impl(x, w, extra_w, act_dtype, T, H, E, k, renorm, scale, topk_w, topk_idx,
                           extra_out, logits_scratch, rule, stream);
 }
 
-// The same with the choice ruled by a correction, groups and a division by (sum + eps).
+// The same with the choice ruled by a correction, groups and a division by (sum + eps), of
+// softmax scores or of sigmoid ones.
 IX_API int ix_router_topk_ruled(const void* x, const float* w, const float* extra_w,
                                 int act_dtype, int T, int H, int E, int k, int renorm,
                                 float scale, const float* correction, int groups, int keep,
-                                float renorm_eps, float* topk_w, int* topk_idx, float* extra_out,
-                                float* logits_scratch, cudaStream_t stream) {
+                                float renorm_eps, int sigmoid, float* topk_w, int* topk_idx,
+                                float* extra_out, float* logits_scratch, cudaStream_t stream) {
   if (groups < 0 || groups > ROUTER_MAX_GROUPS) return IX_ERR_SIZE;
   if (groups > 0 && (E % groups != 0 || keep <= 0 || keep > groups ||
                      (long long)keep * (E / groups) < k))
     return IX_ERR_SIZE;
-  RouteRule rule = {correction, groups, keep, renorm_eps, 1};
+  RouteRule rule = {correction, groups, keep, renorm_eps, 1, sigmoid};
   return router_topk_impl(x, w, extra_w, act_dtype, T, H, E, k, renorm, scale, topk_w, topk_idx,
                           extra_out, logits_scratch, rule, stream);
 }
@@ -563,7 +609,8 @@ static int router_topk_impl(const void* x, const float* w, const float* extra_w,
 __device__ __forceinline__ void dispatch_in_block(const int* topk_idx, int A, int E, int k,
                                                   int* __restrict__ offsets,
                                                   int* __restrict__ rows, int* __restrict__ dest,
-                                                  int* counts) {
+                                                  int* counts, const float* __restrict__ topk_w,
+                                                  float* __restrict__ row_w) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int nwarps = blockDim.x >> 5;
   for (int e = warp; e < E; e += nwarps) {
@@ -609,6 +656,7 @@ __device__ __forceinline__ void dispatch_in_block(const int* topk_idx, int A, in
         const int r = base + __popc(mask & ((1u << lane) - 1u));
         rows[r] = a / k;
         dest[a] = r;
+        if (row_w) row_w[r] = topk_w[a];
       }
       base += __popc(mask);
     }
@@ -617,10 +665,11 @@ __device__ __forceinline__ void dispatch_in_block(const int* topk_idx, int A, in
 
 __global__ void __launch_bounds__(1024)
 moe_dispatch_kernel(const int* __restrict__ topk_idx, int A, int E, int k,
-                    int* __restrict__ offsets, int* __restrict__ rows, int* __restrict__ dest) {
+                    int* __restrict__ offsets, int* __restrict__ rows, int* __restrict__ dest,
+                    const float* __restrict__ topk_w, float* __restrict__ row_w) {
   extern __shared__ int counts[];  // [E + 1]
   IX_PDL_WAIT();
-  dispatch_in_block(topk_idx, A, E, k, offsets, rows, dest, counts);
+  dispatch_in_block(topk_idx, A, E, k, offsets, rows, dest, counts, topk_w, row_w);
 }
 
 // ---------------------------------------------------------------------------
@@ -671,7 +720,8 @@ dispatch_scan_kernel(int* __restrict__ counts, int blocks, int E, int* __restric
 __global__ void __launch_bounds__(DISPATCH_CHUNK)
 dispatch_place_kernel(const int* __restrict__ topk_idx, int A, int E, int k,
                       const int* __restrict__ bases, const int* __restrict__ offsets,
-                      int* __restrict__ rows, int* __restrict__ dest) {
+                      int* __restrict__ rows, int* __restrict__ dest,
+                      const float* __restrict__ topk_w, float* __restrict__ row_w) {
   extern __shared__ int warp_count[];   // [32][E]
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   for (int i = threadIdx.x; i < 32 * E; i += blockDim.x) warp_count[i] = 0;
@@ -688,6 +738,7 @@ dispatch_place_kernel(const int* __restrict__ topk_idx, int A, int E, int k,
     const int r = offsets[e] + bases[(size_t)blockIdx.x * E + e] + before + rank;
     rows[r] = a / k;
     dest[a] = r;
+    if (row_w) row_w[r] = topk_w[a];
   }
 }
 
@@ -699,8 +750,11 @@ IX_API int ix_moe_dispatch_scratch_ints(int T, int E, int k) {
   return (int)(((A + DISPATCH_CHUNK - 1) / DISPATCH_CHUNK) * E);
 }
 
+// row_w (with topk_w [T, k]; both or neither): the weight of every grouped row.
 IX_API int ix_moe_dispatch(const int* topk_idx, int T, int E, int k, int* offsets, int* rows,
-                           int* dest, int* scratch, cudaStream_t stream) {
+                           int* dest, int* scratch, const float* topk_w, float* row_w,
+                           cudaStream_t stream) {
+  if (row_w && !topk_w) return IX_ERR_SIZE;
   if (E <= 0 || k <= 0 || E > ROUTER_MAX_EXPERTS) return IX_ERR_SIZE;
   if (T < 0) return IX_ERR_SIZE;
   const int A = T * k;
@@ -709,11 +763,11 @@ IX_API int ix_moe_dispatch(const int* topk_idx, int T, int E, int k, int* offset
     dispatch_count_kernel<<<blocks, DISPATCH_CHUNK, 0, stream>>>(topk_idx, A, E, scratch);
     dispatch_scan_kernel<<<1, DISPATCH_MAX_E, 0, stream>>>(scratch, blocks, E, offsets);
     dispatch_place_kernel<<<blocks, DISPATCH_CHUNK, 32 * E * sizeof(int), stream>>>(
-        topk_idx, A, E, k, scratch, offsets, rows, dest);
+        topk_idx, A, E, k, scratch, offsets, rows, dest, topk_w, row_w);
     return ix_launch_status();
   }
   const int threads = E >= 32 ? 1024 : 32 * E;
   ix_launch(moe_dispatch_kernel, dim3(1), dim3(threads), (E + 1) * sizeof(int), stream, topk_idx,
-            A, E, k, offsets, rows, dest);
+            A, E, k, offsets, rows, dest, topk_w, row_w);
   return ix_launch_status();
 }

@@ -93,11 +93,12 @@ static inline EncodeTiledFn encode_fn() {
 // 2-D bf16 tensor [rows, cols], cols contiguous, read in boxes of box_rows x box_cols
 // with the 128-byte swizzle (box_cols * 2 bytes must be 128).
 static inline int ix_tensor_map_bf16_2d(CUtensorMap* map, const void* base, long long rows,
-                                        long long cols, int box_cols, int box_rows) {
+                                        long long cols, int box_cols, int box_rows,
+                                        long long row_pitch = 0) {   // elements; 0: cols
   EncodeTiledFn fn = encode_fn();
   if (!fn) return IX_ERR_UNSUPPORTED;
   cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
-  cuuint64_t strides[1] = {(cuuint64_t)cols * 2};
+  cuuint64_t strides[1] = {(cuuint64_t)(row_pitch > 0 ? row_pitch : cols) * 2};
   cuuint32_t box[2] = {(cuuint32_t)box_cols, (cuuint32_t)box_rows};
   cuuint32_t estr[2] = {1, 1};
   CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims,

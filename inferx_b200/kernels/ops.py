@@ -177,22 +177,28 @@ class CombinePending:
     part.  ``add_rmsnorm`` consumes it in the same pass that adds it to the residual;
     ``materialize`` writes it out like ``moe_combine``."""
 
-    def __init__(self, y, dest, topk_w, shared, shared_logit):
+    def __init__(self, y, dest, topk_w, shared, shared_logit, weighted=True):
         self.y, self.dest, self.topk_w = y, dest, topk_w
+        self.weighted = weighted       # False: the rows are added as they are
         self.shared, self.shared_logit = shared, shared_logit
         self.shape = (topk_w.shape[0], y.shape[1])
         self.dtype = y.dtype
 
     def materialize(self):
-        return moe_combine(self.y, self.dest, self.topk_w, self.shared, self.shared_logit)
+        return moe_combine(self.y, self.dest, self.topk_w, self.shared, self.shared_logit,
+                           self.weighted)
+
+    @property
+    def weights(self):
+        return self.topk_w if self.weighted else None
 
 
-def moe_combine_pending(y, dest, topk_w, shared, shared_logit):
+def moe_combine_pending(y, dest, topk_w, shared, shared_logit, weighted=True):
     """``moe_combine`` deferred into the next residual add + norm where that kernel
     exists (bfloat16, width a multiple of 8); the combined tensor otherwise."""
     if y.dtype == torch.bfloat16 and y.shape[1] % 8 == 0 and y.shape[1] <= 8192:
-        return CombinePending(y, dest, topk_w, shared, shared_logit)
-    return moe_combine(y, dest, topk_w, shared, shared_logit)
+        return CombinePending(y, dest, topk_w, shared, shared_logit, weighted)
+    return moe_combine(y, dest, topk_w, shared, shared_logit, weighted)
 
 
 def add_rmsnorm(resid: torch.Tensor, delta, gain: torch.Tensor,
@@ -208,7 +214,7 @@ def add_rmsnorm(resid: torch.Tensor, delta, gain: torch.Tensor,
             T, H = resid.shape
             out = torch.empty((T, H), dtype=out_dtype, device=resid.device)
             code = _lib().ix_combine_add_rmsnorm(
-                _ptr(resid), _ptr(delta.y), _ptr(delta.dest), _ptr(delta.topk_w),
+                _ptr(resid), _ptr(delta.y), _ptr(delta.dest), _ptr(delta.weights),
                 _ptr(delta.shared), _ptr(delta.shared_logit), _ptr(gain), _ptr(out), T, H,
                 delta.topk_w.shape[1], ctypes.c_float(eps), _stream())
             _check(code, "combine_add_rmsnorm")
@@ -270,8 +276,11 @@ def linear(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = 
 
 def gemm_generic(x: torch.Tensor, w: torch.Tensor, rows: Optional[torch.Tensor],
                  offsets: Optional[torch.Tensor], dual: bool,
-                 out_dtype: Optional[torch.dtype] = None, num_out_rows: Optional[int] = None):
-    """CUDA-core product, single (offsets None) or grouped by expert."""
+                 out_dtype: Optional[torch.dtype] = None, num_out_rows: Optional[int] = None,
+                 row_scale: Optional[torch.Tensor] = None):
+    """CUDA-core product, single (offsets None) or grouped by expert.  ``row_scale`` (dual
+    only): see ``grouped_gate_up_swiglu``."""
+    _chk("row_scale", row_scale, torch.float32, optional=True)
     _chk("x", x)
     _chk("w", w)
     _chk("rows", rows, torch.int32, optional=True)
@@ -291,7 +300,8 @@ def gemm_generic(x: torch.Tensor, w: torch.Tensor, rows: Optional[torch.Tensor],
     out = torch.empty((A, N), dtype=out_dtype, device=x.device)
     code = _lib().ix_gemm_generic(
         _ptr(x), _ptr(rows), _ptr(offsets), _ptr(w), _ptr(out), _dtype_code(x),
-        F32 if out_dtype == torch.float32 else BF16, 1 if dual else 0, M, N, K, E, A, _stream())
+        F32 if out_dtype == torch.float32 else BF16, 1 if dual else 0, M, N, K, E, A, _ptr(row_scale),
+        _stream())
     _check(code, "gemm_generic")
     _count()
     return out
@@ -468,14 +478,15 @@ ROUTER_FEW_TOKENS = 128
 def router_topk(x: torch.Tensor, w: torch.Tensor, top_k: int, renormalize: bool, scale: float,
                 extra_w: Optional[torch.Tensor] = None,
                 correction: Optional[torch.Tensor] = None, group_count: int = 0,
-                group_keep: int = 0, renorm_eps: Optional[float] = None
+                group_keep: int = 0, renorm_eps: Optional[float] = None, score: str = "softmax"
                 ) -> Tuple[torch.Tensor, torch.Tensor, Optional[torch.Tensor]]:
     """fp32 router logits, softmax over all experts, top-k (ties to the lower index).
 
     ``correction`` (fp32 [E]) is added to the scores for the choice alone; with
     ``group_count`` > 0 the outputs form that many equal groups of neighbours and only
     outputs of the ``group_keep`` groups with the largest corrected score can be chosen;
-    ``renorm_eps`` >= 0 divides the chosen scores by (their sum + renorm_eps).
+    ``renorm_eps`` >= 0 divides the chosen scores by (their sum + renorm_eps).  ``score``
+    "sigmoid": an output's score is the sigmoid of its own logit instead.
 
     Returns (weights [T,k] fp32, experts [T,k] int32, x.extra_w [T] fp32 or None).
     Few tokens: one warp per (token, expert) computes the logits and one warp per
@@ -493,7 +504,9 @@ def router_topk(x: torch.Tensor, w: torch.Tensor, top_k: int, renormalize: bool,
     ex = torch.empty((T,), dtype=torch.float32, device=x.device) if extra_w is not None else None
     few = T < ROUTER_FEW_TOKENS   # few tokens: logits by many blocks, then a selection kernel
     scratch = torch.empty((T, E), dtype=torch.float32, device=x.device) if few else None
-    ruled = (correction is not None or group_count > 0
+    if score not in ("softmax", "sigmoid"):
+        raise KernelError(f"router_topk: score {score!r}")
+    ruled = (correction is not None or group_count > 0 or score != "softmax"
              or (renorm_eps is not None and renorm_eps >= 0))
     if ruled:
         _chk("correction", correction, torch.float32, optional=True)
@@ -503,7 +516,7 @@ def router_topk(x: torch.Tensor, w: torch.Tensor, top_k: int, renormalize: bool,
             _ptr(x), _ptr(w), _ptr(extra_w), _dtype_code(x), T, H, E, top_k,
             1 if renormalize else 0, ctypes.c_float(scale), _ptr(correction), int(group_count),
             int(group_keep), ctypes.c_float(-1.0 if renorm_eps is None else renorm_eps),
-            _ptr(tw), _ptr(ti), _ptr(ex), _ptr(scratch), _stream())
+            1 if score == "sigmoid" else 0, _ptr(tw), _ptr(ti), _ptr(ex), _ptr(scratch), _stream())
     else:
         code = _lib().ix_router_topk(
             _ptr(x), _ptr(w), _ptr(extra_w), _dtype_code(x), T, H, E, top_k,
@@ -514,8 +527,10 @@ def router_topk(x: torch.Tensor, w: torch.Tensor, top_k: int, renormalize: bool,
     return tw, ti, ex
 
 
-def moe_dispatch(topk_idx: torch.Tensor, num_experts: int):
-    """offsets[E+1], rows[A] (token of each grouped row), dest[A] (grouped row of t*k+slot)."""
+def moe_dispatch(topk_idx: torch.Tensor, num_experts: int,
+                 topk_w: Optional[torch.Tensor] = None):
+    """offsets[E+1], rows[A] (token of each grouped row), dest[A] (grouped row of t*k+slot);
+    with ``topk_w`` [T, k] also the weight of every grouped row [A]."""
     _chk("topk_idx", topk_idx, torch.int32)
     T, k = topk_idx.shape
     dev = topk_idx.device
@@ -524,14 +539,24 @@ def moe_dispatch(topk_idx: torch.Tensor, num_experts: int):
     dest = torch.empty((T * k,), dtype=torch.int32, device=dev)
     n_scratch = _lib().ix_moe_dispatch_scratch_ints(T, num_experts, k)
     scratch = torch.empty((n_scratch,), dtype=torch.int32, device=dev) if n_scratch else None
+    row_w = None
+    if topk_w is not None:
+        _chk("topk_w", topk_w, torch.float32)
+        if topk_w.numel() != T * k:
+            raise KernelError("moe_dispatch: one weight per assignment")
+        row_w = torch.empty((T * k,), dtype=torch.float32, device=dev)
     _check(_lib().ix_moe_dispatch(_ptr(topk_idx), T, num_experts, k, _ptr(offsets), _ptr(rows),
-                                  _ptr(dest), _ptr(scratch), _stream()), "moe_dispatch")
+                                  _ptr(dest), _ptr(scratch), _ptr(topk_w), _ptr(row_w),
+                                  _stream()), "moe_dispatch")
     _count(3 if n_scratch else 1)
-    return offsets, rows, dest
+    return (offsets, rows, dest) if row_w is None else (offsets, rows, dest, row_w)
 
 
 def moe_combine(y: torch.Tensor, dest: torch.Tensor, topk_w: torch.Tensor,
-                shared: Optional[torch.Tensor], shared_logit: Optional[torch.Tensor]):
+                shared: Optional[torch.Tensor], shared_logit: Optional[torch.Tensor],
+                weighted: bool = True):
+    """out[t] = sum_s w[t, s] y[dest[t k + s]] (+ the shared expert's part); with ``weighted``
+    off the rows are added as they are (their weights went into the experts)."""
     _chk("y", y)
     _chk("dest", dest, torch.int32)
     _chk("topk_w", topk_w, torch.float32)
@@ -540,7 +565,8 @@ def moe_combine(y: torch.Tensor, dest: torch.Tensor, topk_w: torch.Tensor,
     T, k = topk_w.shape
     H = y.shape[1]
     out = torch.empty((T, H), dtype=y.dtype, device=y.device)
-    _check(_lib().ix_moe_combine(_ptr(y), _ptr(dest), _ptr(topk_w), _ptr(shared),
+    _check(_lib().ix_moe_combine(_ptr(y), _ptr(dest), _ptr(topk_w if weighted else None),
+                                 _ptr(shared),
                                  _ptr(shared_logit), _ptr(out), _dtype_code(y), T, H, k,
                                  _stream()), "moe_combine")
     _count()
@@ -1049,7 +1075,8 @@ def gemm_small_m(x: torch.Tensor, w: torch.Tensor, rows: Optional[torch.Tensor],
                  offsets: Optional[torch.Tensor], dual: bool, num_out_rows: int,
                  out_dtype: Optional[torch.dtype] = None, rows_per_pass: int = 8,
                  active_groups: int = 0, offsets_settled: bool = False,
-                 glu_clamp: Optional[Tuple[float, float, float]] = None):
+                 glu_clamp: Optional[Tuple[float, float, float]] = None,
+                 row_scale: Optional[torch.Tensor] = None):
     """Weight-streaming product for few rows per weight matrix (bf16 inputs).
     ``offsets_settled``: the kernel that wrote ``offsets`` is at least two launches back
     in this stream (so the launch may read it, and start on its weights, before waiting
@@ -1073,7 +1100,8 @@ def gemm_small_m(x: torch.Tensor, w: torch.Tensor, rows: Optional[torch.Tensor],
         F32 if out_dtype == torch.float32 else BF16, 1 if dual else 0,
         0 if offsets is not None else x.shape[0], N, K, E, rows_per_pass,
         active_groups or min(E, num_out_rows), 1 if offsets_settled else 0,
-        ctypes.c_float(limit), ctypes.c_float(alpha), ctypes.c_float(shift), _stream())
+        ctypes.c_float(limit), ctypes.c_float(alpha), ctypes.c_float(shift), _ptr(row_scale),
+        _stream())
     _check(code, "gemm_small_m")
     _count()
     return out
@@ -1126,7 +1154,8 @@ def check_async_errors():
                               "the output of that call is not valid")
 
 
-def grouped_gemm_tc(a: torch.Tensor, offsets: torch.Tensor, w: torch.Tensor, dual: bool):
+def grouped_gemm_tc(a: torch.Tensor, offsets: torch.Tensor, w: torch.Tensor, dual: bool,
+                    row_scale: Optional[torch.Tensor] = None):
     """Grouped product on tcgen05 tensor cores: ``a`` [rows, K] already grouped by
     expert, ``w`` [E, N or 2N, K]; returns [rows, N] bf16."""
     _chk("a", a, torch.bfloat16)
@@ -1139,7 +1168,7 @@ def grouped_gemm_tc(a: torch.Tensor, offsets: torch.Tensor, w: torch.Tensor, dua
     out = torch.empty((a.shape[0], N), dtype=torch.bfloat16, device=a.device)
     code = _lib().ix_grouped_gemm_tc(_ptr(a), _ptr(offsets), _ptr(w), _ptr(out),
                                      1 if dual else 0, a.shape[0], N, K, E,
-                                     _ptr(_tc_status(a.device)), _stream())
+                                     _ptr(_tc_status(a.device)), _ptr(row_scale), _stream())
     _check(code, "grouped_gemm_tc")
     _count()
     return out
@@ -1154,7 +1183,7 @@ STREAM_GROUPED_MAX_ROWS = 4
 
 def gemm_stream_grouped(x: torch.Tensor, w: torch.Tensor, rows: Optional[torch.Tensor],
                         offsets: torch.Tensor, dual: bool, num_out_rows: int,
-                        rows_per_pass: int = 8):
+                        rows_per_pass: int = 8, row_scale: Optional[torch.Tensor] = None):
     """Grouped weight-streaming product, persistent form (few rows per expert, bf16)."""
     _chk("x", x, torch.bfloat16)
     _chk("w", w, torch.bfloat16)
@@ -1168,7 +1197,8 @@ def gemm_stream_grouped(x: torch.Tensor, w: torch.Tensor, rows: Optional[torch.T
         raise KernelError("gemm_stream_grouped: offsets must have one entry per expert plus one")
     out = torch.empty((num_out_rows, N), dtype=torch.bfloat16, device=x.device)
     code = _lib().ix_gemm_stream_grouped(_ptr(x), _ptr(rows), _ptr(offsets), _ptr(w), _ptr(out),
-                                         1 if dual else 0, N, K, E, rows_per_pass, _stream())
+                                         1 if dual else 0, N, K, E, rows_per_pass, _ptr(row_scale),
+                                         _stream())
     _check(code, "gemm_stream_grouped")
     _count()
     return out
@@ -1185,21 +1215,29 @@ def _streams_weights(x: torch.Tensor, w: torch.Tensor) -> bool:
 
 
 def grouped_gate_up_swiglu(x: torch.Tensor, rows: torch.Tensor, offsets: torch.Tensor,
-                           w_gate_up: torch.Tensor):
+                           w_gate_up: torch.Tensor, row_scale: Optional[torch.Tensor] = None):
     """act[r] = silu(x[rows[r]] . Wg[e]^T) * (x[rows[r]] . Wu[e]^T), e from offsets.
 
-    ``w_gate_up``: [E, 2I, H], per expert the gate rows then the up rows."""
+    ``w_gate_up``: [E, 2I, H], per expert the gate rows then the up rows.  ``row_scale``
+    (fp32 [A]): row r's input counts times row_scale[r]; the products being linear, the
+    factor multiplies both accumulators ahead of the activation."""
     A = rows.numel()
+    if row_scale is not None:
+        _chk("row_scale", row_scale, torch.float32)
+        if row_scale.numel() != A:
+            raise KernelError("grouped_gate_up_swiglu: one factor per grouped row")
     per = A / w_gate_up.shape[0]
     if _stream_grouped_applies(x, w_gate_up, A):
         return gemm_stream_grouped(x, w_gate_up, rows, offsets, True, A,
-                                   rows_per_pass=8 if per <= 2 else 16)
+                                   rows_per_pass=8 if per <= 2 else 16, row_scale=row_scale)
     if per <= SMALL_M_ROWS_PER_GROUP and _streams_weights(x, w_gate_up):
         return gemm_small_m(x, w_gate_up, rows, offsets, True, A,
-                            rows_per_pass=8 if per <= 2 else 16)
+                            rows_per_pass=8 if per <= 2 else 16, row_scale=row_scale)
     if USE_TCGEN05 and _streams_weights(x, w_gate_up) and w_gate_up.shape[0] <= TCGEN05_MAX_EXPERTS:
-        return grouped_gemm_tc(gather_rows(x, rows), offsets, w_gate_up, True)
-    return gemm_generic(x, w_gate_up, rows, offsets, dual=True, num_out_rows=A)
+        return grouped_gemm_tc(gather_rows(x, rows), offsets, w_gate_up, True,
+                               row_scale=row_scale)
+    return gemm_generic(x, w_gate_up, rows, offsets, dual=True, num_out_rows=A,
+                        row_scale=row_scale)
 
 
 def grouped_down(act: torch.Tensor, offsets: torch.Tensor, w_down: torch.Tensor,
@@ -1326,13 +1364,14 @@ def gate_up_glu_clamped(x: torch.Tensor, w_gate_up: torch.Tensor, limit: float, 
 BATCHED_STREAM_MIN_WEIGHTS = 1 << 20
 
 
-def batched_linear(x: torch.Tensor, w: torch.Tensor):
+def batched_linear(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None):
     """out[b] = x[b] . w[b]^T for x [B, M, K] (any strides with unit inner stride) and
     w [B, N, K]: one library call batched over the leading dimension (per-head
     products).  float32 operands are multiplied in true 32-bit.  (For a few rows per
     matrix the grouped weight-streaming kernel, one group per matrix, was measured too:
     equal at 16 heads, slower at 8 and at 32 - a decode step of 0.85 against 0.74 ms at
-    width 4096 -, so the library keeps these products at every size.)"""
+    width 4096 -, so the library keeps these products at every size.)  ``out``: a view [B, M, N] with unit inner
+    stride that takes the result (the heads of a token beside each other, say)."""
     if not (x.is_cuda and w.is_cuda):
         raise KernelError("batched_linear: tensors must be on a CUDA device")
     if x.dtype != w.dtype or x.dim() != 3 or w.dim() != 3 or x.shape[0] != w.shape[0] \
@@ -1342,16 +1381,23 @@ def batched_linear(x: torch.Tensor, w: torch.Tensor):
     if x.dtype == torch.float32 and torch.backends.cuda.matmul.allow_tf32:
         raise KernelError("batched_linear: TF32 is switched on; 32-bit products must be exact")
     B, M, K = x.shape
+    if out is not None and (tuple(out.shape) != (B, M, w.shape[1]) or out.dtype != x.dtype
+                            or out.stride(2) != 1):
+        raise KernelError(f"batched_linear: out must be a view {(B, M, w.shape[1])} of {x.dtype} "
+                          "with unit inner stride")
     if (M <= SMALL_M_DENSE_ROWS and w.shape[1] * K >= BATCHED_STREAM_MIN_WEIGHTS
             and x.is_contiguous() and w.is_contiguous() and _streams_weights(x, w)):
         # a few rows against large matrices: each matrix is a group of the weight-streaming
         # kernel, its rows one pass (the library's batched product reads such weights at a
         # fraction of the memory rate)
         offsets = torch.arange(0, (B + 1) * M, M, dtype=torch.int32, device=x.device)
-        out = gemm_small_m(x.view(B * M, K), w, None, offsets, False, B * M,
-                           rows_per_pass=8 if M <= 8 else 16, active_groups=B)
-        return out.view(B, M, w.shape[1])
+        y = gemm_small_m(x.view(B * M, K), w, None, offsets, False, B * M,
+                         rows_per_pass=8 if M <= 8 else 16, active_groups=B)
+        y = y.view(B, M, w.shape[1])
+        return y if out is None else out.copy_(y)
     LIBRARY_CALLS[0] += 1
+    if out is not None:
+        return torch.bmm(x, w.transpose(1, 2), out=out)
     return torch.bmm(x, w.transpose(1, 2))
 
 
@@ -1415,7 +1461,7 @@ def _mma_latent_applies(q_lat, q_rot) -> bool:
 
 def latent_attention(q_lat: torch.Tensor, q_rot: torch.Tensor, cache: torch.Tensor,
                      block_table: torch.Tensor, step, window: int, scale: float,
-                     kernel: Optional[str] = None):
+                     kernel: Optional[str] = None, fp32_weights: bool = False):
     """Attention of this step's queries over cached latent records.
 
     ``q_lat`` [heads, T, rank] (the query with the key matrix folded in), ``q_rot``
@@ -1424,7 +1470,9 @@ def latent_attention(q_lat: torch.Tensor, q_rot: torch.Tensor, cache: torch.Tens
     the ``window`` - 1 before it; all earlier ones when ``window`` is 0); returns
     sum_j p_j latent_j as [heads, T, rank].  ``step`` carries ``seq_of_token``,
     ``positions``, ``cu_q``, ``q_pos0`` and the host list ``q_lens``.  ``kernel`` picks a
-    form ("mma", "general"); None takes the tensor-core form where it applies."""
+    form ("mma", "general"); None takes the tensor-core form where it applies.  With
+    ``fp32_weights`` the tensor-core form keeps 16 bits of a softmax weight in its product
+    with the latents (two bfloat16 terms) instead of 8; the general form is fp32 anyway."""
     _chk("q_lat", q_lat)
     _chk("q_rot", q_rot, q_lat.dtype)
     _chk("cache", cache, q_lat.dtype)
@@ -1466,7 +1514,8 @@ def latent_attention(q_lat: torch.Tensor, q_rot: torch.Tensor, cache: torch.Tens
             _ptr(cache), _ptr(block_table), block_table.shape[1], _ptr(step.cu_q),
             _ptr(step.q_pos0), S, _ptr(out), ctypes.c_longlong(T * rank),
             ctypes.c_longlong(rank), T, H, rank, dr, page, window, ctypes.c_float(scale), tiles,
-            rows, ct.value, nchunks, _ptr(part_o), _ptr(part_ml), _stream()), "latent_attention (mma)")
+            rows, ct.value, nchunks, _ptr(part_o), _ptr(part_ml), 1 if fp32_weights else 0,
+            _stream()), "latent_attention (mma)")
         if ct.value > 0:
             _count()
         _count()
@@ -1566,7 +1615,7 @@ def add_rmsnorm_sum(resid: torch.Tensor, terms, vector: Optional[torch.Tensor], 
         _ptr(outs[0]), _ptr(outs[1] if len(outs) > 1 else None), _dtype_code(outs[0]), R, W,
         ctypes.c_float(eps), 1 if rows is None else 0,
         _ptr(combine.y if combine else None), _ptr(combine.dest if combine else None),
-        _ptr(combine.topk_w if combine else None), _ptr(combine.shared if combine else None),
+        _ptr(combine.weights if combine else None), _ptr(combine.shared if combine else None),
         _ptr(combine.shared_logit if combine else None),
         combine.topk_w.shape[1] if combine else 0, _stream()), "add_rmsnorm_sum")
     _count()
@@ -2126,3 +2175,236 @@ def identity_rows(x: torch.Tensor, rows: torch.Tensor, offsets: torch.Tensor,
                                    x.shape[1], _stream()), "identity_rows")
     _count()
     return y
+
+
+# ---------------------------------------------------------------------------
+# Parts of decoders that pair chunked attention and a gated recurrence, whose latent queries
+# have a latent of their own and whose logits are squashed
+# ---------------------------------------------------------------------------
+def append_kv_rows(k: torch.Tensor, v: torch.Tensor, k_cache: torch.Tensor,
+                   v_cache: torch.Tensor, slots: torch.Tensor):
+    """Key and value rows of a projection (views of its columns: [T, kv_heads * head size])
+    into the pages at ``slots``; value heads may have a size of their own."""
+    _chk("k_cache", k_cache, k.dtype)
+    _chk("v_cache", v_cache, k.dtype)
+    _chk("slots", slots, torch.int32)
+    P, kvh, page, hd = k_cache.shape
+    vd = v_cache.shape[3]
+    if tuple(v_cache.shape[:3]) != (P, kvh, page) or v.dtype != k.dtype:
+        raise KernelError("append_kv_rows: key and value pages disagree")
+    k_ld, v_ld = _row_view("k", k, kvh * hd), _row_view("v", v, kvh * vd)
+    T = k.shape[0]
+    if v.shape[0] != T or slots.numel() != T:
+        raise KernelError("append_kv_rows: one slot per row")
+    _check(_lib().ix_append_kv_rows(
+        _ptr(k), ctypes.c_longlong(k_ld), _ptr(v), ctypes.c_longlong(v_ld), _ptr(slots),
+        _ptr(k_cache), _ptr(v_cache), _dtype_code(k), T, kvh, hd, vd, page, _stream()),
+        "append_kv_rows")
+    _count()
+
+
+def distance_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
+                       block_table: torch.Tensor, step, scale: float, temp: torch.Tensor,
+                       r1: torch.Tensor, r2: torch.Tensor, chunk: int, out: torch.Tensor,
+                       out_scale: float = 1.0, kernel: Optional[str] = None):
+    """Causal attention of this step's queries over the paged cache with scores
+    (q . k) * scale * temp_h - r1_h ln(1 + r2_h distance), the keys of a query's own run of
+    ``chunk`` positions only (0: all).  ``q`` [T, heads * head size] and ``out`` [T, heads *
+    value size] are views of columns; ``out`` receives the result times ``out_scale``.
+    Scores, penalties and weights are fp32 arithmetic; in bfloat16 with heads of 64 or 128
+    the tensor-core kernels run, in which a weight keeps 16 bits in its product with the
+    values.  ``kernel`` picks a form: "tc", "mma" (both for ragged batches), "decode"
+    (tensor cores), "tiled", "decode_any", "generic" (CUDA cores, any element type)."""
+    _chk("k_cache", k_cache, q.dtype)
+    _chk("v_cache", v_cache, q.dtype)
+    _chk("block_table", block_table, torch.int32)
+    P, kvh, page, hd = k_cache.shape
+    vd = v_cache.shape[3]
+    heads = temp.numel()
+    for name, t in (("temp", temp), ("r1", r1), ("r2", r2)):
+        _chk(name, t, torch.float32)
+        if t.numel() != heads:
+            raise KernelError("distance_attention: temp, r1 and r2 have one number per head")
+    if tuple(v_cache.shape[:3]) != (P, kvh, page) or heads % kvh or out.dtype != q.dtype:
+        raise KernelError("distance_attention: heads and cache disagree")
+    q_ld, o_ld = _row_view("q", q, heads * hd), _row_view("out", out, heads * vd)
+    T, S = q.shape[0], step.num_seqs
+    lib = _lib()
+    bf = q.dtype == torch.bfloat16
+    wide = bf and q_ld % 8 == 0 and o_ld % 8 == 0 and (q.data_ptr() | out.data_ptr()) % 16 == 0
+    tc_sizes = wide and bool(lib.ix_paged_attention_prefill_exact_applies(hd, vd))
+    if kernel is None:
+        nd = int(getattr(step, "num_decode_seqs", 0))
+        if tc_sizes and 0 < nd < S and step.cu_q_prompt is not None:
+            # a mixed batch: its single tokens come first and go to the split-KV kernel
+            _distance_kernel("decode", q[:nd], k_cache, v_cache, block_table[:nd], step, nd, nd,
+                             None, None, step.kv_len[:nd], scale, temp, r1, r2, chunk, out[:nd],
+                             out_scale, q_ld, o_ld)
+            form = "tc" if USE_TCGEN05_ATTENTION and lib.ix_paged_attention_prefill_tc_exact_applies(
+                hd, vd, page) else "mma"
+            _distance_kernel(form, q[nd:], k_cache, v_cache, block_table[nd:], step, T - nd, S - nd,
+                             step.cu_q_prompt, step.q_pos0[nd:], None, scale, temp, r1, r2, chunk,
+                             out[nd:], out_scale, q_ld, o_ld)
+            return out
+        if step.all_decode and T == S:
+            kernel = ("decode" if tc_sizes else
+                      "decode_any" if step.max_kv_len >= DECODE_ANY_MIN_KEYS else "generic")
+        elif tc_sizes:
+            kernel = ("tc" if USE_TCGEN05_ATTENTION
+                      and lib.ix_paged_attention_prefill_tc_exact_applies(hd, vd, page) else "mma")
+        elif (T >= TILED_ATTENTION_MIN_QUERIES * S and lib.ix_paged_attention_tiled_applies(hd)
+              and lib.ix_paged_attention_tiled_applies(vd) and q_ld % 4 == 0 and o_ld % 4 == 0
+              and (q.data_ptr() | out.data_ptr()) % (4 * q.element_size()) == 0):
+            kernel = "tiled"
+        else:
+            kernel = "generic"
+    _distance_kernel(kernel, q, k_cache, v_cache, block_table, step, T, S, step.cu_q, step.q_pos0,
+                     step.kv_len, scale, temp, r1, r2, chunk, out, out_scale, q_ld, o_ld)
+    return out
+
+
+def _distance_kernel(kernel, q, k_cache, v_cache, block_table, step, T, S, cu_q, q_pos0, kv_len,
+                     scale, temp, r1, r2, chunk, out, out_scale, q_ld, o_ld):
+    lib = _lib()
+    P, kvh, page, hd = k_cache.shape
+    vd, heads, maxb = v_cache.shape[3], temp.numel(), block_table.shape[1]
+    ll, f = ctypes.c_longlong, ctypes.c_float
+    vectors = (_ptr(temp), _ptr(r1), _ptr(r2), int(chunk))
+    launches = 1
+    if kernel == "generic":
+        code = lib.ix_distance_attention_generic(
+            _ptr(q), ll(q_ld), _ptr(k_cache), _ptr(v_cache), _ptr(block_table),
+            _ptr(step.seq_of_token), _ptr(step.positions), _ptr(out), ll(o_ld), f(out_scale),
+            _dtype_code(q), T, heads, kvh, hd, vd, page, maxb, f(scale), *vectors, _stream())
+    elif kernel == "tiled":
+        code = lib.ix_distance_attention_tiled(
+            _ptr(q), ll(q_ld), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), _ptr(cu_q),
+            _ptr(q_pos0), _ptr(out), ll(o_ld), f(out_scale), _dtype_code(q), T, S, heads, kvh, hd,
+            vd, page, maxb, f(scale), *vectors, _stream())
+    elif kernel == "mma":
+        code = lib.ix_distance_attention_prefill_exact(
+            _ptr(q), ll(q_ld), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), _ptr(cu_q),
+            _ptr(q_pos0), _ptr(out), ll(o_ld), f(out_scale), T, S, heads, kvh, hd, vd, page, maxb,
+            f(scale), *vectors, _stream())
+    elif kernel == "tc":
+        code = lib.ix_distance_attention_prefill_tc(
+            _ptr(q), ll(q_ld), _ptr(k_cache), _ptr(v_cache), P, _ptr(block_table), _ptr(cu_q),
+            _ptr(q_pos0), _ptr(out), ll(o_ld), f(out_scale), T, S, heads, kvh, hd, page, maxb,
+            f(scale), *vectors, _ptr(_tc_status(q.device)), _stream())
+    elif kernel in ("decode", "decode_any"):
+        span = min(int(step.max_kv_len), chunk) if chunk > 0 else int(step.max_kv_len)
+        if kernel == "decode":
+            splits = lib.ix_attn_decode_splits(S, heads, kvh, span)
+        else:
+            splits = lib.ix_attn_decode_any_splits(S, heads, kvh, hd, vd, span)
+        part_o = part_ml = None
+        if splits > 1:
+            part_o = torch.empty((S, heads, splits, vd), dtype=torch.float32, device=q.device)
+            part_ml = torch.empty((S, heads, splits, 2), dtype=torch.float32, device=q.device)
+            launches = 2
+        if kernel == "decode":
+            code = lib.ix_distance_attention_decode_exact(
+                _ptr(q), ll(q_ld), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), _ptr(kv_len),
+                _ptr(part_o), _ptr(part_ml), _ptr(out), ll(o_ld), f(out_scale), S, heads, kvh, hd,
+                vd, page, maxb, f(scale), splits, *vectors, _stream())
+        else:
+            code = lib.ix_distance_attention_decode_any(
+                _ptr(q), ll(q_ld), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), _ptr(kv_len),
+                _ptr(part_o), _ptr(part_ml), _ptr(out), ll(o_ld), f(out_scale), _dtype_code(q), S,
+                heads, kvh, hd, vd, page, maxb, f(scale), splits, *vectors, _stream())
+    else:
+        raise KernelError(f"distance_attention: no kernel form {kernel!r}")
+    _check(code, f"distance_attention ({kernel})")
+    _count(launches)
+
+
+def min_gru(front: torch.Tensor, z_bias: torch.Tensor, x_bias: torch.Tensor, shift: float,
+            state: torch.Tensor, step, out: torch.Tensor, out_scale: float = 1.0):
+    """z = sigmoid(a + z_bias), u = x + x_bias, c = u + shift (u >= 0) or sigmoid(u) (u < 0);
+    S_t = (1 - z) S_(t-1) + z c along each sequence, entry by entry, from and back to
+    ``state`` [slots, W] (fp32); out = S * silu(g) * out_scale.  ``front`` [T, a | x | g] and
+    ``out`` [T, W] are views of columns."""
+    _chk("z_bias", z_bias, torch.float32)
+    _chk("x_bias", x_bias, torch.float32)
+    _chk("state", state, torch.float32)
+    _chk("cu_q", step.cu_q, torch.int32)
+    _chk("state_slot", step.state_slot, torch.int32)
+    W = z_bias.numel()
+    if x_bias.numel() != W or state.shape[1:] != (W,) or out.dtype != front.dtype:
+        raise KernelError("min_gru: biases, state and rows disagree")
+    ld, o_ld = _row_view("front", front, 3 * W), _row_view("out", out, W)
+    singles = int(getattr(step, "num_decode_seqs", 0))
+    if step.all_decode:
+        singles = step.num_seqs
+    _check(_lib().ix_min_gru(
+        _ptr(front), ctypes.c_longlong(ld), _ptr(z_bias), _ptr(x_bias), ctypes.c_float(shift),
+        _ptr(state), _ptr(step.state_slot), _ptr(step.cu_q), _ptr(out), ctypes.c_longlong(o_ld),
+        ctypes.c_float(out_scale), _dtype_code(front), step.num_seqs, singles, W, _stream()),
+        "min_gru")
+    _count(2 if 0 < singles < step.num_seqs else 1)
+    return out
+
+
+def latent_front(proj: torch.Tensor, q_rank: int, q_gain: torch.Tensor, eps: float, kv_off: int,
+                 positions: torch.Tensor, freq: torch.Tensor, mag: float,
+                 kv_gain: Optional[torch.Tensor], rank: int, rot_dim: int, rot_dims: int,
+                 cache: Optional[torch.Tensor], slots: Optional[torch.Tensor]):
+    """From a product that makes the queries' latent (columns 0 .. q_rank) beside the
+    down-projection (columns from ``kv_off`` on): the RMS-normed query latent [T, q_rank], and
+    the record [normed latent | rotated key part] into ``cache`` at ``slots`` (no cache: the
+    product has no down-projection)."""
+    _chk("proj", proj)
+    _chk("q_gain", q_gain, torch.float32)
+    _chk("positions", positions, torch.int32)
+    _chk("freq", freq, torch.float32)
+    _chk("kv_gain", kv_gain, torch.float32, optional=True)
+    _chk("cache", cache, proj.dtype, optional=True)
+    _chk("slots", slots, torch.int32, optional=True)
+    T, ld = proj.shape
+    if q_gain.numel() != q_rank or freq.numel() * 2 != rot_dims:
+        raise KernelError("latent_front: one gain per query latent entry, one frequency per pair")
+    if cache is not None and (cache.shape[1] != 1 or cache.shape[3] != rank + rot_dim
+                              or kv_gain is None or kv_gain.numel() != rank or slots is None
+                              or slots.numel() != T):
+        raise KernelError("latent_front: cache records must be [1, page, rank + rot_dim], with "
+                          "one gain per latent entry and one slot per row")
+    c_q = torch.empty((T, q_rank), dtype=proj.dtype, device=proj.device)
+    _check(_lib().ix_latent_front(
+        _ptr(proj), ctypes.c_longlong(ld), q_rank, _ptr(q_gain), kv_off, _ptr(positions),
+        _ptr(freq), ctypes.c_float(mag), _ptr(kv_gain), ctypes.c_float(eps), _ptr(slots),
+        _ptr(cache), _ptr(c_q), _dtype_code(proj), T, rot_dim, rot_dims, rank, _stream()),
+        "latent_front")
+    _count()
+    return c_q
+
+
+def latent_queries(q: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor, mag: float,
+                   heads: int, dim: int, rot_dim: int, rot_dims: int):
+    """Head by head [dim plain | rot_dim rotated] queries, split: the rotated parts turned,
+    [T, heads, rot_dim], and the plain ones heads outermost, [heads, T, dim]."""
+    _chk("q", q)
+    _chk("positions", positions, torch.int32)
+    _chk("freq", freq, torch.float32)
+    T, ld = q.shape
+    if heads * (dim + rot_dim) > ld or freq.numel() * 2 != rot_dims:
+        raise KernelError("latent_queries: rows narrower than the heads, or not one frequency "
+                          "per rotated pair")
+    q_rot = torch.empty((T, heads, rot_dim), dtype=q.dtype, device=q.device)
+    q_plain = torch.empty((heads, T, dim), dtype=q.dtype, device=q.device)
+    _check(_lib().ix_latent_prepare(
+        _ptr(q), ctypes.c_longlong(ld), 0, 0, _ptr(positions), _ptr(freq), ctypes.c_float(mag),
+        _ptr(None), ctypes.c_float(1.0), _ptr(None), _ptr(None), _ptr(q_rot), _ptr(q_plain),
+        _dtype_code(q), T, heads, dim, rot_dim, rot_dims, 1, _stream()), "latent_queries")
+    _count()
+    return q_rot, q_plain
+
+
+def softcap_rows(x: torch.Tensor, cap: float):
+    """x <- cap * tanh(x / cap), fp32, in place."""
+    _chk("x", x, torch.float32)
+    if not cap > 0:
+        raise KernelError(f"softcap_rows: cap {cap} must be positive")
+    _check(_lib().ix_softcap_rows(_ptr(x), ctypes.c_longlong(x.numel()), ctypes.c_float(cap),
+                                  _stream()), "softcap_rows")
+    _count()
+    return x
