@@ -1,0 +1,297 @@
+"""The Dominex design on the GPU: every new kernel and kernel option alone against its plain
+statement (tests/host_ops.py), then the engine against the plain model
+(tests/plain_dominex.py): whole prompts, prefill against token-by-token decoding, portions
+down to two tokens, unequal batches with pages and slots used again, long decoding with
+recorded steps over the borders of runs, and greedy generation through the engine's own
+entry point."""
+import json
+import math
+import os
+import subprocess
+import sys
+from types import SimpleNamespace
+
+import numpy as np
+import pytest
+import torch
+
+import dominex_cases as dk
+import host_ops
+import model_cases as mc
+import plain_dominex as plain
+import traces
+from conftest import ROOT
+from inferx_b200.engine.replay import ReplaySession
+
+pytestmark = pytest.mark.gpu
+
+DTYPES = [torch.float32, torch.bfloat16]
+CASES = [("DA", dk.DA, 0, [5, 9, 27, 44, 3, 60], 4), ("DB", dk.DB, 1, [1, 6, 13, 31, 45], 8),
+         ("DC", dk.DC, 3, [21, 1, 50, 2, 110], 16)]
+
+
+def _ops():
+    from inferx_b200.kernels import ops
+    return ops
+
+
+def _tol(dtype):
+    return dict(rtol=2e-5, atol=2e-5) if dtype == torch.float32 else dict(rtol=1.6e-2, atol=1.6e-2)
+
+
+def _step(q_lens, starts, slots=None):
+    """A batch description: sequence s brings q_lens[s] tokens from position starts[s];
+    single tokens come first."""
+    assert list(q_lens) == sorted(q_lens, key=lambda n: n != 1), "single tokens come first"
+    seq_of, pos, cu = [], [], [0]
+    for s, (n, a) in enumerate(zip(q_lens, starts)):
+        seq_of += [s] * n
+        pos += list(range(a, a + n))
+        cu.append(cu[-1] + n)
+    nd = sum(1 for n in q_lens if n == 1)
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32)
+    return SimpleNamespace(
+        seq_of_token=i32(seq_of), positions=i32(pos), cu_q=i32(cu), q_pos0=i32(list(starts)),
+        q_lens=list(q_lens), num_seqs=len(q_lens), num_tokens=len(seq_of),
+        kv_len=i32([a + n for n, a in zip(q_lens, starts)]),
+        max_kv_len=max(a + n for n, a in zip(q_lens, starts)), max_q_len=max(q_lens),
+        all_decode=nd == len(q_lens), num_decode_seqs=nd, cu_q_prompt=i32([c - nd for c in cu[nd:]]),
+        state_slot=i32(slots if slots is not None else list(range(len(q_lens)))))
+
+
+def _cuda(ns):
+    return SimpleNamespace(**{k: (v.cuda() if torch.is_tensor(v) else v)
+                              for k, v in vars(ns).items()})
+
+
+def _kv_case(seed, H, G, D, VD, page, q_lens, starts, dtype, chunk=0):
+    """(step, block table, key pages, value pages, q rows): pages in a shuffled order, those
+    that hold no key a query of this step can see given back."""
+    g = torch.Generator().manual_seed(seed)
+    step = _step(q_lens, starts)
+    S = len(q_lens)
+    need = [-(-(a + n) // page) for n, a in zip(q_lens, starts)]
+    total = sum(need) + 3
+    perm = torch.randperm(total, generator=g).to(torch.int32)
+    bt = torch.full((S, max(need)), -1, dtype=torch.int32)
+    at = 0
+    for s, n in enumerate(need):
+        bt[s, :n] = perm[at:at + n]
+        at += n
+        if chunk > 0:
+            bt[s, :starts[s] // chunk * chunk // page] = -1
+    kc = (torch.randn(total, G, page, D, generator=g) * 0.4).to(dtype)
+    vc = torch.randn(total, G, page, VD, generator=g).to(dtype)
+    q = (torch.randn(sum(q_lens), H * D, generator=g) * 0.4).to(dtype)
+    return step, bt, kc, vc, q
+
+
+def _head_vectors(H, seed):
+    g = torch.Generator().manual_seed(seed)
+    return (0.5 + torch.rand(H, generator=g), torch.rand(H, generator=g) * 1.5,
+            torch.rand(H, generator=g) * 0.6)
+
+
+def _wide(t, lead, tail, seed=0):
+    """``t`` as a view of columns of a wider tensor on the device."""
+    w = torch.randn(t.shape[0], lead + t.shape[1] + tail,
+                    generator=torch.Generator().manual_seed(seed)).to(t.dtype)
+    w[:, lead:lead + t.shape[1]] = t
+    return w.cuda()[:, lead:lead + t.shape[1]]
+
+
+# -- kernels alone -------------------------------------------------------------------
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("G,D,VD,page,lead", [(2, 16, 24, 4, 8), (1, 7, 9, 8, 3), (3, 64, 128, 16, 0),
+                                              (2, 64, 64, 16, 5)])
+def test_key_and_value_rows_into_pages(dtype, G, D, VD, page, lead):
+    g = torch.Generator().manual_seed(G * D)
+    T, pages = 13, 6
+    k, v = (torch.randn(T, G * n, generator=g).to(dtype) for n in (D, VD))
+    slots = torch.randperm(pages * page, generator=g)[:T].to(torch.int32)
+    kc, vc = (torch.zeros(pages, G, page, n, dtype=dtype) for n in (D, VD))
+    dk_, dv_ = kc.cuda(), vc.cuda()
+    host_ops.append_kv_rows(k, v, kc, vc, slots)
+    _ops().append_kv_rows(_wide(k, lead, 16), _wide(v, lead, 8, 1), dk_, dv_, slots.cuda())
+    assert torch.equal(dk_.cpu(), kc) and torch.equal(dv_.cpu(), vc)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("W,lead", [(31, 3), (56, 8), (16, 0), (384, 4), (2050, 2)])
+@pytest.mark.parametrize("q_lens", [[1, 1, 1], [1, 1, 3, 40, 2], [700], [9, 520, 1025]])
+def test_gated_recurrence(dtype, W, lead, q_lens):
+    """Single tokens, portions shorter and longer than a stretch of the walk, and both kinds
+    in one batch; the state comes from and goes back to each sequence's slot."""
+    g = torch.Generator().manual_seed(W + len(q_lens))
+    T, S = sum(q_lens), len(q_lens)
+    front = (torch.randn(T, 3 * W, generator=g) * 2.0).to(dtype)
+    zb, xb = torch.randn(W, generator=g) - 1.5, torch.randn(W, generator=g)
+    slots = torch.randperm(S + 2, generator=g)[:S].tolist()
+    step = _step(q_lens, [5] * S, slots)
+    state = torch.randn(S + 2, W, generator=g)
+    ref_state, dev_state = state.clone(), state.cuda()
+    ref = host_ops.min_gru(front, zb, xb, 0.5, ref_state, step, torch.empty(T, W), 1.3)
+    wide = torch.full((T, W + 2 * lead + 2), 7.0, dtype=dtype, device="cuda")
+    off = 2 * lead
+    _ops().min_gru(_wide(front, off, 6), zb.cuda(), xb.cuda(), 0.5, dev_state, _cuda(step),
+                   wide[:, off:off + W], 1.3)
+    torch.testing.assert_close(wide[:, off:off + W].float().cpu(), ref, **_tol(dtype))
+    tol = 3e-5 if dtype == torch.float32 else 1e-4
+    torch.testing.assert_close(dev_state.cpu(), ref_state, rtol=tol, atol=tol)
+    others = [i for i in range(S + 2) if i not in slots]
+    assert torch.equal(dev_state.cpu()[others], state[others])
+    assert bool((wide[:, :off] == 7).all()) and bool((wide[:, off + W:] == 7).all())
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_gated_recurrence_carries_what_was_written_far_back(dtype):
+    """Gates that are almost shut after the first token: its candidate must survive a thousand
+    tokens of a walk in pieces, and a cut anywhere gives the same state."""
+    W, n = 40, 1300
+    front = torch.zeros(n, 3 * W)
+    front[:, :W] = -14.0
+    front[0, :W] = 14.0
+    front[:, W:2 * W] = -3.0
+    front[0, W:2 * W] = torch.linspace(1.0, 50.0, W)
+    front[:, 2 * W:] = 2.0
+    front = front.to(dtype)
+    zero = torch.zeros(W)
+    finals = []
+    for cuts in ([n], [1, n - 1], [2, 511, 514, n - 1027], [700, 600]):
+        state, out, at = torch.zeros(1, W).cuda(), torch.empty(n, W, dtype=dtype, device="cuda"), 0
+        for c in cuts:
+            _ops().min_gru(front[at:at + c].cuda(), zero.cuda(), zero.cuda(), 0.5, state,
+                           _cuda(_step([c], [at])), out[at:at + c], 1.0)
+            at += c
+        finals.append((state.cpu(), out.float().cpu()))
+    ref_state = torch.zeros(1, W)
+    ref = host_ops.min_gru(front, zero, zero, 0.5, ref_state, _step([n], [0]), torch.empty(n, W))
+    assert float(ref_state.max()) > 40.0
+    for st, out in finals:
+        torch.testing.assert_close(st, ref_state, rtol=1e-4, atol=1e-4)
+        torch.testing.assert_close(out, ref, **_tol(dtype))
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("q_rank,rank,dr,rot,own", [(28, 24, 8, 8, True), (9, 11, 2, 2, True),
+                                                    (1536, 512, 64, 64, True), (112, 0, 0, 0, False),
+                                                    (20, 16, 6, 4, True)])
+def test_query_latent_and_record(dtype, q_rank, rank, dr, rot, own):
+    g = torch.Generator().manual_seed(q_rank)
+    T, page, pages = 7, 4, 5
+    proj = (torch.randn(T, q_rank + rank + dr + 3, generator=g) * 2.0).to(dtype)
+    qg = 1.0 + 0.3 * torch.randn(q_rank, generator=g)
+    kg = 1.0 + 0.3 * torch.randn(max(rank, 1), generator=g)
+    pos = torch.tensor([0, 1, 2, 900, 901, 65, 7], dtype=torch.int32)
+    freq = torch.rand(rot // 2, generator=g)
+    slots = torch.randperm(page * pages, generator=g)[:T].to(torch.int32)
+    cache = torch.zeros(pages, 1, page, rank + dr, dtype=dtype) if own else None
+    dev = cache.cuda() if own else None
+    args = (q_rank, qg, 1e-5, q_rank, pos, freq, 1.0, kg if own else None, rank, dr, rot)
+    ref = host_ops.latent_front(proj, *args, cache, slots if own else None)
+    out = _ops().latent_front(proj.cuda(), *[a.cuda() if torch.is_tensor(a) else a for a in args],
+                              dev, slots.cuda() if own else None)
+    torch.testing.assert_close(out.cpu().float(), ref.float(), **_tol(dtype))
+    if own:
+        torch.testing.assert_close(dev.cpu().float(), cache.float(), **_tol(dtype))
+    # the queries a latent is widened to, split and turned
+    H, dim = 3, 5
+    rd = max(rot, 2)
+    q = torch.randn(T, H * (dim + rd), generator=g).to(dtype)
+    f2 = torch.rand(rd // 2, generator=g)
+    want = host_ops.latent_queries(q, pos, f2, 1.0, H, dim, rd, rd)
+    got = _ops().latent_queries(q.cuda(), pos.cuda(), f2.cuda(), 1.0, H, dim, rd, rd)
+    for a, b in zip(got, want):
+        torch.testing.assert_close(a.cpu().float(), b.float(), **_tol(dtype))
+
+
+@pytest.mark.parametrize("n", [1, 640, 3 * 509])
+def test_squashed_logits(n):
+    x = torch.randn(3, n, generator=torch.Generator().manual_seed(n)) * 40.0
+    want = host_ops.softcap_rows(x.clone(), 15.0)
+    got = _ops().softcap_rows(x.cuda(), 15.0).cpu()
+    torch.testing.assert_close(got, want, rtol=1e-5, atol=1e-5)
+    assert float(got.abs().max()) <= 15.0
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("T", [3, 130, 1500])
+@pytest.mark.parametrize("E,k", [(2, 2), (16, 1), (60, 4), (130, 6)])
+def test_sigmoid_router(dtype, T, E, k):
+    g = torch.Generator().manual_seed(E + T)
+    x = torch.randn(T, 64, generator=g).to(dtype)
+    w = torch.randn(E, 64, generator=g) * 0.3
+    tw, ti, _ = _ops().router_topk(x.cuda(), w.cuda(), k, False, 1.0, score="sigmoid")
+    logits = x.double() @ w.double().T
+    want, _ = torch.sort(torch.sigmoid(logits), dim=-1, descending=True)
+    torch.testing.assert_close(tw.cpu(), want[:, :k].float(), rtol=1e-4, atol=1e-5)
+    torch.testing.assert_close(torch.sigmoid(torch.gather(logits, 1, ti.cpu().long())).float(),
+                               tw.cpu(), rtol=1e-4, atol=1e-5)
+    assert all(len(set(r)) == k for r in ti.cpu().tolist())
+
+
+def test_sigmoid_router_orders_saturated_scores_by_their_logits():
+    """Scores that are all one in fp32 are still chosen by the larger logit."""
+    E = 40
+    w = torch.zeros(E, 32)
+    w[:, 0] = torch.linspace(20.0, 60.0, E)[torch.randperm(E, generator=torch.Generator().manual_seed(1))]
+    x = torch.zeros(200, 32)
+    x[:, 0] = 1.0
+    for rows in (4, 200):
+        tw, ti, _ = _ops().router_topk(x[:rows].cuda(), w.cuda(), 3, False, 1.0, score="sigmoid")
+        want = torch.topk(w[:, 0], 3).indices.tolist()
+        assert all(r == want for r in ti.cpu().tolist()) and bool((tw == 1.0).all())
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("T,E,k,H,I", [(1, 8, 2, 256, 64), (3, 6, 2, 64, 32), (40, 5, 3, 72, 40),
+                                       (130, 4, 2, 128, 96), (700, 16, 1, 256, 64), (9, 3, 3, 45, 21)])
+def test_weights_on_the_experts_inputs(dtype, T, E, k, H, I):
+    """Dispatch with the weights of the grouped rows, gate/up product with a factor per row,
+    plain sum of the experts' rows: every kernel that serves the product."""
+    g = torch.Generator().manual_seed(T)
+    ops = _ops()
+    x = torch.randn(T, H, generator=g).to(dtype)
+    gu = (torch.randn(E, 2 * I, H, generator=g) / math.sqrt(H) * 2.0).to(dtype)
+    dn = (torch.randn(E, H, I, generator=g) / math.sqrt(I)).to(dtype)
+    idx = torch.stack([torch.randperm(E, generator=g)[:k] for _ in range(T)]).to(torch.int32)
+    tw = torch.rand(T, k, generator=g)
+    ro, rr, rd, rw = host_ops.moe_dispatch(idx, E, topk_w=tw)
+    do, dr, dd, dw = ops.moe_dispatch(idx.cuda(), E, topk_w=tw.cuda())
+    for a, b in ((do, ro), (dr, rr), (dd, rd), (dw, rw)):
+        assert torch.equal(a.cpu(), b)
+    want = host_ops.grouped_gate_up_swiglu(x.float(), rr, ro, gu.float(), row_scale=rw)
+    got = ops.grouped_gate_up_swiglu(x.cuda(), dr, do, gu.cuda(), row_scale=dw)
+    torch.testing.assert_close(got.float().cpu(), want, **_tol(dtype))
+    # the weight went in ahead of the activation, not behind it
+    behind = host_ops.grouped_gate_up_swiglu(x.float(), rr, ro, gu.float()) * rw[:, None]
+    assert float((behind - want).abs().max()) > 0.05
+    forms = [lambda: ops.gemm_generic(x.cuda(), gu.cuda(), dr, do, dual=True,
+                                      num_out_rows=T * k, row_scale=dw)]
+    if dtype == torch.bfloat16 and H % 8 == 0:
+        forms += [lambda: ops.gemm_small_m(x.cuda(), gu.cuda(), dr, do, True, T * k, row_scale=dw),
+                  lambda: ops.gemm_small_m(x.cuda(), gu.cuda(), dr, do, True, T * k,
+                                           rows_per_pass=16, row_scale=dw),
+                  lambda: ops.grouped_gemm_tc(ops.gather_rows(x.cuda(), dr), do, gu.cuda(), True,
+                                              row_scale=dw)]
+        if H >= 256:
+            forms += [lambda: ops.gemm_stream_grouped(x.cuda(), gu.cuda(), dr, do, True, T * k,
+                                                      row_scale=dw)]
+    for form in forms:
+        torch.testing.assert_close(form().float().cpu(), want, **_tol(dtype))
+    ops.check_async_errors()
+    y = ops.grouped_down(got, do, dn.cuda())
+    plain_sum = ops.moe_combine(y, dd, tw.cuda(), None, None, weighted=False).float().cpu()
+    ref = torch.zeros(T, H)
+    for s in range(k):
+        ref += y.float().cpu()[rd.view(T, k)[:, s].long()]
+    torch.testing.assert_close(plain_sum, ref, **_tol(dtype))
+    gain = 1.0 + 0.1 * torch.randn(H, generator=g)
+    for fn in (lambda r, p: ops.add_rmsnorm(r, p, gain.cuda(), 1e-5, dtype),
+               lambda r, p: ops.add_rmsnorm_sum(r, [p], None, (gain.cuda(),), 1e-5, dtype)[0]):
+        resid = torch.randn(T, H, generator=g)
+        dev = resid.cuda()
+        n = fn(dev, ops.moe_combine_pending(y, dd, tw.cuda(), None, None, weighted=False))
+        torch.testing.assert_close(dev.cpu(), resid + ref, rtol=2e-2, atol=2e-2)
+        torch.testing.assert_close(n.float().cpu(), host_ops.add_rmsnorm(
+            (resid + ref).clone(), None, gain, 1e-5, torch.float32), rtol=3e-2, atol=3e-2)
