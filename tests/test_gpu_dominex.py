@@ -167,9 +167,11 @@ def test_gated_recurrence_carries_what_was_written_far_back(dtype):
     ref_state = torch.zeros(1, W)
     ref = host_ops.min_gru(front, zero, zero, 0.5, ref_state, _step([n], [0]), torch.empty(n, W))
     assert float(ref_state.max()) > 40.0
+    # 1 - z of a gate of 8e-7 is rounded to fp32 at every token: n * 2^-25 in all
+    tol = dict(rtol=1e-4, atol=1e-4) if dtype == torch.float32 else _tol(dtype)
     for st, out in finals:
         torch.testing.assert_close(st, ref_state, rtol=1e-4, atol=1e-4)
-        torch.testing.assert_close(out, ref, **_tol(dtype))
+        torch.testing.assert_close(out, ref, **tol)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -295,3 +297,79 @@ def test_weights_on_the_experts_inputs(dtype, T, E, k, H, I):
         torch.testing.assert_close(dev.cpu(), resid + ref, rtol=2e-2, atol=2e-2)
         torch.testing.assert_close(n.float().cpu(), host_ops.add_rmsnorm(
             (resid + ref).clone(), None, gain, 1e-5, torch.float32), rtol=3e-2, atol=3e-2)
+
+
+def _forms(dtype, D, VD, page, ragged):
+    tensor = dtype == torch.bfloat16 and D in (64, 128) and VD in (64, 128)
+    if not ragged:
+        return ["generic", "decode_any"] + (["decode"] if tensor else [])
+    out = ["generic"]
+    if D % 4 == 0 and VD % 4 == 0:
+        out.append("tiled")
+    if tensor:
+        out.append("mma")
+        if D == VD and page in (8, 16, 32, 64):
+            out.append("tc")
+    return out
+
+
+def _distance(form, q, kc, vc, bt, step, scale, vec, chunk, VD, out_scale=1.0, lead=8):
+    """One kernel form on views of columns; returns [T, heads * VD] on the host."""
+    T, H = q.shape[0], vec[0].numel()
+    wide = torch.full((T, lead + H * VD + 16), 5.0, dtype=q.dtype, device="cuda")
+    out = wide[:, lead:lead + H * VD]
+    _ops().distance_attention(_wide(q, lead, 24), kc.cuda(), vc.cuda(), bt.cuda(), _cuda(step),
+                              scale, *[v.cuda() for v in vec], chunk, out, out_scale, kernel=form)
+    _ops().check_async_errors()
+    assert bool((wide[:, :lead] == 5).all()) and bool((wide[:, lead + H * VD:] == 5).all())
+    return out.float().cpu()
+
+
+def _reference(q, kc, vc, bt, step, scale, vec, chunk, VD, out_scale=1.0):
+    return host_ops.distance_attention(q.float(), kc.float(), vc.float(), bt, step, scale, *vec,
+                                       chunk, torch.empty(q.shape[0], vec[0].numel() * VD),
+                                       out_scale)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,G,D,VD,page", [(6, 2, 16, 24, 4), (1, 1, 7, 9, 8), (8, 2, 64, 64, 16),
+                                           (4, 4, 128, 128, 16), (16, 1, 64, 128, 16),
+                                           (20, 1, 128, 64, 8), (3, 3, 64, 64, 64)])
+@pytest.mark.parametrize("chunk", [0, 1, 33, 64, 100, 1000])
+def test_distance_attention_of_portions(dtype, H, G, D, VD, page, chunk):
+    """Ragged portions that start anywhere and cross the borders of runs, over pages of which
+    those before the run were given back; every form that takes the sizes."""
+    q_lens, starts = [5, 150, 2, 70], [96, 31, 199, 0]
+    step, bt, kc, vc, q = _kv_case(H * D + chunk, H, G, D, VD, page, q_lens, starts, dtype, chunk)
+    vec = _head_vectors(H, H)
+    ref = _reference(q, kc, vc, bt, step, D ** -0.5, vec, chunk, VD, 0.7)
+    for form in _forms(dtype, D, VD, page, True) + [None]:
+        got = _distance(form, q, kc, vc, bt, step, D ** -0.5, vec, chunk, VD, 0.7)
+        torch.testing.assert_close(got, ref, **_tol(dtype), msg=lambda m: f"{form}: {m}")
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,G,D,VD,page", [(6, 2, 16, 24, 4), (1, 1, 7, 9, 8), (8, 2, 64, 64, 16),
+                                           (4, 4, 128, 128, 16), (16, 1, 64, 128, 16),
+                                           (20, 1, 128, 64, 8)])
+@pytest.mark.parametrize("chunk", [0, 1, 110, 500])
+def test_distance_attention_of_single_tokens(dtype, H, G, D, VD, page, chunk):
+    """One token a sequence at the first, last and inner places of runs, in splits."""
+    starts = [0, 109, 110, 111, 999, 1000, 730]
+    step, bt, kc, vc, q = _kv_case(H * D + chunk, H, G, D, VD, page, [1] * 7, starts, dtype, chunk)
+    vec = _head_vectors(H, H + 1)
+    ref = _reference(q, kc, vc, bt, step, D ** -0.5, vec, chunk, VD)
+    for form in _forms(dtype, D, VD, page, False) + [None]:
+        got = _distance(form, q, kc, vc, bt, step, D ** -0.5, vec, chunk, VD)
+        torch.testing.assert_close(got, ref, **_tol(dtype), msg=lambda m: f"{form}: {m}")
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("D,VD", [(64, 64), (128, 64), (16, 24)])
+def test_distance_attention_of_a_mixed_batch(dtype, D, VD):
+    step, bt, kc, vc, q = _kv_case(3, 4, 2, D, VD, 16, [1, 1, 1, 40, 3], [50, 0, 129, 100, 62],
+                                   dtype, 48)
+    vec = _head_vectors(4, 9)
+    ref = _reference(q, kc, vc, bt, step, 0.2, vec, 48, VD)
+    got = _distance(None, q, kc, vc, bt, step, 0.2, vec, 48, VD)
+    torch.testing.assert_close(got, ref, **_tol(dtype))
