@@ -373,3 +373,106 @@ def test_distance_attention_of_a_mixed_batch(dtype, D, VD):
     ref = _reference(q, kc, vc, bt, step, 0.2, vec, 48, VD)
     got = _distance(None, q, kc, vc, bt, step, 0.2, vec, 48, VD)
     torch.testing.assert_close(got, ref, **_tol(dtype))
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("D,VD", [(64, 64), (128, 128), (64, 128), (12, 8), (7, 9)])
+@pytest.mark.parametrize("ragged", [True, False])
+def test_a_run_s_first_key_is_seen_and_the_key_before_it_is_not(dtype, D, VD, ragged):
+    """One key that outweighs all others, at the first place of the query's run, directly
+    before it, at page borders and far back: the query's output is that key's value, or
+    holds nothing of it.  The penalty is weak (a far key must still win)."""
+    chunk, page = 110, 16
+    for pos, key, seen in [(219, 110, True), (219, 109, False), (220, 219, False), (220, 220, True),
+                           (221, 220, True), (1099, 990, True), (1099, 989, False),
+                           (329, 256, True), (329, 255, True), (330, 0, False)]:
+        n = 3 if ragged else 1
+        start = pos - n + 1
+        step, bt, kc, vc, q = _kv_case(7, 2, 1, D, VD, page, [n], [start], dtype)
+        kc.mul_(0.05)
+        q.mul_(0.05)
+        u = torch.zeros(D)
+        u[0] = 6.0
+        at = (int(bt[0, key // page]), 0, key % page)
+        kc[at] = u.to(dtype)
+        q[n - 1] = u.repeat(2).to(dtype)
+        vc[at] = 40.0
+        vec = (torch.tensor([1.0, 1.5]), torch.tensor([0.3, 0.02]), torch.tensor([0.2, 0.1]))
+        for form in _forms(dtype, D, VD, page, ragged):
+            got = _distance(form, q, kc, vc, bt, step, 1.0, vec, chunk, VD)[n - 1]
+            if seen:
+                assert float((got - 40.0).abs().max()) < 0.5, (form, pos, key)
+            else:
+                assert float(got.abs().max()) < 10.0, (form, pos, key)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("ragged", [True, False])
+def test_the_penalty_decides_between_equal_keys(dtype, ragged):
+    """All keys alike: the weights are the penalties' alone, (1 + r2 d)^(-r1) normalised, and a
+    negative r1 prefers the far keys."""
+    H, D, page, pos = 4, 64, 16, 300
+    n = 2 if ragged else 1
+    step, bt, kc, vc, q = _kv_case(5, H, 1, D, D, page, [n], [pos - n + 1], dtype)
+    kc.fill_(0.25)
+    q.fill_(0.5)
+    vc.zero_()
+    for p in range(pos + 1):
+        vc[int(bt[0, p // page]), 0, p % page] = p / 64.0
+    vec = (torch.tensor([1.0, 2.0, -1.0, 1.0]), torch.tensor([2.0, 0.5, -1.5, 0.0]),
+           torch.tensor([0.7, 3.0, 0.5, 1.0]))
+    d = torch.arange(pos, -1, -1, dtype=torch.float64)
+    vals = vc[bt[0, torch.arange(pos + 1) // page].long(), 0, torch.arange(pos + 1) % page, 0].double()
+    for form in _forms(dtype, D, D, page, ragged):
+        got = _distance(form, q, kc, vc, bt, step, 0.1, vec, 0, D)[n - 1].view(H, D)
+        for h in range(H):
+            w = (1.0 + float(vec[2][h]) * d) ** (-float(vec[1][h]))
+            want = float((w * vals).sum() / w.sum())
+            tol = 2e-5 if dtype == torch.float32 else 6e-3
+            assert float((got[h] - want).abs().max()) <= tol * max(1.0, abs(want)), (form, h)
+
+
+def test_prompt_forms_do_not_depend_on_the_cut():
+    """The tcgen05 and the tiled form walk key tiles at multiples of 64 of the absolute
+    position.  The tiled form gives the same bits however a sequence was cut; in the tcgen05
+    form a row's running reference moves with its warp's, which changes roundings only."""
+    for dtype, form, D in ((torch.bfloat16, "tc", 128), (torch.float32, "tiled", 40)):
+        step, bt, kc, vc, q = _kv_case(11, 4, 2, D, D, 16, [300], [0], dtype)
+        vec = _head_vectors(4, 2)
+        for chunk in (0, 90):
+            whole = _distance(form, q, kc, vc, bt, step, 0.1, vec, chunk, D)
+            for a, b in ((0, 37), (37, 164), (164, 166), (166, 300)):
+                part = _distance(form, q[a:b], kc, vc, bt, _step([b - a], [a]), 0.1, vec, chunk, D)
+                if form == "tiled":
+                    assert torch.equal(part, whole[a:b]), (chunk, a)
+                else:
+                    torch.testing.assert_close(part, whole[a:b], rtol=8e-3, atol=1e-5)
+                    assert float((part == whole[a:b]).float().mean()) > 0.98
+
+
+@pytest.mark.parametrize("rank,dr", [(64, 16), (128, 32), (256, 64), (512, 64)])
+@pytest.mark.parametrize("H", [4, 16, 70])
+@pytest.mark.parametrize("q_lens,starts", [([1, 1, 1], [0, 700, 77]), ([1, 5, 90], [300, 2, 40])])
+def test_latent_attention_with_16_bit_weights(rank, dr, H, q_lens, starts):
+    """Two-term weights: closer to the fp32-arithmetic kernel than the 8-bit ones, and within
+    one rounding of the result."""
+    g = torch.Generator().manual_seed(rank + H)
+    step = _step(q_lens, starts)
+    page, S, T = 16, len(q_lens), sum(q_lens)
+    need = [-(-(a + n) // page) for n, a in zip(q_lens, starts)]
+    bt = torch.full((S, max(need)), -1, dtype=torch.int32)
+    perm, at = torch.randperm(sum(need), generator=g).to(torch.int32), 0
+    for s, n in enumerate(need):
+        bt[s, :n] = perm[at:at + n]
+        at += n
+    cache = torch.randn(sum(need), 1, page, rank + dr, generator=g).bfloat16().cuda()
+    q_lat = (torch.randn(H, T, rank, generator=g) * 0.4).bfloat16().cuda()
+    q_rot = (torch.randn(T, H, dr, generator=g) * 0.4).bfloat16().cuda()
+    st = _cuda(step)
+    run = lambda **kw: _ops().latent_attention(q_lat, q_rot, cache, bt.cuda(), st, 0, 0.1, **kw)
+    exact = _ops().latent_attention(q_lat.float(), q_rot.float(), cache.float(), bt.cuda(), st, 0,
+                                    0.1, kernel="general").cpu()
+    wide = run(kernel="mma", fp32_weights=True).float().cpu()
+    narrow = run(kernel="mma").float().cpu()
+    torch.testing.assert_close(wide, exact, rtol=5e-3, atol=1e-4)
+    assert float((wide - exact).pow(2).mean()) <= float((narrow - exact).pow(2).mean())
