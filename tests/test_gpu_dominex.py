@@ -476,3 +476,167 @@ def test_latent_attention_with_16_bit_weights(rank, dr, H, q_lens, starts):
     narrow = run(kernel="mma").float().cpu()
     torch.testing.assert_close(wide, exact, rtol=5e-3, atol=1e-4)
     assert float((wide - exact).pow(2).mean()) <= float((narrow - exact).pow(2).mean())
+
+
+# -- the engine ------------------------------------------------------------------------
+def _folder_dtype(dtype):
+    return "float32" if dtype == "float32" else "bfloat16"
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name,cfg,seed,lengths,page", CASES)
+@pytest.mark.parametrize("kind", list(mc.TRACE_KINDS))
+def test_replay_matches_plain(tmp_path, dtype, name, cfg, seed, lengths, page, kind):
+    d = dk.make_model_dir(cfg, tmp_path / "m", seed, dtype=_folder_dtype(dtype))
+    reqs = dk.make_requests(cfg, lengths, seed)
+    ref = dk.reference_rows(d, reqs)
+    steps = mc.TRACE_KINDS[kind](reqs)
+    sess = ReplaySession(d, dtype, traces.peak_tokens(steps), page_size=page, max_live=4)
+    rows = mc.run_trace(sess, steps)
+    sess.executor.poll_errors()
+    rows = dk.rows_to_compare(dtype, d, reqs, rows)
+    mc.compare(rows, ref, dk.bound_for(dtype, d, reqs), f"{name}/{kind}/{dtype}")
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_long_decoding_with_recorded_steps(tmp_path, dtype):
+    """250 decoded tokens over many borders of two kinds of runs: pages before a run are given
+    back and used again, the recurrences are carried through recorded steps."""
+    cfg = dk.DA
+    d = dk.make_model_dir(cfg, tmp_path / "m", 3, dtype=_folder_dtype(dtype))
+    reqs = dk.make_requests(cfg, [270], 3)
+    ref = dk.reference_rows(d, reqs)
+    steps = traces.tail_decode(reqs, 250)
+    sess = ReplaySession(d, dtype, traces.peak_tokens(steps), page_size=4, use_graphs=True)
+    rows = mc.run_trace(sess, steps)
+    assert len(rows) == 270 and sess.executor.graph_replays >= 200
+    rows = dk.rows_to_compare(dtype, d, reqs, rows, share=0.03)
+    mc.compare(rows, ref, dk.bound_for(dtype, d, reqs), f"long decode {dtype}")
+
+
+@pytest.mark.parametrize("dtype,kind", [("bfloat16", "whole"), ("bfloat16", "mixed"),
+                                        ("float32", "tail"), ("float32", "mixed")])
+def test_long_prompts(tmp_path, dtype, kind):
+    """Prompts of several hundred tokens at head sizes 48 to 128: many key tiles and runs, the
+    recurrence in several stretches, attention over many pages."""
+    cfg = dk.DD
+    d = dk.make_model_dir(cfg, tmp_path / "m", 11, dtype=_folder_dtype(dtype))
+    reqs = dk.make_requests(cfg, [700, 260], 11)
+    ref = dk.reference_rows(d, reqs)
+    steps = mc.TRACE_KINDS[kind](reqs)
+    sess = ReplaySession(d, dtype, traces.peak_tokens(steps), page_size=16, max_live=4)
+    rows = mc.run_trace(sess, steps)
+    sess.executor.poll_errors()
+    mc.compare(rows, ref, dk.bound_for(dtype, d, reqs), f"long/{kind}/{dtype}")
+
+
+def test_prefill_equals_decoding_in_32_bit(tmp_path):
+    """The same sequence whole, token by token and in portions of two: the three runs
+    agree with each other far inside their distance to the plain model."""
+    cfg = dk.DB
+    d = dk.make_model_dir(cfg, tmp_path / "m", 6)
+    reqs = dk.make_requests(cfg, [75], 6)
+    runs = []
+    for steps in (traces.whole(reqs), traces.tail_decode(reqs, 74),
+                  traces.portions(reqs, sizes=(2,))):
+        sess = ReplaySession(d, "float32", 128, page_size=8, max_live=1)
+        rows = mc.run_trace(sess, steps)
+        runs.append(torch.stack([rows[("r0", p)] for p in range(75)]))
+    scale = float(runs[0].abs().max())
+    for other in runs[1:]:
+        assert float((other - runs[0]).abs().max()) / scale < 2e-5
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_unequal_batch_equals_each_alone(tmp_path, dtype):
+    """Four requests of unequal lengths in one step, and then a token of each, against each
+    alone in a pool whose pages and slots other requests have used."""
+    cfg = dk.DD
+    d = dk.make_model_dir(cfg, tmp_path / "m", 8, dtype=_folder_dtype(dtype))
+    reqs = dk.make_requests(cfg, [70, 3, 131, 48], 8)
+
+    def steps(groups):
+        out = []
+        for ids in groups:
+            for part in (slice(0, -1), slice(-1, None)):
+                out.append({"step": len(out), "end": ids if part.start == -1 else [],
+                            "entries": [{"id": r, "tokens": reqs[r][part],
+                                         "want": [len(reqs[r][part]) - 1]} for r in ids]})
+        return out
+    results = []
+    for groups in ([list(reqs)], [[r] for r in reqs] * 2):
+        sess = ReplaySession(d, dtype, 320, page_size=16, max_live=4)
+        results.append(mc.run_trace(sess, steps(groups)))
+    bound = 2e-5 if dtype == "float32" else dk.bound_for(dtype, d, reqs)
+    mc.compare(results[1], results[0], bound, "alone")
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_trace_run_program(tmp_path, dtype):
+    cfg = dk.DA
+    d = dk.make_model_dir(cfg, tmp_path / "m", 5, dtype="bfloat16")
+    reqs = dk.make_requests(cfg, [70, 33, 20, 9, 50, 41], 5)
+    ref = dk.reference_rows(d, reqs)
+    steps = traces.mixed(reqs, max_live=4, seed=1)
+    out = tmp_path / "out"
+    p = subprocess.run(
+        [sys.executable, os.path.join(ROOT, "bin", "trace_run"), "--model", d, "--dtype", dtype,
+         "--out", str(out), "--max-tokens", str(traces.peak_tokens(steps))],
+        input="".join(json.dumps(s) + "\n" for s in steps), capture_output=True, text=True,
+        timeout=600)
+    assert p.returncode == 0, p.stderr[-2000:]
+    outs = []
+    for s in steps:
+        n = sum(len(e["want"]) for e in s["entries"])
+        outs.append(None if n == 0 else torch.from_numpy(
+            np.fromfile(out / f"{s['step']}.f32", dtype="<f4").reshape(n, cfg["vocab"]).copy()))
+    rows = dk.rows_to_compare(dtype, d, reqs, traces.collect(steps, outs), share=0.1)
+    mc.compare(rows, ref, dk.bound_for(dtype, d, reqs), f"trace_run/{dtype}")
+
+
+def test_greedy_generation_through_the_engine(tmp_path):
+    from inferx_b200 import Engine, EngineConfig, Request, SamplingParams
+    d = dk.make_model_dir(dk.DA, tmp_path / "m", 4)
+    c, w = plain.read_model_folder(d)
+    prompts = list(dk.make_requests(dk.DA, [7, 19, 3, 30, 11], 8).values())
+    eng = Engine.create(EngineConfig(model=d, dtype="float32", block_size=4, max_num_seqs=3,
+                                     num_gpu_blocks_override=96, prefill_chunk=6,
+                                     max_model_len=64))
+    done = eng.generate([Request(p, SamplingParams(max_tokens=12, ignore_eos=True))
+                         for p in prompts])
+    for p, c_out in zip(prompts, done):
+        seq = list(p)
+        for tok in c_out.output_tokens:
+            lg = plain.forward(c, w, seq)[-1]
+            top = torch.topk(lg, 2).values
+            # the engine's choice is the plain model's, unless the two best are a tie in fp32
+            assert tok == int(lg.argmax()) or float(top[0] - top[1]) < 1e-4 * float(lg.abs().max())
+            seq.append(tok)
+        assert len(c_out.output_tokens) == 12
+
+
+def test_command_line(tmp_path):
+    """The generation program takes a folder of the design like any other: greedy output is
+    the plain model's, and sampling with a seed gives the same tokens twice."""
+    d = dk.make_model_dir(dk.DB, tmp_path / "m", 9)
+    c, w = plain.read_model_folder(d)
+    base = [sys.executable, os.path.join(ROOT, "bin", "inferx-generate"), d, "--dtype", "fp32",
+            "--block-size", "4", "--max-model-len", "64", "--max-num-seqs", "2",
+            "--num-gpu-blocks-override", "48", "--log-level", "warning", "--ignore-eos"]
+
+    def run(*args):
+        p = subprocess.run(base + list(args), capture_output=True, text=True, timeout=600)
+        assert p.returncode == 0, p.stderr[-2000:]
+        return [json.loads(ln)["output_ids"] for ln in p.stdout.splitlines() if ln.startswith("{")]
+    outs = run("--prompt-ids", "5,17,3,80,41", "--prompt-ids", "9 8 7", "--max-tokens", "6")
+    for ids, prompt in zip(outs, ([5, 17, 3, 80, 41], [9, 8, 7])):
+        seq = list(prompt)
+        for tok in ids:
+            lg = plain.forward(c, w, seq)[-1]
+            top = torch.topk(lg, 2).values
+            assert tok == int(lg.argmax()) or float(top[0] - top[1]) < 1e-4 * float(lg.abs().max())
+            seq.append(tok)
+        assert len(ids) == 6
+    sampled = [run("--prompt-ids", "9 8 7", "--max-tokens", "8", "--temperature", "0.9", "--top-k",
+                   "20", "--top-p", "0.9", "--seed", "3") for _ in range(2)]
+    assert sampled[0] == sampled[1] and len(sampled[0][0]) == 8
