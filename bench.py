@@ -948,6 +948,55 @@ def fudulix_configs(z, layers):
     return new, twin
 
 
+# `--designs --design dominex`: the Dominex design, one line per kind of layer beside the model
+# that has the closest kind at equal sizes.  "parallel" layers (attention with a distance
+# penalty beside a gated recurrence as wide as the stream, a mixture of experts) beside
+# Mapovik's (attention beside a state-space mixer, a mixture of the same experts chosen by a
+# table); "latent" layers (query latents, every second layer reading the records of the one
+# before it) beside Zuzisun's latent attention of the same heads, latent and rotated part,
+# both without a feed-forward.  Runs of 8,192 positions: every key of the timed steps is seen.
+DOMINEX_SIZES = {
+    "1k": dict(width=1024, heads=8, kv=2, experts=16, top=2, ff=512, dim=96, rot=32, vdim=128,
+               rank=256, q_rank=384),
+    "2k": dict(width=2048, heads=16, kv=4, experts=32, top=4, ff=1024, dim=128, rot=64, vdim=128,
+               rank=512, q_rank=768),
+    "4k": dict(width=4096, heads=32, kv=8, experts=32, top=4, ff=1408, dim=128, rot=64, vdim=128,
+               rank=512, q_rank=1536),
+}
+DOMINEX_CHUNK = 8192
+
+
+def dominex_configs(z, layers, kind):
+    import math
+    W = z["width"]
+    new = {"architecture": "Dominex", "vocab": DESIGN_VOCAB, "width": W,
+           "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6}, "logit_softcap": 30.0}
+    if kind == "parallel":
+        mlp = {"kind": "moe", "expert": {"ff": z["ff"]},
+               "router": {"experts": z["experts"], "top": z["top"]}}
+        attn = {"heads": z["heads"], "kv_heads": z["kv"], "dim": 128, "vdim": 128,
+                "scale": 1.0 / math.sqrt(128.0)}
+        new["layers"] = [{"type": "parallel", "mlp": mlp, "mixer": {
+            "left": dict(attn, mask={"size": DOMINEX_CHUNK}), "right": {"width": W},
+            "left_scale": 0.7, "right_scale": 0.7}}] * layers
+        twin = {"architecture": "Mapovik", "vocab": DESIGN_VOCAB, "width": W,
+                "norm": {"eps": 1e-6}, "residual_mult": 1.0, "logit_scale": 1.0,
+                "layers": [{"type": "parallel", "mlp": mlp, "mixer": {
+                    "left": attn, "right": {"heads": W // 64, "vdim": 64, "state": 128,
+                                            "groups": 2, "conv": 4, "norm_groups": 2}}}] * layers}
+        return new, twin
+    latent = {"heads": z["heads"], "dim": z["dim"], "rot_dim": z["rot"], "vdim": z["vdim"],
+              "kv_rank": z["rank"], "scale": 1.0 / math.sqrt(z["dim"] + z["rot"]),
+              "rot": {"base": 10000.0, "dims": z["rot"]}}
+    new["layers"] = [{"type": "latent_attention", "mlp": None, "mixer": dict(
+        latent, q_rank=z["q_rank"], **({"kv_from": i - 1} if i % 2 else {}))}
+        for i in range(layers)]
+    twin = {"architecture": "Zuzisun", "vocab": DESIGN_VOCAB, "width": W,
+            "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6, "groups": 8},
+            "layers": [{"type": "latent_attention", "mixer": latent, "mlp": None}] * layers}
+    return new, twin
+
+
 def designs(args):
     """One JSON line per size: prompt tokens/s (one prompt of --prefill-tokens, default
     2048) and decode tokens/s (--batch sequences at --context) of both designs, device
@@ -959,17 +1008,27 @@ def designs(args):
     tinapel = args.design == "tinapel"
     mapovik = args.design == "mapovik"
     fudulix = args.design == "fudulix"
-    sizes = (FUDULIX_SIZES if fudulix else MAPOVIK_SIZES if mapovik
+    dominex = args.design == "dominex"
+    sizes = (DOMINEX_SIZES if dominex else FUDULIX_SIZES if fudulix else MAPOVIK_SIZES if mapovik
              else TINAPEL_SIZES if tinapel else DESIGN_SIZES)
     first, second = (("fudulix", "qwen2_moe") if fudulix else ("mapovik", "tinapel") if mapovik
                      else ("tinapel", "qwen2_moe") if tinapel else ("zuzisun", "qwen2_dense"))
-    for name in (args.design_sizes.split(",") if args.design_sizes else list(sizes)):
+    names = args.design_sizes.split(",") if args.design_sizes else list(sizes)
+    kinds = [None]
+    if dominex:
+        kinds = ([k for k in args.design_pattern.split(",")] if "wkv" not in args.design_pattern
+                 else ["parallel", "latent"])
+    for name, kind in ((n, k) for n in names for k in kinds):
         z = sizes[name]
         C = args.context or 4096
         row = {"size": name, "layers": layers, "width": z["width"], "heads": z["heads"],
                "ff": z["ff"], "prompt_tokens": prompt, "batch": B,
                "context": C, "dtype": "bf16", "data": "synthetic, random weights"}
-        if fudulix:
+        if dominex:
+            first, second = "dominex", {"parallel": "mapovik", "latent": "zuzisun"}[kind]
+            row["layer_kind"] = kind
+            pair = dominex_configs(z, layers, kind)
+        elif fudulix:
             row["window"] = FUDULIX_WINDOW
             pair = fudulix_configs(z, layers)
         elif mapovik:
@@ -1049,12 +1108,13 @@ def main(argv=None):
                          "beside the closest Qwen2-MoE at equal sizes (random weights); --layers (4), "
                          "--batch, --context (4096), --prefill-tokens (2048) apply")
     ap.add_argument("--design-sizes", default="", help="with --designs: of 1k,2k,4k (all)")
-    ap.add_argument("--design", default="zuzisun", choices=["zuzisun", "tinapel", "mapovik", "fudulix"],
+    ap.add_argument("--design", default="zuzisun", choices=["zuzisun", "tinapel", "mapovik", "fudulix", "dominex"],
                     help="with --designs: which design stands beside its closest model")
     ap.add_argument("--design-pattern", default="wkv,gla,attention,attention",
                     help="with --design tinapel: the mixers of the layers, repeated; with "
                          "--design mapovik of parallel, delta (default "
-                         "parallel,delta,delta,parallel)")
+                         "parallel,delta,delta,parallel); with --design dominex the kinds of "
+                         "layers to report, of parallel, latent (both)")
     args = ap.parse_args(argv)
     if args.impl == "reference":
         return reference_arm()

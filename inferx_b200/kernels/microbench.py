@@ -15,6 +15,7 @@
     python -m inferx_b200.kernels.microbench recurrent --tokens 64 --batch 64 --hidden 2048 --head-dim 64
     python -m inferx_b200.kernels.microbench attn_prefill --tokens 2048 --softcap 30
     python -m inferx_b200.kernels.microbench prepared --tokens 2048 --hidden 2048 --heads 16 --kv-heads 4 --inter 4096 --experts 32 --batch 8 --window 1024
+    python -m inferx_b200.kernels.microbench paired --tokens 2048 --hidden 2048 --heads 16 --kv-heads 4 --inter 1024 --experts 32 --batch 8
 
 Each case runs one kernel face at Qwen1.5-MoE-A2.7B sizes (or the sizes given),
 cycling through enough copies of its inputs that consecutive iterations do not
@@ -625,11 +626,193 @@ def prepared(args):
     return out
 
 
+def paired(args):
+    """The kernels of decoders that pair attention and a gated recurrence, each beside the
+    like kernel of another model of this engine at the same sizes: ``--tokens`` rows of
+    ``--hidden`` (the recurrence is as wide), ``--heads`` over ``--kv-heads`` heads of
+    ``--head-dim``, ``--experts`` experts of ``--inter``, ``--top-k`` chosen, a latent of
+    ``--rank`` + ``--rot-dim``; attention of one prompt of ``--tokens`` tokens, and of
+    ``--batch`` single tokens at ``--context``.  GB/s over the bytes the operation has to
+    move, attention and products also as TFLOP/s."""
+    from . import ops
+    T, W, H, G, D = args.tokens, args.hidden, args.heads, args.kv_heads, args.head_dim
+    E, K, I, page, B, C = args.experts, args.top_k, args.inter, args.page, args.batch, args.context
+    rank, dr = args.rank, args.rot_dim
+    dt, dev = torch.bfloat16, "cuda"
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    out = {"case": "paired", "tokens": T, "hidden": W, "heads": H, "kv_heads": G, "head_dim": D,
+           "experts": E, "top_k": K, "inter": I, "batch": B, "context": C}
+
+    def report(name, us, nbytes=0, flops=0):
+        out[name] = {"us": round(us, 2)}
+        if nbytes:
+            out[name]["GBps"] = round(nbytes / us / 1e3, 1)
+        if flops:
+            out[name]["TFLOPs"] = round(flops / us / 1e6, 2)
+
+    def batch(q_lens, starts):
+        S, cu = len(q_lens), [0]
+        for q in q_lens:
+            cu.append(cu[-1] + q)
+        one = max(q_lens) == 1
+        return types.SimpleNamespace(
+            cu_q=i32(cu), q_pos0=i32(starts), q_lens=q_lens, num_seqs=S, num_tokens=cu[-1],
+            seq_of_token=i32([s for s, q in enumerate(q_lens) for _ in range(q)]),
+            positions=i32([a + t for a, q in zip(starts, q_lens) for t in range(q)]),
+            kv_len=i32([a + q for a, q in zip(starts, q_lens)]), state_slot=i32(list(range(S))),
+            max_kv_len=max(a + q for a, q in zip(starts, q_lens)), max_q_len=max(q_lens),
+            all_decode=one, num_decode_seqs=S if one else 0, cu_q_prompt=i32(cu))
+    prompt, single = batch([T], [0]), batch([1] * B, [C - 1] * B)
+
+    # recurrence over a prompt and over single tokens, beside the state-space recurrence
+    front_w = (H + 2 * G) * D + 3 * W
+    n = max(2, min(8, _copies(T * 4 * W * 2)))
+    zb = torch.zeros(W, device=dev)
+    state = torch.zeros(B, W, device=dev)
+    fronts = [torch.randn(T, front_w, device=dev, dtype=dt) for _ in range(n)]
+    both = [torch.empty(T, H * D + W, device=dev, dtype=dt) for _ in range(n)]
+    off = front_w - 3 * W
+    report("min_gru (prompt)", _time(lambda i: ops.min_gru(
+        fronts[i][:, off:], zb, zb, 0.5, state, prompt, both[i][:, H * D:], 0.7), n, args.iters),
+        T * W * 8)
+    few = [torch.randn(B, front_w, device=dev, dtype=dt) for _ in range(8)]
+    fewo = torch.empty(B, H * D + W, device=dev, dtype=dt)
+    report("min_gru (single tokens)", _time(lambda i: ops.min_gru(
+        few[i][:, off:], zb, zb, 0.5, state, single, fewo[:, H * D:], 0.7), 8, args.iters),
+        B * W * 16)
+    hs, st, gr = W // 64, 128, 2
+    xbc = torch.randn(T, W + 2 * gr * st, device=dev, dtype=dt) * 0.3
+    dt_raw, hv = torch.randn(T, hs, device=dev, dtype=dt), torch.zeros(hs, device=dev)
+    sst = torch.zeros(B, hs, st, 64, device=dev)
+    report("ssd_recurrence (prompt, like)", _time(lambda i: ops.ssd_recurrence(
+        xbc, dt_raw, hv, hv, hv, sst, prompt, hs, 64, st, gr), 1, args.iters),
+        T * (W * 2 + 2 * gr * st * 2 + W * 4))
+    # rows into pages, beside the split of a q | k | v row
+    pages = -(-T // page)
+    kp = torch.randn(pages, G, page, D, device=dev, dtype=dt) * 0.3
+    vp = torch.randn(pages, G, page, D, device=dev, dtype=dt)
+    slots = torch.arange(T, dtype=torch.int32, device=dev)
+    dq, dk = H * D, G * D
+    report("append_kv_rows", _time(lambda i: ops.append_kv_rows(
+        fronts[i][:, dq:dq + dk], fronts[i][:, dq + dk:dq + 2 * dk], kp, vp, slots), n,
+        args.iters), T * dk * 8)
+    qkv = [f[:, :dq + 2 * dk].contiguous() for f in fronts]
+    report("qkv_rope_append (like)", _time(lambda i: ops.qkv_rope_append(
+        qkv[i], None, prompt.positions, None, 0, H, G, D, kp, vp, slots), n, args.iters),
+        T * (dq + 2 * dk) * 4)
+    # attention
+    scale = 1.0 / math.sqrt(D)
+    bt = torch.arange(pages, dtype=torch.int32, device=dev).view(1, pages)
+    vec = [torch.ones(H, device=dev), torch.full((H,), 0.8, device=dev),
+           torch.full((H,), 0.3, device=dev)]
+    flops = 4.0 * H * D * (T * (T + 1) // 2)
+    q3 = qkv[0][:, :dq].contiguous().view(T, H, D)
+    for form in ("tc", "mma", "tiled"):
+        report(f"prompt attention with a distance penalty: {form}", _time(
+            lambda i: ops.distance_attention(fronts[i][:, :dq], kp, vp, bt, prompt, scale, *vec,
+                                             4 * T, both[i][:, :dq], 0.7, kernel=form),
+            n, max(3, args.iters // (20 if form == "tiled" else 2))), 0, flops)
+    report("prompt attention: tcgen05 16-bit weights (like)", _time(
+        lambda i: ops.paged_attention_prefill_exact(q3, kp, vp, bt, prompt.cu_q, prompt.q_pos0, 0,
+                                                    scale, kernel="tc"), 1, args.iters), 0, flops)
+    report("prompt attention: tcgen05 8-bit weights (like)", _time(
+        lambda i: ops.paged_attention_prefill(q3, kp, vp, bt, prompt.cu_q, prompt.q_pos0, 0, scale,
+                                              max_kv_len=T), 1, args.iters), 0, flops)
+    per = -(-C // page)
+    nc = min(_copies(B * C * G * D * 4), 8)
+    kcs = [torch.randn(B * per, G, page, D, device=dev, dtype=dt) * 0.3 for _ in range(nc)]
+    vcs = [torch.randn(B * per, G, page, D, device=dev, dtype=dt) for _ in range(nc)]
+    btd = torch.randperm(B * per, device=dev).to(torch.int32).view(B, per)
+    qd = few[0][:, :dq].contiguous().view(B, H, D)
+    nbytes = B * C * G * D * 4
+    for form in ("decode", "decode_any"):
+        report(f"single-token attention with a distance penalty: {form}", _time(
+            lambda i: ops.distance_attention(few[0][:, :dq], kcs[i], vcs[i], btd, single, scale,
+                                             *vec, 4 * C, fewo[:, :dq], 0.7, kernel=form),
+            nc, args.iters), nbytes)
+    report("single-token attention: mma.sync 16-bit weights (like)", _time(
+        lambda i: ops.paged_attention_decode_exact(qd, kcs[i], vcs[i], btd, single.kv_len, C, 0,
+                                                   scale), nc, args.iters), nbytes)
+    report("single-token attention: TMA 8-bit weights (like)", _time(
+        lambda i: ops.paged_attention_decode(qd, kcs[i], vcs[i], btd, single.kv_len, C, 0, scale),
+        nc, args.iters), nbytes)
+    del kcs, vcs
+    _paired_latent_and_experts(args, ops, prompt, single, report)
+    return out
+
+
+def _paired_latent_and_experts(args, ops, prompt, single, report):
+    T, W, H, page, B, C = args.tokens, args.hidden, args.heads, args.page, args.batch, args.context
+    E, K, I, rank, dr = args.experts, args.top_k, args.inter, args.rank, args.rot_dim
+    D, dt, dev = args.head_dim, torch.bfloat16, "cuda"
+    # query latent and record, beside the preparation of a whole latent projection
+    qr = 3 * W // 8
+    pos, slots = prompt.positions, torch.arange(T, dtype=torch.int32, device=dev)
+    freq = torch.rand(dr // 2, device=dev)
+    gq, gk = torch.ones(qr, device=dev), torch.ones(rank, device=dev)
+    pages = -(-T // page)
+    rec = torch.zeros(pages, 1, page, rank + dr, device=dev, dtype=dt)
+    n = max(2, min(8, _copies(T * (qr + rank + dr) * 4)))
+    projs = [torch.randn(T, qr + rank + dr, device=dev, dtype=dt) for _ in range(n)]
+    report("latent_front", _time(lambda i: ops.latent_front(
+        projs[i], qr, gq, 1e-6, qr, pos, freq, 1.0, gk, rank, dr, dr, rec, slots), n, args.iters),
+        T * (qr + rank + dr) * 4)
+    n = max(2, min(8, _copies(T * H * (D + dr) * 4)))
+    qs = [torch.randn(T, H * (D + dr), device=dev, dtype=dt) for _ in range(n)]
+    report("latent_queries", _time(lambda i: ops.latent_queries(
+        qs[i], pos, freq, 1.0, H, D, dr, dr), n, args.iters), T * H * (D + dr) * 4)
+    wide = [torch.randn(T, H * (D + dr) + rank + dr, device=dev, dtype=dt) for _ in range(n)]
+    report("latent_prepare (like)", _time(lambda i: ops.latent_prepare(
+        wide[i], 0, H * (D + dr), pos, freq, 1.0, gk, 1e-6, H, D, dr, dr, rank, rec, slots), n,
+        args.iters), T * (H * (D + dr) + rank + dr) * 4)
+    # latent attention with two-term weights, beside one-term ones
+    scale = 1.0 / math.sqrt(D + dr)
+    for name, step, Tq, S, L in (("prompt", prompt, T, 1, T), ("single tokens", single, B, B, C)):
+        per = -(-L // page)
+        nc = 1 if S == 1 else min(_copies(S * L * (rank + dr) * 2), 8)
+        caches = [torch.randn(S * per, 1, page, rank + dr, device=dev, dtype=dt) * 0.3
+                  for _ in range(nc)]
+        bt = torch.randperm(S * per, device=dev).to(torch.int32).view(S, per)
+        ql = torch.randn(H, Tq, rank, device=dev, dtype=dt) * 0.3
+        qrot = torch.randn(Tq, H, dr, device=dev, dtype=dt) * 0.3
+        seen = T * (T + 1) // 2 if S == 1 else S * L
+        for label, flag in (("16-bit weights", True), ("8-bit weights (like)", False)):
+            report(f"latent attention, {name}: {label}", _time(
+                lambda i: ops.latent_attention(ql, qrot, caches[i], bt, step, 0, scale,
+                                               fp32_weights=flag), nc, args.iters),
+                S * L * (rank + dr) * 2 if S > 1 else 0, 2.0 * H * (2 * rank + dr) * seen)
+    # router, dispatch and the gate/up product with a factor per row, beside the plain ones
+    for name, rows in (("prompt", T), ("single tokens", B)):
+        x = torch.randn(rows, W, device=dev, dtype=dt)
+        rw = torch.randn(E, W, device=dev) * 0.02
+        for label, kw in (("sigmoid", {"score": "sigmoid"}), ("softmax (like)", {})):
+            report(f"router_topk, {name}: {label}", _time(
+                lambda i: ops.router_topk(x, rw, K, False, 1.0, **kw), 1, args.iters))
+        tw, ti, _ = ops.router_topk(x, rw, K, False, 1.0, score="sigmoid")
+        report(f"moe_dispatch, {name}: with row weights", _time(
+            lambda i: ops.moe_dispatch(ti, E, topk_w=tw), 1, args.iters))
+        report(f"moe_dispatch, {name}: plain (like)", _time(
+            lambda i: ops.moe_dispatch(ti, E), 1, args.iters))
+        off, rr, _, rs = ops.moe_dispatch(ti, E, topk_w=tw)
+        nw = max(1, min(4, _copies(E * 2 * I * W * 2)))
+        gu = [torch.randn(E, 2 * I, W, device=dev, dtype=dt) * 0.02 for _ in range(nw)]
+        flops = 4.0 * rows * K * I * W
+        for label, kw in (("row weights", {"row_scale": rs}), ("plain (like)", {})):
+            report(f"gate/up product, {name}: {label}", _time(
+                lambda i: ops.grouped_gate_up_swiglu(x, rr, off, gu[i], **kw), nw, args.iters),
+                0, flops)
+        del gu
+    for rows, vocab in ((B, 32000), (512, 32000)):
+        lg = torch.randn(rows, vocab, device=dev)
+        report(f"softcap_rows, {rows} rows", _time(lambda i: ops.softcap_rows(lg, 30.0), 1,
+                                                   args.iters), rows * vocab * 8)
+
+
 def main(argv=None):
     ap = argparse.ArgumentParser(description=__doc__.split("\n\n")[0])
     ap.add_argument("case", choices=["attn_decode", "grouped", "dense", "attn_prefill", "router",
                                      "qkv", "latent_attn", "rowwise", "recurrent", "delta",
-                                     "prepared"])
+                                     "prepared", "paired"])
     ap.add_argument("--softcap", type=float, default=0.0,
                     help="attn_decode, attn_prefill: squash scores to softcap * tanh(s / softcap)")
     ap.add_argument("--rank", type=int, default=512, help="latent_attn: entries of the latent")
