@@ -155,56 +155,82 @@ __global__ void min_gru_step_kernel(const TA* __restrict__ front, long long ld,
   MgVec<TA, V>::store(out + (size_t)t * o_ld + c, y);
 }
 
-// Portions: a block owns MG_CH neighbouring channels of one sequence; its threads are
-// MG_CH / V channel lanes times MG_TL time lanes, a time lane MG_L neighbouring tokens of a
-// stretch of MG_TL * MG_L.  Every thread forms the map of its tokens, the maps of the time
-// lanes before it are joined (shuffles inside a warp, shared memory between warps), and the
-// thread walks its tokens from the state it then knows.
-#define MG_CH 16
+// Portions: a block owns CL * V neighbouring channels of one sequence; its threads are CL
+// channel lanes times NW * 32 / CL time lanes, a time lane MG_L neighbouring tokens of a
+// stretch.  Every thread forms the map of its tokens, the maps of the time lanes before it
+// are joined (shuffles inside a warp, shared memory between warps), and the thread walks its
+// tokens from the state it then knows.
+//   MODE 0: the block takes the whole portion, stretch by stretch (portions of a few
+//           hundred tokens: narrow tiles of channels, many time lanes);
+//   MODE 1: long portions are cut into segments of seg_len tokens, blockIdx.z picks one; the
+//           map of the segment alone goes to maps[s][1 + segment] as (A, B) per channel, and
+//           the state ahead of the portion to maps[s][0] as (0, S);
+//   MODE 2: the segment's block joins the maps ahead of it and walks its tokens.
+// z and x are read twice then, the second time from L2, and the segments fill the device.
 #define MG_L 8
-#define MG_THREADS 512
 
-template <typename TA, int V>
-__global__ void __launch_bounds__(MG_THREADS)
+template <typename TA, int V, int CL, int NW, int MODE>
+__global__ void __launch_bounds__(NW * 32)
 min_gru_scan_kernel(const TA* __restrict__ front, long long ld, const float* __restrict__ z_bias,
                     const float* __restrict__ x_bias, float shift, float* __restrict__ state,
                     const int* __restrict__ slots, const int* __restrict__ cu_q,
-                    TA* __restrict__ out, long long o_ld, float out_scale, int W) {
-  constexpr int CL = MG_CH / V;                 // channel lanes
+                    TA* __restrict__ out, long long o_ld, float out_scale, int W, int seg_len,
+                    int segments, float2* __restrict__ maps) {
+  constexpr int CH = CL * V;                    // channels of the block
   constexpr int TW = 32 / CL;                   // time lanes of a warp
-  constexpr int NW = MG_THREADS / 32;
   constexpr int SPAN = NW * TW * MG_L;          // tokens of a stretch
-  __shared__ float wa[NW][MG_CH], wb[NW][MG_CH];
-  __shared__ float carry[MG_CH];
+  __shared__ float wa[NW][CH], wb[NW][CH];
+  __shared__ float carry[CH], carry_a[CH];
   IX_PDL_WAIT();
   const int s = blockIdx.y;
-  const int tok0 = cu_q[s], n = cu_q[s + 1] - tok0;
+  const int tok0 = cu_q[s], total = cu_q[s + 1] - tok0;
+  const int first = MODE == 0 ? 0 : (int)blockIdx.z * seg_len;
+  const int n = MODE == 0 ? total : min(total, first + seg_len);
+  if (first >= n) return;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int cl = lane % CL, tw = lane / CL;
   const int tl = warp * TW + tw;
-  const int c = blockIdx.x * MG_CH + cl * V;
+  const int c0 = blockIdx.x * CH;
+  const int c = c0 + cl * V;
   const bool live = c < W;                      // W is a multiple of V
   float* st = state + (size_t)slots[s] * W;
-  if (threadIdx.x < MG_CH)
-    carry[threadIdx.x] = blockIdx.x * MG_CH + threadIdx.x < W ? st[blockIdx.x * MG_CH + threadIdx.x] : 0.f;
+  float2* my_maps = MODE == 0 ? nullptr : maps + (size_t)s * (segments + 1) * W;
+  for (int i = threadIdx.x; i < CH; i += NW * 32) {
+    const bool ok = c0 + i < W;
+    float x = 0.f;
+    if (MODE == 0 && ok) x = st[c0 + i];
+    if (MODE == 1 && blockIdx.z == 0 && ok) my_maps[c0 + i] = make_float2(0.f, st[c0 + i]);
+    if (MODE == 2 && ok) {
+#pragma unroll 4
+      for (int g = 0; g <= (int)blockIdx.z; ++g) {
+        const float2 m = my_maps[(size_t)g * W + c0 + i];
+        x = fmaf(m.x, x, m.y);
+      }
+    }
+    carry[i] = x;                               // MODE 1: B of what came before, A beside it
+    if (MODE == 1) carry_a[i] = 1.f;
+  }
   float zb[V], xb[V];
 #pragma unroll
   for (int i = 0; i < V; ++i) {
     zb[i] = live ? z_bias[c + i] : 0.f;
     xb[i] = live ? x_bias[c + i] : 0.f;
   }
-  for (int base = 0; base < n; base += SPAN) {
+  for (int base = first; base < n; base += SPAN) {
     const int t0 = base + tl * MG_L;
     const int m = live ? max(0, min(MG_L, n - t0)) : 0;
-    const TA* row = front + (size_t)(tok0 + t0) * ld + c;
-    float a[MG_L][V], b[MG_L][V], g[MG_L][V];
+    // Loads and maps without a branch, so that all loads are out before the first is used:
+    // tokens past the end and channels past the width read a valid place and count as the
+    // identity map.
+    const TA* row = front + (size_t)tok0 * ld + (live ? c : 0);
+    float a[MG_L][V], b[MG_L][V], g[MODE == 1 ? 1 : MG_L][V];
 #pragma unroll
-    for (int i = 0; i < MG_L; ++i)
-      if (i < m) {
-        MgVec<TA, V>::load(row + (size_t)i * ld, a[i]);
-        MgVec<TA, V>::load(row + (size_t)i * ld + W, b[i]);
-        MgVec<TA, V>::load(row + (size_t)i * ld + 2 * W, g[i]);
-      }
+    for (int i = 0; i < MG_L; ++i) {
+      const TA* p = row + (size_t)min(t0 + i, n - 1) * ld;
+      MgVec<TA, V>::load(p, a[i]);
+      MgVec<TA, V>::load(p + W, b[i]);
+      if (MODE != 1) MgVec<TA, V>::load(p + 2 * W, g[MODE == 1 ? 0 : i]);
+    }
     float A[V], B[V];
 #pragma unroll
     for (int v = 0; v < V; ++v) {
@@ -213,16 +239,15 @@ min_gru_scan_kernel(const TA* __restrict__ front, long long ld, const float* __r
     }
 #pragma unroll
     for (int i = 0; i < MG_L; ++i)
-      if (i < m)
 #pragma unroll
-        for (int v = 0; v < V; ++v) {
-          float ma, mb;
-          mg_map<TA>(a[i][v], b[i][v], zb[v], xb[v], shift, ma, mb);
-          a[i][v] = ma;
-          b[i][v] = mb;
-          A[v] *= ma;
-          B[v] = fmaf(ma, B[v], mb);
-        }
+      for (int v = 0; v < V; ++v) {
+        float ma, mb;
+        mg_map<TA>(a[i][v], b[i][v], zb[v], xb[v], shift, ma, mb);
+        a[i][v] = i < m ? ma : 1.f;
+        b[i][v] = i < m ? mb : 0.f;
+        A[v] *= a[i][v];
+        B[v] = fmaf(a[i][v], B[v], b[i][v]);
+      }
     // inclusive maps over the warp's time lanes
 #pragma unroll
     for (int o = CL; o < 32; o <<= 1)
@@ -241,19 +266,36 @@ min_gru_scan_kernel(const TA* __restrict__ front, long long ld, const float* __r
         wa[warp][cl * V + v] = A[v];
         wb[warp][cl * V + v] = B[v];
       }
-    // exclusive inside the warp
-    float S[V];
+    if (MODE == 1) {          // the stretch's map behind the one of the stretches before
+      __syncthreads();
+      for (int i = threadIdx.x; i < CH; i += NW * 32) {
+        float x = carry[i], y = carry_a[i];
 #pragma unroll
-    for (int v = 0; v < V; ++v) {
-      float ea = __shfl_up_sync(0xffffffffu, A[v], CL);
-      float eb = __shfl_up_sync(0xffffffffu, B[v], CL);
-      if (tw == 0) {
-        ea = 1.f;
-        eb = 0.f;
+        for (int w = 0; w < NW; ++w) {
+          x = fmaf(wa[w][i], x, wb[w][i]);
+          y *= wa[w][i];
+        }
+        carry[i] = x;
+        carry_a[i] = y;
       }
-      A[v] = ea;
-      B[v] = eb;
+      __syncthreads();
+      continue;
     }
+    // exclusive inside the warp
+    if (TW > 1) {
+#pragma unroll
+      for (int v = 0; v < V; ++v) {
+        A[v] = __shfl_up_sync(0xffffffffu, A[v], CL);
+        B[v] = __shfl_up_sync(0xffffffffu, B[v], CL);
+      }
+    }
+    if (tw == 0)
+#pragma unroll
+      for (int v = 0; v < V; ++v) {
+        A[v] = 1.f;
+        B[v] = 0.f;
+      }
+    float S[V];
     __syncthreads();          // the warps' maps and the carried state are there
 #pragma unroll
     for (int v = 0; v < V; ++v) {
@@ -263,16 +305,15 @@ min_gru_scan_kernel(const TA* __restrict__ front, long long ld, const float* __r
     }
     TA* o = out + (size_t)(tok0 + t0) * o_ld + c;
 #pragma unroll
-    for (int i = 0; i < MG_L; ++i)
-      if (i < m) {
-        float y[V];
+    for (int i = 0; i < MG_L; ++i) {
+      float y[V];
 #pragma unroll
-        for (int v = 0; v < V; ++v) {
-          S[v] = fmaf(a[i][v], S[v], b[i][v]);
-          y[v] = mg_gate<TA>(S[v], g[i][v], out_scale);
-        }
-        MgVec<TA, V>::store(o + (size_t)i * o_ld, y);
+      for (int v = 0; v < V; ++v) {
+        S[v] = fmaf(a[i][v], S[v], b[i][v]);
+        y[v] = mg_gate<TA>(S[v], g[MODE == 1 ? 0 : i][v], out_scale);
       }
+      if (i < m) MgVec<TA, V>::store(o + (size_t)i * o_ld, y);
+    }
     __syncthreads();          // everyone has read the carried state
     // the thread of the stretch's last token knows the state behind it
     if (m > 0 && (t0 + m == n || (tl == NW * TW - 1)))
@@ -280,24 +321,67 @@ min_gru_scan_kernel(const TA* __restrict__ front, long long ld, const float* __r
       for (int v = 0; v < V; ++v) carry[cl * V + v] = S[v];
   }
   __syncthreads();
-  if (threadIdx.x < MG_CH && blockIdx.x * MG_CH + threadIdx.x < W)
-    st[blockIdx.x * MG_CH + threadIdx.x] = carry[threadIdx.x];
+  for (int i = threadIdx.x; i < CH; i += NW * 32) {
+    if (c0 + i >= W) break;
+    if (MODE == 1) my_maps[(size_t)(blockIdx.z + 1) * W + c0 + i] = make_float2(carry_a[i], carry[i]);
+    else if (n == total) st[c0 + i] = carry[i];
+  }
+}
+
+#define MG_SHORT 512       // portions up to this many tokens take MODE 0
+#define MG_STRETCH 64      // tokens of a stretch in MODE 1 and 2
+#define MG_MAX_SEGMENTS 32
+
+// Segments a step whose longest portion has max_q tokens is cut into (1: not cut); the scratch
+// is float2 [sequences that are no single tokens][segments + 1][W].
+IX_API int ix_min_gru_segments(int max_q) {
+  if (max_q <= MG_SHORT) return 1;
+  int len = (max_q + MG_MAX_SEGMENTS - 1) / MG_MAX_SEGMENTS;
+  len = (len + MG_STRETCH - 1) / MG_STRETCH * MG_STRETCH;
+  return (max_q + len - 1) / len;
+}
+
+template <typename TA, int V>
+static void launch_min_gru_scan(const void* front, long long ld, const float* z_bias,
+                                const float* x_bias, float shift, float* state, const int* slots,
+                                const int* cu_q, void* out, long long o_ld, float out_scale,
+                                int W, int S, int max_q, int segments, float* maps,
+                                cudaStream_t stream) {
+  if (segments <= 1) {
+    constexpr int CL = 16 / V;
+    ix_launch(min_gru_scan_kernel<TA, V, CL, 16, 0>, dim3((W + 15) / 16, S), dim3(512), 0, stream,
+              (const TA*)front, ld, z_bias, x_bias, shift, state, slots, cu_q, (TA*)out, o_ld,
+              out_scale, W, 0, 1, (float2*)nullptr);
+    return;
+  }
+  int len = (max_q + segments - 1) / segments;
+  len = (len + MG_STRETCH - 1) / MG_STRETCH * MG_STRETCH;
+  const dim3 grid((W + 32 * V - 1) / (32 * V), S, segments);
+  ix_launch(min_gru_scan_kernel<TA, V, 32, 8, 1>, grid, dim3(256), 0, stream, (const TA*)front, ld,
+            z_bias, x_bias, shift, state, slots, cu_q, (TA*)out, o_ld, out_scale, W, len, segments,
+            (float2*)maps);
+  ix_launch(min_gru_scan_kernel<TA, V, 32, 8, 2>, grid, dim3(256), 0, stream, (const TA*)front, ld,
+            z_bias, x_bias, shift, state, slots, cu_q, (TA*)out, o_ld, out_scale, W, len, segments,
+            (float2*)maps);
 }
 
 // front: rows of pitch ld, columns [z: W | x: W | g: W]; state [slots, W] fp32; slots and cu_q
-// are those of the S sequences; the first `singles` of them bring one token each.
+// are those of the S sequences; the first `singles` of them bring one token each, the longest
+// of the rest max_q.  segments > 1 (see ix_min_gru_segments): maps is the scratch.
 IX_API int ix_min_gru(const void* front, long long ld, const float* z_bias, const float* x_bias,
                       float shift, float* state, const int* slots, const int* cu_q, void* out,
                       long long o_ld, float out_scale, int act_dtype, int S, int singles, int W,
-                      cudaStream_t stream) {
+                      int max_q, int segments, float* maps, cudaStream_t stream) {
   if (S <= 0) return IX_OK;
   if (W <= 0 || singles < 0 || singles > S || S > 65535 || ld < 3LL * W || o_ld < W)
+    return IX_ERR_SIZE;
+  if (segments < 1 || (segments > 1 && (!maps || max_q <= 0 ||
+                                        segments != ix_min_gru_segments(max_q))))
     return IX_ERR_SIZE;
   const int esize = act_dtype == IX_F32 ? 4 : 2;
   const bool pairs = W % 2 == 0 && ld % 2 == 0 && o_ld % 2 == 0 &&
                      (((uintptr_t)front | (uintptr_t)out) % (2 * esize)) == 0;
   const int rest = S - singles;
-  const dim3 scan_grid((W + MG_CH - 1) / MG_CH, rest > 0 ? rest : 1);
 #define IX_MG(V)                                                                                \
   IX_DISPATCH_DTYPE(act_dtype, TA, {                                                            \
     if (singles > 0)                                                                            \
@@ -305,9 +389,9 @@ IX_API int ix_min_gru(const void* front, long long ld, const float* z_bias, cons
                 stream, (const TA*)front, ld, z_bias, x_bias, shift, state, slots, cu_q,        \
                 (TA*)out, o_ld, out_scale, W);                                                  \
     if (rest > 0)                                                                               \
-      ix_launch(min_gru_scan_kernel<TA, V>, scan_grid, dim3(MG_THREADS), 0, stream,             \
-                (const TA*)front, ld, z_bias, x_bias, shift, state, slots + singles,            \
-                cu_q + singles, (TA*)out, o_ld, out_scale, W);                                  \
+      launch_min_gru_scan<TA, V>(front, ld, z_bias, x_bias, shift, state, slots + singles,      \
+                                 cu_q + singles, out, o_ld, out_scale, W, rest, max_q, segments, \
+                                 maps, stream);                                                 \
   })
   if (pairs) IX_MG(2);
   else IX_MG(1);

@@ -2336,12 +2336,17 @@ def min_gru(front: torch.Tensor, z_bias: torch.Tensor, x_bias: torch.Tensor, shi
     singles = int(getattr(step, "num_decode_seqs", 0))
     if step.all_decode:
         singles = step.num_seqs
+    rest, max_q = step.num_seqs - singles, int(step.max_q_len)
+    segments = _lib().ix_min_gru_segments(max_q) if rest > 0 else 1
+    maps = None
+    if segments > 1:      # long portions: the maps of their segments, joined by a second kernel
+        maps = torch.empty((rest, segments + 1, W, 2), dtype=torch.float32, device=front.device)
     _check(_lib().ix_min_gru(
         _ptr(front), ctypes.c_longlong(ld), _ptr(z_bias), _ptr(x_bias), ctypes.c_float(shift),
         _ptr(state), _ptr(step.state_slot), _ptr(step.cu_q), _ptr(out), ctypes.c_longlong(o_ld),
-        ctypes.c_float(out_scale), _dtype_code(front), step.num_seqs, singles, W, _stream()),
-        "min_gru")
-    _count(2 if 0 < singles < step.num_seqs else 1)
+        ctypes.c_float(out_scale), _dtype_code(front), step.num_seqs, singles, W, max_q,
+        segments, _ptr(maps), _stream()), "min_gru")
+    _count((1 if singles else 0) + (0 if rest <= 0 else 2 if segments > 1 else 1))
     return out
 
 
