@@ -66,7 +66,7 @@ def _served(choice):
         latent(8, 48, 16, 32, 128, 160, 0.125, 10000.0, kv_from=1, mlp=moe(2, 2, 64)),
         parallel(4, 4, 128, 128, 0.088, 96, 320, (1.0, 0.8), mlp=moe(1, 1, 128)),
         parallel(16, 1, 64, 128, 0.12, 33, 192, (0.8, 1.0), mlp=moe(3, 3, 64)),
-        latent(16, 64, 32, 64, 64, 96, 0.1, 500.0, mlp=moe(2, 2, 160)),
+        latent(16, 64, 32, 64, 64, 104, 0.1, 500.0, mlp=moe(2, 2, 160)),
     ])
 
 
