@@ -76,6 +76,10 @@ def _register_builtin():
     from .dominex_config import DominexConfig
     register_architecture(DominexConfig.ARCHITECTURE, DominexConfig.from_json,
                           dominex.build_spec, replace=True)
+    from ..models import biguzen
+    from .biguzen_config import BiguzenConfig
+    register_architecture(BiguzenConfig.ARCHITECTURE, BiguzenConfig.from_json,
+                          biguzen.build_spec, replace=True)
 
 
 _register_builtin()

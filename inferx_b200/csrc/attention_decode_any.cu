@@ -14,9 +14,9 @@
 // number of splits alone.
 //
 // `keep_first` > 0 keeps the sequence's first keep_first keys visible beside the window: the
-// walk goes over them and then over the window, as one range that is split.  `sink` adds
-// one to the softmax's denominator (a key of score 0 without a value), where the result
-// is normalised: in this kernel when the sequence is not split, else in the merge.
+// walk goes over them and then over the window, as one range that is split.  A sink
+// per head (a key of that score without a value) and a gate per (token, head) enter where
+// the result is normalised: in this kernel when the sequence is not split, else in the merge.
 //
 // A third form (attention_distance.cuh) multiplies a score by its head's temperature, takes
 // r1 ln(1 + r2 distance) off and may confine the query to its own run of positions.
@@ -36,7 +36,7 @@ attn_decode_any_kernel(const TA* __restrict__ q, const TA* __restrict__ kc,
                        const int* __restrict__ kv_len, float* __restrict__ part_o,
                        float* __restrict__ part_ml, TA* __restrict__ out, int heads, int kvh,
                        int hd, int vd, int page_size, int maxb, int window, float scale,
-                       float softcap, int splits, int keep_first, int sink, IxRows rows,
+                       float softcap, int splits, int keep_first, IxRows rows,
                        IxDistance dist) {
   extern __shared__ float sm[];
   float* sm_acc = sm;                               // [G][DA_WARPS][vd]
@@ -194,14 +194,15 @@ attn_decode_any_kernel(const TA* __restrict__ q, const TA* __restrict__ kc,
     }
     const size_t hrow = (size_t)s * heads + h0 + g;
     if (splits == 1) {
-      if (sink && M != -INFINITY) {
-        const float top = fmaxf(M, 0.f);
+      if (rows.sink && M != -INFINITY) {
+        const float sk = rows.sink[h0 + g];
+        const float top = fmaxf(M, sk);
         const float c = expf(M - top);
         o *= c;
-        L = L * c + expf(-top);
+        L = L * c + expf(sk - top);
       }
       out[(size_t)s * rows.o_ld + (size_t)(h0 + g) * vd + d] =
-          from_f32<TA>(L > 0.f ? o / L * rows.o_scale : 0.f);
+          from_f32<TA>(L > 0.f ? o / L * ix_result_factor<TA>(rows, s, h0 + g) : 0.f);
     } else {
       part_o[(hrow * splits + split) * vd + d] = o;
       if (d == 0) {
@@ -216,7 +217,7 @@ template <typename TA>
 __global__ void attn_decode_any_merge_kernel(const float* __restrict__ part_o,
                                              const float* __restrict__ part_ml,
                                              TA* __restrict__ out, int heads, int vd,
-                                             int splits, int sink, IxRows rows) {
+                                             int splits, IxRows rows) {
   IX_PDL_WAIT();
   const size_t hrow = blockIdx.x;   // s * heads + h
   const float* ml = part_ml + hrow * splits * 2;
@@ -226,18 +227,20 @@ __global__ void attn_decode_any_merge_kernel(const float* __restrict__ part_o,
   for (int j = 0; j < splits; ++j)
     if (ml[2 * j] != -INFINITY) L = fmaf(ml[2 * j + 1], expf(ml[2 * j] - M), L);
   float c = 1.f;
-  if (sink && M != -INFINITY) {
-    const float top = fmaxf(M, 0.f);
+  if (rows.sink && M != -INFINITY) {
+    const float sk = rows.sink[hrow % heads];
+    const float top = fmaxf(M, sk);
     c = expf(M - top);
-    L = L * c + expf(-top);
+    L = L * c + expf(sk - top);
   }
+  const float factor = ix_result_factor<TA>(rows, hrow / heads, (int)(hrow % heads));
   for (int d = threadIdx.x; d < vd; d += blockDim.x) {
     float o = 0.f;
     for (int j = 0; j < splits; ++j)
       if (ml[2 * j] != -INFINITY)
         o = fmaf(part_o[(hrow * splits + j) * vd + d], expf(ml[2 * j] - M), o);
     out[hrow / heads * rows.o_ld + hrow % heads * vd + d] =
-        from_f32<TA>(L > 0.f ? o * c / L * rows.o_scale : 0.f);
+        from_f32<TA>(L > 0.f ? o * c / L * factor : 0.f);
   }
 }
 
@@ -272,7 +275,7 @@ static int decode_any_checked(const void* q, const void* k_cache, const void* v_
                               const int* block_table, const int* kv_len, float* part_o,
                               float* part_ml, void* out, int act_dtype, int S, int heads, int kvh,
                               int hd, int vd, int page_size, int max_blocks, int window,
-                              float scale, float softcap, int splits, int keep_first, int sink,
+                              float scale, float softcap, int splits, int keep_first,
                               IxRows rows, IxDistance dist, cudaStream_t stream) {
   if (S <= 0) return IX_OK;
   if (heads <= 0 || kvh <= 0 || heads % kvh != 0 || page_size <= 0 || max_blocks <= 0)
@@ -295,7 +298,7 @@ static int decode_any_checked(const void* q, const void* k_cache, const void* v_
       cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);      \
     ix_launch(kern, grid, dim3(DA_THREADS), smem, stream, (const TA*)q, (const TA*)k_cache,    \
               (const TA*)v_cache, block_table, kv_len, part_o, part_ml, (TA*)out, heads, kvh,  \
-              hd, vd, page_size, max_blocks, window, scale, softcap, splits, keep_first, sink, \
+              hd, vd, page_size, max_blocks, window, scale, softcap, splits, keep_first, \
               rows, dist);                                                                     \
   })
 #define DA_D(DD)                                                                               \
@@ -315,7 +318,7 @@ static int decode_any_checked(const void* q, const void* k_cache, const void* v_
   if (rc != 0 || splits == 1) return rc;
   IX_DISPATCH_DTYPE(act_dtype, TA, {
     ix_launch(attn_decode_any_merge_kernel<TA>, dim3(S * heads), dim3(vd >= 128 ? 128 : 64), 0,
-              stream, (const float*)part_o, (const float*)part_ml, (TA*)out, heads, vd, splits, sink,
+              stream, (const float*)part_o, (const float*)part_ml, (TA*)out, heads, vd, splits,
               rows);
   });
   return ix_launch_status();
@@ -326,11 +329,13 @@ IX_API int ix_paged_attention_decode_any(const void* q, const void* k_cache, con
                                          float* part_ml, void* out, int act_dtype, int S, int heads,
                                          int kvh, int hd, int vd, int page_size, int max_blocks,
                                          int window, float scale, float softcap, int splits,
-                                         int keep_first, int sink, cudaStream_t stream) {
+                                         int keep_first, const float* sink, const void* gate,
+                                         long long gate_ld, cudaStream_t stream) {
   return decode_any_checked(q, k_cache, v_cache, block_table, kv_len, part_o, part_ml, out,
                             act_dtype, S, heads, kvh, hd, vd, page_size, max_blocks, window, scale,
-                            softcap, splits, keep_first, sink,
-                            IxRows{(long long)heads * hd, (long long)heads * vd, 1.f},
+                            softcap, splits, keep_first,
+                            IxRows{(long long)heads * hd, (long long)heads * vd, 1.f, sink, gate,
+                                   gate_ld},
                             ix_no_distance(), stream);
 }
 
@@ -344,6 +349,6 @@ IX_API int ix_distance_attention_decode_any(
   if (!temp || !r1 || !r2 || chunk < 0) return IX_ERR_SIZE;
   return decode_any_checked(q, k_cache, v_cache, block_table, kv_len, part_o, part_ml, out,
                             act_dtype, S, heads, kvh, hd, vd, page_size, max_blocks, 0, scale, 0.f,
-                            splits, 0, 0, IxRows{q_ld, o_ld, o_scale},
+                            splits, 0, IxRows{q_ld, o_ld, o_scale},
                             IxDistance{temp, r1, r2, chunk}, stream);
 }

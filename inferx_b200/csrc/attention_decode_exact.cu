@@ -20,7 +20,8 @@
 //  * value heads of a size of their own (64 or 128, as the keys');
 //  * `keep_first`: the sequence's first keep_first keys stay visible beside the window;
 //    the walk goes over them and then over the window as one range that is split;
-//  * `sink`: one is added to the denominator where the result is normalised.
+//  * a sink per head joins the denominator, and a gate per (token, head) multiplies the
+//    result, where it is normalised (IxRows).
 //  * DIST: a score is multiplied by its head's temperature and loses r1 ln(1 + r2 distance),
 //    and the query may be confined to its own run of positions (attention_distance.cuh).
 //
@@ -77,7 +78,7 @@ attn_decode_exact_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc
                          const int* __restrict__ kv_len, float* __restrict__ part_o,
                          float* __restrict__ part_ml, bf16* __restrict__ out, int heads, int kvh,
                          int page_size, int page_shift, int maxb, int window, float scale_log2e,
-                         int splits, int keep_first, int sink, IxRows rows,
+                         int splits, int keep_first, IxRows rows,
                          IxDistance dist) {
   constexpr int CH = HD / 8, CHV = VD / 8, KS = HD / 16, DT = VD / 8;
   constexpr int K_TILE = DX_BN * HD * 2, V_TILE = DX_BN * VD * 2;
@@ -322,14 +323,15 @@ attn_decode_exact_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc
     }
     const size_t hrow = (size_t)s * heads + h0 + r;
     if (splits == 1) {
-      if (sink && M != -INFINITY) {        // one more term, 2^(0 - max), in the denominator
-        const float top = fmaxf(M, 0.f);
+      if (rows.sink && M != -INFINITY) {   // one more term, 2^(sink - max), in the denominator
+        const float sk = rows.sink[h0 + r] * 1.4426950408889634f;
+        const float top = fmaxf(M, sk);
         const float c = dx_exp2(M - top);
         ov *= c;
-        L = L * c + dx_exp2(-top);
+        L = L * c + dx_exp2(sk - top);
       }
       out[(size_t)s * rows.o_ld + (size_t)(h0 + r) * VD + d] =
-          __float2bfloat16_rn(L > 0.f ? ov / L * rows.o_scale : 0.f);
+          __float2bfloat16_rn(L > 0.f ? ov / L * ix_result_factor<bf16>(rows, s, h0 + r) : 0.f);
     } else {
       part_o[(hrow * splits + split) * VD + d] = ov;
       if (d == 0) {
@@ -343,7 +345,7 @@ attn_decode_exact_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc
 __global__ void attn_decode_exact_merge_kernel(const float* __restrict__ part_o,
                                                const float* __restrict__ part_ml,
                                                bf16* __restrict__ out, int heads, int vd,
-                                               int splits, int sink, IxRows rows) {
+                                               int splits, IxRows rows) {
   IX_PDL_WAIT();
   const size_t hrow = blockIdx.x;   // s * heads + h
   const float* ml = part_ml + hrow * splits * 2;
@@ -353,18 +355,20 @@ __global__ void attn_decode_exact_merge_kernel(const float* __restrict__ part_o,
   for (int j = 0; j < splits; ++j)
     if (ml[2 * j] != -INFINITY) L += ml[2 * j + 1] * dx_exp2(ml[2 * j] - M);
   float c = 1.f;
-  if (sink && M != -INFINITY) {
-    const float top = fmaxf(M, 0.f);
+  if (rows.sink && M != -INFINITY) {
+    const float sk = rows.sink[hrow % heads] * 1.4426950408889634f;
+    const float top = fmaxf(M, sk);
     c = dx_exp2(M - top);
-    L = L * c + dx_exp2(-top);
+    L = L * c + dx_exp2(sk - top);
   }
+  const float factor = ix_result_factor<bf16>(rows, hrow / heads, (int)(hrow % heads));
   for (int d = threadIdx.x; d < vd; d += blockDim.x) {
     float o = 0.f;
     for (int j = 0; j < splits; ++j)
       if (ml[2 * j] != -INFINITY)
         o += part_o[(hrow * splits + j) * vd + d] * dx_exp2(ml[2 * j] - M);
     out[hrow / heads * rows.o_ld + hrow % heads * vd + d] =
-        __float2bfloat16_rn(L > 0.f ? o * c / L * rows.o_scale : 0.f);
+        __float2bfloat16_rn(L > 0.f ? o * c / L * factor : 0.f);
   }
 }
 
@@ -372,7 +376,7 @@ template <int HD, int VD>
 static int launch_decode_exact(const void* q, const void* kc, const void* vc, const int* bt,
                                const int* kv_len, float* part_o, float* part_ml, void* out, int S,
                                int heads, int kvh, int page_size, int maxb, int window,
-                               float scale, int splits, int keep_first, int sink, IxRows rows,
+                               float scale, int splits, int keep_first, IxRows rows,
                                IxDistance dist, cudaStream_t stream) {
   const int rep = heads / kvh;
   const float sl2 = scale * 1.4426950408889634f;
@@ -389,7 +393,7 @@ static int launch_decode_exact(const void* q, const void* kc, const void* vc, co
     if (e != cudaSuccess) return (int)e;                                                        \
     ix_launch(kern, grid, dim3(DX_THREADS), smem, stream, (const bf16*)q, (const bf16*)kc,      \
               (const bf16*)vc, bt, kv_len, part_o, part_ml, (bf16*)out, heads, kvh, page_size,  \
-              page_shift, maxb, window, sl2, splits, keep_first, sink, rows, dist);             \
+              page_shift, maxb, window, sl2, splits, keep_first, rows, dist);             \
   } while (0)
   if (dist.temp) {
     if (rep <= 8) DX_LAUNCH(true, true);
@@ -402,7 +406,7 @@ static int launch_decode_exact(const void* q, const void* kc, const void* vc, co
   int rc = ix_launch_status();
   if (rc != 0 || splits == 1) return rc;
   ix_launch(attn_decode_exact_merge_kernel, dim3(S * heads), dim3(VD >= 128 ? 128 : 64), 0,
-            stream, (const float*)part_o, (const float*)part_ml, (bf16*)out, heads, VD, splits, sink,
+            stream, (const float*)part_o, (const float*)part_ml, (bf16*)out, heads, VD, splits,
             rows);
   return ix_launch_status();
 }
@@ -416,7 +420,7 @@ static int decode_exact_checked(const void* q, const void* k_cache, const void* 
                                 const int* block_table, const int* kv_len, float* part_o,
                                 float* part_ml, void* out, int S, int heads, int kvh, int hd,
                                 int vd, int page_size, int max_blocks, int window, float scale,
-                                int splits, int keep_first, int sink, IxRows rows,
+                                int splits, int keep_first, IxRows rows,
                                 IxDistance dist, cudaStream_t stream) {
   if (S <= 0) return IX_OK;
   if (heads <= 0 || kvh <= 0 || heads % kvh != 0 || page_size <= 0 || max_blocks <= 0 ||
@@ -430,7 +434,7 @@ static int decode_exact_checked(const void* q, const void* k_cache, const void* 
   if (hd == H_ && vd == V_)                                                                   \
     return launch_decode_exact<H_, V_>(q, k_cache, v_cache, block_table, kv_len, part_o,      \
                                        part_ml, out, S, heads, kvh, page_size, max_blocks,    \
-                                       window, scale, splits, keep_first, sink, rows, dist,   \
+                                       window, scale, splits, keep_first, rows, dist,   \
                                        stream);
   DX_GO(64, 64)
   DX_GO(64, 128)
@@ -445,12 +449,13 @@ IX_API int ix_paged_attention_decode_exact(const void* q, const void* k_cache,
                                            const int* kv_len, float* part_o, float* part_ml,
                                            void* out, int S, int heads, int kvh, int hd, int vd,
                                            int page_size, int max_blocks, int window, float scale,
-                                           int splits, int keep_first, int sink,
-                                           cudaStream_t stream) {
+                                           int splits, int keep_first, const float* sink,
+                                           const void* gate, long long gate_ld, cudaStream_t stream) {
   return decode_exact_checked(q, k_cache, v_cache, block_table, kv_len, part_o, part_ml, out, S,
                               heads, kvh, hd, vd, page_size, max_blocks, window, scale, splits,
-                              keep_first, sink,
-                              IxRows{(long long)heads * hd, (long long)heads * vd, 1.f},
+                              keep_first,
+                              IxRows{(long long)heads * hd, (long long)heads * vd, 1.f, sink, gate,
+                                     gate_ld},
                               ix_no_distance(), stream);
 }
 
@@ -463,7 +468,7 @@ IX_API int ix_distance_attention_decode_exact(
     int chunk, cudaStream_t stream) {
   if (!temp || !r1 || !r2 || chunk < 0) return IX_ERR_SIZE;
   return decode_exact_checked(q, k_cache, v_cache, block_table, kv_len, part_o, part_ml, out, S,
-                              heads, kvh, hd, vd, page_size, max_blocks, 0, scale, splits, 0, 0,
+                              heads, kvh, hd, vd, page_size, max_blocks, 0, scale, splits, 0,
                               IxRows{q_ld, o_ld, o_scale}, IxDistance{temp, r1, r2, chunk},
                               stream);
 }

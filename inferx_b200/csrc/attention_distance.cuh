@@ -18,13 +18,29 @@ struct IxDistance {
 
 // Where a kernel reads queries and writes results: token t of q starts at t * q_ld, of the
 // output at t * o_ld (elements); results are multiplied by o_scale before they are rounded.
+// What else happens to a (token, head) pair's result where it is normalised and written:
+// `sink` (null: none) holds a number per query head whose exponential joins the softmax's
+// denominator, a key with that score and no value; `gate` (null: none) holds a number per
+// (token, head), row t at t * gate_ld, in the activations' type: the result is multiplied by
+// its sigmoid.
 struct IxRows {
   long long q_ld, o_ld;
   float o_scale;
+  const float* sink;
+  const void* gate;
+  long long gate_ld;
 };
 
 __host__ __device__ __forceinline__ IxDistance ix_no_distance() {
   return IxDistance{nullptr, nullptr, nullptr, 0};
+}
+
+// o_scale times the head's gate, where there is one.
+template <typename TA>
+__device__ __forceinline__ float ix_result_factor(const IxRows& rows, long long token, int head) {
+  if (!rows.gate) return rows.o_scale;
+  const float z = to_f32(reinterpret_cast<const TA*>(rows.gate)[token * rows.gate_ld + head]);
+  return rows.o_scale / (1.0f + expf(-z));
 }
 
 // The first key a query at position `pos` can see.

@@ -17,8 +17,8 @@
 //
 // Two options of windowed attention: `keep_first` > 0 keeps the sequence's first
 // keep_first keys visible beside the window (they are walked first, as if they stood
-// directly before the window), and `sink` adds one to the softmax's denominator (a key
-// of score 0 that has no value).
+// directly before the window), and a sink per head joins the softmax's denominator (a
+// key of that score that has no value); IxRows has it, and a gate per (token, head).
 //
 // A third form (attention_distance.cuh) multiplies a score by its head's temperature, takes
 // r1 ln(1 + r2 distance) off and may confine a query to its own run of positions.
@@ -36,7 +36,7 @@ paged_attention_generic_kernel(const TA* __restrict__ q, const TA* __restrict__ 
                                const int* __restrict__ positions, TA* __restrict__ out, int heads,
                                int kvh, int hd, int vd, int page_size, int max_blocks,
                                int window, float scale, float softcap, int keep_first,
-                               int sink, IxRows rows, IxDistance dist) {
+                               IxRows rows, IxDistance dist) {
   extern __shared__ float smem[];
   float* qs = smem;        // [hd]
   float* sc = smem + hd;   // [ATT_TILE]
@@ -113,15 +113,17 @@ paged_attention_generic_kernel(const TA* __restrict__ q, const TA* __restrict__ 
   }
   TA* orow = out + (size_t)t * rows.o_ld + (size_t)h * vd;
   float inv_l = 1.0f / l;
-  if (sink) {          // one more term, exp(0 - max), in the denominator
-    const float top = fmaxf(m, 0.f);
+  if (rows.sink) {     // one more term, exp(sink - max), in the denominator
+    const float sk = rows.sink[h];
+    const float top = fmaxf(m, sk);
     const float c = expf(m - top);
-    inv_l = c / (l * c + expf(-top));
+    inv_l = c / (l * c + expf(sk - top));
   }
+  const float factor = ix_result_factor<TA>(rows, t, h);
 #pragma unroll
   for (int i = 0; i < ATT_MAX_DPT; ++i) {
     const int d = threadIdx.x + i * ATT_THREADS;
-    if (d < vd) orow[d] = from_f32<TA>(acc[i] * inv_l * rows.o_scale);
+    if (d < vd) orow[d] = from_f32<TA>(acc[i] * inv_l * factor);
   }
 }
 
@@ -133,7 +135,7 @@ static int generic_checked(const void* q, const void* k_cache, const void* v_cac
                            const int* block_table, const int* seq_of_token, const int* positions,
                            void* out, int act_dtype, int T, int heads, int kvh, int hd, int vd,
                            int page_size, int max_blocks, int window, float scale, float softcap,
-                           int keep_first, int sink, IxRows rows, IxDistance dist,
+                           int keep_first, IxRows rows, IxDistance dist,
                            cudaStream_t stream) {
   if (T <= 0) return IX_OK;
   if (heads <= 0 || kvh <= 0 || heads % kvh != 0 || page_size <= 0 || max_blocks <= 0)
@@ -148,7 +150,7 @@ static int generic_checked(const void* q, const void* k_cache, const void* v_cac
                     (paged_attention_generic_kernel<TA><<<grid, ATT_THREADS, smem, stream>>>(
                         (const TA*)q, (const TA*)k_cache, (const TA*)v_cache, block_table,
                         seq_of_token, positions, (TA*)out, heads, kvh, hd, vd, page_size,
-                        max_blocks, window, scale, softcap, keep_first, sink, rows, dist)));
+                        max_blocks, window, scale, softcap, keep_first, rows, dist)));
   return ix_launch_status();
 }
 
@@ -157,10 +159,13 @@ IX_API int ix_paged_attention_generic(const void* q, const void* k_cache, const 
                                       const int* positions, void* out, int act_dtype, int T,
                                       int heads, int kvh, int hd, int vd, int page_size,
                                       int max_blocks, int window, float scale, float softcap,
-                                      int keep_first, int sink, cudaStream_t stream) {
+                                      int keep_first, const float* sink, const void* gate,
+                                      long long gate_ld, cudaStream_t stream) {
   return generic_checked(q, k_cache, v_cache, block_table, seq_of_token, positions, out, act_dtype,
                          T, heads, kvh, hd, vd, page_size, max_blocks, window, scale, softcap,
-                         keep_first, sink, IxRows{(long long)heads * hd, (long long)heads * vd, 1.f},
+                         keep_first,
+                         IxRows{(long long)heads * hd, (long long)heads * vd, 1.f, sink, gate,
+                                gate_ld},
                          ix_no_distance(), stream);
 }
 
@@ -173,6 +178,6 @@ IX_API int ix_distance_attention_generic(
     const float* r2, int chunk, cudaStream_t stream) {
   if (!temp || !r1 || !r2 || chunk < 0) return IX_ERR_SIZE;
   return generic_checked(q, k_cache, v_cache, block_table, seq_of_token, positions, out, act_dtype,
-                         T, heads, kvh, hd, vd, page_size, max_blocks, 0, scale, 0.f, 0, 0,
+                         T, heads, kvh, hd, vd, page_size, max_blocks, 0, scale, 0.f, 0,
                          IxRows{q_ld, o_ld, o_scale}, IxDistance{temp, r1, r2, chunk}, stream);
 }

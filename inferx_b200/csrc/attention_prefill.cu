@@ -278,7 +278,8 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc,
 // (each weight enters as its bfloat16 rounding plus the bfloat16 rounding of the rest, two
 // tensor-core products into the same fp32 accumulator), value heads of a size of their own
 // (64 or 128 each), optionally the sequence's first `keep_first` keys visible beside the
-// window and one added to the softmax's denominator (`sink`).  For decoders that want their
+// window, a sink per head in the softmax's denominator and a gate per (token, head) on the
+// result (IxRows).  For decoders that want their
 // attention weights in 32-bit arithmetic: the scores are exact products of bfloat16 numbers
 // summed in fp32, maxima, exponentials and sums are fp32, and the weights lose nothing a
 // bfloat16 value would not lose many times over.  DIST: a score is multiplied by its head's
@@ -291,7 +292,7 @@ attn_prefill_exact_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k
                     const int* __restrict__ cu_q, const int* __restrict__ q_pos0,
                     bf16* __restrict__ out, int S, int heads, int kvh, int page_size,
                     int page_shift, int maxb, int window, float scale_log2e,
-                          int keep_first, int sink, IxRows rows, IxDistance dist) {
+                          int keep_first, IxRows rows, IxDistance dist) {
   constexpr int CH = HD / 8;            // 16-byte chunks per row
   constexpr int KS = HD / 16;           // k-steps of Q K^T
   constexpr int CHV = VD / 8;           // 16-byte chunks per value row
@@ -511,15 +512,20 @@ attn_prefill_exact_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k
     l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 1);
     l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
   }
-  float inv_a = l_run[0] > 0.f ? rows.o_scale / l_run[0] : 0.f;
-  float inv_b = l_run[1] > 0.f ? rows.o_scale / l_run[1] : 0.f;
-  if (sink) {      // one more term in the denominator: 2^(0 - max), maxima being in log2 units
+  const float fac_a =
+      row_a < rows_valid ? ix_result_factor<bf16>(rows, tok0 + q0 + row_a, h) : 0.f;
+  const float fac_b =
+      row_b < rows_valid ? ix_result_factor<bf16>(rows, tok0 + q0 + row_b, h) : 0.f;
+  float inv_a = l_run[0] > 0.f ? fac_a / l_run[0] : 0.f;
+  float inv_b = l_run[1] > 0.f ? fac_b / l_run[1] : 0.f;
+  if (rows.sink) {   // one more term in the denominator: 2^(sink - max), all in log2 units
+    const float sk = rows.sink[h] * 1.4426950408889634f;
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
       if (!(l_run[r] > 0.f)) continue;
-      const float top = fmaxf(m_run[r], 0.f);
+      const float top = fmaxf(m_run[r], sk);
       const float c = fast_exp2(m_run[r] - top);
-      const float inv = rows.o_scale * c / (l_run[r] * c + fast_exp2(-top));
+      const float inv = (r == 0 ? fac_a : fac_b) * c / (l_run[r] * c + fast_exp2(sk - top));
       if (r == 0) inv_a = inv; else inv_b = inv;
     }
   }
@@ -587,7 +593,7 @@ template <int HD, int VD, bool DIST>
 static int launch_prefill_exact(const void* q, const void* kc, const void* vc, const int* bt,
                                 const int* cu_q, const int* q_pos0, void* out, int T, int S,
                                 int heads, int kvh, int page_size, int maxb, int window,
-                                float scale, int keep_first, int sink, IxRows rows,
+                                float scale, int keep_first, IxRows rows,
                                 IxDistance dist, cudaStream_t stream) {
   const size_t smem = (size_t)(PF_BM + 2 * PF_BN) * HD * 2 + (size_t)2 * PF_BN * VD * 2;
   auto kern = attn_prefill_exact_kernel<HD, VD, DIST>;
@@ -605,7 +611,7 @@ static int launch_prefill_exact(const void* q, const void* kc, const void* vc, c
   kern<<<grid, PF_THREADS, smem, stream>>>((const bf16*)q, (const bf16*)kc, (const bf16*)vc, bt,
                                            cu_q, q_pos0, (bf16*)out, S, heads, kvh, page_size,
                                            page_shift, maxb, window,
-                                           scale * 1.4426950408889634f, keep_first, sink, rows,
+                                           scale * 1.4426950408889634f, keep_first, rows,
                                            dist);
   return ix_launch_status();
 }
@@ -619,7 +625,7 @@ static int prefill_exact_checked(const void* q, const void* k_cache, const void*
                                  const int* block_table, const int* cu_q, const int* q_pos0,
                                  void* out, int T, int S, int heads, int kvh, int hd, int vd,
                                  int page_size, int max_blocks, int window, float scale,
-                                 int keep_first, int sink, IxRows rows, IxDistance dist,
+                                 int keep_first, IxRows rows, IxDistance dist,
                                  cudaStream_t stream) {
   if (T <= 0 || S <= 0) return IX_OK;
   if (heads <= 0 || kvh <= 0 || heads % kvh != 0 || page_size <= 0 || max_blocks <= 0 ||
@@ -634,11 +640,11 @@ static int prefill_exact_checked(const void* q, const void* k_cache, const void*
                ? launch_prefill_exact<H_, V_, true>(q, k_cache, v_cache, block_table, cu_q,    \
                                                     q_pos0, out, T, S, heads, kvh, page_size,  \
                                                     max_blocks, window, scale, keep_first,     \
-                                                    sink, rows, dist, stream)                  \
+                                                    rows, dist, stream)                        \
                : launch_prefill_exact<H_, V_, false>(q, k_cache, v_cache, block_table, cu_q,   \
                                                      q_pos0, out, T, S, heads, kvh, page_size, \
                                                      max_blocks, window, scale, keep_first,    \
-                                                     sink, rows, dist, stream);
+                                                     rows, dist, stream);
   PF_EXACT(64, 64)
   PF_EXACT(64, 128)
   PF_EXACT(128, 64)
@@ -652,10 +658,12 @@ IX_API int ix_paged_attention_prefill_exact(const void* q, const void* k_cache,
                                             const int* cu_q, const int* q_pos0, void* out, int T,
                                             int S, int heads, int kvh, int hd, int vd,
                                             int page_size, int max_blocks, int window, float scale,
-                                            int keep_first, int sink, cudaStream_t stream) {
+                                            int keep_first, const float* sink, const void* gate,
+                                            long long gate_ld, cudaStream_t stream) {
   return prefill_exact_checked(q, k_cache, v_cache, block_table, cu_q, q_pos0, out, T, S, heads,
-                               kvh, hd, vd, page_size, max_blocks, window, scale, keep_first, sink,
-                               IxRows{(long long)heads * hd, (long long)heads * vd, 1.f},
+                               kvh, hd, vd, page_size, max_blocks, window, scale, keep_first,
+                               IxRows{(long long)heads * hd, (long long)heads * vd, 1.f, sink, gate,
+                                      gate_ld},
                                ix_no_distance(), stream);
 }
 
@@ -668,7 +676,7 @@ IX_API int ix_distance_attention_prefill_exact(
     cudaStream_t stream) {
   if (!temp || !r1 || !r2 || chunk < 0) return IX_ERR_SIZE;
   return prefill_exact_checked(q, k_cache, v_cache, block_table, cu_q, q_pos0, out, T, S, heads,
-                               kvh, hd, vd, page_size, max_blocks, 0, scale, 0, 0,
+                               kvh, hd, vd, page_size, max_blocks, 0, scale, 0,
                                IxRows{q_ld, o_ld, o_scale}, IxDistance{temp, r1, r2, chunk},
                                stream);
 }

@@ -95,7 +95,7 @@ __device__ __forceinline__ float fa_max3(float a, float b, float c) {
 // that left over: the second term takes the 32 columns of the score buffer that the first
 // leaves free, and a second product adds it into the same accumulator (16 bits of the
 // weight).  The sequence's first `keep_first` keys stay visible beside the window (their
-// tiles are walked first) and `sink` adds one to the softmax's denominator.  One run of
+// tiles are walked first) and a sink per head joins the softmax's denominator.  One run of
 // keys per query tile (nsplit 1).
 // DIST (with EXACT): a score is multiplied by its head's temperature and loses r1 ln(1 + r2
 // distance), and a query may be confined to its own run of positions (attention_distance.cuh).
@@ -112,7 +112,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                        int kvh, int page_size, int page_shift, int maxb, int window,
                        float scale_log2e, int* __restrict__ status, int nsplit,
                        float* __restrict__ part_o, float* __restrict__ part_ml, float cap_c1,
-                       float cap_over_scale, int keep_first, int sink, IxRows rows,
+                       float cap_over_scale, int keep_first, IxRows rows,
                        IxDistance dist) {
   constexpr int HALVES = HD / 64;
   constexpr int Q_BYTES = FA_BM * HD * 2;
@@ -467,11 +467,15 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
       }
     } else if (n_tiles > 0) {
       tc_fence_after();
-      float inv = l_run > 0.f ? rows.o_scale / l_run : 0.f;
-      if (EXACT && sink && l_run > 0.f) {   // one more term, 2^(0 - reference), in the denominator
-        const float top = fmaxf(m_ref, 0.f);
+      const float factor = EXACT && row < rows_valid
+                               ? ix_result_factor<bf16>(rows, tok0 + q0 + row, h)
+                               : rows.o_scale;
+      float inv = l_run > 0.f ? factor / l_run : 0.f;
+      if (EXACT && rows.sink && l_run > 0.f) {   // one more term, 2^(sink - reference)
+        const float sk = rows.sink[h] * 1.4426950408889634f;
+        const float top = fmaxf(m_ref, sk);
         const float c = fa_exp2(m_ref - top);
-        inv = rows.o_scale * c / (l_run * c + fa_exp2(-top));
+        inv = factor * c / (l_run * c + fa_exp2(sk - top));
       }
       bf16* dst = out + (size_t)(tok0 + q0 + row) * rows.o_ld + (size_t)h * HD;
 #pragma unroll
@@ -540,7 +544,7 @@ static int launch_prefill_tc(const void* q, const void* kc, const void* vc, long
                              int S, int heads, int kvh, int page_size, int page_shift, int maxb,
                              int window, float scale, float softcap, int* status, int nsplit,
                              float* part_o, float* part_ml, cudaStream_t stream,
-                             int keep_first = 0, int sink = 0, IxRows rows = {0, 0, 1.f},
+                             int keep_first = 0, IxRows rows = {0, 0, 1.f},
                              IxDistance dist = ix_no_distance()) {
   CUtensorMap map_q, map_k, map_v;
   if (rows.q_ld == 0) rows.q_ld = rows.o_ld = (long long)heads * HD;
@@ -564,7 +568,7 @@ static int launch_prefill_tc(const void* q, const void* kc, const void* vc, long
                                            part_ml,
                                            softcap > 0.f ? 2.f * scale * 1.4426950408889634f / softcap
                                                          : 0.f,
-                                           softcap > 0.f ? softcap / scale : 0.f, keep_first, sink,
+                                           softcap > 0.f ? softcap / scale : 0.f, keep_first,
                                            rows, dist);
   rc = ix_launch_status();
   if (rc != IX_OK || nsplit == 1) return rc;
@@ -657,7 +661,8 @@ static int prefill_tc_checked(const void* q, const void* k_cache, const void* v_
 }
 
 // The EXACT form: weights of 16 bits in their product with the values, the sequence's first
-// `keep_first` keys kept beside the window, `sink` for one more term in the denominator.
+// `keep_first` keys kept beside the window, `sink` (per head) for one more term in the
+// denominator, `gate` (per token and head) for a factor sigmoid(gate) on the result.
 IX_API int ix_paged_attention_prefill_tc_exact_applies(int hd, int vd, int page_size) {
   return hd == vd && (hd == 64 || hd == 128) &&
          (page_size == 8 || page_size == 16 || page_size == 32 || page_size == 64);
@@ -667,7 +672,8 @@ IX_API int ix_paged_attention_prefill_tc_exact(
     const void* q, const void* k_cache, const void* v_cache, int num_pages,
     const int* block_table, const int* cu_q, const int* q_pos0, void* out, int T, int S,
     int heads, int kvh, int hd, int page_size, int max_blocks, int window, float scale,
-    int keep_first, int sink, int* status, cudaStream_t stream) {
+    int keep_first, const float* sink, const void* gate, long long gate_ld, int* status,
+    cudaStream_t stream) {
   if (T <= 0 || S <= 0) return IX_OK;
   if (heads <= 0 || kvh <= 0 || heads % kvh != 0 || max_blocks <= 0 || window < 0 ||
       keep_first < 0 || num_pages <= 0 || status == nullptr || heads > 65535 || !(scale > 0.f))
@@ -679,15 +685,16 @@ IX_API int ix_paged_attention_prefill_tc_exact(
   while ((1 << page_shift) < page_size) ++page_shift;
   const long long cache_rows = (long long)num_pages * kvh * page_size;
   if (cache_rows > 0x7fffffffLL) return IX_ERR_SIZE;
+  const IxRows rows = {(long long)heads * hd, (long long)heads * hd, 1.f, sink, gate, gate_ld};
   if (hd == 128)
     return launch_prefill_tc<128, true>(q, k_cache, v_cache, cache_rows, block_table, cu_q,
                                         q_pos0, out, T, S, heads, kvh, page_size, page_shift,
                                         max_blocks, window, scale, 0.f, status, 1, nullptr,
-                                        nullptr, stream, keep_first, sink);
+                                        nullptr, stream, keep_first, rows);
   return launch_prefill_tc<64, true>(q, k_cache, v_cache, cache_rows, block_table, cu_q, q_pos0,
                                      out, T, S, heads, kvh, page_size, page_shift, max_blocks,
                                      window, scale, 0.f, status, 1, nullptr, nullptr, stream,
-                                     keep_first, sink);
+                                     keep_first, rows);
 }
 
 // The EXACT form with a temperature and a distance penalty per head (attention_distance.cuh).
@@ -717,9 +724,9 @@ IX_API int ix_distance_attention_prefill_tc(
     return launch_prefill_tc<128, true, true>(q, k_cache, v_cache, cache_rows, block_table, cu_q,
                                               q_pos0, out, T, S, heads, kvh, page_size, page_shift,
                                               max_blocks, 0, scale, 0.f, status, 1, nullptr,
-                                              nullptr, stream, 0, 0, rows, dist);
+                                              nullptr, stream, 0, rows, dist);
   return launch_prefill_tc<64, true, true>(q, k_cache, v_cache, cache_rows, block_table, cu_q,
                                            q_pos0, out, T, S, heads, kvh, page_size, page_shift,
                                            max_blocks, 0, scale, 0.f, status, 1, nullptr, nullptr,
-                                           stream, 0, 0, rows, dist);
+                                           stream, 0, rows, dist);
 }

@@ -14,7 +14,7 @@
 //
 // With `keep_first` > 0 the sequence's first keep_first keys stay visible beside the
 // window: their tiles (also at multiples of 64) are walked before the window's.  With
-// `sink` one is added to the softmax's denominator.
+// a sink per head its exponential joins the softmax's denominator (IxRows).
 //
 // A third form (attention_distance.cuh) multiplies a score by its head's temperature, takes
 // r1 ln(1 + r2 distance) off and may confine a query to its own run of positions; the
@@ -59,7 +59,7 @@ paged_attention_tiled_kernel(const TA* __restrict__ q, const TA* __restrict__ kc
                              const int* __restrict__ cu_q, const int* __restrict__ q_pos0,
                              TA* __restrict__ out, int S, int heads, int kvh, int hd, int vd,
                              int page_size, int max_blocks, int window, float scale,
-                             float softcap, int keep_first, int sink, IxRows rows,
+                             float softcap, int keep_first, IxRows rows,
                              IxDistance dist) {
   extern __shared__ __align__(16) float tsm[];
   __shared__ float band[TA_BQ + TA_BK];          // penalty per distance, see below
@@ -255,11 +255,13 @@ paged_attention_tiled_kernel(const TA* __restrict__ q, const TA* __restrict__ kc
   for (int i = 0; i < 4; ++i) {
     const int r = 4 * ow + i;
     if (r >= rows_valid) continue;
-    float inv_l = rows.o_scale / l_run[r];
-    if (sink) {        // one more term, exp(0 - max), in the denominator
-      const float top = fmaxf(m_run[r], 0.f);
+    const float factor = ix_result_factor<TA>(rows, tok0 + r, h);
+    float inv_l = factor / l_run[r];
+    if (rows.sink) {   // one more term, exp(sink - max), in the denominator
+      const float sk = rows.sink[h];
+      const float top = fmaxf(m_run[r], sk);
       const float c = expf(m_run[r] - top);
-      inv_l = rows.o_scale * c / (l_run[r] * c + expf(-top));
+      inv_l = factor * c / (l_run[r] * c + expf(sk - top));
     }
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
@@ -281,7 +283,7 @@ static int tiled_checked(const void* q, const void* k_cache, const void* v_cache
                          const int* block_table, const int* cu_q, const int* q_pos0, void* out,
                          int act_dtype, int T, int S, int heads, int kvh, int hd, int vd,
                          int page_size, int max_blocks, int window, float scale, float softcap,
-                         int keep_first, int sink, IxRows rows, IxDistance dist,
+                         int keep_first, IxRows rows, IxDistance dist,
                          cudaStream_t stream) {
   if (T <= 0) return IX_OK;
   if (S <= 0 || heads <= 0 || kvh <= 0 || heads % kvh != 0 || page_size <= 0 || max_blocks <= 0 ||
@@ -308,7 +310,7 @@ static int tiled_checked(const void* q, const void* k_cache, const void* v_cache
     kern<<<grid, TA_THREADS, smem, stream>>>((const TA*)q, (const TA*)k_cache, (const TA*)v_cache,
                                              block_table, cu_q, q_pos0, (TA*)out, S, heads, kvh,
                                              hd, vd, page_size, max_blocks, window, scale,
-                                             softcap, keep_first, sink, rows, dist);
+                                             softcap, keep_first, rows, dist);
   });
   return ix_launch_status();
 }
@@ -317,12 +319,13 @@ IX_API int ix_paged_attention_tiled(const void* q, const void* k_cache, const vo
                                     const int* block_table, const int* cu_q, const int* q_pos0,
                                     void* out, int act_dtype, int T, int S, int heads, int kvh,
                                     int hd, int vd, int page_size, int max_blocks, int window,
-                                    float scale, float softcap, int keep_first, int sink,
-                                    cudaStream_t stream) {
+                                    float scale, float softcap, int keep_first, const float* sink,
+                                    const void* gate, long long gate_ld, cudaStream_t stream) {
   return tiled_checked(q, k_cache, v_cache, block_table, cu_q, q_pos0, out, act_dtype, T, S, heads,
-                       kvh, hd, vd, page_size, max_blocks, window, scale, softcap, keep_first, sink,
-                       IxRows{(long long)heads * hd, (long long)heads * vd, 1.f}, ix_no_distance(),
-                       stream);
+                       kvh, hd, vd, page_size, max_blocks, window, scale, softcap, keep_first,
+                       IxRows{(long long)heads * hd, (long long)heads * vd, 1.f, sink, gate,
+                              gate_ld},
+                       ix_no_distance(), stream);
 }
 
 // With a temperature and a distance penalty per head (see attention_distance.cuh).
@@ -334,6 +337,6 @@ IX_API int ix_distance_attention_tiled(
     cudaStream_t stream) {
   if (!temp || !r1 || !r2 || chunk < 0) return IX_ERR_SIZE;
   return tiled_checked(q, k_cache, v_cache, block_table, cu_q, q_pos0, out, act_dtype, T, S, heads,
-                       kvh, hd, vd, page_size, max_blocks, 0, scale, 0.f, 0, 0,
+                       kvh, hd, vd, page_size, max_blocks, 0, scale, 0.f, 0,
                        IxRows{q_ld, o_ld, o_scale}, IxDistance{temp, r1, r2, chunk}, stream);
 }

@@ -36,6 +36,18 @@ template <typename T> __device__ __forceinline__ T from_f32(float v);
 template <> __device__ __forceinline__ float from_f32<float>(float v) { return v; }
 template <> __device__ __forceinline__ bf16 from_f32<bf16>(float v) { return __float2bfloat16_rn(v); }
 
+// Activation of a product that has no gate beside it.
+enum { IX_ACT_NONE = 0, IX_ACT_GELU = 1, IX_ACT_RELU2 = 2 };   // gelu: the exact (erf) form
+
+__device__ __forceinline__ float ix_act(float v, int act) {
+  if (act == IX_ACT_GELU) return 0.5f * v * (1.0f + erff(v * 0.70710678118654752f));
+  if (act == IX_ACT_RELU2) {
+    v = fmaxf(v, 0.f);
+    return v * v;
+  }
+  return v;
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

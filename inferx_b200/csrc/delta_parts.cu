@@ -12,7 +12,7 @@
 //   gated delta rule    S = diag(g) S;  u = beta (v - S^T k);  S += k u^T;  o = S^T q
 //   gate + group norm   out = groupnorm(y * silu(z)) * gain
 //   normed pair mean    out = (l / rms(l) * gl + r / rms(r) * gr) / 2
-//   relu squared, table routing, scaling of rows
+//   activations (relu squared, gelu), table routing, scaling of rows
 //
 // Everything but the stored activations is fp32 with the accurate library functions.
 #include "common.cuh"
@@ -211,6 +211,7 @@ IX_API int ix_stream_concat(const float* resid, const void* delta, int delta_dty
 
 template <typename TA>
 __global__ void causal_conv_kernel(const TA* __restrict__ x, long long ldx,
+                                   const float* __restrict__ in_bias,
                                    const float* __restrict__ w, const float* __restrict__ bias,
                                    const float* __restrict__ state,
                                    const int* __restrict__ cu_q,
@@ -225,11 +226,12 @@ __global__ void causal_conv_kernel(const TA* __restrict__ x, long long ldx,
   const int begin = cu_q[s];
   const float* st = state + (size_t)state_slot[s] * (taps - 1) * C;
   float acc = bias ? bias[c] : 0.f;
+  const float ib = in_bias ? in_bias[c] : 0.f;
   for (int j = 0; j < taps; ++j) {
     const int src = t - (taps - 1) + j;          // token index of this tap's input
     float v;
     if (src >= begin) {
-      v = to_f32(x[(size_t)src * ldx + c]);
+      v = to_f32(x[(size_t)src * ldx + c]) + ib;
     } else {
       // begin - src inputs back from the step's first token: 1 is the newest kept one
       const int back = begin - src;               // 1 .. taps-1
@@ -257,7 +259,8 @@ __device__ __forceinline__ float2 pair_f32(__nv_bfloat162 v) {
 
 template <typename TA, int TAPS>
 __global__ void __launch_bounds__(CONV_THREADS)
-causal_conv_run_kernel(const TA* __restrict__ x, long long ldx, const float* __restrict__ w,
+causal_conv_run_kernel(const TA* __restrict__ x, long long ldx,
+                       const float* __restrict__ in_bias, const float* __restrict__ w,
                        const float* __restrict__ bias, const float* __restrict__ state,
                        const int* __restrict__ cu_q, const int* __restrict__ seq_of_token,
                        const int* __restrict__ state_slot, TA* __restrict__ out, int T, int C,
@@ -273,6 +276,7 @@ causal_conv_run_kernel(const TA* __restrict__ x, long long ldx, const float* __r
     wv[1][j] = w[(size_t)(c + 1) * TAPS + j];
   }
   const float b0 = bias ? bias[c] : 0.f, b1 = bias ? bias[c + 1] : 0.f;
+  const float ib0 = in_bias ? in_bias[c] : 0.f, ib1 = in_bias ? in_bias[c + 1] : 0.f;
   // the run's inputs are all on their way before the first is used
   typedef typename ConvPair<TA>::type P2;
   P2 raw[CONV_RUN];
@@ -291,8 +295,8 @@ causal_conv_run_kernel(const TA* __restrict__ x, long long ldx, const float* __r
       for (int j = 0; j < TAPS - 1; ++j) {
         const int src = t - (TAPS - 1) + j;
         if (src >= begin) {
-          win[0][j] = to_f32(x[(size_t)src * ldx + c]);
-          win[1][j] = to_f32(x[(size_t)src * ldx + c + 1]);
+          win[0][j] = to_f32(x[(size_t)src * ldx + c]) + ib0;
+          win[1][j] = to_f32(x[(size_t)src * ldx + c + 1]) + ib1;
         } else {
           const int back = begin - src;
           win[0][j] = st[(size_t)(TAPS - 1 - back) * C + c];
@@ -301,7 +305,7 @@ causal_conv_run_kernel(const TA* __restrict__ x, long long ldx, const float* __r
       }
     }
     const float2 cur = pair_f32(raw[i]);
-    const float cur0 = cur.x, cur1 = cur.y;
+    const float cur0 = cur.x + ib0, cur1 = cur.y + ib1;
     float a0 = b0, a1 = b1;
 #pragma unroll
     for (int j = 0; j < TAPS - 1; ++j) {
@@ -339,7 +343,7 @@ causal_conv_run_kernel(const TA* __restrict__ x, long long ldx, const float* __r
 // reads from the old state lies above what it has written.
 template <typename TA>
 __global__ void conv_state_update_kernel(const TA* __restrict__ x, long long ldx,
-                                         float* __restrict__ state, const int* __restrict__ cu_q,
+                                         const float* __restrict__ in_bias, float* __restrict__ state, const int* __restrict__ cu_q,
                                          const int* __restrict__ state_slot, int C, int taps) {
   IX_PDL_WAIT();
   const int s = blockIdx.x;
@@ -347,17 +351,20 @@ __global__ void conv_state_update_kernel(const TA* __restrict__ x, long long ldx
   if (c >= C) return;
   const int begin = cu_q[s], n = cu_q[s + 1] - begin;
   if (n <= 0) return;
+  const float ib = in_bias ? in_bias[c] : 0.f;
   float* st = state + (size_t)state_slot[s] * (taps - 1) * C;
   for (int i = 0; i < taps - 1; ++i) {
     const int src = n - (taps - 1) + i;           // index among this step's tokens
-    const float v = src >= 0 ? to_f32(x[(size_t)(begin + src) * ldx + c])
+    const float v = src >= 0 ? to_f32(x[(size_t)(begin + src) * ldx + c]) + ib
                              : st[(size_t)(i + n) * C + c];
     st[(size_t)i * C + c] = v;
   }
 }
 
-IX_API int ix_causal_conv(const void* x, int dtype, long long ldx, const float* w,
-                          const float* bias, float* state, const int* cu_q,
+// in_bias (fp32 [C], or null) is added to every input of the step before it is used or kept
+// (not to the zeros before a sequence's start).
+IX_API int ix_causal_conv(const void* x, int dtype, long long ldx, const float* in_bias,
+                          const float* w, const float* bias, float* state, const int* cu_q,
                           const int* seq_of_token, const int* state_slot, void* out, int T, int S,
                           int C, int taps, int act, cudaStream_t stream) {
   if (T <= 0 || S <= 0) return IX_OK;
@@ -370,7 +377,7 @@ IX_API int ix_causal_conv(const void* x, int dtype, long long ldx, const float* 
   const dim3 rgrid((T + CONV_RUN - 1) / CONV_RUN, (C / 2 + CONV_THREADS - 1) / CONV_THREADS);
 #define CONV_GO(TAPS)                                                                        \
   ix_launch(causal_conv_run_kernel<TA, TAPS>, rgrid, dim3(CONV_THREADS), 0, stream,          \
-            (const TA*)x, ldx, w, bias, (const float*)state, cu_q, seq_of_token, state_slot, \
+            (const TA*)x, ldx, in_bias, w, bias, (const float*)state, cu_q, seq_of_token, state_slot, \
             (TA*)out, T, C, act)
   IX_DISPATCH_DTYPE(dtype, TA, {
     if (run && taps == 2) CONV_GO(2);
@@ -378,11 +385,11 @@ IX_API int ix_causal_conv(const void* x, int dtype, long long ldx, const float* 
     else if (run && taps == 4) CONV_GO(4);
     else
       ix_launch(causal_conv_kernel<TA>, dim3(T, cb), dim3(CONV_THREADS), 0, stream,
-                (const TA*)x, ldx, w, bias, (const float*)state, cu_q, seq_of_token,
+                (const TA*)x, ldx, in_bias, w, bias, (const float*)state, cu_q, seq_of_token,
                 state_slot, (TA*)out, C, taps, act);
     if (taps > 1)
       ix_launch(conv_state_update_kernel<TA>, dim3(S, cb), dim3(CONV_THREADS), 0, stream,
-                (const TA*)x, ldx, state, cu_q, state_slot, C, taps);
+                (const TA*)x, ldx, in_bias, state, cu_q, state_slot, C, taps);
   });
 #undef CONV_GO
   return ix_launch_status();
@@ -1122,23 +1129,44 @@ IX_API int ix_normed_pair_mean(const void* l, const void* r, int dtype, const fl
 // relu squared; table routing; rows times a constant.
 // ---------------------------------------------------------------------------
 template <typename TA>
-__global__ void relu_squared_kernel(const TA* __restrict__ x, TA* __restrict__ out, size_t n) {
+__global__ void activate_kernel(const TA* x, TA* out, size_t n, int act) {
   IX_PDL_WAIT();
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n;
+       i += (size_t)gridDim.x * blockDim.x)
+    out[i] = from_f32<TA>(ix_act(to_f32(x[i]), act));
+}
+
+// four entries an access
+template <typename TA>
+__global__ void __launch_bounds__(256)
+activate_vec_kernel(const TA* x, TA* out, size_t quads, int act) {
+  IX_PDL_WAIT();
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < quads;
        i += (size_t)gridDim.x * blockDim.x) {
-    const float v = fmaxf(to_f32(x[i]), 0.f);
-    out[i] = from_f32<TA>(v * v);
+    const float4 v = ld4(x + 4 * i);
+    st4(out + 4 * i, make_float4(ix_act(v.x, act), ix_act(v.y, act), ix_act(v.z, act),
+                                 ix_act(v.w, act)));
   }
 }
 
-IX_API int ix_relu_squared(const void* x, void* out, int dtype, long long n,
-                           cudaStream_t stream) {
+// out = act(x) for n entries, act an IX_ACT_*; out may be x.
+IX_API int ix_activate(const void* x, void* out, int dtype, long long n, int act,
+                       cudaStream_t stream) {
   if (n <= 0) return IX_OK;
-  const long long want = (n + 255) / 256;
+  if (act < IX_ACT_NONE || act > IX_ACT_RELU2) return IX_ERR_UNSUPPORTED;
+  const size_t four = dtype == IX_F32 ? 16 : 8;
+  const bool vec = n % 4 == 0 && (((uintptr_t)x | (uintptr_t)out) % four) == 0;
+  const long long items = vec ? n / 4 : n;
+  const long long want = (items + 255) / 256;
   const int blocks = (int)(want > 148 * 16 ? 148 * 16 : want);
-  IX_DISPATCH_DTYPE(dtype, TA,
-                    ix_launch(relu_squared_kernel<TA>, dim3(blocks), dim3(256), 0, stream,
-                              (const TA*)x, (TA*)out, (size_t)n));
+  IX_DISPATCH_DTYPE(dtype, TA, {
+    if (vec)
+      ix_launch(activate_vec_kernel<TA>, dim3(blocks), dim3(256), 0, stream, (const TA*)x,
+                (TA*)out, (size_t)items, act);
+    else
+      ix_launch(activate_kernel<TA>, dim3(blocks), dim3(256), 0, stream, (const TA*)x, (TA*)out,
+                (size_t)n, act);
+  });
   return ix_launch_status();
 }
 

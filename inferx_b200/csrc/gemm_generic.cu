@@ -72,7 +72,7 @@ gemm_tiles_kernel(const TA* __restrict__ x, const int* __restrict__ rows,
                   const int* __restrict__ offsets, const TA* __restrict__ w,
                   TO* __restrict__ out, int M_single, int N, int K, int E,
                   long long w_expert_stride, int up_row_offset, int vec,
-                  const float* __restrict__ row_scale) {
+                  const float* __restrict__ row_scale, int plain) {
   constexpr int BN = DUAL ? 64 : 128;
   constexpr int RM = BM / 16;            // rows a thread owns: 4 or 8
   constexpr int RN = BN / 16;            // columns a thread owns: 4 or 8
@@ -222,6 +222,8 @@ gemm_tiles_kernel(const TA* __restrict__ x, const int* __restrict__ rows,
         const float w = row_scale ? row_scale[r] : 1.0f;
         const float g = row_scale ? val * w : val;
         val = g / (1.0f + expf(-g)) * (row_scale ? acc2[i][j] * w : acc2[i][j]);
+      } else {
+        val = ix_act(val, plain);
       }
       out[(size_t)r * N + c] = from_f32<TO>(val);
     }
@@ -239,7 +241,8 @@ __global__ void __launch_bounds__(GR_WARPS * 32)
 gemm_rows_kernel(const TA* __restrict__ x, const int* __restrict__ rows,
                  const int* __restrict__ offsets, const TA* __restrict__ w,
                  TO* __restrict__ out, int M_single, int N, int K, long long w_expert_stride,
-                 int up_row_offset, int vec, const float* __restrict__ row_scale) {
+                 int up_row_offset, int vec, const float* __restrict__ row_scale,
+                 int plain) {
   constexpr int COLS = DUAL ? 2 : 4;     // output columns a warp owns
   constexpr int WR = DUAL ? 4 : 4;       // weight rows it streams (gate and up when DUAL)
   const int e = blockIdx.y;
@@ -309,6 +312,8 @@ gemm_rows_kernel(const TA* __restrict__ x, const int* __restrict__ rows,
             const float w = row_scale ? row_scale[r0 + i] : 1.0f;
             const float g = row_scale ? val * w : val;
             val = g / (1.0f + expf(-g)) * (row_scale ? acc[i][j + 2] * w : acc[i][j + 2]);
+          } else {
+            val = ix_act(val, plain);
           }
           out[(size_t)(r0 + i) * N + c] = from_f32<TO>(val);
         }
@@ -323,7 +328,7 @@ gemm_rows_kernel(const TA* __restrict__ x, const int* __restrict__ rows,
 template <typename TA, typename TO, bool DUAL>
 static int launch_generic(const void* x, const int* rows, const int* offsets, const void* w,
                           void* out, int M, int N, int K, int E, int max_rows,
-                          const float* row_scale, cudaStream_t stream) {
+                          const float* row_scale, int plain, cudaStream_t stream) {
   const long long w_rows = DUAL ? 2LL * N : N;
   const long long stride = w_rows * K;
   const int esize = (int)sizeof(TA);
@@ -336,7 +341,7 @@ static int launch_generic(const void* x, const int* rows, const int* offsets, co
     dim3 grid((N + GR_WARPS * COLS - 1) / (GR_WARPS * COLS), E);
     gemm_rows_kernel<TA, TO, DUAL><<<grid, GR_WARPS * 32, 0, stream>>>(
         (const TA*)x, rows, offsets, (const TA*)w, (TO*)out, Ms, N, K, stride, N, vec,
-        row_scale);
+        row_scale, plain);
     return ix_launch_status();
   }
   constexpr int BN = DUAL ? 64 : 128;
@@ -349,26 +354,26 @@ static int launch_generic(const void* x, const int* rows, const int* offsets, co
   if (small_m)
     gemm_tiles_kernel<TA, TO, DUAL, 64><<<grid, GT_THREADS, 0, stream>>>(
         (const TA*)x, rows, offsets, (const TA*)w, (TO*)out, Ms, N, K, E, stride, N, vec,
-        row_scale);
+        row_scale, plain);
   else
     gemm_tiles_kernel<TA, TO, DUAL, 128><<<grid, GT_THREADS, 0, stream>>>(
         (const TA*)x, rows, offsets, (const TA*)w, (TO*)out, Ms, N, K, E, stride, N, vec,
-        row_scale);
+        row_scale, plain);
   return ix_launch_status();
 }
 
 IX_API int ix_gemm_generic(const void* x, const int* rows, const int* offsets, const void* w,
                            void* out, int in_dtype, int out_dtype, int dual, int M, int N, int K,
-                           int E, int max_rows, const float* row_scale,
+                           int E, int max_rows, const float* row_scale, int plain,
                            cudaStream_t stream) {
-  if (row_scale && !dual) return IX_ERR_UNSUPPORTED;
+  if ((row_scale && !dual) || (plain && dual)) return IX_ERR_UNSUPPORTED;
   if (N <= 0 || K <= 0 || E <= 0) return IX_ERR_SIZE;
   if (max_rows <= 0) return IX_OK;
 #define IX_GG(TA, TO)                                                                        \
   return dual ? launch_generic<TA, TO, true>(x, rows, offsets, w, out, M, N, K, E, max_rows,  \
-                                             row_scale, stream)                               \
+                                             row_scale, plain, stream)                               \
               : launch_generic<TA, TO, false>(x, rows, offsets, w, out, M, N, K, E, max_rows, \
-                                              row_scale, stream)
+                                              row_scale, plain, stream)
   if (in_dtype == IX_F32 && out_dtype == IX_F32) IX_GG(float, float);
   if (in_dtype == IX_BF16 && out_dtype == IX_BF16) IX_GG(bf16, bf16);
   if (in_dtype == IX_BF16 && out_dtype == IX_F32) IX_GG(bf16, float);

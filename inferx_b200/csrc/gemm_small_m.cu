@@ -52,6 +52,7 @@ __device__ __forceinline__ void mma_bf16_16816(float* c, unsigned a0, unsigned a
 struct DualAct {     // the gated unit's form; limit <= 0: silu(g) * u
   float limit, alpha, shift;
   const float* row_scale;   // one factor per output row on both products, or null
+  int plain;                // without a gate: the activation of the single product (IX_ACT_*)
 };
 __device__ __forceinline__ float dual_act(float g, float u, int row, const DualAct& a) {
   if (a.row_scale) {        // the row's input times w: both products times w
@@ -193,6 +194,7 @@ gemm_small_m_kernel(const bf16* __restrict__ x, const int* __restrict__ rows,
           if (j < N && r < hi) {
             float v = acc[i][c];
             if (DUAL) v = dual_act(v, acc2[i][c], r, act);
+            else v = ix_act(v, act.plain);
             out[(size_t)r * N + j] = from_f32<TO>(v);
           }
         }
@@ -219,6 +221,7 @@ gemm_small_m_kernel(const bf16* __restrict__ x, const int* __restrict__ rows,
         const int r = r0 + i * 8 + 2 * tt + (c & 1);
         if (j < N && r < hi) {
           if (DUAL) v = dual_act(v, v2, r, act);
+          else v = ix_act(v, act.plain);
           out[(size_t)r * N + j] = from_f32<TO>(v);
         }
       }
@@ -266,13 +269,14 @@ static int launch_small_m(const void* x, const int* rows, const int* offsets, co
 // act_limit > 0 (dual only): the clamped gated unit with that limit, sigmoid slope
 // act_alpha and act_shift added to the clamped linear branch; otherwise silu(g) * u.
 // row_scale (dual only; fp32 per output row, or null): the row's input counts times this.
+// plain_act (not dual): an IX_ACT_* applied to the product.
 IX_API int ix_gemm_small_m_act(const void* x, const int* rows, const int* offsets, const void* w,
                                void* out, int out_dtype, int dual, int M, int N, int K, int E,
                                int rows_per_pass, int active_groups, int offsets_settled,
                                float act_limit, float act_alpha, float act_shift,
-                               const float* row_scale, cudaStream_t stream) {
-  const DualAct act = {act_limit, act_alpha, act_shift, row_scale};
-  if (row_scale && !dual) return IX_ERR_UNSUPPORTED;
+                               const float* row_scale, int plain_act, cudaStream_t stream) {
+  const DualAct act = {act_limit, act_alpha, act_shift, row_scale, plain_act};
+  if ((row_scale && !dual) || (plain_act && dual)) return IX_ERR_UNSUPPORTED;
   if (N <= 0 || K <= 0 || E <= 0) return IX_ERR_SIZE;
   if (K % 8 != 0) return IX_ERR_UNSUPPORTED;
   if (!offsets && E != 1) return IX_ERR_SIZE;
@@ -303,5 +307,5 @@ IX_API int ix_gemm_small_m(const void* x, const int* rows, const int* offsets, c
                            int rows_per_pass, int active_groups, int offsets_settled,
                            cudaStream_t stream) {
   return ix_gemm_small_m_act(x, rows, offsets, w, out, out_dtype, dual, M, N, K, E, rows_per_pass,
-                             active_groups, offsets_settled, 0.f, 1.f, 0.f, nullptr, stream);
+                             active_groups, offsets_settled, 0.f, 1.f, 0.f, nullptr, IX_ACT_NONE, stream);
 }

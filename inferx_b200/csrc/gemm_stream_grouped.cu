@@ -56,7 +56,8 @@ __global__ void __launch_bounds__(GS_THREADS, 2)
 gemm_stream_grouped_kernel(const bf16* __restrict__ x, const int* __restrict__ rows,
                            const int* __restrict__ offsets, const bf16* __restrict__ w,
                            bf16* __restrict__ out, int N, int K, int E,
-                           long long w_expert_stride, const float* __restrict__ row_scale) {
+                           long long w_expert_stride, const float* __restrict__ row_scale,
+                           int plain) {
   constexpr int D = DUAL ? 3 : (NT > 1 ? 4 : 6);      // k-steps in flight per warp
   __shared__ int act[GS_MAX_EXPERTS];
   __shared__ int n_act_s;
@@ -206,6 +207,8 @@ gemm_stream_grouped_kernel(const bf16* __restrict__ x, const int* __restrict__ r
                   v2 *= row_scale[r];
                 }
                 v = v / (1.0f + __expf(-v)) * v2;
+              } else {
+                v = ix_act(v, plain);
               }
               out[(size_t)r * N + j] = __float2bfloat16_rn(v);
             }
@@ -221,7 +224,7 @@ gemm_stream_grouped_kernel(const bf16* __restrict__ x, const int* __restrict__ r
 template <bool DUAL, int NT>
 static int launch_stream_grouped(const void* x, const int* rows, const int* offsets,
                                  const void* w, void* out, int N, int K, int E,
-                                 const float* row_scale, cudaStream_t stream) {
+                                 const float* row_scale, int plain, cudaStream_t stream) {
   static int sms = 0;
   if (sms == 0) {
     int dev = 0;
@@ -233,25 +236,26 @@ static int launch_stream_grouped(const void* x, const int* rows, const int* offs
   const long long w_rows = DUAL ? 2LL * N : N;
   ix_launch(gemm_stream_grouped_kernel<DUAL, NT>, dim3(2 * sms), dim3(GS_THREADS), 0, stream,
             (const bf16*)x, rows, offsets, (const bf16*)w, (bf16*)out, N, K, E, w_rows * K,
-            row_scale);
+            row_scale, plain);
   return ix_launch_status();
 }
 
 // x: [*, K] bf16; rows: source row of each grouped row, or null when x is already
 // grouped; offsets: [E + 1]; w: [E, N (or 2N when dual), K] bf16; out: [rows, N] bf16.
 // rows_per_pass: 8 or 16 activation rows handled per pass over an expert's weights.
+// plain (not dual): an IX_ACT_* applied to the product.
 IX_API int ix_gemm_stream_grouped(const void* x, const int* rows, const int* offsets,
                                   const void* w, void* out, int dual, int N, int K, int E,
-                                  int rows_per_pass, const float* row_scale,
+                                  int rows_per_pass, const float* row_scale, int plain,
                                   cudaStream_t stream) {
-  if (row_scale && !dual) return IX_ERR_UNSUPPORTED;
+  if ((row_scale && !dual) || (plain && dual)) return IX_ERR_UNSUPPORTED;
   if (N <= 0 || K <= 0 || E <= 0 || offsets == nullptr) return IX_ERR_SIZE;
   if (K % 8 != 0 || K < 256 || E > GS_MAX_EXPERTS) return IX_ERR_UNSUPPORTED;
   if (((uintptr_t)x | (uintptr_t)w | (uintptr_t)out) & 15) return IX_ERR_ALIGN;
   if (rows_per_pass > 8) {
-    if (dual) return launch_stream_grouped<true, 2>(x, rows, offsets, w, out, N, K, E, row_scale, stream);
-    return launch_stream_grouped<false, 2>(x, rows, offsets, w, out, N, K, E, row_scale, stream);
+    if (dual) return launch_stream_grouped<true, 2>(x, rows, offsets, w, out, N, K, E, row_scale, plain, stream);
+    return launch_stream_grouped<false, 2>(x, rows, offsets, w, out, N, K, E, row_scale, plain, stream);
   }
-  if (dual) return launch_stream_grouped<true, 1>(x, rows, offsets, w, out, N, K, E, row_scale, stream);
-  return launch_stream_grouped<false, 1>(x, rows, offsets, w, out, N, K, E, row_scale, stream);
+  if (dual) return launch_stream_grouped<true, 1>(x, rows, offsets, w, out, N, K, E, row_scale, plain, stream);
+  return launch_stream_grouped<false, 1>(x, rows, offsets, w, out, N, K, E, row_scale, plain, stream);
 }

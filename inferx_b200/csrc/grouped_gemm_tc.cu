@@ -110,7 +110,7 @@ grouped_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a,
                        const __grid_constant__ CUtensorMap map_w,
                        const int* __restrict__ offsets, bf16* __restrict__ out, int N, int K,
                        int E, int w_rows_per_expert, int* __restrict__ status,
-                       const float* __restrict__ row_scale) {
+                       const float* __restrict__ row_scale, int plain) {
   constexpr bool DUAL = MODE != 0;      // two weight tiles and two accumulators an item
   constexpr bool SWIGLU = MODE == 1;
   constexpr int F_ITEM = MODE == 2 ? 2 * TC_BF : TC_BF;   // output features of an item
@@ -296,6 +296,13 @@ grouped_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a,
             u[DUAL ? i : 0] *= w_row;
           }
         }
+        if (!SWIGLU && plain) {
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            g[i] = ix_act(g[i], plain);
+            if (MODE == 2) u[DUAL ? i : 0] = ix_act(u[DUAL ? i : 0], plain);
+          }
+        }
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
           float a = g[i];
@@ -355,7 +362,7 @@ IX_API int ix_gather_rows(const void* src, const int* rows, void* dst, int n_row
 template <int MODE, int BT>
 static int launch_tc(const void* a, const int* offsets, const void* w, void* out, int A_rows,
                      int N, int K, int E, long long w_rows, int* status,
-                     const float* row_scale, cudaStream_t stream) {
+                     const float* row_scale, int plain, cudaStream_t stream) {
   CUtensorMap map_a, map_w;
   int rc = ix_tensor_map_bf16_2d(&map_a, a, A_rows, K, TC_BK, TC_BOX_T);
   if (rc != IX_OK) return rc;
@@ -379,14 +386,14 @@ static int launch_tc(const void* a, const int* offsets, const void* w, void* out
   cudaError_t e2 = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e2 != cudaSuccess) return (int)e2;
   kern<<<grid, TC_THREADS, smem, stream>>>(map_a, map_w, offsets, (bf16*)out, N, K, E,
-                                           (int)w_rows, status, row_scale);
+                                           (int)w_rows, status, row_scale, plain);
   return ix_launch_status();
 }
 
 IX_API int ix_grouped_gemm_tc(const void* a, const int* offsets, const void* w, void* out,
                               int dual, int A_rows, int N, int K, int E, int* status,
-                              const float* row_scale, cudaStream_t stream) {
-  if (row_scale && !dual) return IX_ERR_UNSUPPORTED;
+                              const float* row_scale, int plain, cudaStream_t stream) {
+  if ((row_scale && !dual) || (plain && dual)) return IX_ERR_UNSUPPORTED;
   if (A_rows <= 0) return IX_OK;
   if (N <= 0 || K <= 0 || E <= 0 || status == nullptr) return IX_ERR_SIZE;
   if (K % 8 != 0 || E > TC_MAX_EXPERTS) return IX_ERR_UNSUPPORTED;
@@ -406,10 +413,10 @@ IX_API int ix_grouped_gemm_tc(const void* a, const int* offsets, const void* w, 
   const int bt = per <= 128.0 ? 128 : per <= 160.0 ? 160 : per <= 192.0 ? 192 : 256;
 #define IX_TC(D)                                                                              \
   do {                                                                                        \
-    if (bt == 128) return launch_tc<D, 128>(a, offsets, w, out, A_rows, N, K, E, w_rows, status, row_scale, stream); \
-    if (bt == 160) return launch_tc<D, 160>(a, offsets, w, out, A_rows, N, K, E, w_rows, status, row_scale, stream); \
-    if (bt == 192) return launch_tc<D, 192>(a, offsets, w, out, A_rows, N, K, E, w_rows, status, row_scale, stream); \
-    return launch_tc<D, 256>(a, offsets, w, out, A_rows, N, K, E, w_rows, status, row_scale, stream);   \
+    if (bt == 128) return launch_tc<D, 128>(a, offsets, w, out, A_rows, N, K, E, w_rows, status, row_scale, plain, stream); \
+    if (bt == 160) return launch_tc<D, 160>(a, offsets, w, out, A_rows, N, K, E, w_rows, status, row_scale, plain, stream); \
+    if (bt == 192) return launch_tc<D, 192>(a, offsets, w, out, A_rows, N, K, E, w_rows, status, row_scale, plain, stream); \
+    return launch_tc<D, 256>(a, offsets, w, out, A_rows, N, K, E, w_rows, status, row_scale, plain, stream);   \
   } while (0)
   if (dual) IX_TC(1);
   // plain: two feature tiles an item when the features fill them (measured at 60 experts

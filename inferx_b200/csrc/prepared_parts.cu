@@ -10,7 +10,7 @@
 //    q and k head by position * frequency, pairs being neighbours or half a rotation
 //    apart, cos and sin times a factor; division of every q and k head by its root mean
 //    square (optional); values blended with another layer's, (1 - lambda) v + lambda v0
-//    (optional); q written densely, k and v into their pages.
+//    (optional); q written densely, k and v into their pages (no k and v: kvh 0).
 //  * ix_glu_bias_act: act(g + b_g) * (u + b_u) over rows laid out g | u, act the tanh form
 //    of gelu or silu.
 //  * ix_identity_rows: grouped rows of experts that return their input.
@@ -248,11 +248,11 @@ IX_API int ix_attention_prepare(const void* qkv, long long ld, int dtype, const 
                                 int page_size, void* k_dense, void* v_dense, int T,
                                 cudaStream_t stream) {
   if (T <= 0) return IX_OK;
-  if (heads <= 0 || kvh <= 0 || hd <= 0 || vd <= 0 || rot < 0 || rot > hd || (rot & 1) ||
+  if (heads <= 0 || kvh < 0 || hd <= 0 || vd <= 0 || rot < 0 || rot > hd || (rot & 1) ||
       page_size <= 0)
     return IX_ERR_SIZE;
   if ((q_gain == nullptr) != (k_gain == nullptr) || (rot > 0 && !freq) || (earlier && !lam) ||
-      (k_cache && (!v_cache || !slots)))
+      (k_cache && (!v_cache || !slots)) || (kvh == 0 && (q_gain || k_cache)))
     return IX_ERR_SIZE;
   const size_t smem = ((size_t)(heads + kvh) * hd + rot) * sizeof(float);
   if (smem > 200 * 1024) return IX_ERR_SMEM;

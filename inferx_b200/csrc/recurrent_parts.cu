@@ -547,7 +547,8 @@ IX_API int ix_linear_recurrence(const void* q, long long ldq, const void* k, lon
 
 // ---------------------------------------------------------------------------
 // head norm + gate.  One warp per (token, head).  `gain` covers all heads
-// (gain_per_head) or is shared by them.  gate_form 0: silu(gate); 1: sigmoid(gate).
+// (gain_per_head) or is shared by them.  gate_form 0: silu(gate); 1: sigmoid(gate).  With
+// `nq` ([T, H]; null: o as it is) a head's row is first divided by max(|nq|, floor) + den_eps.
 // ---------------------------------------------------------------------------
 #define HNG_WARPS 4
 
@@ -555,7 +556,8 @@ template <typename TG, typename TA>
 __global__ void head_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ gain,
                                       int gain_per_head, const TG* __restrict__ gate,
                                       long long ldg, TA* __restrict__ out, int H, int V,
-                                      float eps, int gate_form) {
+                                      float eps, int gate_form, const float* __restrict__ nq,
+                                      const float* __restrict__ floor_, float den_eps) {
   IX_PDL_WAIT();
   const int t = blockIdx.x;
   const int h = blockIdx.y * HNG_WARPS + (threadIdx.x >> 5);
@@ -563,8 +565,16 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, const float* 
   if (h >= H) return;
   const float* row = o + ((size_t)t * H + h) * V;
   float ss = 0.f;
-  for (int c = lane; c < V; c += 32) ss += row[c] * row[c];
-  const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)V + eps);
+  float den = 1.f;
+  if (nq) {
+    const size_t at = (size_t)t * H + h;
+    den = 1.0f / (fmaxf(fabsf(nq[at]), floor_[at]) + den_eps);
+  }
+  for (int c = lane; c < V; c += 32) {
+    const float x = row[c] * den;
+    ss += x * x;
+  }
+  const float inv = den / sqrtf(warp_sum(ss) / (float)V + eps);
   const float* g = gain + (gain_per_head ? (size_t)h * V : 0);
   const TG* gt = gate + (size_t)t * ldg + (size_t)h * V;
   TA* dst = out + ((size_t)t * H + h) * V;
@@ -579,11 +589,13 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, const float* 
 // lanes share a head, each with four values (16-byte reads of o and the gain, 8-byte ones
 // of the gate), 32 / GL heads a warp.  The sum of squares is added by a shuffle tree inside
 // the lanes of a head.
-template <int GL>
+template <int GL, bool SIGMOID>
 __global__ void head_norm_gate_bf16_vec_kernel(const float* __restrict__ o,
                                                const float* __restrict__ gain, int gain_per_head,
                                                const bf16* __restrict__ gate, long long ldg,
-                                               bf16* __restrict__ out, int H, int V, float eps) {
+                                               bf16* __restrict__ out, int H, int V, float eps,
+                                               const float* __restrict__ nq,
+                                               const float* __restrict__ floor_, float den_eps) {
   IX_PDL_WAIT();
   const int t = blockIdx.x;
   const int lane = threadIdx.x & 31;
@@ -593,6 +605,11 @@ __global__ void head_norm_gate_bf16_vec_kernel(const float* __restrict__ o,
   const bool ok = h < H;
   float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
   if (ok) x = reinterpret_cast<const float4*>(o + ((size_t)t * H + h) * V)[sub];
+  if (nq && ok) {
+    const size_t at = (size_t)t * H + h;
+    const float den = 1.0f / (fmaxf(fabsf(nq[at]), floor_[at]) + den_eps);
+    x.x *= den; x.y *= den; x.z *= den; x.w *= den;
+  }
   float ss = x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
 #pragma unroll
   for (int d = GL / 2; d > 0; d >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, d);
@@ -602,10 +619,10 @@ __global__ void head_norm_gate_bf16_vec_kernel(const float* __restrict__ o,
   const uint2 zr = reinterpret_cast<const uint2*>(gate + (size_t)t * ldg + (size_t)h * V)[sub];
   const float2 z01 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&zr.x));
   const float2 z23 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&zr.y));
-  const float r0 = x.x * inv * g.x * (z01.x / (1.0f + expf(-z01.x)));
-  const float r1 = x.y * inv * g.y * (z01.y / (1.0f + expf(-z01.y)));
-  const float r2 = x.z * inv * g.z * (z23.x / (1.0f + expf(-z23.x)));
-  const float r3 = x.w * inv * g.w * (z23.y / (1.0f + expf(-z23.y)));
+  const float r0 = x.x * inv * g.x * ((SIGMOID ? 1.0f : z01.x) / (1.0f + expf(-z01.x)));
+  const float r1 = x.y * inv * g.y * ((SIGMOID ? 1.0f : z01.y) / (1.0f + expf(-z01.y)));
+  const float r2 = x.z * inv * g.z * ((SIGMOID ? 1.0f : z23.x) / (1.0f + expf(-z23.x)));
+  const float r3 = x.w * inv * g.w * ((SIGMOID ? 1.0f : z23.y) / (1.0f + expf(-z23.y)));
   uint2 w;
   *reinterpret_cast<__nv_bfloat162*>(&w.x) = __floats2bfloat162_rn(r0, r1);
   *reinterpret_cast<__nv_bfloat162*>(&w.y) = __floats2bfloat162_rn(r2, r3);
@@ -615,20 +632,27 @@ __global__ void head_norm_gate_bf16_vec_kernel(const float* __restrict__ o,
 IX_API int ix_head_norm_gate(const float* o, const float* gain, int gain_per_head,
                              const void* gate, int gate_dtype, long long ldg, void* out,
                              int out_dtype, int T, int H, int V, float eps, int gate_form,
+                             const float* nq, const float* floor_, float den_eps,
                              cudaStream_t stream) {
   if (T <= 0) return IX_OK;
+  if ((nq == nullptr) != (floor_ == nullptr)) return IX_ERR_SIZE;
   if (H <= 0 || V <= 0 || ldg < (long long)H * V) return IX_ERR_SIZE;
   const int groups = (H + HNG_WARPS - 1) / HNG_WARPS;
   if (groups > 65535) return IX_ERR_SIZE;
   if (gate_dtype != out_dtype) return IX_ERR_UNSUPPORTED;
   const int gl = V / 4;
-  if (gate_form == 0 && out_dtype == IX_BF16 && V % 4 == 0 && gl <= 32 && (gl & (gl - 1)) == 0 && ldg % 4 == 0 &&
+  if (out_dtype == IX_BF16 && V % 4 == 0 && gl <= 32 && (gl & (gl - 1)) == 0 && ldg % 4 == 0 &&
       (((uintptr_t)o | (uintptr_t)gain) & 15) == 0 && (((uintptr_t)gate | (uintptr_t)out) & 7) == 0) {
     const int hpb = HNG_WARPS * (32 / gl);
     const int vgroups = (H + hpb - 1) / hpb;
 #define IX_HNG(GL)                                                                            \
-  ix_launch(head_norm_gate_bf16_vec_kernel<GL>, dim3(T, vgroups), dim3(32 * HNG_WARPS), 0,    \
-            stream, o, gain, gain_per_head, (const bf16*)gate, ldg, (bf16*)out, H, V, eps)
+  do {                                                                                        \
+    auto kern = gate_form ? head_norm_gate_bf16_vec_kernel<GL, true>                          \
+                          : head_norm_gate_bf16_vec_kernel<GL, false>;                        \
+    ix_launch(kern, dim3(T, vgroups), dim3(32 * HNG_WARPS), 0, stream, o, gain,               \
+              gain_per_head, (const bf16*)gate, ldg, (bf16*)out, H, V, eps, nq, floor_,       \
+              den_eps);                                                                       \
+  } while (0)
     if (gl == 32) IX_HNG(32);
     else if (gl == 16) IX_HNG(16);
     else if (gl == 8) IX_HNG(8);
@@ -641,6 +665,7 @@ IX_API int ix_head_norm_gate(const float* o, const float* gain, int gain_per_hea
   IX_DISPATCH_DTYPE(out_dtype, TA,
                     ix_launch(head_norm_gate_kernel<TA, TA>, dim3(T, groups),
                               dim3(32 * HNG_WARPS), 0, stream, o, gain, gain_per_head,
-                              (const TA*)gate, ldg, (TA*)out, H, V, eps, gate_form));
+                              (const TA*)gate, ldg, (TA*)out, H, V, eps, gate_form, nq, floor_,
+                              den_eps));
   return ix_launch_status();
 }

@@ -71,7 +71,7 @@ __device__ __forceinline__ void select_topk(float* p, int E, int k, int renorm, 
 // How the chosen experts are picked and weighted beyond the plain top-k: `correction`
 // ([E] or null) is added to the scores for the choice alone; with `groups` > 0 the E
 // outputs form that many equal groups of neighbours, a group's value is its largest
-// corrected score, and only outputs of the `keep` groups with the largest values can be
+// corrected score (`pair_sum`: the sum of its two largest), and only outputs of the `keep` groups with the largest values can be
 // chosen (ties to the lower group); `renorm_eps` >= 0 divides the chosen scores by (their
 // sum + renorm_eps).  `active` 0: the plain rule above.
 struct RouteRule {
@@ -80,6 +80,7 @@ struct RouteRule {
   int keep;
   float renorm_eps;
   int active;
+  int pair_sum;
   int sigmoid;      // scores are sigmoid(logit), each on its own, instead of the softmax
 };
 
@@ -124,10 +125,14 @@ __device__ __forceinline__ void select_topk_ruled(float* p, int E, int k, int re
   unsigned allowed = 0xffffffffu;
   const int gsize = rule.groups > 0 ? E / rule.groups : E;
   if (rule.groups > 0) {
-    float gv = -INFINITY;
+    float gv = -INFINITY, second = -INFINITY;
     if (lane < rule.groups)
-      for (int e = lane * gsize; e < (lane + 1) * gsize; ++e)
-        gv = fmaxf(gv, p[e] + (rule.correction ? rule.correction[e] : 0.f));
+      for (int e = lane * gsize; e < (lane + 1) * gsize; ++e) {
+        const float c = p[e] + (rule.correction ? rule.correction[e] : 0.f);
+        second = fmaxf(second, fminf(gv, c));
+        gv = fmaxf(gv, c);
+      }
+    if (rule.pair_sum && gsize > 1) gv += second;
     allowed = 0u;
     for (int r = 0; r < rule.keep; ++r) {
       const bool open = lane < rule.groups && !((allowed >> lane) & 1u);
@@ -490,7 +495,7 @@ IX_API int ix_router_topk(const void* x, const float* w, const float* extra_w, i
                           int T, int H, int E, int k, int renorm, float scale, float* topk_w,
                           int* topk_idx, float* extra_out, float* logits_scratch,
                           cudaStream_t stream) {
-  RouteRule rule = {nullptr, 0, 0, -1.f, 0, 0};
+  RouteRule rule = {nullptr, 0, 0, -1.f, 0, 0, 0};
   return router_topk_impl(x, w, extra_w, act_dtype, T, H, E, k, renorm, scale, topk_w, topk_idx,
                           extra_out, logits_scratch, rule, stream);
 }
@@ -500,13 +505,14 @@ IX_API int ix_router_topk(const void* x, const float* w, const float* extra_w, i
 IX_API int ix_router_topk_ruled(const void* x, const float* w, const float* extra_w,
                                 int act_dtype, int T, int H, int E, int k, int renorm,
                                 float scale, const float* correction, int groups, int keep,
-                                float renorm_eps, int sigmoid, float* topk_w, int* topk_idx,
+                                float renorm_eps, int sigmoid, int pair_sum, float* topk_w,
+                                int* topk_idx,
                                 float* extra_out, float* logits_scratch, cudaStream_t stream) {
   if (groups < 0 || groups > ROUTER_MAX_GROUPS) return IX_ERR_SIZE;
   if (groups > 0 && (E % groups != 0 || keep <= 0 || keep > groups ||
                      (long long)keep * (E / groups) < k))
     return IX_ERR_SIZE;
-  RouteRule rule = {correction, groups, keep, renorm_eps, 1, sigmoid};
+  RouteRule rule = {correction, groups, keep, renorm_eps, 1, pair_sum, sigmoid};
   return router_topk_impl(x, w, extra_w, act_dtype, T, H, E, k, renorm, scale, topk_w, topk_idx,
                           extra_out, logits_scratch, rule, stream);
 }

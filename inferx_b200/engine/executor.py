@@ -159,7 +159,8 @@ class Executor:
         self.device = storage.device
         self.vocab = model.spec.vocab_size
         self.caches = storage.layer_caches(model.spec.schedule,
-                                           getattr(model, "cache_unit", None))
+                                           getattr(model, "cache_unit", None),
+                                           getattr(model, "state_unit", None))
         # state of parts that are not layers of the schedule (the embedding's) follows
         for unit in getattr(model, "extra_cache_units", ()):
             self.caches.append(storage.unit_cache(unit))

@@ -252,6 +252,38 @@ def silu_mul(gu: torch.Tensor):
     return out
 
 
+# activations of products without a gate (csrc/common.cuh)
+_ACTIVATIONS = {None: 0, "gelu": 1, "relu_squared": 2}
+
+
+def activate(x: torch.Tensor, activation: str, out: Optional[torch.Tensor] = None):
+    """act(x): "gelu" (the exact, erf form) or "relu_squared"; ``out`` may be ``x``."""
+    _chk("x", x)
+    out = torch.empty_like(x) if out is None else out
+    _chk("out", out, x.dtype)
+    if out.numel() != x.numel():
+        raise KernelError("activate: out must have the input's size")
+    _check(_lib().ix_activate(_ptr(x), _ptr(out), _dtype_code(x), ctypes.c_longlong(x.numel()),
+                              _ACTIVATIONS[activation], _stream()), "activate")
+    _count()
+    return out
+
+
+def linear_act(x: torch.Tensor, w: torch.Tensor, activation: str):
+    """act(x[M,K] . w[N,K]^T): in the product's epilogue where this library's kernels run it,
+    else in place over the library's result."""
+    _chk("x", x)
+    _chk("w", w, x.dtype)
+    M = x.shape[0]
+    if M <= SMALL_M_DENSE_ROWS and _streams_weights(x, w):
+        return gemm_small_m(x, w.unsqueeze(0), None, None, False, M, rows_per_pass=M,
+                            activation=activation)
+    if x.dtype == torch.float32:
+        return gemm_generic(x, w.unsqueeze(0), None, None, dual=False, activation=activation)
+    y = linear(x, w)
+    return activate(y, activation, out=y)
+
+
 def linear(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None):
     """x[M,K] . w[N,K]^T.  bfloat16: cuBLAS, fp32 accumulation.  float32: own FFMA kernel."""
     _chk("x", x)
@@ -277,9 +309,9 @@ def linear(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = 
 def gemm_generic(x: torch.Tensor, w: torch.Tensor, rows: Optional[torch.Tensor],
                  offsets: Optional[torch.Tensor], dual: bool,
                  out_dtype: Optional[torch.dtype] = None, num_out_rows: Optional[int] = None,
-                 row_scale: Optional[torch.Tensor] = None):
+                 row_scale: Optional[torch.Tensor] = None, activation: Optional[str] = None):
     """CUDA-core product, single (offsets None) or grouped by expert.  ``row_scale`` (dual
-    only): see ``grouped_gate_up_swiglu``."""
+    only): see ``grouped_gate_up_swiglu``; ``activation`` (not dual): see ``linear_act``."""
     _chk("row_scale", row_scale, torch.float32, optional=True)
     _chk("x", x)
     _chk("w", w)
@@ -301,7 +333,7 @@ def gemm_generic(x: torch.Tensor, w: torch.Tensor, rows: Optional[torch.Tensor],
     code = _lib().ix_gemm_generic(
         _ptr(x), _ptr(rows), _ptr(offsets), _ptr(w), _ptr(out), _dtype_code(x),
         F32 if out_dtype == torch.float32 else BF16, 1 if dual else 0, M, N, K, E, A, _ptr(row_scale),
-        _stream())
+        _ACTIVATIONS[activation], _stream())
     _check(code, "gemm_generic")
     _count()
     return out
@@ -403,10 +435,36 @@ def qkv_project_rope_append(x: torch.Tensor, w: torch.Tensor, bias: Optional[tor
     return q
 
 
+_ZERO_SINKS = {}
+
+
+def _sink_and_gate(q: torch.Tensor, sink, gate):
+    """(keep-alive tensors, launch arguments) of a per-head sink and of a gate per (token,
+    head).  ``sink``: fp32 [heads], True (a score of zero in every head) or None / False;
+    ``gate``: a view [T, heads] with unit inner stride in q's element type, or None."""
+    T, heads = q.shape[0], q.shape[1]
+    if sink is True:
+        key = (str(q.device), heads)
+        if key not in _ZERO_SINKS:
+            _ZERO_SINKS[key] = torch.zeros(heads, dtype=torch.float32, device=q.device)
+        sink = _ZERO_SINKS[key]
+    elif sink is False:
+        sink = None
+    _chk("sink", sink, torch.float32, optional=True)
+    if sink is not None and sink.numel() != heads:
+        raise KernelError(f"attention: {sink.numel()} sinks for {heads} heads")
+    ld = 0
+    if gate is not None:
+        ld = _row_view("attention: gate", gate, heads)
+        if gate.shape[0] != T or gate.dtype != q.dtype:
+            raise KernelError("attention: one gate per (token, head), in the queries' type")
+    return sink, (_ptr(sink), _ptr(gate), ctypes.c_longlong(ld))
+
+
 def paged_attention_generic(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                             block_table: torch.Tensor, seq_of_token: torch.Tensor,
                             positions: torch.Tensor, window: int, scale: float,
-                            softcap: float = 0.0, keep_first: int = 0, sink: bool = False):
+                            softcap: float = 0.0, keep_first: int = 0, sink=None, gate=None):
     _chk("q", q)
     _chk("k_cache", k_cache, q.dtype)
     _chk("v_cache", v_cache, q.dtype)
@@ -419,11 +477,12 @@ def paged_attention_generic(q: torch.Tensor, k_cache: torch.Tensor, v_cache: tor
     if chd != hd or tuple(v_cache.shape[:3]) != (P, kvh, page):
         raise KernelError("paged_attention: cache head size differs from the query's")
     out = torch.empty((T, heads, vd), dtype=q.dtype, device=q.device)
+    sink, extra = _sink_and_gate(q, sink, gate)
     code = _lib().ix_paged_attention_generic(
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), _ptr(seq_of_token),
         _ptr(positions), _ptr(out), _dtype_code(q), T, heads, kvh, hd, vd, page,
         block_table.shape[1], window, ctypes.c_float(scale), ctypes.c_float(softcap),
-        int(keep_first), 1 if sink else 0, _stream())
+        int(keep_first), *extra, _stream())
     _check(code, "paged_attention_generic")
     _count()
     return out
@@ -432,7 +491,7 @@ def paged_attention_generic(q: torch.Tensor, k_cache: torch.Tensor, v_cache: tor
 def paged_attention_tiled(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                           block_table: torch.Tensor, cu_q: torch.Tensor, q_pos0: torch.Tensor,
                           window: int, scale: float, softcap: float = 0.0, keep_first: int = 0,
-                          sink: bool = False):
+                          sink=None, gate=None):
     """CUDA-core attention for a ragged batch, tiled (32 queries of a sequence against 64
     keys at a time in shared memory, fp32 math): sequence s brings the queries
     q[cu_q[s]:cu_q[s+1]] at positions q_pos0[s], q_pos0[s]+1, ...  Any element type, head
@@ -453,11 +512,11 @@ def paged_attention_tiled(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch
     if cu_q.numel() != S + 1 or block_table.shape[0] != S:
         raise KernelError("paged_attention_tiled: cu_q, q_pos0 and block_table disagree")
     out = torch.empty((T, heads, vd), dtype=q.dtype, device=q.device)
+    sink, extra = _sink_and_gate(q, sink, gate)
     code = _lib().ix_paged_attention_tiled(
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), _ptr(cu_q), _ptr(q_pos0),
         _ptr(out), _dtype_code(q), T, S, heads, kvh, hd, vd, page, block_table.shape[1], window,
-        ctypes.c_float(scale), ctypes.c_float(softcap), int(keep_first), 1 if sink else 0,
-        _stream())
+        ctypes.c_float(scale), ctypes.c_float(softcap), int(keep_first), *extra, _stream())
     _check(code, "paged_attention_tiled")
     _count()
     return out
@@ -478,13 +537,14 @@ ROUTER_FEW_TOKENS = 128
 def router_topk(x: torch.Tensor, w: torch.Tensor, top_k: int, renormalize: bool, scale: float,
                 extra_w: Optional[torch.Tensor] = None,
                 correction: Optional[torch.Tensor] = None, group_count: int = 0,
-                group_keep: int = 0, renorm_eps: Optional[float] = None, score: str = "softmax"
-                ) -> Tuple[torch.Tensor, torch.Tensor, Optional[torch.Tensor]]:
+                group_keep: int = 0, renorm_eps: Optional[float] = None, score: str = "softmax",
+                group_value: str = "max") -> Tuple[torch.Tensor, torch.Tensor, Optional[torch.Tensor]]:
     """fp32 router logits, softmax over all experts, top-k (ties to the lower index).
 
     ``correction`` (fp32 [E]) is added to the scores for the choice alone; with
     ``group_count`` > 0 the outputs form that many equal groups of neighbours and only
-    outputs of the ``group_keep`` groups with the largest corrected score can be chosen;
+    outputs of the ``group_keep`` groups of the largest value can be chosen, a group's value
+    being its largest corrected score, or (``group_value`` "pair_sum") the sum of its two;
     ``renorm_eps`` >= 0 divides the chosen scores by (their sum + renorm_eps).  ``score``
     "sigmoid": an output's score is the sigmoid of its own logit instead.
 
@@ -516,7 +576,7 @@ def router_topk(x: torch.Tensor, w: torch.Tensor, top_k: int, renormalize: bool,
             _ptr(x), _ptr(w), _ptr(extra_w), _dtype_code(x), T, H, E, top_k,
             1 if renormalize else 0, ctypes.c_float(scale), _ptr(correction), int(group_count),
             int(group_keep), ctypes.c_float(-1.0 if renorm_eps is None else renorm_eps),
-            1 if score == "sigmoid" else 0, _ptr(tw), _ptr(ti), _ptr(ex), _ptr(scratch), _stream())
+            1 if score == "sigmoid" else 0, 1 if group_value == "pair_sum" else 0, _ptr(tw), _ptr(ti), _ptr(ex), _ptr(scratch), _stream())
     else:
         code = _lib().ix_router_topk(
             _ptr(x), _ptr(w), _ptr(extra_w), _dtype_code(x), T, H, E, top_k,
@@ -841,7 +901,7 @@ def paged_attention_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: tor
 def paged_attention_prefill_exact(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                                   block_table: torch.Tensor, cu_q: torch.Tensor,
                                   q_pos0: torch.Tensor, window: int, scale: float,
-                                  keep_first: int = 0, sink: bool = False,
+                                  keep_first: int = 0, sink=None, gate=None,
                                   kernel: Optional[str] = None):
     """Tensor-core attention for a ragged batch of bfloat16 queries whose softmax weights
     keep 16 bits in their product with the values (each weight enters as two bfloat16 terms
@@ -866,6 +926,7 @@ def paged_attention_prefill_exact(q: torch.Tensor, k_cache: torch.Tensor, v_cach
     if cu_q.numel() != S + 1 or block_table.shape[0] != S:
         raise KernelError("paged_attention_prefill_exact: cu_q, q_pos0 and block_table disagree")
     out = torch.empty((T, heads, vd), dtype=q.dtype, device=q.device)
+    sink, extra = _sink_and_gate(q, sink, gate)
     tc_ok = bool(_lib().ix_paged_attention_prefill_tc_exact_applies(hd, vd, page))
     if kernel is None:
         kernel = "tc" if USE_TCGEN05_ATTENTION and tc_ok else "mma"
@@ -876,14 +937,14 @@ def paged_attention_prefill_exact(q: torch.Tensor, k_cache: torch.Tensor, v_cach
         _check(_lib().ix_paged_attention_prefill_tc_exact(
             _ptr(q), _ptr(k_cache), _ptr(v_cache), P, _ptr(block_table), _ptr(cu_q),
             _ptr(q_pos0), _ptr(out), T, S, heads, kvh, hd, page, block_table.shape[1], window,
-            ctypes.c_float(scale), int(keep_first), 1 if sink else 0,
+            ctypes.c_float(scale), int(keep_first), *extra,
             _ptr(_tc_status(q.device)), _stream()), "paged_attention_prefill_tc_exact")
         _count()
         return out
     _check(_lib().ix_paged_attention_prefill_exact(
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), _ptr(cu_q), _ptr(q_pos0),
         _ptr(out), T, S, heads, kvh, hd, vd, page, block_table.shape[1], window,
-        ctypes.c_float(scale), int(keep_first), 1 if sink else 0, _stream()),
+        ctypes.c_float(scale), int(keep_first), *extra, _stream()),
         "paged_attention_prefill_exact")
     _count()
     return out
@@ -892,7 +953,7 @@ def paged_attention_prefill_exact(q: torch.Tensor, k_cache: torch.Tensor, v_cach
 def paged_attention_decode_exact(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                                  block_table: torch.Tensor, kv_len: torch.Tensor, max_kv_len: int,
                                  window: int, scale: float, splits: Optional[int] = None,
-                                 keep_first: int = 0, sink: bool = False):
+                                 keep_first: int = 0, sink=None, gate=None):
     """Split-KV tensor-core attention (mma.sync) for a batch in which sequence s brings the
     one bfloat16 query q[s] at position kv_len[s] - 1, with softmax weights that keep 16 bits
     in their product with the values; key and value heads of 64 or 128 entries each."""
@@ -917,10 +978,11 @@ def paged_attention_decode_exact(q: torch.Tensor, k_cache: torch.Tensor, v_cache
     if splits > 1:
         part_o = torch.empty((S, heads, splits, vd), dtype=torch.float32, device=q.device)
         part_ml = torch.empty((S, heads, splits, 2), dtype=torch.float32, device=q.device)
+    sink, extra = _sink_and_gate(q, sink, gate)
     _check(lib.ix_paged_attention_decode_exact(
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), _ptr(kv_len), _ptr(part_o),
         _ptr(part_ml), _ptr(out), S, heads, kvh, hd, vd, page, block_table.shape[1], window,
-        ctypes.c_float(scale), splits, int(keep_first), 1 if sink else 0, _stream()),
+        ctypes.c_float(scale), splits, int(keep_first), *extra, _stream()),
         "paged_attention_decode_exact")
     _count(2 if splits > 1 else 1)
     return out
@@ -933,10 +995,12 @@ USE_EXACT_TC_ATTENTION = True
 def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                     block_table: torch.Tensor, step, window: int, scale: float,
                     softcap: float = 0.0, fp32_weights: bool = False, keep_first: int = 0,
-                    sink: bool = False):
+                    sink=None, gate=None):
     """Causal attention of this step's queries over the paged cache.  ``keep_first``: with
-    a window, the sequence's first tokens stay visible beside it; ``sink``: one is added
-    to the softmax's denominator (both run on the fp32-arithmetic kernels).  With ``softcap``
+    a window, the sequence's first tokens stay visible beside it; ``sink`` (fp32 [heads], or
+    True for zeros): its exponential joins the softmax's denominator, a key with that score
+    and no value; ``gate`` (a view [T, heads]): a head's result is multiplied by its sigmoid
+    (all of these run on the fp32-arithmetic kernels).  With ``softcap``
     > 0 a score s becomes softcap * tanh(s / softcap) before the softmax.  With
     ``fp32_weights``, or value pages whose head size differs from the keys', the
     fp32-arithmetic kernels run whatever the element type.
@@ -947,9 +1011,12 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     tuned kernels do not take, to the general kernel."""
     hd = q.shape[2]
     page = k_cache.shape[2]
-    if fp32_weights or v_cache.shape[3] != hd or sink or (keep_first and window > 0):
+    if isinstance(sink, bool):
+        sink = sink or None
+    if (fp32_weights or v_cache.shape[3] != hd or sink is not None or gate is not None
+            or (keep_first and window > 0)):
         return _paged_attention_softcap(q, k_cache, v_cache, block_table, step, window, scale,
-                                        softcap, keep_first if window > 0 else 0, sink)
+                                        softcap, keep_first if window > 0 else 0, sink, gate)
     if softcap > 0 and not (scale > 0 and USE_TMA_DECODE and _tma_decode_applies(q, page)
                             and USE_TCGEN05_ATTENTION and _tc_prefill_applies(q, page)):
         # of the tuned kernels only the TMA decode form and the tcgen05 prompt form squash
@@ -980,7 +1047,7 @@ def paged_attention_decode_any(q: torch.Tensor, k_cache: torch.Tensor, v_cache: 
                                block_table: torch.Tensor, kv_len: torch.Tensor, max_kv_len: int,
                                window: int, scale: float, softcap: float = 0.0,
                                splits: Optional[int] = None, keep_first: int = 0,
-                               sink: bool = False):
+                               sink=None, gate=None):
     """Split-KV attention in fp32 arithmetic for a batch in which sequence s brings the one
     query q[s] at position kv_len[s] - 1: any head size up to 512, value heads of a size
     of their own, any element type.  Returns [S, heads, value size]."""
@@ -1004,11 +1071,12 @@ def paged_attention_decode_any(q: torch.Tensor, k_cache: torch.Tensor, v_cache: 
     if splits > 1:
         part_o = torch.empty((S, heads, splits, vd), dtype=torch.float32, device=q.device)
         part_ml = torch.empty((S, heads, splits, 2), dtype=torch.float32, device=q.device)
+    sink, extra = _sink_and_gate(q, sink, gate)
     _check(lib.ix_paged_attention_decode_any(
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), _ptr(kv_len), _ptr(part_o),
         _ptr(part_ml), _ptr(out), _dtype_code(q), S, heads, kvh, hd, vd, page,
         block_table.shape[1], window, ctypes.c_float(scale), ctypes.c_float(softcap), splits,
-        int(keep_first), 1 if sink else 0, _stream()), "paged_attention_decode_any")
+        int(keep_first), *extra, _stream()), "paged_attention_decode_any")
     _count(2 if splits > 1 else 1)
     return out
 
@@ -1019,7 +1087,7 @@ DECODE_ANY_MIN_KEYS = 128
 
 
 def _paged_attention_softcap(q, k_cache, v_cache, block_table, step, window, scale, softcap,
-                             keep_first=0, sink=False):
+                             keep_first=0, sink=None, gate=None):
     """The fp32-arithmetic kernels (squashed scores or not)."""
     hd = q.shape[2]
     if (USE_EXACT_TC_ATTENTION and softcap == 0.0 and scale > 0 and q.dtype == torch.bfloat16
@@ -1028,13 +1096,13 @@ def _paged_attention_softcap(q, k_cache, v_cache, block_table, step, window, sca
             and _lib().ix_paged_attention_decode_exact_applies(hd, v_cache.shape[3])):
         return paged_attention_decode_exact(q, k_cache, v_cache, block_table, step.kv_len,
                                             step.max_kv_len, window, scale,
-                                            keep_first=keep_first, sink=sink)
+                                            keep_first=keep_first, sink=sink, gate=gate)
     if (getattr(step, "all_decode", False) and getattr(step, "kv_len", None) is not None
             and step.num_tokens == step.num_seqs and step.max_kv_len >= DECODE_ANY_MIN_KEYS
             and max(hd, v_cache.shape[3]) <= 512):
         return paged_attention_decode_any(q, k_cache, v_cache, block_table, step.kv_len,
                                           step.max_kv_len, window, scale, softcap,
-                                          keep_first=keep_first, sink=sink)
+                                          keep_first=keep_first, sink=sink, gate=gate)
     if (USE_EXACT_TC_ATTENTION and softcap == 0.0 and scale > 0 and q.dtype == torch.bfloat16
             and _lib().ix_paged_attention_prefill_exact_applies(hd, v_cache.shape[3])
             and getattr(step, "cu_q", None) is not None):
@@ -1045,21 +1113,24 @@ def _paged_attention_softcap(q, k_cache, v_cache, block_table, step, window, sca
             # the prompt portions to the tiled one
             single = paged_attention_decode_exact(
                 q[:nd], k_cache, v_cache, block_table[:nd], step.kv_len[:nd], step.max_kv_len,
-                window, scale, keep_first=keep_first, sink=sink)
+                window, scale, keep_first=keep_first, sink=sink,
+                gate=None if gate is None else gate[:nd])
             rest = paged_attention_prefill_exact(
                 q[nd:], k_cache, v_cache, block_table[nd:], step.cu_q_prompt, step.q_pos0[nd:],
-                window, scale, keep_first, sink)
+                window, scale, keep_first, sink,
+                gate=None if gate is None else gate[nd:])
             return torch.cat([single, rest], dim=0)
         return paged_attention_prefill_exact(q, k_cache, v_cache, block_table, step.cu_q,
-                                             step.q_pos0, window, scale, keep_first, sink)
+                                             step.q_pos0, window, scale, keep_first, sink, gate=gate)
     if (step.num_tokens >= TILED_ATTENTION_MIN_QUERIES * step.num_seqs
             and _lib().ix_paged_attention_tiled_applies(hd)
             and _lib().ix_paged_attention_tiled_applies(v_cache.shape[3])
             and getattr(step, "cu_q", None) is not None):
         return paged_attention_tiled(q, k_cache, v_cache, block_table, step.cu_q, step.q_pos0,
-                                     window, scale, softcap, keep_first, sink)
+                                     window, scale, softcap, keep_first, sink, gate)
     return paged_attention_generic(q, k_cache, v_cache, block_table, step.seq_of_token,
-                                   step.positions, window, scale, softcap, keep_first, sink)
+                                   step.positions, window, scale, softcap, keep_first, sink,
+                                   gate)
 
 
 USE_TCGEN05 = True           # prompt-sized grouped products go to the tcgen05 kernel
@@ -1076,7 +1147,7 @@ def gemm_small_m(x: torch.Tensor, w: torch.Tensor, rows: Optional[torch.Tensor],
                  out_dtype: Optional[torch.dtype] = None, rows_per_pass: int = 8,
                  active_groups: int = 0, offsets_settled: bool = False,
                  glu_clamp: Optional[Tuple[float, float, float]] = None,
-                 row_scale: Optional[torch.Tensor] = None):
+                 row_scale: Optional[torch.Tensor] = None, activation: Optional[str] = None):
     """Weight-streaming product for few rows per weight matrix (bf16 inputs).
     ``offsets_settled``: the kernel that wrote ``offsets`` is at least two launches back
     in this stream (so the launch may read it, and start on its weights, before waiting
@@ -1101,7 +1172,7 @@ def gemm_small_m(x: torch.Tensor, w: torch.Tensor, rows: Optional[torch.Tensor],
         0 if offsets is not None else x.shape[0], N, K, E, rows_per_pass,
         active_groups or min(E, num_out_rows), 1 if offsets_settled else 0,
         ctypes.c_float(limit), ctypes.c_float(alpha), ctypes.c_float(shift), _ptr(row_scale),
-        _stream())
+        _ACTIVATIONS[activation], _stream())
     _check(code, "gemm_small_m")
     _count()
     return out
@@ -1155,7 +1226,7 @@ def check_async_errors():
 
 
 def grouped_gemm_tc(a: torch.Tensor, offsets: torch.Tensor, w: torch.Tensor, dual: bool,
-                    row_scale: Optional[torch.Tensor] = None):
+                    row_scale: Optional[torch.Tensor] = None, activation: Optional[str] = None):
     """Grouped product on tcgen05 tensor cores: ``a`` [rows, K] already grouped by
     expert, ``w`` [E, N or 2N, K]; returns [rows, N] bf16."""
     _chk("a", a, torch.bfloat16)
@@ -1168,7 +1239,8 @@ def grouped_gemm_tc(a: torch.Tensor, offsets: torch.Tensor, w: torch.Tensor, dua
     out = torch.empty((a.shape[0], N), dtype=torch.bfloat16, device=a.device)
     code = _lib().ix_grouped_gemm_tc(_ptr(a), _ptr(offsets), _ptr(w), _ptr(out),
                                      1 if dual else 0, a.shape[0], N, K, E,
-                                     _ptr(_tc_status(a.device)), _ptr(row_scale), _stream())
+                                     _ptr(_tc_status(a.device)), _ptr(row_scale),
+                                     _ACTIVATIONS[activation], _stream())
     _check(code, "grouped_gemm_tc")
     _count()
     return out
@@ -1183,7 +1255,8 @@ STREAM_GROUPED_MAX_ROWS = 4
 
 def gemm_stream_grouped(x: torch.Tensor, w: torch.Tensor, rows: Optional[torch.Tensor],
                         offsets: torch.Tensor, dual: bool, num_out_rows: int,
-                        rows_per_pass: int = 8, row_scale: Optional[torch.Tensor] = None):
+                        rows_per_pass: int = 8, row_scale: Optional[torch.Tensor] = None,
+                        activation: Optional[str] = None):
     """Grouped weight-streaming product, persistent form (few rows per expert, bf16)."""
     _chk("x", x, torch.bfloat16)
     _chk("w", w, torch.bfloat16)
@@ -1198,7 +1271,7 @@ def gemm_stream_grouped(x: torch.Tensor, w: torch.Tensor, rows: Optional[torch.T
     out = torch.empty((num_out_rows, N), dtype=torch.bfloat16, device=x.device)
     code = _lib().ix_gemm_stream_grouped(_ptr(x), _ptr(rows), _ptr(offsets), _ptr(w), _ptr(out),
                                          1 if dual else 0, N, K, E, rows_per_pass, _ptr(row_scale),
-                                         _stream())
+                                         _ACTIVATIONS[activation], _stream())
     _check(code, "gemm_stream_grouped")
     _count()
     return out
@@ -1238,6 +1311,23 @@ def grouped_gate_up_swiglu(x: torch.Tensor, rows: torch.Tensor, offsets: torch.T
                                row_scale=row_scale)
     return gemm_generic(x, w_gate_up, rows, offsets, dual=True, num_out_rows=A,
                         row_scale=row_scale)
+
+
+def grouped_up(x: torch.Tensor, rows: torch.Tensor, offsets: torch.Tensor, w_up: torch.Tensor,
+               activation: str):
+    """act[r] = activation(x[rows[r]] . Wu[e]^T), e from offsets: experts without a gate,
+    ``w_up`` [E, I, H]."""
+    A = rows.numel()
+    per = A / w_up.shape[0]
+    if _stream_grouped_applies(x, w_up, A):
+        return gemm_stream_grouped(x, w_up, rows, offsets, False, A,
+                                   rows_per_pass=8 if per <= 2 else 16, activation=activation)
+    if per <= SMALL_M_ROWS_PER_GROUP and _streams_weights(x, w_up):
+        return gemm_small_m(x, w_up, rows, offsets, False, A,
+                            rows_per_pass=8 if per <= 2 else 16, activation=activation)
+    if USE_TCGEN05 and _streams_weights(x, w_up) and w_up.shape[0] <= TCGEN05_MAX_EXPERTS:
+        return grouped_gemm_tc(gather_rows(x, rows), offsets, w_up, False, activation=activation)
+    return gemm_generic(x, w_up, rows, offsets, dual=False, num_out_rows=A, activation=activation)
 
 
 def grouped_down(act: torch.Tensor, offsets: torch.Tensor, w_down: torch.Tensor,
@@ -1790,11 +1880,13 @@ _GATE_FORMS = {"silu": 0, "sigmoid": 1}
 
 
 def head_norm_gate(o: torch.Tensor, gain: torch.Tensor, gate: torch.Tensor, eps: float,
-                   out_dtype: torch.dtype, gate_form: str = "silu"):
+                   out_dtype: torch.dtype, gate_form: str = "silu", den=None):
     """out[t, h] = o[t, h] / sqrt(mean(o[t, h]^2) + eps) * gain * act(gate[t, h]) (act:
     silu, or sigmoid with ``gate_form`` "sigmoid") for
     o fp32 [T, heads, vdim]; ``gain`` fp32 [vdim] (shared by the heads) or [heads * vdim];
-    ``gate`` a view [T, heads * vdim] with unit inner stride in ``out_dtype``."""
+    ``gate`` a view [T, heads * vdim] with unit inner stride in ``out_dtype``.  ``den`` (nq,
+    floor, den_eps) with nq and floor fp32 [T, heads]: a head's row is first divided by
+    max(|nq|, floor) + den_eps."""
     _chk("o", o, torch.float32)
     _chk("gain", gain, torch.float32)
     T, H, V = o.shape
@@ -1802,10 +1894,16 @@ def head_norm_gate(o: torch.Tensor, gain: torch.Tensor, gate: torch.Tensor, eps:
     if gain.numel() not in (V, H * V) or gate.dtype != out_dtype or gate.shape[0] != T:
         raise KernelError("head_norm_gate: gain or gate do not fit the heads")
     out = torch.empty((T, H * V), dtype=out_dtype, device=o.device)
+    nq, floor, den_eps = den if den is not None else (None, None, 0.0)
+    _chk("nq", nq, torch.float32, optional=True)
+    _chk("floor", floor, torch.float32, optional=True)
+    if nq is not None and (nq.numel() != T * H or floor is None or floor.numel() != T * H):
+        raise KernelError("head_norm_gate: one denominator per (token, head)")
     _check(_lib().ix_head_norm_gate(
         _ptr(o), _ptr(gain), 1 if (gain.numel() == H * V and H > 1) else 0, _ptr(gate),
         _dtype_code(gate), ctypes.c_longlong(ldg), _ptr(out), _dtype_code(out), T, H, V,
-        ctypes.c_float(eps), _GATE_FORMS[gate_form], _stream()), "head_norm_gate")
+        ctypes.c_float(eps), _GATE_FORMS[gate_form], _ptr(nq), _ptr(floor),
+        ctypes.c_float(den_eps), _stream()), "head_norm_gate")
     _count()
     return out
 
@@ -1868,16 +1966,20 @@ def stream_concat(resid: torch.Tensor, delta, delta_scale: float,
 
 
 def causal_conv(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor],
-                state: torch.Tensor, step, silu: bool = True):
+                state: torch.Tensor, step, silu: bool = True,
+                in_bias: Optional[torch.Tensor] = None):
     """Causal convolution over time per channel with the activation: x [T, C] (a view with
     unit inner stride), ``w`` fp32 [C, taps] whose last column multiplies the current
     token, ``bias`` fp32 [C] or None, ``state`` fp32 [slots, taps - 1, C]: a request's last
     taps - 1 inputs, read for the tokens before this step's first and moved on (None with
-    one tap, which keeps nothing).  Returns
+    one tap, which keeps nothing).  ``in_bias`` fp32 [C] is added to every input first.  Returns
     [T, C] in x's element type."""
     _chk("w", w, torch.float32)
     _chk("bias", bias, torch.float32, optional=True)
+    _chk("in_bias", in_bias, torch.float32, optional=True)
     C, taps = w.shape
+    if in_bias is not None and in_bias.numel() != C:
+        raise KernelError("causal_conv: one input bias per channel")
     _chk("state", state, torch.float32, optional=taps == 1)
     ldx = _row_view("causal_conv: x", x, C)
     T = x.shape[0]
@@ -1886,8 +1988,8 @@ def causal_conv(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor],
         raise KernelError("causal_conv: state or bias do not fit the channels and taps")
     out = torch.empty((T, C), dtype=x.dtype, device=x.device)
     _check(_lib().ix_causal_conv(
-        _ptr(x), _dtype_code(x), ctypes.c_longlong(ldx), _ptr(w), _ptr(bias), _ptr(state),
-        _ptr(step.cu_q), _ptr(step.seq_of_token), _ptr(step.state_slot), _ptr(out), T,
+        _ptr(x), _dtype_code(x), ctypes.c_longlong(ldx), _ptr(in_bias), _ptr(w), _ptr(bias),
+        _ptr(state), _ptr(step.cu_q), _ptr(step.seq_of_token), _ptr(step.state_slot), _ptr(out), T,
         step.num_seqs, C, taps, 1 if silu else 0, _stream()), "causal_conv")
     _count(2 if taps > 1 else 1)
     return out
@@ -2009,12 +2111,7 @@ def normed_pair_mean(left: torch.Tensor, right: torch.Tensor, gain_left: torch.T
 
 def relu_squared(x: torch.Tensor):
     """max(x, 0)^2 in x's element type."""
-    _chk("x", x)
-    out = torch.empty_like(x)
-    _check(_lib().ix_relu_squared(_ptr(x), _ptr(out), _dtype_code(x),
-                                  ctypes.c_longlong(x.numel()), _stream()), "relu_squared")
-    _count()
-    return out
+    return activate(x, "relu_squared")
 
 
 def table_route(token_ids: torch.Tensor, table: torch.Tensor, num_experts: int):
@@ -2413,3 +2510,158 @@ def softcap_rows(x: torch.Tensor, cap: float):
                                   _stream()), "softcap_rows")
     _count()
     return x
+
+
+# ---------------------------------------------------------------------------
+# Several residual streams (csrc/stream_parts.cu) and the matrix memory (csrc/matrix_memory.cu)
+# ---------------------------------------------------------------------------
+def check_stream_limits(streams: int, where: str = ""):
+    most = _lib().ix_stream_max()
+    if streams > most:
+        raise KernelError(f"{where}: {streams} streams exceed the kernel's {most}")
+
+
+def embed_streams(table: torch.Tensor, ids: torch.Tensor, streams: int):
+    """fp32 [T, streams, W]: the table's row of every token in each stream."""
+    _chk("table", table)
+    _chk("ids", ids, torch.int32)
+    T, W = ids.numel(), table.shape[1]
+    out = torch.empty((T, streams, W), dtype=torch.float32, device=table.device)
+    _check(_lib().ix_embed_streams(_ptr(table), _dtype_code(table), _ptr(ids), _ptr(out), T, W,
+                                   streams, _stream()), "embed_streams")
+    _count()
+    return out
+
+
+def stream_step(streams: torch.Tensor, update, read: torch.Tensor, norm, out_dtype: torch.dtype,
+                rows: Optional[torch.Tensor] = None):
+    """streams fp32 [T, n, W].  ``update`` (None: none; else ``y`` [T, W] fp32 or bfloat16 or a
+    mixture's output that was not written, ``mix`` fp32 [n, n], ``put`` fp32 [n]): x_t <- sum_s
+    mix[s, t] x_s + put[t] y, kept unless ``rows`` picks rows to gather.  Returns the reading
+    sum_s read[s] x_s: in fp32 with ``norm`` None, else tanh(alpha u) * gain + bias with
+    ``norm`` = (alpha, gain, bias) in ``out_dtype``."""
+    _chk("streams", streams, torch.float32)
+    _chk("read", read, torch.float32)
+    _chk("rows", rows, torch.int32, optional=True)
+    T, n, W = streams.shape
+    if read.numel() != n:
+        raise KernelError("stream_step: one reading weight per stream")
+    y = combine = mix = put = None
+    if update is not None:
+        y, mix, put = update.y, update.mix, update.put
+        _chk("mix", mix, torch.float32)
+        _chk("put", put, torch.float32)
+        if tuple(mix.shape) != (n, n) or put.numel() != n:
+            raise KernelError("stream_step: mix must be [n, n] and put [n]")
+        if isinstance(y, CombinePending):
+            combine, y = y, None
+            if combine.shape != (T, W):
+                raise KernelError("stream_step: the mixture's output does not fit the streams")
+        else:
+            if hasattr(y, "materialize"):
+                y = y.materialize()
+            _chk("y", y)
+            if tuple(y.shape) != (T, W):
+                raise KernelError("stream_step: y does not fit the streams")
+    alpha = gain = bias = None
+    if norm is not None:
+        alpha, gain, bias = norm
+        for name, t in (("alpha", alpha), ("gain", gain), ("bias", bias)):
+            _chk(name, t, torch.float32)
+        if gain.numel() != W or bias.numel() != W or alpha.numel() != 1:
+            raise KernelError("stream_step: gain and bias must have the streams' width")
+    else:
+        out_dtype = torch.float32
+    R = T if rows is None else rows.numel()
+    out = torch.empty((R, W), dtype=out_dtype, device=streams.device)
+    src = combine.y if combine is not None else y
+    c = combine
+    _check(_lib().ix_stream_step(
+        _ptr(streams), _ptr(y), F32 if src is None else _dtype_code(src),
+        _ptr(c.y if c else None), _ptr(c.dest if c else None), _ptr(c.weights if c else None),
+        _ptr(c.shared if c else None), _ptr(c.shared_logit if c else None),
+        c.topk_w.shape[1] if c else 0, _ptr(mix), _ptr(put), _ptr(read), _ptr(alpha), _ptr(gain),
+        _ptr(bias), _ptr(rows), _ptr(out), _dtype_code(out), R, W, n, 1 if rows is None else 0,
+        _stream()), "stream_step")
+    _count()
+    return out
+
+
+def check_matrix_memory_limits(dim: int, where: str = ""):
+    most = _lib().ix_mm_max_dim()
+    if dim > most:
+        raise KernelError(f"{where}: {dim} key entries per head exceed the matrix memory "
+                          f"kernels' {most}")
+
+
+# Steps of single tokens up to this many take one kernel for the gates' products and the gates
+# (a warp per token and head); beyond, a matrix product and a scan.
+MEMORY_GATES_SINGLE_TOKENS = 128
+
+
+def memory_gates(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, cap: float,
+                 m_state: torch.Tensor, step):
+    """fp32 [3, T, H]: exp(f + m_(t-1) - m_t), exp(i - m_t) and exp(-m_t) of every token and
+    head, with the log gates i = cap tanh(z_i / cap), f = logsigmoid(cap tanh(z_f / cap)), z =
+    x . w^T + bias (``w`` [2 H, W]: the input gates' rows, then the forget gates') and m_t =
+    max(f + m_(t-1), i) along each sequence from and back to ``m_state`` fp32 [slots, H]."""
+    _chk("x", x)
+    _chk("w", w, x.dtype)
+    _chk("bias", bias, torch.float32)
+    _chk("m_state", m_state, torch.float32)
+    T, W = x.shape
+    H = w.shape[0] // 2
+    if w.shape[1] != W or bias.numel() != 2 * H or m_state.shape[1] != H:
+        raise KernelError("memory_gates: weights, biases and state disagree")
+    gates = torch.empty((3, T, H), dtype=torch.float32, device=x.device)
+    if step.all_decode and T == step.num_seqs and T <= MEMORY_GATES_SINGLE_TOKENS:
+        _check(_lib().ix_mm_gates_single(
+            _ptr(x), _ptr(w), _dtype_code(x), _ptr(bias), ctypes.c_float(cap), _ptr(m_state),
+            _ptr(step.state_slot), _ptr(gates), T, W, H, _stream()), "mm_gates_single")
+        _count()
+        return gates
+    z = linear(x, w, out_dtype=torch.float32)
+    _check(_lib().ix_mm_gates_scan(
+        _ptr(z), _ptr(bias), ctypes.c_float(cap), _ptr(m_state), _ptr(step.state_slot),
+        _ptr(step.cu_q), _ptr(gates), T, step.num_seqs, H, _stream()), "mm_gates_scan")
+    _count()
+    return gates
+
+
+def matrix_memory(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: torch.Tensor,
+                  state: torch.Tensor, normaliser: torch.Tensor, step, heads: int, dim: int,
+                  vdim: int, q_scale: float):
+    """S_t = keep S_(t-1) + put k v^T and n_t = keep n_(t-1) + put k along each sequence, from
+    and back to ``state`` [slots, heads, dim, vdim] and ``normaliser`` [slots, heads, dim]
+    (fp32); ``gates`` as ``memory_gates`` leaves them; q, k [T, heads * dim] and v [T, heads *
+    vdim] are views with unit inner stride, q counts times ``q_scale``.  Returns S_t^T q fp32
+    [T, heads, vdim] and n_t . q fp32 [T, heads]."""
+    ldq = _row_view("matrix_memory: q", q, heads * dim)
+    ldk = _row_view("matrix_memory: k", k, heads * dim)
+    ldv = _row_view("matrix_memory: v", v, heads * vdim)
+    _chk("gates", gates, torch.float32)
+    _chk("state", state, torch.float32)
+    _chk("normaliser", normaliser, torch.float32)
+    T = q.shape[0]
+    if not (q.dtype == k.dtype == v.dtype) or k.shape[0] != T or v.shape[0] != T \
+            or tuple(gates.shape) != (3, T, heads) \
+            or tuple(state.shape[1:]) != (heads, dim, vdim) \
+            or tuple(normaliser.shape[1:]) != (heads, dim):
+        raise KernelError("matrix_memory: q, k, v, gates and state do not fit together")
+    num = torch.empty((T, heads, vdim), dtype=torch.float32, device=q.device)
+    nq = torch.empty((T, heads), dtype=torch.float32, device=q.device)
+    views = (_ptr(q), ctypes.c_longlong(ldq), _ptr(k), ctypes.c_longlong(ldk), _ptr(v),
+             ctypes.c_longlong(ldv), _dtype_code(q), _ptr(gates), _ptr(state), _ptr(normaliser))
+    S = step.num_seqs
+    singles = S if step.all_decode else int(getattr(step, "num_decode_seqs", 0))
+    if singles:
+        _check(_lib().ix_mm_single(*views, _ptr(step.state_slot), _ptr(num), _ptr(nq), T, singles,
+                                   heads, dim, vdim, ctypes.c_float(q_scale), _stream()),
+               "mm_single")
+        _count()
+    if singles < S:
+        _check(_lib().ix_mm_walk(*views, _ptr(step.cu_q), _ptr(step.state_slot), _ptr(num),
+                                 _ptr(nq), T, S, singles, heads, dim, vdim,
+                                 ctypes.c_float(q_scale), _stream()), "mm_walk")
+        _count()
+    return num, nq

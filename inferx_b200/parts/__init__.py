@@ -1,6 +1,7 @@
 # importing a module registers the kinds it defines
 from . import (attention, embedding, feed_forward, gated_pair, latent_attention,  # noqa: F401
-               linear_recurrence, norm, position, state_space, token_shift)
+               linear_recurrence, matrix_memory, norm, position, state_space, streams,
+               token_shift)
 from .base import (BuildContext, GroupView, LayerCache, PagedKvNeed, StateNeed,  # noqa: F401
                    StepContext)
 from .block import Block, DecoderModel  # noqa: F401

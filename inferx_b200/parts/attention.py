@@ -13,6 +13,7 @@ import torch
 
 from ..weights.loader import TensorDecl
 from .base import PagedKvNeed, StateNeed
+from .matrix_memory import padded_rows
 from .registry import build_part, register_part
 
 
@@ -207,8 +208,10 @@ class PreparedAttentionMixer:
     and the cache, a short causal convolution, a norm of the whole q and k rows, the
     rotation, a division of every q and k head by its root mean square and a blend of the
     values with those an earlier layer left for this step - each only where the spec asks
-    for it.  The window may keep a request's first tokens visible and the softmax may have
-    one added to its denominator.  Keys and values live in the framework's pages (the
+    for it; the projections may have biases.  The window may keep a request's first tokens visible,
+    the softmax may have one (or a learned number per head, exponentiated) added to its
+    denominator, and a head's result may be multiplied by a gate of its own.  A layer may
+    project queries alone and read another layer's keys and values.  Keys and values live in the framework's pages (the
     value pages as wide as the value heads); the convolutions' last inputs in the state
     slots.  Norms, angles, scores and weights are fp32 in every element type."""
 
@@ -223,6 +226,13 @@ class PreparedAttentionMixer:
         self.vdim = int(s.value_dim or s.head_dim)
         self.dq, self.dk = s.heads * s.head_dim, s.kv_heads * s.head_dim
         self.dv = s.kv_heads * self.vdim
+        self.own_kv = bool(s.own_kv)
+        if not self.own_kv:
+            if s.projection_norm or s.value_mix != "none":
+                raise ValueError(f"{prefix}: a layer without keys and values of its own neither "
+                                 "norms whole projections nor mixes values")
+            self.dk = self.dv = 0
+        self.width = self.dq + self.dk + self.dv      # of a token's projected row
         self.taps = int(s.conv_taps) if s.conv_taps and s.conv_taps > 1 else 1
         self.has_conv = bool(s.conv_taps)
         self.position = build_part("position", s.position, ctx, prefix)
@@ -231,6 +241,7 @@ class PreparedAttentionMixer:
                              "frequencies")
         self.names = dict(s.names)
         self.qkv_w = self.o_w = self.conv_w = self.q_gain = self.k_gain = self.lam = None
+        self.in_bias = self.sink = None
 
     def check_limits(self):
         check = getattr(self.ctx.ops, "check_attention_limits", None)
@@ -245,33 +256,54 @@ class PreparedAttentionMixer:
     def _n(self, key):
         return f"{self.prefix}.{self.names[key]}"
 
+    def _projections(self):
+        """(name, rows) of the projections whose rows a token's projected row is made of."""
+        both = [("k", self.dk), ("v", self.dv)] if self.own_kv else []
+        return [("q", self.dq)] + both
+
     def tensors(self):
         s = self.spec
-        decls = [TensorDecl(self._n("q"), (self.dq, s.hidden)),
-                 TensorDecl(self._n("k"), (self.dk, s.hidden)),
-                 TensorDecl(self._n("v"), (self.dv, s.hidden)),
-                 TensorDecl(self._n("o"), (s.hidden, s.heads * self.vdim))]
-        if self.has_conv:
-            decls += [TensorDecl(self._n("q_conv"), (self.dq, s.conv_taps), keep="float32"),
-                      TensorDecl(self._n("k_conv"), (self.dk, s.conv_taps), keep="float32"),
-                      TensorDecl(self._n("v_conv"), (self.dv, s.conv_taps), keep="float32")]
+        decls = [TensorDecl(self._n(n), (rows, s.hidden)) for n, rows in self._projections()]
+        decls.append(TensorDecl(self._n("o"), (s.hidden, s.heads * self.vdim)))
+        for n, rows in self._projections():
+            if s.bias:
+                decls.append(TensorDecl(self._n(f"{n}_bias"), (rows,), keep="float32",
+                                        init="bias"))
+            if self.has_conv:
+                decls.append(TensorDecl(self._n(f"{n}_conv"), (rows, s.conv_taps),
+                                        keep="float32"))
+        if s.learned_sink:
+            decls.append(TensorDecl(self._n("sink"), (s.heads,), keep="float32", init="bias"))
+        if s.head_gate:
+            decls.append(TensorDecl(self._n("g"), (s.heads, s.hidden)))
         if s.projection_norm:
             decls += [TensorDecl(self._n("q_norm"), (self.dq,), keep="float32", init="gain"),
                       TensorDecl(self._n("k_norm"), (self.dk,), keep="float32", init="gain")]
         # the layer that leaves its values has the scalar too (it is not used there); a layer
         # that mixes nothing may have it in its checkpoint all the same
-        decls.append(TensorDecl(self._n("mix"), (), keep="float32", init="bias",
-                                optional=s.value_mix == "none"))
+        if "mix" in self.names:
+            decls.append(TensorDecl(self._n("mix"), (), keep="float32", init="bias",
+                                    optional=s.value_mix == "none"))
         return decls
 
     def bind(self, w):
         s = self.spec
-        self.qkv_w = torch.cat([w[self._n("q")], w[self._n("k")], w[self._n("v")]],
-                               dim=0).contiguous()
+        names = [n for n, _ in self._projections()]
+        matrices = [w[self._n(n)] for n in names]
+        if s.head_gate:                     # one more number per head beside q, k and v
+            self.qkv_w = padded_rows(matrices + [w[self._n("g")]])
+        else:
+            self.qkv_w = torch.cat(matrices, dim=0).contiguous()
         self.o_w = w[self._n("o")]
         if self.has_conv:
-            self.conv_w = torch.cat([w[self._n("q_conv")], w[self._n("k_conv")],
-                                     w[self._n("v_conv")]], dim=0).contiguous()
+            self.conv_w = torch.cat([w[self._n(f"{n}_conv")] for n in names], dim=0).contiguous()
+        if s.bias:
+            self.in_bias = torch.cat([w[self._n(f"{n}_bias")] for n in names], dim=0).contiguous()
+            if not self.has_conv:           # a convolution of one tap that changes nothing
+                self.conv_w = torch.ones((self.width, 1), dtype=torch.float32,
+                                         device=self.in_bias.device)
+        if s.learned_sink:
+            self.sink = w[self._n("sink")].contiguous()
         if s.projection_norm:
             self.q_gain, self.k_gain = w[self._n("q_norm")], w[self._n("k_norm")]
         if s.value_mix == "mix":
@@ -279,21 +311,27 @@ class PreparedAttentionMixer:
 
     def cache_needs(self):
         s = self.spec
-        needs = [PagedKvNeed(s.kv_heads, s.head_dim, s.window,
-                             entry_dims=(s.head_dim, self.vdim),
-                             keep_first=s.keep_first if s.window > 0 else 0)]
+        needs = []
+        if self.own_kv:
+            window = s.window if s.cache_window is None else s.cache_window
+            needs.append(PagedKvNeed(s.kv_heads, s.head_dim, window,
+                                     entry_dims=(s.head_dim, self.vdim),
+                                     keep_first=s.keep_first if window > 0 else 0))
         if self.taps > 1:
-            needs.append(StateNeed(CONV_INPUTS, (self.taps - 1, self.dq + self.dk + self.dv),
-                                   torch.float32))
+            needs.append(StateNeed(CONV_INPUTS, (self.taps - 1, self.width), torch.float32))
         return needs
 
     def forward(self, x, step, cache):
         s, ops = self.spec, self.ctx.ops
         group = step.groups[cache.group]
-        qkv = ops.linear(x, self.qkv_w)                     # [T, q | k | v]
-        if self.has_conv:
+        front = ops.linear(x, self.qkv_w)                   # [T, q | k | v (| gates)]
+        qkv, gate = front, None
+        if s.head_gate:
+            qkv, gate = front[:, :self.width], front[:, self.width:self.width + s.heads]
+        if self.conv_w is not None:
             qkv = ops.causal_conv(qkv, self.conv_w, None, cache.state.get(CONV_INPUTS), step,
-                                  silu=False)
+                                  silu=False, **({} if self.in_bias is None
+                                                 else {"in_bias": self.in_bias}))
         key = f"value_mix:{s.value_mix_key}"
         earlier = None
         if s.value_mix == "mix":
@@ -304,8 +342,8 @@ class PreparedAttentionMixer:
         if self.position is not None:
             freq, magnitude, rot, interleaved = self.position.pair_table()
         q = ops.attention_prepare(
-            qkv, step.positions, freq, magnitude, rot, interleaved, s.heads, s.kv_heads,
-            s.head_dim, self.vdim, self.q_gain, self.k_gain, s.norm_eps, s.head_unit_norm,
+            qkv, step.positions, freq, magnitude, rot, interleaved, s.heads,
+            s.kv_heads if self.own_kv else 0, s.head_dim, self.vdim, self.q_gain, self.k_gain, s.norm_eps, s.head_unit_norm,
             earlier, self.lam, cache.k if cache.writes else None,
             cache.v if cache.writes else None, group.slots if cache.writes else None)
         if s.value_mix == "source":
@@ -313,7 +351,9 @@ class PreparedAttentionMixer:
             step.shared[key] = qkv[:, self.dq + self.dk:]
         attn = ops.paged_attention(q, cache.k, cache.v, group.block_table, step, s.window,
                                    s.scale, fp32_weights=True,
-                                   keep_first=s.keep_first if s.window > 0 else 0, sink=s.sink)
+                                   keep_first=s.keep_first if s.window > 0 else 0,
+                                   sink=s.sink if self.sink is None else self.sink,
+                                   **({} if gate is None else {"gate": gate}))
         return ops.linear(attn.view(step.num_tokens, s.heads * self.vdim), self.o_w)
 
 

@@ -162,6 +162,16 @@ class PendingSum:
 
 
 @dataclass
+class StreamUpdate:
+    """A sublayer's output on its way into several residual streams: x_t <- sum_s mix[s, t]
+    x_s + put[t] y, all streams at once from the old ones.  ``y`` may be a mixture's output
+    that was not written (anything with ``materialize``)."""
+    y: Any
+    mix: torch.Tensor           # fp32 [n, n], from and to
+    put: torch.Tensor           # fp32 [n]
+
+
+@dataclass
 class LayerCache:
     """What one run of a layer gets from the cache: the paged tensors of the layer it
     reads (its own unless the schedule says otherwise) by entry name, the group whose

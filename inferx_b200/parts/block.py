@@ -20,6 +20,7 @@ from ..weights import loader as wl
 from ..weights.loader import TensorDecl
 from .base import BuildContext, LayerCache, PendingSum, StepContext
 from .registry import build_part, register_part
+from .streams import read_streams
 
 
 class PreNormBlock:
@@ -199,6 +200,8 @@ class DecoderModel:
                 for part in b.parts():
                     if hasattr(part, "check_limits"):
                         part.check_limits()
+            if hasattr(self.embedding, "check_limits"):
+                self.embedding.check_limits()
 
     # -- weights -----------------------------------------------------------
     def _own_tensors(self) -> List[TensorDecl]:
@@ -268,6 +271,12 @@ class DecoderModel:
         """The cache unit a schedule entry reads and writes."""
         return self._unit_index[(entry.cache_layer, getattr(entry, "cache_copy", 0))]
 
+    def state_unit(self, entry) -> int:
+        """The cache unit that holds the entry's state per request: the layer's own, also where
+        its records are another layer's."""
+        return self._unit_index.get((entry.layer, getattr(entry, "cache_copy", 0)),
+                                    self.cache_unit(entry))
+
     def _project_stream(self, resid, pending, before, embedded):
         """The stream becomes W [x; x0]: what is pending is added while the two halves are
         laid side by side in the run's element type, and the product leaves in fp32."""
@@ -334,10 +343,14 @@ class DecoderModel:
             pending = self.blocks[entry.layer].forward(resid, pending, step, cache)
         if logit_rows is None or logit_rows.numel() == 0:
             return None
-        if hasattr(pending, "materialize") and not getattr(self.final_norm, "accepts_pending",
-                                                            False):
-            pending = pending.materialize()
-        n = self.final_norm.forward(resid, pending, rows=logit_rows)
+        if getattr(self.embedding, "streams", 0):     # several streams: their sum is normed
+            n = read_streams(ops, self.final_norm, resid, pending, self.embedding.ones,
+                             rows=logit_rows)
+        else:
+            if hasattr(pending, "materialize") and not getattr(self.final_norm,
+                                                                "accepts_pending", False):
+                pending = pending.materialize()
+            n = self.final_norm.forward(resid, pending, rows=logit_rows)
         logits = ops.linear(n, self.head, out_dtype=torch.float32)
         scale = float(getattr(self.spec, "logit_scale", 1.0))
         if scale != 1.0:

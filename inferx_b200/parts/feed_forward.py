@@ -147,6 +147,14 @@ class MoeFeedForward:
         self.correction = None
         self.score = getattr(spec, "score", "softmax")
         self.weight_input = bool(getattr(spec, "weight_input", False))
+        self.group_value = getattr(spec, "group_value", "max")
+        self.activation = getattr(spec, "expert_activation", None)
+        if self.group_value not in ("max", "pair_sum"):
+            raise ValueError(f"{prefix}: group value {self.group_value!r}")
+        if self.activation not in (None, "gelu", "relu_squared"):
+            raise ValueError(f"{prefix}: expert activation {self.activation!r}")
+        if self.activation is not None and self.weight_input:
+            raise ValueError(f"{prefix}: weights on the experts' inputs need gated experts")
         if self.score not in ("softmax", "sigmoid"):
             raise ValueError(f"{prefix}: router score {self.score!r}")
         if self.weight_input and self.identity:
@@ -185,6 +193,11 @@ class MoeFeedForward:
     def _router_name(self):
         return f"{self.prefix}.{getattr(self.spec, 'router_name', 'gate.weight')}"
 
+    def _shared_gate_tensor(self):
+        s = self.spec
+        suffix = getattr(s, "shared_gate_suffix", ".weight")
+        return f"{self.prefix}.{s.shared_gate_name}{suffix}"
+
     def _expert_names(self, e: int):
         names = getattr(self.spec, "expert_names", (
             "experts.{e}.gate_proj.weight", "experts.{e}.up_proj.weight",
@@ -198,16 +211,13 @@ class MoeFeedForward:
             decls.append(TensorDecl(f"{p}.{self.correction_name}", (self.outputs,),
                                     keep="float32", init="bias"))
         for e in range(s.num_experts):
-            g, u, d = self._expert_names(e)
-            decls += [
-                TensorDecl(g, (s.expert_intermediate, s.hidden)),
-                TensorDecl(u, (s.expert_intermediate, s.hidden)),
-                TensorDecl(d, (s.hidden, s.expert_intermediate)),
-            ]
+            *up, d = self._expert_names(e)
+            decls += [TensorDecl(n, (s.expert_intermediate, s.hidden)) for n in up]
+            decls.append(TensorDecl(d, (s.hidden, s.expert_intermediate)))
         if self.shared is not None:
             decls += self.shared.tensors()
             if s.shared_gated:
-                decls.append(TensorDecl(f"{p}.{s.shared_gate_name}.weight", (1, s.hidden),
+                decls.append(TensorDecl(self._shared_gate_tensor(), (1, s.hidden),
                                         keep="float32"))
         return decls
 
@@ -216,14 +226,15 @@ class MoeFeedForward:
         self.router_w = w[self._router_name()]
         if self.correction_name:
             self.correction = w[f"{p}.{self.correction_name}"]
-        gu = torch.empty((s.num_experts, 2 * s.expert_intermediate, s.hidden),
+        I = s.expert_intermediate
+        gu = torch.empty((s.num_experts, (1 if self.activation else 2) * I, s.hidden),
                          dtype=self.ctx.dtype, device=self.ctx.device)
-        dn = torch.empty((s.num_experts, s.hidden, s.expert_intermediate),
-                         dtype=self.ctx.dtype, device=self.ctx.device)
+        dn = torch.empty((s.num_experts, s.hidden, I), dtype=self.ctx.dtype,
+                         device=self.ctx.device)
         for e in range(s.num_experts):
-            g, u, d = self._expert_names(e)
-            gu[e, :s.expert_intermediate] = w[g]
-            gu[e, s.expert_intermediate:] = w[u]
+            *up, d = self._expert_names(e)
+            for j, n in enumerate(up):      # gate rows, then up rows
+                gu[e, j * I:(j + 1) * I] = w[n]
             dn[e] = w[d]
         self.expert_gate_up, self.expert_down = gu, dn
         if self.shared is not None:
@@ -231,7 +242,7 @@ class MoeFeedForward:
             self._shared_bytes = sum(w[d.name].numel() * w[d.name].element_size()
                                      for d in self.shared.tensors())
             if s.shared_gated:
-                self.shared_gate_w = w[f"{p}.{s.shared_gate_name}.weight"].reshape(-1).contiguous()
+                self.shared_gate_w = w[self._shared_gate_tensor()].reshape(-1).contiguous()
 
     # In a step of few tokens the kernels leave the GPU partly idle; the shared
     # expert (which needs nothing from the router) then runs beside the routed experts,
@@ -309,8 +320,9 @@ class MoeFeedForward:
                 x, self.router_w, s.top_k, s.renormalize, s.routed_scale,
                 extra_w=self.shared_gate_w, correction=self.correction,
                 group_count=self.group_count, group_keep=self.group_keep,
-                renorm_eps=self.renorm_eps, **({} if self.score == "softmax"
-                                               else {"score": self.score}))
+                renorm_eps=self.renorm_eps,
+                **({} if self.score == "softmax" else {"score": self.score}),
+                **({} if self.group_value == "max" else {"group_value": self.group_value}))
         else:
             topk_w, topk_idx, shared_logit = ops.router_topk(
                 x, self.router_w, s.top_k, s.renormalize, s.routed_scale,
@@ -328,7 +340,9 @@ class MoeFeedForward:
             side.wait_event(ready)
             with torch.cuda.stream(side):
                 shared = self.shared.forward(x, step)
-        if row_w is None:
+        if self.activation is not None:
+            act = ops.grouped_up(x, rows, offsets, self.expert_gate_up, self.activation)
+        elif row_w is None:
             act = ops.grouped_gate_up_swiglu(x, rows, offsets, self.expert_gate_up)
         else:
             act = ops.grouped_gate_up_swiglu(x, rows, offsets, self.expert_gate_up,
@@ -371,6 +385,31 @@ class ReluSquaredFeedForward:
         ops = self.ctx.ops
         act = ops.relu_squared(ops.linear(x, self.up_w))
         return ops.linear(act, self.down_w, out_dtype=torch.float32)
+
+
+class ActivatedMlpFeedForward:
+    """``down(act(up h))``, no biases; the activation sits in the product's epilogue where the
+    step is small enough for this library's own kernels."""
+
+    def __init__(self, spec, ctx, prefix: str):
+        self.spec, self.ctx, self.prefix = spec, ctx, prefix
+        if spec.activation not in ("gelu", "relu_squared"):
+            raise ValueError(f"{prefix}: activation {spec.activation!r}")
+        self.up_w = self.down_w = None
+
+    def tensors(self):
+        s, p = self.spec, self.prefix
+        u, d = s.names
+        return [TensorDecl(f"{p}.{u}", (s.intermediate, s.hidden)),
+                TensorDecl(f"{p}.{d}", (s.hidden, s.intermediate))]
+
+    def bind(self, w):
+        u, d = self.spec.names
+        self.up_w, self.down_w = w[f"{self.prefix}.{u}"], w[f"{self.prefix}.{d}"]
+
+    def forward(self, x, step=None):
+        ops = self.ctx.ops
+        return ops.linear(ops.linear_act(x, self.up_w, self.spec.activation), self.down_w)
 
 
 class TableMoeFeedForward:
@@ -437,5 +476,6 @@ register_part("feed_forward", "swiglu", SwiGluFeedForward)
 register_part("feed_forward", "moe", MoeFeedForward)
 register_part("feed_forward", "clamped_glu", ClampedGluFeedForward)
 register_part("feed_forward", "relu_squared", ReluSquaredFeedForward)
+register_part("feed_forward", "mlp_activated", ActivatedMlpFeedForward)
 register_part("feed_forward", "glu_biased", BiasedGluFeedForward)
 register_part("feed_forward", "moe_table", TableMoeFeedForward)

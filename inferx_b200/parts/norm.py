@@ -130,3 +130,42 @@ class GroupedRmsNorm:
 
 
 register_part("norm", "grouped_rmsnorm", GroupedRmsNorm)
+
+
+class DynamicTanh:
+    """tanh(alpha x) * gain + bias entry by entry, with a scalar alpha: no mean, no variance.
+    Reads a plain residual stream (the pending contribution added in the same pass) or one of
+    several streams beside each other (``forward_streams``: their update, the weighted reading
+    and the tanh in one pass)."""
+    accepts_pending = True
+    accepts_scaled = True
+
+    def __init__(self, spec, ctx, prefix: str):
+        self.spec, self.ctx = spec, ctx
+        self.name = f"{prefix}{getattr(spec, 'suffix', '')}"
+        self.gain = self.bias = self.alpha = None
+        self.one = torch.ones(1, dtype=torch.float32, device=ctx.device)
+
+    def tensors(self):
+        n = self.spec.size
+        return [TensorDecl(self.name, (n,), keep="float32", init="gain"),
+                TensorDecl(f"{self.name}.b", (n,), keep="float32", init="bias"),
+                TensorDecl(f"{self.name}.alpha", (), keep="float32", init="gain")]
+
+    def bind(self, weights):
+        self.gain, self.bias = weights[self.name], weights[f"{self.name}.b"]
+        self.alpha = weights[f"{self.name}.alpha"].reshape(1).contiguous()
+
+    def forward_streams(self, streams, update, read, rows=None):
+        return self.ctx.ops.stream_step(streams, update, read, (self.alpha, self.gain, self.bias),
+                                        self.ctx.dtype, rows=rows)
+
+    def forward(self, resid, delta, rows=None):
+        from .base import StreamUpdate
+        if hasattr(delta, "terms"):
+            delta = delta.materialize()
+        update = None if delta is None else StreamUpdate(delta, self.one.view(1, 1), self.one)
+        return self.forward_streams(resid.unsqueeze(1), update, self.one, rows=rows)
+
+
+register_part("norm", "dynamic_tanh", DynamicTanh)

@@ -115,8 +115,8 @@ register_part("position", "sinusoid_added", SinusoidAdded)
 
 class ScaledRotary:
     """Rotation of pairs of a head's first ``rotary_dim`` entries, in either pairing, with
-    the frequencies stretched by wavelength or by a ramp over the pair index (the spec
-    says how).  ``pair_table()`` gives (frequency per pair as fp32 [rotary_dim / 2], the
+    the frequencies stretched by wavelength, by a ramp over the pair index or all by one factor
+    (the spec says how).  ``pair_table()`` gives (frequency per pair as fp32 [rotary_dim / 2], the
     factor on cos and sin, rotary_dim, whether pairs are neighbours).  The frequencies are
     formed in float64 and rounded once; the kernel multiplies position and frequency, and
     takes cos and sin, in fp32."""
@@ -156,8 +156,10 @@ class ScaledRotary:
             ramp = [min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0) for i in range(r // 2)]
             f = [v / factor * t + v * (1.0 - t) for v, t in zip(f, ramp)]
             self.magnitude = 0.1 * math.log(factor) + 1.0
+        elif sc is not None and sc[0] == "linear":
+            f = [v / sc[1] for v in f]
         elif sc is not None:
-            raise ValueError(f"rotary scaling {sc[0]!r} is not 'wavelength' or 'ramp'")
+            raise ValueError(f"rotary scaling {sc[0]!r} is not 'wavelength', 'ramp' or 'linear'")
         self.freq = torch.tensor(f, dtype=torch.float64).to(torch.float32).to(ctx.device)
 
     def tensors(self):

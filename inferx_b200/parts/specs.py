@@ -49,6 +49,15 @@ class LayerNormSpec:
 
 
 @dataclass(frozen=True)
+class DynamicTanhSpec:
+    """tanh(alpha * x) * w + b entry by entry: no mean, no variance.  The scalar alpha and the
+    vector b are tensors beside the weight, ``<name>.alpha`` and ``<name>.b``."""
+    size: int
+    suffix: str = ""
+    kind: str = "dynamic_tanh"
+
+
+@dataclass(frozen=True)
 class RopeSpec:
     """Half-split (NeoX) rotary encoding of the first ``rotary_dim`` of each head.  Every
     frequency is divided by ``scaling_factor`` (linear position scaling; 1: none)."""
@@ -322,6 +331,45 @@ class MinGruSpec:
 
 
 @dataclass(frozen=True)
+class MatrixMemorySpec:
+    """Matrix memory with exponential gates.  Per head: log gates i = cap tanh((W_i h + b_i) /
+    cap) and f = logsigmoid(cap tanh((W_f h + b_f) / cap)) with cap = ``gate_cap``; running
+    maximum m_t = max(f + m_(t-1), i), m = 0 at the start; S_t = exp(f + m_(t-1) - m_t) S_(t-1)
+    + exp(i - m_t) k v^T, n_t likewise with k alone; o = S_t^T q / (max(|n_t . q|, exp(-m_t)) +
+    ``den_eps``) with q times ``q_scale``.  o is divided by its root mean square per head
+    (``norm_eps``), multiplied by a gain over all heads and by sigmoid(W_g h), projected.
+    State per request, fp32: S [heads, dim, vdim], n [heads, dim], m [heads]."""
+    hidden: int
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+    q_scale: float
+    norm_eps: float
+    den_eps: float = 1e-6
+    kind: str = "matrix_memory"
+
+
+@dataclass(frozen=True)
+class HyperConnectionSpec:
+    """How a layer's two sublayers read and write ``streams`` residual streams: per sublayer
+    u = sum_s in[s] x_s, then x_t <- sum_s mix[s, t] x_s + out[t] y.  ``sublayers`` are the
+    names inside the layer's prefix (mixer, feed-forward), ``names`` the tensors inside."""
+    streams: int
+    sublayers: tuple = ("hc1", "hc2")
+    names: tuple = ("in", "out", "mix")
+    kind: str = "hyper_connection"
+
+
+@dataclass(frozen=True)
+class StreamCopiesSpec:
+    """The residual stream is ``streams`` streams, all equal to the token's embedding at the
+    start; the model's last norm reads their sum."""
+    streams: int
+    kind: str = "stream_copies"
+
+
+@dataclass(frozen=True)
 class ScaledPairSpec:
     """Two mixers side by side reading the same input; the result is
     ``left_scale`` * left + ``right_scale`` * right."""
@@ -342,6 +390,17 @@ class ReluSquaredSpec:
     intermediate: int
     names: tuple = ("up", "down")
     kind: str = "relu_squared"
+
+
+@dataclass(frozen=True)
+class ActivatedMlpSpec:
+    """down(act(up h)) without biases, ``activation`` "relu_squared" or "gelu" (the exact,
+    erf form)."""
+    hidden: int
+    intermediate: int
+    activation: str
+    names: tuple = ("up", "down")
+    kind: str = "mlp_activated"
 
 
 @dataclass(frozen=True)
@@ -372,7 +431,7 @@ class ScaledRopeSpec:
     (2 pi t)) / (2 ln theta), lo = max(floor(pair(fast)), 0), hi = min(ceil(pair(slow)),
     rotary_dim - 1) and r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1) the frequency is
     f_i / factor * r_i + f_i (1 - r_i), and cos and sin are multiplied by
-    0.1 ln(factor) + 1."""
+    0.1 ln(factor) + 1; ("linear", factor): every f is divided by the factor."""
     head_dim: int
     rotary_dim: int
     theta: float
@@ -392,11 +451,16 @@ class PreparedAttentionSpec:
     (``head_unit_norm``), and the value mixing: with ``value_mix`` "mix" the values become
     (1 - lambda) v + lambda v0, v0 being the values of the same token left by the layer
     whose ``value_mix`` is "source" (the first of the model that mixes) and lambda a
-    scalar of the checkpoint; what is mixed is what the cache holds.  A query at position
+    scalar of the checkpoint; what is mixed is what the cache holds.  ``bias``: the
+    projections have biases, added before the convolution.  A query at position
     i sees key j <= i when i - j < ``window`` (0: all) or j < ``keep_first``.  With
     ``sink`` one is added to the softmax's denominator (a key of score 0 without a
-    value).  Scores are (q . k) * scale; scores, weights and their products with the values
-    are 32-bit arithmetic in every element type."""
+    value); with ``learned_sink`` the exponential of a number per head of the checkpoint.
+    ``head_gate``: head h's result is multiplied by sigmoid(W_g x)_h.  Scores are (q . k) *
+    scale; scores, weights and their products with the values are 32-bit arithmetic in every
+    element type.  ``own_kv`` off: the layer projects queries alone and reads the keys and
+    values another layer keeps (the schedule names it); that layer's ``cache_window`` then
+    says for how many tokens they are kept (0: all, None: its own window)."""
     hidden: int
     heads: int
     kv_heads: int
@@ -413,6 +477,11 @@ class PreparedAttentionSpec:
     head_unit_norm: bool = False
     value_mix: str = "none"          # "none" | "source" | "mix"
     value_mix_key: str = "values"    # layers that mix with one another share the key
+    bias: bool = False
+    learned_sink: bool = False
+    head_gate: bool = False
+    own_kv: bool = True
+    cache_window: Optional[int] = None
     names: tuple = (("q", "q"), ("k", "k"), ("v", "v"), ("o", "o"), ("q_norm", "q.norm"),
                     ("k_norm", "k.norm"), ("q_conv", "q.conv"), ("k_conv", "k.conv"),
                     ("v_conv", "v.conv"), ("mix", "vmix"))
@@ -468,8 +537,10 @@ class MoeSpec:
     shared_gated: bool        # its output scaled by sigmoid(x . w_gate)
     shared_name: str = "shared_expert"
     shared_gate_name: str = "shared_expert_gate"
+    shared_gate_suffix: str = ".weight"
     # tensor names inside the part's prefix: the router's matrix, and one expert's
-    # prefix with {e} for its number followed by its gate, up and down matrices
+    # prefix with {e} for its number followed by its gate, up and down matrices (up and down
+    # alone for experts without a gate)
     router_name: str = "gate.weight"
     expert_names: tuple = ("experts.{e}.gate_proj.weight", "experts.{e}.up_proj.weight",
                            "experts.{e}.down_proj.weight")
@@ -491,6 +562,11 @@ class MoeSpec:
     score: str = "softmax"
     # The weight multiplies the expert's input instead of its output: expert(w h).
     weight_input: bool = False
+    # What a group is worth: the "max" of its choice scores, or the sum of its two largest.
+    group_value: str = "max"         # "max" | "pair_sum"
+    # Experts without a gate: down(act(up h)) with this activation ("gelu", "relu_squared");
+    # None: down(silu(gate h) * (up h)).
+    expert_activation: Optional[str] = None
     kind: str = "moe"
 
 
@@ -500,7 +576,9 @@ class LayerSpec:
     x += mixer(norm(x)); x += ffn(norm(x)); "sublayer_norm" is x += norm(mixer(x));
     x += norm(ffn(x)), where ``input_norm`` follows the mixer and ``post_norm`` the
     feed-forward (``ffn`` and ``post_norm`` may be None: a layer without feed-forward);
-    "parallel" is x += mixer(input_norm(x)) + ffn(post_norm(x)), both of the same x."""
+    "parallel" is x += mixer(input_norm(x)) + ffn(post_norm(x)), both of the same x;
+    "hyper_connected" is the pre-norm order on several streams (``connection`` says how a
+    sublayer reads and writes them)."""
     prefix: str  # tensor-name prefix, e.g. "model.layers.3"
     input_norm: Any
     mixer: Any
@@ -517,6 +595,8 @@ class LayerSpec:
     mixer_input_name: str = "shift"
     # "pre_norm" only: each sublayer's output is multiplied by this before it is added
     residual_scale: float = 1.0
+    # "hyper_connected" only: a HyperConnectionSpec
+    connection: Any = None
 
 
 @dataclass(frozen=True)

@@ -94,8 +94,10 @@ def append_kv(k, v, k_cache, v_cache, slots):
 
 
 def paged_attention_generic(q, k_cache, v_cache, block_table, seq_of_token, positions, window,
-                            scale, softcap=0.0, keep_first=0, sink=False):
+                            scale, softcap=0.0, keep_first=0, sink=None, gate=None):
     T, heads, hd = q.shape
+    if isinstance(sink, bool):        # True: a sink of zero in every head
+        sink = torch.zeros(heads) if sink else None
     P, kvh, page, _ = k_cache.shape
     rep = heads // kvh
     out = torch.zeros(T, heads, v_cache.shape[3], dtype=torch.float32)
@@ -115,22 +117,25 @@ def paged_attention_generic(q, k_cache, v_cache, block_table, seq_of_token, posi
             sc = (keys @ _f(q[t, h])) * scale
             if softcap > 0:
                 sc = softcap * torch.tanh(sc / softcap)
-            top = torch.clamp(sc.max(), min=0.0) if sink else sc.max()
+            top = sc.max() if sink is None else torch.maximum(sc.max(), _f(sink[h]))
             p = torch.exp(sc - top)
-            # the sink: a key of score 0 that has no value
-            den = p.sum() + (torch.exp(-top) if sink else 0.0)
+            # the sink: a key of that score that has no value
+            den = p.sum() + (0.0 if sink is None else torch.exp(_f(sink[h]) - top))
             out[t, h] = (p[:, None] * vals).sum(0) / den
+            if gate is not None:
+                out[t, h] *= torch.sigmoid(_f(gate[t, h]))
     return out.to(q.dtype)
 
 
 def paged_attention(q, k_cache, v_cache, block_table, step, window, scale, softcap=0.0,
-                    fp32_weights=False, keep_first=0, sink=False):
+                    fp32_weights=False, keep_first=0, sink=None, gate=None):
     return paged_attention_generic(q, k_cache, v_cache, block_table, step.seq_of_token,
-                                   step.positions, window, scale, softcap, keep_first, sink)
+                                   step.positions, window, scale, softcap, keep_first, sink,
+                                   gate)
 
 
 def router_topk(x, w, top_k, renormalize, scale, extra_w=None, correction=None, group_count=0,
-                group_keep=0, renorm_eps=-1.0, score="softmax"):
+                group_keep=0, renorm_eps=-1.0, score="softmax", group_value="max"):
     logits = _f(x) @ w.T
     p = torch.sigmoid(logits) if score == "sigmoid" else torch.softmax(logits, dim=-1)
     T, E = p.shape
@@ -141,7 +146,8 @@ def router_topk(x, w, top_k, renormalize, scale, extra_w=None, correction=None, 
             pick = logits.clone()         # the same order, also where the sigmoid is flat
         if group_count:
             size = E // group_count
-            best = pick.view(T, group_count, size).max(-1).values
+            best = pick.view(T, group_count, size).sort(-1, descending=True).values
+            best = best[..., :2].sum(-1) if group_value == "pair_sum" else best[..., 0]
             kept = torch.zeros(T, group_count, dtype=torch.bool)
             work = best.clone()
             for _ in range(group_keep):
@@ -531,8 +537,11 @@ def linear_recurrence(q, k, v, decay, bonus, state, step, heads, dim, vdim, q_sc
     return out
 
 
-def head_norm_gate(o, weight, gate, eps, out_dtype, gate_form="silu"):
+def head_norm_gate(o, weight, gate, eps, out_dtype, gate_form="silu", den=None):
     T, H, V = o.shape
+    if den is not None:
+        nq, floor, den_eps = den
+        o = o / (torch.maximum(nq.abs(), floor) + den_eps)[:, :, None]
     n = o / torch.sqrt((o * o).mean(-1, keepdim=True) + eps)
     n = n * (weight.reshape(H, V) if weight.numel() == H * V else weight)
     g = _f(gate).reshape(T, H, V)
@@ -575,8 +584,9 @@ def stream_concat(resid, delta, delta_scale, vector, first, out_dtype):
     return torch.cat([x, first], -1).to(out_dtype)
 
 
-def causal_conv(x, w, bias, state, step, silu=True):
+def causal_conv(x, w, bias, state, step, silu=True, in_bias=None):
     T, C = x.shape
+    shift = 0.0 if in_bias is None else in_bias
     taps = w.shape[1]
     out = torch.zeros(T, C)
     for s in range(step.num_seqs):
@@ -585,7 +595,7 @@ def causal_conv(x, w, bias, state, step, silu=True):
             continue
         slot = int(step.state_slot[s])
         past = state[slot] if taps > 1 else torch.zeros(0, C)
-        rows = torch.cat([past, _f(x[a:b])], 0)                   # [taps - 1 + n, C]
+        rows = torch.cat([past, _f(x[a:b]) + shift], 0)                   # [taps - 1 + n, C]
         acc = torch.zeros(b - a, C) if bias is None else bias[None, :].repeat(b - a, 1)
         for j in range(taps):
             acc = acc + rows[j:j + b - a] * w[:, j]
@@ -836,3 +846,91 @@ def latent_queries(q, positions, freq, mag, heads, dim, rot_dim, rot_dims):
 def softcap_rows(x, cap):
     x.copy_(cap * torch.tanh(x / cap))
     return x
+
+
+# ---------------------------------------------------------------------------------------
+# several residual streams, the matrix memory, and products with an activation but no gate
+def _activate(v, activation):
+    if activation == "gelu":
+        return 0.5 * v * (1.0 + torch.erf(v * 0.7071067811865476))
+    assert activation == "relu_squared"
+    return torch.relu(v) ** 2
+
+
+def activate(x, activation, out=None):
+    y = _activate(_f(x), activation).to(x.dtype)
+    if out is None:
+        return y
+    out.copy_(y)
+    return out
+
+
+def linear_act(x, w, activation):
+    return _activate(_f(x) @ _f(w).T, activation).to(x.dtype)
+
+
+def grouped_up(x, rows, offsets, w_up, activation):
+    E, i, H = w_up.shape
+    out = torch.zeros(rows.numel(), i, dtype=torch.float32)
+    for e in range(E):
+        lo, hi = int(offsets[e]), int(offsets[e + 1])
+        if hi > lo:
+            out[lo:hi] = _activate(_f(x[rows[lo:hi].long()]) @ _f(w_up[e]).T, activation)
+    return out.to(x.dtype)
+
+
+def embed_streams(table, ids, streams):
+    return _f(table[ids.long()])[:, None, :].repeat(1, streams, 1)
+
+
+def stream_step(streams, update, read, norm, out_dtype, rows=None):
+    x = streams
+    if update is not None:
+        y = update.y.materialize() if hasattr(update.y, "materialize") else update.y
+        x = torch.einsum("tsw,so->tow", streams, update.mix) + \
+            update.put[None, :, None] * _f(y)[:, None, :]
+        if rows is None:
+            streams.copy_(x)
+    if rows is not None:
+        x = x[rows.long()]
+    u = (read[None, :, None] * x).sum(1)
+    if norm is None:
+        return u
+    alpha, gain, bias = norm
+    return (torch.tanh(alpha * u) * gain + bias).to(out_dtype)
+
+
+def memory_gates(x, w, bias, cap, m_state, step):
+    T, H = x.shape[0], w.shape[0] // 2
+    z = _f(x) @ _f(w).T + bias
+    i = cap * torch.tanh(z[:, :H] / cap)
+    f = torch.nn.functional.logsigmoid(cap * torch.tanh(z[:, H:] / cap))
+    out = torch.zeros(3, T, H)
+    for s in range(step.num_seqs):
+        slot = int(step.state_slot[s])
+        m = m_state[slot].clone()
+        for t in range(int(step.cu_q[s]), int(step.cu_q[s + 1])):
+            new = torch.maximum(f[t] + m, i[t])
+            out[0, t], out[1, t] = torch.exp(f[t] + m - new), torch.exp(i[t] - new)
+            out[2, t] = torch.exp(-new)
+            m = new
+        m_state[slot] = m
+    return out
+
+
+def matrix_memory(q, k, v, gates, state, normaliser, step, heads, dim, vdim, q_scale):
+    T = q.shape[0]
+    qf = _f(q).reshape(T, heads, dim) * q_scale
+    kf, vf = _f(k).reshape(T, heads, dim), _f(v).reshape(T, heads, vdim)
+    num, nq = torch.zeros(T, heads, vdim), torch.zeros(T, heads)
+    for s in range(step.num_seqs):
+        slot = int(step.state_slot[s])
+        S, n = state[slot].clone(), normaliser[slot].clone()
+        for t in range(int(step.cu_q[s]), int(step.cu_q[s + 1])):
+            kk = gates[1, t][:, None] * kf[t]
+            S = gates[0, t][:, None, None] * S + kk[:, :, None] * vf[t][:, None, :]
+            n = gates[0, t][:, None] * n + kk
+            num[t] = torch.einsum("hkv,hk->hv", S, qf[t])
+            nq[t] = (n * qf[t]).sum(-1)
+        state[slot], normaliser[slot] = S, n
+    return num, nq
