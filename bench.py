@@ -997,6 +997,51 @@ def dominex_configs(z, layers, kind):
     return new, twin
 
 
+# `--designs --design biguzen`: the Biguzen design, one line per kind of layer beside the model
+# that has the closest kind at equal sizes.  "memory" layers (matrix memory with exponential
+# gates) beside Tinapel's gated linear attention with a state of the same size; "attention"
+# layers (biases, convolutions, sink, head gates; every second layer reading the keys and
+# values of the one before it) beside Fudulix's attention with convolutions over the same
+# window.  Both kinds carry a mixture of as many experts of the same inner width and a shared
+# one; Biguzen's experts have no gate (two matrices where the twins have three), and it
+# carries four residual streams where they have one.
+BIGUZEN_SIZES = TINAPEL_SIZES
+BIGUZEN_WINDOW = 1024
+
+
+def biguzen_configs(z, layers, kind):
+    import math
+    W = z["width"]
+    moe = {"kind": "moe", "expert": {"ff": z["ff"]}, "shared": {"ff": z["shared"]}}
+    mlp = dict(moe, router={"experts": z["experts"], "top": z["top"], "scale": 1.5,
+                            "groups": {"count": 4, "keep": 2}})
+    new = {"architecture": "Biguzen", "vocab": DESIGN_VOCAB, "width": W, "streams": 4,
+           "norm": {"eps": 1e-6}}
+    if kind == "memory":
+        heads = {"heads": W // 128, "dim": 64, "vdim": 128}
+        new["layers"] = [{"type": "mlstm", "mixer": dict(heads, gate_cap=15.0),
+                          "mlp": mlp}] * layers
+        twin = {"architecture": "Tinapel", "vocab": DESIGN_VOCAB, "width": W,
+                "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6},
+                "layers": [{"type": "gla", "mixer": dict(heads, tau=8.0, rank=64), "mlp": dict(
+                    moe, router={"experts": z["experts"], "top": z["top"], "scale": 1.0})}]
+                * layers}
+        return new, twin
+    attn = {"heads": z["heads"], "kv_heads": z["kv"], "dim": 128, "vdim": 128,
+            "scale": 1.0 / math.sqrt(128.0), "conv": 4, "mask": {"size": BIGUZEN_WINDOW}}
+    new["layers"] = [{"type": "attention", "mlp": mlp, "mixer": dict(
+        attn, rot={"dims": 64, "base": 10000.0, "scaling": {"factor": 2.0}},
+        **({"kv_from": i - 1} if i % 2 else {}))} for i in range(layers)]
+    twin = {"architecture": "Fudulix", "vocab": DESIGN_VOCAB, "width": W, "norm": {"eps": 1e-6},
+            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 7}},
+            "layers": [{"type": "attention_2", "mixer": dict(
+                attn, v_mix=False, mask={"size": BIGUZEN_WINDOW, "keep_first": 0},
+                rot={"dims": 64, "base": 10000.0}), "mlp": dict(
+                    moe, router={"experts": z["experts"], "top": z["top"],
+                                 "groups": {"count": 4, "keep": 2}})}] * layers}
+    return new, twin
+
+
 def designs(args):
     """One JSON line per size: prompt tokens/s (one prompt of --prefill-tokens, default
     2048) and decode tokens/s (--batch sequences at --context) of both designs, device
@@ -1009,22 +1054,27 @@ def designs(args):
     mapovik = args.design == "mapovik"
     fudulix = args.design == "fudulix"
     dominex = args.design == "dominex"
-    sizes = (DOMINEX_SIZES if dominex else FUDULIX_SIZES if fudulix else MAPOVIK_SIZES if mapovik
+    biguzen = args.design == "biguzen"
+    sizes = (BIGUZEN_SIZES if biguzen else DOMINEX_SIZES if dominex else FUDULIX_SIZES if fudulix else MAPOVIK_SIZES if mapovik
              else TINAPEL_SIZES if tinapel else DESIGN_SIZES)
     first, second = (("fudulix", "qwen2_moe") if fudulix else ("mapovik", "tinapel") if mapovik
                      else ("tinapel", "qwen2_moe") if tinapel else ("zuzisun", "qwen2_dense"))
     names = args.design_sizes.split(",") if args.design_sizes else list(sizes)
     kinds = [None]
-    if dominex:
+    if dominex or biguzen:
         kinds = ([k for k in args.design_pattern.split(",")] if "wkv" not in args.design_pattern
-                 else ["parallel", "latent"])
+                 else ["memory", "attention"] if biguzen else ["parallel", "latent"])
     for name, kind in ((n, k) for n in names for k in kinds):
         z = sizes[name]
         C = args.context or 4096
         row = {"size": name, "layers": layers, "width": z["width"], "heads": z["heads"],
                "ff": z["ff"], "prompt_tokens": prompt, "batch": B,
                "context": C, "dtype": "bf16", "data": "synthetic, random weights"}
-        if dominex:
+        if biguzen:
+            first, second = "biguzen", {"memory": "tinapel", "attention": "fudulix"}[kind]
+            row.update(layer_kind=kind, window=BIGUZEN_WINDOW if kind == "attention" else 0)
+            pair = biguzen_configs(z, layers, kind)
+        elif dominex:
             first, second = "dominex", {"parallel": "mapovik", "latent": "zuzisun"}[kind]
             row["layer_kind"] = kind
             pair = dominex_configs(z, layers, kind)
@@ -1108,13 +1158,15 @@ def main(argv=None):
                          "beside the closest Qwen2-MoE at equal sizes (random weights); --layers (4), "
                          "--batch, --context (4096), --prefill-tokens (2048) apply")
     ap.add_argument("--design-sizes", default="", help="with --designs: of 1k,2k,4k (all)")
-    ap.add_argument("--design", default="zuzisun", choices=["zuzisun", "tinapel", "mapovik", "fudulix", "dominex"],
+    ap.add_argument("--design", default="zuzisun", choices=["zuzisun", "tinapel", "mapovik", "fudulix", "dominex",
+                                                              "biguzen"],
                     help="with --designs: which design stands beside its closest model")
     ap.add_argument("--design-pattern", default="wkv,gla,attention,attention",
                     help="with --design tinapel: the mixers of the layers, repeated; with "
                          "--design mapovik of parallel, delta (default "
                          "parallel,delta,delta,parallel); with --design dominex the kinds of "
-                         "layers to report, of parallel, latent (both)")
+                         "layers to report, of parallel, latent (both); with --design biguzen "
+                         "of memory, attention (both)")
     args = ap.parse_args(argv)
     if args.impl == "reference":
         return reference_arm()

@@ -61,15 +61,15 @@ class CacheStorage:
     def layer_caches(self, schedule, unit_of=None, state_unit_of=None) -> List[LayerCache]:
         """One ``LayerCache`` per schedule entry.  ``unit_of(entry)`` gives the index of the
         entry's cache among the needs this storage was built from (the layer it names,
-        when absent).  A layer that reads another's pages and has state of its own
-        (``state_unit_of(entry)``) keeps that."""
+        when absent).  State is never shared: a layer that reads another's pages has the
+        state of ``state_unit_of(entry)``, its own unit."""
         out = []
         for e in schedule:
             src = unit_of(e) if unit_of is not None else e.cache_layer
             own = state_unit_of(e) if state_unit_of is not None else src
             out.append(LayerCache(
                 group=self.group_of_layer.get(src, -1), pages=self.paged.get(src, {}),
-                writes=e.writes_cache, state=self.state.get(own) or self.state.get(src, {})))
+                writes=e.writes_cache, state=self.state.get(own, {})))
         return out
 
     def unit_cache(self, unit: int) -> LayerCache:

@@ -25,7 +25,8 @@ __device__ __forceinline__ float mm_log_sigmoid(float z) {
 // ---------------------------------------------------------------------------
 // Steps of single tokens: one warp per (token, head) forms both dot products and moves the
 // running maximum on.  x [T, W] and w [2 H, W] (input gates' rows, then forget gates') of one
-// type; gates [3, T, H]: keep, put, floor.
+// type; gates [4, T, H]: keep, put, floor and
+// the logarithm of keep.
 // ---------------------------------------------------------------------------
 #define MG_WARPS 4
 
@@ -79,6 +80,7 @@ mm_gates_single_kernel(const TA* __restrict__ x, const TA* __restrict__ w,
     gates[at] = expf(f + before - m);
     gates[plane + at] = expf(i - m);
     gates[2 * plane + at] = expf(-m);
+    gates[3 * plane + at] = f + before - m;
   }
 }
 
@@ -156,6 +158,7 @@ mm_gates_scan_kernel(const float* __restrict__ z, const float* __restrict__ bias
       gates[at] = expf(f + before - m);
       gates[plane + at] = expf(i - m);
       gates[2 * plane + at] = expf(-m);
+      gates[3 * plane + at] = f + before - m;
     }
     carry = last[MS_THREADS / 32 - 1];
     __syncthreads();
@@ -277,7 +280,7 @@ mm_single_kernel(const TA* __restrict__ q, long long ldq, const TA* __restrict__
 }
 
 // q, k [T, H K] and v [T, H V] are views with row pitches; sequences 0 .. singles - 1 bring one
-// token each (token s of the step).  gates [3, T, H] as the gate kernels leave them.  num fp32
+// token each (token s of the step).  gates [4, T, H] as the gate kernels leave them.  num fp32
 // [T, H, V], nq fp32 [T, H].
 IX_API int ix_mm_single(const void* q, long long ldq, const void* k, long long ldk,
                         const void* v, long long ldv, int dtype, const float* gates, float* S,

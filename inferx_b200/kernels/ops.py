@@ -2601,8 +2601,8 @@ MEMORY_GATES_SINGLE_TOKENS = 128
 
 def memory_gates(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, cap: float,
                  m_state: torch.Tensor, step):
-    """fp32 [3, T, H]: exp(f + m_(t-1) - m_t), exp(i - m_t) and exp(-m_t) of every token and
-    head, with the log gates i = cap tanh(z_i / cap), f = logsigmoid(cap tanh(z_f / cap)), z =
+    """fp32 [4, T, H]: exp(f + m_(t-1) - m_t), exp(i - m_t), exp(-m_t) and the first one's
+    logarithm of every token and head, with the log gates i = cap tanh(z_i / cap), f = logsigmoid(cap tanh(z_f / cap)), z =
     x . w^T + bias (``w`` [2 H, W]: the input gates' rows, then the forget gates') and m_t =
     max(f + m_(t-1), i) along each sequence from and back to ``m_state`` fp32 [slots, H]."""
     _chk("x", x)
@@ -2613,7 +2613,7 @@ def memory_gates(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, cap: floa
     H = w.shape[0] // 2
     if w.shape[1] != W or bias.numel() != 2 * H or m_state.shape[1] != H:
         raise KernelError("memory_gates: weights, biases and state disagree")
-    gates = torch.empty((3, T, H), dtype=torch.float32, device=x.device)
+    gates = torch.empty((4, T, H), dtype=torch.float32, device=x.device)
     if step.all_decode and T == step.num_seqs and T <= MEMORY_GATES_SINGLE_TOKENS:
         _check(_lib().ix_mm_gates_single(
             _ptr(x), _ptr(w), _dtype_code(x), _ptr(bias), ctypes.c_float(cap), _ptr(m_state),
@@ -2628,14 +2628,21 @@ def memory_gates(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, cap: floa
     return gates
 
 
+# Portions of prompts: three launches in chunks of 64 tokens, or one that walks them token by
+# token; up to this many tokens the walk is as fast.
+MEMORY_CHUNK_MIN_TOKENS = 32
+
+
 def matrix_memory(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: torch.Tensor,
                   state: torch.Tensor, normaliser: torch.Tensor, step, heads: int, dim: int,
-                  vdim: int, q_scale: float):
+                  vdim: int, q_scale: float, form: Optional[str] = None):
     """S_t = keep S_(t-1) + put k v^T and n_t = keep n_(t-1) + put k along each sequence, from
     and back to ``state`` [slots, heads, dim, vdim] and ``normaliser`` [slots, heads, dim]
     (fp32); ``gates`` as ``memory_gates`` leaves them; q, k [T, heads * dim] and v [T, heads *
-    vdim] are views with unit inner stride, q counts times ``q_scale``.  Returns S_t^T q fp32
-    [T, heads, vdim] and n_t . q fp32 [T, heads]."""
+    vdim] are views with unit inner stride, q counts times ``q_scale``.  ``form`` of sequences
+    that bring several tokens: "walk" (token by token), "chunks" (bfloat16 on the tensor cores)
+    or None (chunks from MEMORY_CHUNK_MIN_TOKENS tokens a sequence on, where they apply).
+    Returns S_t^T q fp32 [T, heads, vdim] and n_t . q fp32 [T, heads]."""
     ldq = _row_view("matrix_memory: q", q, heads * dim)
     ldk = _row_view("matrix_memory: k", k, heads * dim)
     ldv = _row_view("matrix_memory: v", v, heads * vdim)
@@ -2644,7 +2651,7 @@ def matrix_memory(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: torc
     _chk("normaliser", normaliser, torch.float32)
     T = q.shape[0]
     if not (q.dtype == k.dtype == v.dtype) or k.shape[0] != T or v.shape[0] != T \
-            or tuple(gates.shape) != (3, T, heads) \
+            or tuple(gates.shape) != (4, T, heads) \
             or tuple(state.shape[1:]) != (heads, dim, vdim) \
             or tuple(normaliser.shape[1:]) != (heads, dim):
         raise KernelError("matrix_memory: q, k, v, gates and state do not fit together")
@@ -2660,6 +2667,25 @@ def matrix_memory(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: torc
                "mm_single")
         _count()
     if singles < S:
+        applies = q.dtype == torch.bfloat16 and bool(_lib().ix_mm_chunks_applies(dim, vdim))
+        if form is None:
+            form = ("chunks" if applies and int(step.max_q_len) >= MEMORY_CHUNK_MIN_TOKENS
+                    else "walk")
+        if form not in ("walk", "chunks") or (form == "chunks" and not applies):
+            raise KernelError(f"matrix_memory: no form {form!r} for {q.dtype}, heads of {dim} / "
+                              f"{vdim}")
+        if form == "chunks":
+            tokens = T - singles         # single tokens come first, one each
+            size = _lib().ix_mm_chunks_scratch_floats
+            size.restype = ctypes.c_longlong
+            scratch = torch.empty((size(tokens, S - singles, heads, dim, vdim),),
+                                  dtype=torch.float32, device=q.device)
+            _check(_lib().ix_mm_chunks(
+                *views[:6], *views[7:], _ptr(step.cu_q), _ptr(step.state_slot), _ptr(num),
+                _ptr(nq), T, tokens, S, singles, int(step.max_q_len), heads, dim, vdim,
+                ctypes.c_float(q_scale), _ptr(scratch), _stream()), "mm_chunks")
+            _count(3)
+            return num, nq
         _check(_lib().ix_mm_walk(*views, _ptr(step.cu_q), _ptr(step.state_slot), _ptr(num),
                                  _ptr(nq), T, S, singles, heads, dim, vdim,
                                  ctypes.c_float(q_scale), _stream()), "mm_walk")

@@ -905,14 +905,14 @@ def memory_gates(x, w, bias, cap, m_state, step):
     z = _f(x) @ _f(w).T + bias
     i = cap * torch.tanh(z[:, :H] / cap)
     f = torch.nn.functional.logsigmoid(cap * torch.tanh(z[:, H:] / cap))
-    out = torch.zeros(3, T, H)
+    out = torch.zeros(4, T, H)
     for s in range(step.num_seqs):
         slot = int(step.state_slot[s])
         m = m_state[slot].clone()
         for t in range(int(step.cu_q[s]), int(step.cu_q[s + 1])):
             new = torch.maximum(f[t] + m, i[t])
             out[0, t], out[1, t] = torch.exp(f[t] + m - new), torch.exp(i[t] - new)
-            out[2, t] = torch.exp(-new)
+            out[2, t], out[3, t] = torch.exp(-new), f[t] + m - new
             m = new
         m_state[slot] = m
     return out
