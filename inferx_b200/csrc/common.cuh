@@ -39,8 +39,30 @@ template <> __device__ __forceinline__ bf16 from_f32<bf16>(float v) { return __f
 // Activation of a product that has no gate beside it.
 enum { IX_ACT_NONE = 0, IX_ACT_GELU = 1, IX_ACT_RELU2 = 2 };   // gelu: the exact (erf) form
 
+// erf by the rational approximation 7.1.28 of Abramowitz and Stegun, "Handbook of Mathematical
+// Functions" (absolute error 3e-7): 1 - 1 / (1 + a1 x + ... + a6 x^6)^16 for x >= 0; for results
+// that are rounded to bfloat16.  Far out the power overflows and its reciprocal is 0.
+__device__ __forceinline__ float ix_erf_bf16(float x) {
+  const float a = fabsf(x);
+  float p = fmaf(0.0000430638f, a, 0.0002765672f);
+  p = fmaf(p, a, 0.0001520143f);
+  p = fmaf(p, a, 0.0092705272f);
+  p = fmaf(p, a, 0.0422820123f);
+  p = fmaf(p, a, 0.0705230784f);
+  p = fmaf(p, a, 1.0f);
+  p *= p; p *= p; p *= p; p *= p;
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(p));
+  return copysignf(1.0f - r, x);
+}
+
+// TO: what the result is rounded to.
+template <typename TO>
 __device__ __forceinline__ float ix_act(float v, int act) {
-  if (act == IX_ACT_GELU) return 0.5f * v * (1.0f + erff(v * 0.70710678118654752f));
+  if (act == IX_ACT_GELU) {
+    const float z = v * 0.70710678118654752f;
+    return 0.5f * v * (1.0f + (sizeof(TO) == 2 ? ix_erf_bf16(z) : erff(z)));
+  }
   if (act == IX_ACT_RELU2) {
     v = fmaxf(v, 0.f);
     return v * v;

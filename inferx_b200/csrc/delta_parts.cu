@@ -1133,7 +1133,7 @@ __global__ void activate_kernel(const TA* x, TA* out, size_t n, int act) {
   IX_PDL_WAIT();
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n;
        i += (size_t)gridDim.x * blockDim.x)
-    out[i] = from_f32<TA>(ix_act(to_f32(x[i]), act));
+    out[i] = from_f32<TA>(ix_act<TA>(to_f32(x[i]), act));
 }
 
 // four entries an access
@@ -1144,8 +1144,8 @@ activate_vec_kernel(const TA* x, TA* out, size_t quads, int act) {
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < quads;
        i += (size_t)gridDim.x * blockDim.x) {
     const float4 v = ld4(x + 4 * i);
-    st4(out + 4 * i, make_float4(ix_act(v.x, act), ix_act(v.y, act), ix_act(v.z, act),
-                                 ix_act(v.w, act)));
+    st4(out + 4 * i, make_float4(ix_act<TA>(v.x, act), ix_act<TA>(v.y, act),
+                                 ix_act<TA>(v.z, act), ix_act<TA>(v.w, act)));
   }
 }
 

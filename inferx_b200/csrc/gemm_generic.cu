@@ -223,7 +223,7 @@ gemm_tiles_kernel(const TA* __restrict__ x, const int* __restrict__ rows,
         const float g = row_scale ? val * w : val;
         val = g / (1.0f + expf(-g)) * (row_scale ? acc2[i][j] * w : acc2[i][j]);
       } else {
-        val = ix_act(val, plain);
+        val = ix_act<TO>(val, plain);
       }
       out[(size_t)r * N + c] = from_f32<TO>(val);
     }
@@ -313,7 +313,7 @@ gemm_rows_kernel(const TA* __restrict__ x, const int* __restrict__ rows,
             const float g = row_scale ? val * w : val;
             val = g / (1.0f + expf(-g)) * (row_scale ? acc[i][j + 2] * w : acc[i][j + 2]);
           } else {
-            val = ix_act(val, plain);
+            val = ix_act<TO>(val, plain);
           }
           out[(size_t)(r0 + i) * N + c] = from_f32<TO>(val);
         }

@@ -194,7 +194,7 @@ gemm_small_m_kernel(const bf16* __restrict__ x, const int* __restrict__ rows,
           if (j < N && r < hi) {
             float v = acc[i][c];
             if (DUAL) v = dual_act(v, acc2[i][c], r, act);
-            else v = ix_act(v, act.plain);
+            else v = ix_act<TO>(v, act.plain);
             out[(size_t)r * N + j] = from_f32<TO>(v);
           }
         }
@@ -221,7 +221,7 @@ gemm_small_m_kernel(const bf16* __restrict__ x, const int* __restrict__ rows,
         const int r = r0 + i * 8 + 2 * tt + (c & 1);
         if (j < N && r < hi) {
           if (DUAL) v = dual_act(v, v2, r, act);
-          else v = ix_act(v, act.plain);
+          else v = ix_act<TO>(v, act.plain);
           out[(size_t)r * N + j] = from_f32<TO>(v);
         }
       }

@@ -208,7 +208,7 @@ gemm_stream_grouped_kernel(const bf16* __restrict__ x, const int* __restrict__ r
                 }
                 v = v / (1.0f + __expf(-v)) * v2;
               } else {
-                v = ix_act(v, plain);
+                v = ix_act<bf16>(v, plain);
               }
               out[(size_t)r * N + j] = __float2bfloat16_rn(v);
             }

@@ -299,8 +299,8 @@ grouped_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a,
         if (!SWIGLU && plain) {
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
-            g[i] = ix_act(g[i], plain);
-            if (MODE == 2) u[DUAL ? i : 0] = ix_act(u[DUAL ? i : 0], plain);
+            g[i] = ix_act<bf16>(g[i], plain);
+            if (MODE == 2) u[DUAL ? i : 0] = ix_act<bf16>(u[DUAL ? i : 0], plain);
           }
         }
 #pragma unroll

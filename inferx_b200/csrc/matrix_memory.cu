@@ -6,15 +6,16 @@
 //   memory         S_t = keep S_(t-1) + put k_t v_t^T,  n_t = keep n_(t-1) + put k_t
 //   read-out       num_t = S_t^T q_t,  nq_t = n_t . q_t
 //
-// The head's output num / (max(|nq|, floor) + eps) is formed by the norm that follows
-// (ix_head_norm_gate).  S [slots, H, K, V], n [slots, H, K] and m [slots, H] are fp32 state per
+// The head's output num / (max(|nq|, floor) + eps) is formed with the norm and the gate that
+// follow: in these kernels where a block has the whole head (MmFinish), else by
+// ix_head_norm_gate.  S [slots, H, K, V], n [slots, H, K] and m [slots, H] are fp32 state per
 // request.  Three kernels make the gates: one for steps of single tokens, which also takes the
 // dot products; a scan over each sequence otherwise (the two numbers of a token combine
 // associatively: the sum of the f's and the largest i carried to the end).  The memory is
 // walked by one of three forms: single tokens (the memory streams through the chip once),
 // token by token with the memory in registers (any sizes and types), and in chunks
 // (matrix_memory_chunks.cu).
-#include "common.cuh"
+#include "matrix_memory.cuh"
 
 __device__ __forceinline__ float mm_cap(float z, float cap) { return cap * tanhf(z / cap); }
 // logsigmoid(z) = min(z, 0) - log(1 + exp(-|z|))
@@ -46,6 +47,7 @@ mm_gates_single_kernel(const TA* __restrict__ x, const TA* __restrict__ w,
   const TA* wf = w + (size_t)(H + h) * W;
   float zi = 0.f, zf = 0.f;
   if (VEC) {                        // bf16, W a multiple of 8: 16-byte accesses
+#pragma unroll 4
     for (int c = lane * 8; c < W; c += 256) {
       const uint4 a = *reinterpret_cast<const uint4*>(xr + c);
       const uint4 b = *reinterpret_cast<const uint4*>(wi + c);
@@ -109,7 +111,7 @@ IX_API int ix_mm_gates_single(const void* x, const void* w, int dtype, const flo
 // end is max(m before it + F, M); spans join as (F1 + F2, max(M1 + F2, M2)).  keep uses the
 // m of the token before as that token's own thread formed it.
 // ---------------------------------------------------------------------------
-#define MS_THREADS 256
+#define MS_THREADS 1024
 
 __global__ void __launch_bounds__(MS_THREADS)
 mm_gates_scan_kernel(const float* __restrict__ z, const float* __restrict__ bias, float cap,
@@ -186,13 +188,15 @@ IX_API int ix_mm_gates_scan(const float* z, const float* bias, float cap, float*
 #define MD_COLS 128
 #define MD_ROWS 8       // rows a warp has in flight
 
+// With `fin.gain` (V at most MD_COLS: the block has the head's whole output) the block divides
+// by the normaliser, norms, gates and writes the head's row of the activations itself.
 template <typename TA, bool VEC>
 __global__ void __launch_bounds__(MD_WARPS * 32)
 mm_single_kernel(const TA* __restrict__ q, long long ldq, const TA* __restrict__ k, long long ldk,
                  const TA* __restrict__ v, long long ldv, const float* __restrict__ gates,
                  float* __restrict__ S, float* __restrict__ N, const int* __restrict__ state_slot,
                  float* __restrict__ num, float* __restrict__ nq, int T, int H, int K, int V,
-                 float q_scale) {
+                 float q_scale, MmFinish fin) {
   extern __shared__ __align__(16) float sm[];
   float* q_s = sm;             // [K]
   float* k_s = sm + K;         // [K], times put
@@ -260,11 +264,11 @@ mm_single_kernel(const TA* __restrict__ q, long long ldq, const TA* __restrict__
     }
   }
   __syncthreads();
-  for (int c = tid; c < MD_COLS && v0 + c < V; c += MD_WARPS * 32) {
-    float total = 0.f;
+  float total = 0.f;                 // of column tid (MD_COLS threads have one)
+  if (tid < MD_COLS && v0 + tid < V) {
 #pragma unroll
-    for (int w = 0; w < MD_WARPS; ++w) total += part[w * MD_COLS + c];
-    num[at * V + v0 + c] = total;
+    for (int w = 0; w < MD_WARPS; ++w) total += part[w * MD_COLS + tid];
+    if (!fin.gain) num[at * V + v0 + tid] = total;
   }
   if (blockIdx.x == 0) {
     float* nr = N + slot_head * K;
@@ -275,18 +279,33 @@ mm_single_kernel(const TA* __restrict__ q, long long ldq, const TA* __restrict__
       nr[i] = x;
     }
     a = block_sum(a, scratch);
-    if (tid == 0) nq[at] = a;
+    if (fin.gain) {
+      const float y = total / (fmaxf(fabsf(a), gates[2 * plane + at]) + fin.den_eps);
+      const float ss = block_sum(y * y, scratch);     // 0 beyond V
+      if (tid < V) {
+        const size_t c = (size_t)h * V + tid;
+        const float z = to_f32(reinterpret_cast<const TA*>(fin.gate)[(size_t)t * fin.gate_ld + c]);
+        reinterpret_cast<TA*>(fin.out)[(size_t)t * H * V + c] =
+            from_f32<TA>(y / sqrtf(ss / (float)V + fin.eps) * fin.gain[c] / (1.0f + expf(-z)));
+      }
+    } else if (tid == 0) {
+      nq[at] = a;
+    }
   }
 }
 
 // q, k [T, H K] and v [T, H V] are views with row pitches; sequences 0 .. singles - 1 bring one
 // token each (token s of the step).  gates [4, T, H] as the gate kernels leave them.  num fp32
-// [T, H, V], nq fp32 [T, H].
+// [T, H, V], nq fp32 [T, H]; or, with `gain`, the finished rows in `out` (see MmFinish).
 IX_API int ix_mm_single(const void* q, long long ldq, const void* k, long long ldk,
                         const void* v, long long ldv, int dtype, const float* gates, float* S,
                         float* N, const int* state_slot, float* num, float* nq, int T,
-                        int singles, int H, int K, int V, float q_scale, cudaStream_t stream) {
+                        int singles, int H, int K, int V, float q_scale, const float* gain,
+                        const void* gate, long long gate_ld, float eps, float den_eps, void* out,
+                        cudaStream_t stream) {
   if (singles <= 0) return IX_OK;
+  if (gain && (V > MD_COLS || !gate || !out)) return IX_ERR_UNSUPPORTED;
+  const MmFinish fin = {gain, gate, gate_ld, eps, den_eps, out};
   if (H <= 0 || K <= 0 || V <= 0 || H > 65535 || singles > 65535 || singles > T)
     return IX_ERR_SIZE;
   const size_t smem = ((size_t)((2 * K + 3) & ~3) + MD_WARPS * MD_COLS) * sizeof(float);
@@ -296,7 +315,8 @@ IX_API int ix_mm_single(const void* q, long long ldq, const void* k, long long l
   IX_DISPATCH_DTYPE(dtype, TA, {
     auto kern = vec ? mm_single_kernel<TA, true> : mm_single_kernel<TA, false>;
     ix_launch(kern, grid, dim3(MD_WARPS * 32), smem, stream, (const TA*)q, ldq, (const TA*)k, ldk,
-              (const TA*)v, ldv, gates, S, N, state_slot, num, nq, T, H, K, V, q_scale);
+              (const TA*)v, ldv, gates, S, N, state_slot, num, nq, T, H, K, V, q_scale,
+              fin);
   });
   return ix_launch_status();
 }

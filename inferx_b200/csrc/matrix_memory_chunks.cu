@@ -17,7 +17,7 @@
 // (the weighted keys, the weighted scores, the start state) they enter as two bfloat16 terms
 // each (16 bits) into the same fp32 accumulator, and q, k and v as they are.  A chunk's scratch
 // number is tokens before the sequence / 64 + the sequence's number + the chunk's: no two meet.
-#include "common.cuh"
+#include "matrix_memory.cuh"
 
 #define MC_L 64               // tokens a chunk
 #define MC_THREADS 128
@@ -51,17 +51,31 @@ __device__ __forceinline__ unsigned mc_pack_rest(float a, float b, unsigned hi) 
   return mc_pack(a - __low2float(h), b - __high2float(h));
 }
 
+// 16 or 8 bytes to shared memory without registers in between; `bytes` of them are read, the
+// rest is zero
+__device__ __forceinline__ void mc_async16(void* dst, const void* src, int bytes) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(mc_smem(dst)), "l"(src),
+               "r"(bytes) : "memory");
+}
+__device__ __forceinline__ void mc_async8(void* dst, const void* src, int bytes) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 8, %2;" ::"r"(mc_smem(dst)), "l"(src),
+               "r"(bytes) : "memory");
+}
+__device__ __forceinline__ void mc_async_wait() {
+  asm volatile("cp.async.commit_group;\ncp.async.wait_group 0;" ::: "memory");
+}
+
 // `rows` of MC_L rows (the rest zero) of `cols` entries into shared rows of `pitch` entries,
-// columns cols .. padded zero.  vec: rows start on 16-byte marks and cols is a multiple of 8.
+// columns cols .. padded zero.  vec: rows start on 16-byte marks and cols is a multiple of 8; the
+// copies are then asynchronous (mc_async_wait).
 __device__ __forceinline__ void mc_load(bf16* dst, int pitch, const bf16* src, long long ld,
                                         int rows, int cols, int padded, bool vec) {
   if (vec) {
     const int per = padded >> 3;
     for (int i = threadIdx.x; i < MC_L * per; i += MC_THREADS) {
       const int r = i / per, c = (i - r * per) * 8;
-      uint4 x = make_uint4(0, 0, 0, 0);
-      if (r < rows && c < cols) x = *reinterpret_cast<const uint4*>(src + (size_t)r * ld + c);
-      *reinterpret_cast<uint4*>(dst + r * pitch + c) = x;
+      const bool ok = r < rows && c < cols;
+      mc_async16(dst + r * pitch + c, ok ? src + (size_t)r * ld + c : src, ok ? 16 : 0);
     }
   } else {
     for (int i = threadIdx.x; i < MC_L * padded; i += MC_THREADS) {
@@ -129,6 +143,7 @@ mm_chunk_own_kernel(const bf16* __restrict__ k, long long ldk, const bf16* __res
   mc_load(v_s, pv, v + (size_t)at.t0 * ldv + (size_t)h * V + v0, ldv, at.n, min(VT, V - v0), VT,
           vec_v);
   if (warp == 0) mc_gates(G, put, gates, plane, (size_t)at.t0 * H + h, H, at.n);
+  mc_async_wait();
   __syncthreads();
   const float g_end = G[MC_L - 1];
   // the keys times their weight at the chunk's end, in two terms
@@ -195,7 +210,7 @@ mm_chunk_own_kernel(const bf16* __restrict__ k, long long ldk, const bf16* __res
 // columns of one row of the memory (or one entry of the normaliser) along the sequence.
 // A scratch cell of four fp32 numbers becomes four high terms and four low terms.
 // ---------------------------------------------------------------------------
-#define MJ_THREADS 256
+#define MJ_THREADS 128
 #define MJ_AHEAD 8
 
 __global__ void __launch_bounds__(MJ_THREADS)
@@ -265,13 +280,13 @@ mm_chunk_join_kernel(float* __restrict__ scr_s, float* __restrict__ scr_n,
 // out: grid (V tiles, chunks, heads * sequences); warp w owns the chunk's tokens 16 w .. 16 w + 15
 // ---------------------------------------------------------------------------
 template <int VT>
-__global__ void __launch_bounds__(MC_THREADS)
+__global__ void __launch_bounds__(MC_THREADS, 3)
 mm_chunk_out_kernel(const bf16* __restrict__ q, long long ldq, const bf16* __restrict__ k,
                     long long ldk, const bf16* __restrict__ v, long long ldv,
                     const float* __restrict__ gates, const int* __restrict__ cu_q,
                     const float* __restrict__ scr_s, const float* __restrict__ scr_n,
                     float* __restrict__ num, float* __restrict__ nq, int T, int H, int K, int V,
-                    int s0, float q_scale, int vec_q, int vec_k, int vec_v) {
+                    int s0, float q_scale, int vec_q, int vec_k, int vec_v, MmFinish fin) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   __shared__ float G[MC_L], put[MC_L];
   const int Kp = (K + 15) & ~15, Vp = (V + 7) & ~7;
@@ -292,16 +307,16 @@ mm_chunk_out_kernel(const bf16* __restrict__ q, long long ldq, const bf16* __res
   mc_load(v_s, pv, v + (size_t)at.t0 * ldv + (size_t)h * V + v0, ldv, at.n, min(VT, V - v0), VT,
           vec_v);
   const uint4* start = reinterpret_cast<const uint4*>(scr_s + cell * K * Vp);
-#pragma unroll 4
   for (int i = tid; i < Kp * (VT / 4); i += MC_THREADS) {
     const int r = i / (VT / 4), c = (i % (VT / 4)) * 4;
-    uint4 w = make_uint4(0, 0, 0, 0);
-    if (r < K && v0 + c < Vp) w = start[(size_t)r * (Vp >> 2) + ((v0 + c) >> 2)];
-    *reinterpret_cast<uint2*>(s_hi + r * pv + c) = make_uint2(w.x, w.y);
-    *reinterpret_cast<uint2*>(s_lo + r * pv + c) = make_uint2(w.z, w.w);
+    const bool ok = r < K && v0 + c < Vp;
+    const uint4* w = ok ? start + (size_t)r * (Vp >> 2) + ((v0 + c) >> 2) : start;
+    mc_async8(s_hi + r * pv + c, w, ok ? 8 : 0);
+    mc_async8(s_lo + r * pv + c, reinterpret_cast<const uint2*>(w) + 1, ok ? 8 : 0);
   }
   for (int i = tid; i < Kp; i += MC_THREADS) n_s[i] = i < K ? scr_n[cell * K + i] : 0.f;
   if (warp == 0) mc_gates(G, put, gates, plane, (size_t)at.t0 * H + h, H, at.n);
+  mc_async_wait();
   __syncthreads();
   if (warp * 16 >= at.n) return;                        // (no barrier follows)
   const int g = lane >> 2, t2 = (lane & 3) * 2;
@@ -401,10 +416,68 @@ mm_chunk_out_kernel(const bf16* __restrict__ q, long long ldq, const bf16* __res
     sum_a += __shfl_xor_sync(0xffffffffu, sum_a, 2);
     sum_b += __shfl_xor_sync(0xffffffffu, sum_b, 1);
     sum_b += __shfl_xor_sync(0xffffffffu, sum_b, 2);
-    if ((lane & 3) == 0) {
+    if (!fin.gain && (lane & 3) == 0) {
       if (ra < at.n) nq[(size_t)(at.t0 + ra) * H + h] = sum_a * q_scale;
       if (rb < at.n) nq[(size_t)(at.t0 + rb) * H + h] = sum_b * q_scale;
     }
+  }
+  if (fin.gain) {        // one tile holds the head's whole output
+    const size_t fa = (size_t)(at.t0 + min(ra, at.n - 1)), fb = (size_t)(at.t0 + min(rb, at.n - 1));
+    const float da = q_scale / (fmaxf(fabsf(sum_a * q_scale), gates[2 * plane + fa * H + h]) +
+                                fin.den_eps);
+    const float db = q_scale / (fmaxf(fabsf(sum_b * q_scale), gates[2 * plane + fb * H + h]) +
+                                fin.den_eps);
+    float qa = 0.f, qb = 0.f;
+#pragma unroll
+    for (int j = 0; j < VT / 8; ++j) {       // columns beyond V are zero
+      o[j][0] *= da; o[j][1] *= da;
+      o[j][2] *= db; o[j][3] *= db;
+      qa += o[j][0] * o[j][0] + o[j][1] * o[j][1];
+      qb += o[j][2] * o[j][2] + o[j][3] * o[j][3];
+    }
+    qa += __shfl_xor_sync(0xffffffffu, qa, 1);
+    qa += __shfl_xor_sync(0xffffffffu, qa, 2);
+    qb += __shfl_xor_sync(0xffffffffu, qb, 1);
+    qb += __shfl_xor_sync(0xffffffffu, qb, 2);
+    const float ia = 1.0f / sqrtf(qa / (float)V + fin.eps), ib = 1.0f / sqrtf(qb / (float)V + fin.eps);
+    const bf16* gate = reinterpret_cast<const bf16*>(fin.gate) + (size_t)h * V;
+    bf16* dst = reinterpret_cast<bf16*>(fin.out) + (size_t)h * V;
+    const float* gain = fin.gain + (size_t)h * V;
+    const size_t width = (size_t)H * V;
+    const bool two = (V & 1) == 0 && (fin.gate_ld & 1) == 0 &&
+                     (((uintptr_t)fin.gate | (uintptr_t)fin.out) & 3) == 0;
+#pragma unroll
+    for (int j = 0; j < VT / 8; ++j) {
+      const int c = j * 8 + t2;
+      if (c >= V) continue;
+      if (two) {
+        const __nv_bfloat162 za = *reinterpret_cast<const __nv_bfloat162*>(gate + fa * fin.gate_ld + c);
+        const __nv_bfloat162 zb = *reinterpret_cast<const __nv_bfloat162*>(gate + fb * fin.gate_ld + c);
+        const float g0 = gain[c], g1 = gain[c + 1];
+        if (ra < at.n)
+          *reinterpret_cast<unsigned*>(dst + fa * width + c) =
+              mc_pack(o[j][0] * ia * g0 / (1.0f + expf(-__low2float(za))),
+                      o[j][1] * ia * g1 / (1.0f + expf(-__high2float(za))));
+        if (rb < at.n)
+          *reinterpret_cast<unsigned*>(dst + fb * width + c) =
+              mc_pack(o[j][2] * ib * g0 / (1.0f + expf(-__low2float(zb))),
+                      o[j][3] * ib * g1 / (1.0f + expf(-__high2float(zb))));
+      } else {
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          if (c + e >= V) continue;
+          const float za = __bfloat162float(gate[fa * fin.gate_ld + c + e]);
+          const float zb = __bfloat162float(gate[fb * fin.gate_ld + c + e]);
+          if (ra < at.n)
+            dst[fa * width + c + e] =
+                __float2bfloat16_rn(o[j][e] * ia * gain[c + e] / (1.0f + expf(-za)));
+          if (rb < at.n)
+            dst[fb * width + c + e] =
+                __float2bfloat16_rn(o[j][2 + e] * ib * gain[c + e] / (1.0f + expf(-zb)));
+        }
+      }
+    }
+    return;
   }
   float* oa = num + ((size_t)(at.t0 + ra) * H + h) * V;
   float* ob = num + ((size_t)(at.t0 + rb) * H + h) * V;
@@ -440,12 +513,17 @@ IX_API long long ix_mm_chunks_scratch_floats(int T, int S, int H, int K, int V) 
   return cells * K * ((V + 7) & ~7) + cells * K + cells + 8;
 }
 
-// Sequences s0 .. S - 1, `tokens` of them all together, the longest of max_q tokens.
+// Sequences s0 .. S - 1, `tokens` of them all together, the longest of max_q tokens.  num and nq,
+// or, with `gain` (V at most 128), the finished rows in `out` (MmFinish).
 IX_API int ix_mm_chunks(const void* q, long long ldq, const void* k, long long ldk,
                         const void* v, long long ldv, const float* gates, float* S_state,
                         float* N, const int* cu_q, const int* state_slot, float* num, float* nq,
                         int T, int tokens, int S, int s0, int max_q, int H, int K, int V,
-                        float q_scale, float* scratch, cudaStream_t stream) {
+                        float q_scale, float* scratch, const float* gain, const void* gate,
+                        long long gate_ld, float eps, float den_eps, void* out,
+                        cudaStream_t stream) {
+  if (gain && (V > 128 || !gate || !out)) return IX_ERR_UNSUPPORTED;
+  const MmFinish fin = {gain, gate, gate_ld, eps, den_eps, out};
   const int seqs = S - s0;
   if (seqs <= 0 || tokens <= 0) return IX_OK;
   if (s0 < 0 || H <= 0 || K <= 0 || K > MC_MAX_K || V <= 0 || max_q <= 0 || !scratch)
@@ -466,13 +544,13 @@ IX_API int ix_mm_chunks(const void* q, long long ldq, const void* k, long long l
   do {                                                                                         \
     const dim3 grid((V + VT - 1) / VT, chunks, H * seqs);                                      \
     const size_t own = (size_t)MC_L * (2 * (Kp + 8) + VT + 8) * 2;                             \
-    const size_t fin = ((size_t)MC_L * (2 * (Kp + 8) + VT + 8) + (size_t)2 * Kp * (VT + 8)) * 2 \
+    const size_t tail = ((size_t)MC_L * (2 * (Kp + 8) + VT + 8) + (size_t)2 * Kp * (VT + 8)) * 2 \
                        + (size_t)Kp * 4;                                                       \
     cudaError_t e = cudaFuncSetAttribute(mm_chunk_own_kernel<VT>,                              \
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, (int)own); \
     if (e == cudaSuccess)                                                                      \
       e = cudaFuncSetAttribute(mm_chunk_out_kernel<VT>,                                        \
-                               cudaFuncAttributeMaxDynamicSharedMemorySize, (int)fin);         \
+                               cudaFuncAttributeMaxDynamicSharedMemorySize, (int)tail);        \
     if (e != cudaSuccess) return (int)e;                                                       \
     mm_chunk_own_kernel<VT><<<grid, MC_THREADS, own, stream>>>(                                \
         (const bf16*)k, ldk, (const bf16*)v, ldv, gates, cu_q, scr_s, scr_n, scr_p, T, H, K, V, \
@@ -481,9 +559,9 @@ IX_API int ix_mm_chunks(const void* q, long long ldq, const void* k, long long l
     mm_chunk_join_kernel<<<dim3((items + MJ_THREADS - 1) / MJ_THREADS, H, seqs), MJ_THREADS, 0, \
                            stream>>>(scr_s, scr_n, scr_p, S_state, N, cu_q, state_slot, H, K, V, \
                                      s0);                                                      \
-    mm_chunk_out_kernel<VT><<<grid, MC_THREADS, fin, stream>>>(                                \
+    mm_chunk_out_kernel<VT><<<grid, MC_THREADS, tail, stream>>>(                               \
         (const bf16*)q, ldq, (const bf16*)k, ldk, (const bf16*)v, ldv, gates, cu_q, scr_s,     \
-        scr_n, num, nq, T, H, K, V, s0, q_scale, vq, vk, vv);                                  \
+        scr_n, num, nq, T, H, K, V, s0, q_scale, vq, vk, vv, fin);                             \
   } while (0)
   if (V <= 64) MC_GO(64);
   else MC_GO(128);

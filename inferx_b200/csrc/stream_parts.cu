@@ -125,6 +125,7 @@ stream_step_kernel(float* __restrict__ streams, const TY* __restrict__ y, StComb
     if (updates) {
       if (cmb.rows) {
         const TY* er = reinterpret_cast<const TY*>(cmb.rows);
+#pragma unroll 4
         for (int j = 0; j < cmb.k; ++j) {
           const float w = cmb.weight ? cmb.weight[t * cmb.k + j] : 1.0f;
           const StVec<VW> f = st_load<VW>(er + (size_t)cmb.dest[t * cmb.k + j] * W + c);

@@ -15,6 +15,7 @@
     python -m inferx_b200.kernels.microbench recurrent --tokens 64 --batch 64 --hidden 2048 --head-dim 64
     python -m inferx_b200.kernels.microbench attn_prefill --tokens 2048 --softcap 30
     python -m inferx_b200.kernels.microbench prepared --tokens 2048 --hidden 2048 --heads 16 --kv-heads 4 --inter 4096 --experts 32 --batch 8 --window 1024
+    python -m inferx_b200.kernels.microbench streams --tokens 2048 --hidden 2048 --heads 16 --kv-heads 4 --inter 1024 --experts 32 --batch 8 --window 1024
     python -m inferx_b200.kernels.microbench paired --tokens 2048 --hidden 2048 --heads 16 --kv-heads 4 --inter 1024 --experts 32 --batch 8
 
 Each case runs one kernel face at Qwen1.5-MoE-A2.7B sizes (or the sizes given),
@@ -808,11 +809,196 @@ def _paired_latent_and_experts(args, ops, prompt, single, report):
                                                    args.iters), rows * vocab * 8)
 
 
+def streams(args):
+    """The kernels of decoders with several residual streams and a matrix memory, each beside the
+    like kernel of another model of this engine at the same sizes: ``--tokens`` rows of
+    ``--hidden`` in four streams, memory heads of 64 key and 128 value entries, attention of
+    ``--heads`` over ``--kv-heads`` heads of ``--head-dim`` over a ``--window``, ``--experts``
+    experts of ``--inter``, ``--top-k`` chosen; one prompt of ``--tokens`` tokens, and ``--batch``
+    single tokens at ``--context``.  GB/s over the bytes the operation has to move, attention and
+    products as TFLOP/s."""
+    from . import ops
+    from ..parts.base import StreamUpdate
+    T, W, H, G, D = args.tokens, args.hidden, args.heads, args.kv_heads, args.head_dim
+    E, topk, I, page, B, C = args.experts, args.top_k, args.inter, args.page, args.batch, args.context
+    win, ns = args.window, 4
+    dt, dev = torch.bfloat16, "cuda"
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    rnd = lambda *s: torch.randn(*s, device=dev)
+    out = {"case": "streams", "tokens": T, "hidden": W, "heads": H, "kv_heads": G, "head_dim": D,
+           "window": win, "experts": E, "top_k": topk, "inter": I, "batch": B, "context": C}
+
+    def report(name, fn, n, nbytes=0, flops=0, iters=args.iters):
+        us = _time(fn, n, iters)
+        out[name] = {"us": round(us, 2)}
+        if nbytes:
+            out[name]["GBps"] = round(nbytes / us / 1e3, 1)
+        if flops:
+            out[name]["TFLOPs"] = round(flops / us / 1e6, 2)
+
+    def batch(q_lens, starts):
+        S, cu = len(q_lens), [0]
+        for q in q_lens:
+            cu.append(cu[-1] + q)
+        one = max(q_lens) == 1
+        return types.SimpleNamespace(
+            cu_q=i32(cu), q_pos0=i32(starts), q_lens=q_lens, num_seqs=S, num_tokens=cu[-1],
+            seq_of_token=i32([s for s, q in enumerate(q_lens) for _ in range(q)]),
+            positions=i32([a + t for a, q in zip(starts, q_lens) for t in range(q)]),
+            kv_len=i32([a + q for a, q in zip(starts, q_lens)]), state_slot=i32(list(range(S))),
+            max_kv_len=max(a + q for a, q in zip(starts, q_lens)), max_q_len=max(q_lens),
+            all_decode=one, num_decode_seqs=S if one else 0, cu_q_prompt=i32(cu),
+            token_ids=i32([0] * cu[-1]))
+    prompt, single = batch([T], [0]), batch([1] * B, [C - 1] * B)
+
+    # streams, for the prompt's rows and for the single tokens'
+    gain, bias, alpha = rnd(W), rnd(W), torch.ones(1, device=dev)
+    mix, put, read = rnd(ns, ns) * 0.3, rnd(ns), rnd(ns)
+    n = max(2, min(4, _copies(T * ns * W * 4)))
+    xs = [rnd(T, ns, W) for _ in range(n)]
+    ys = [rnd(T, W).to(dt) for _ in range(n)]
+    resid = [x[:, 0].contiguous() for x in xs]
+    for name, rows in (("prompt", T), ("single tokens", B)):
+        report(f"stream_step ({name})", lambda i: ops.stream_step(
+            xs[i][:rows], StreamUpdate(ys[i][:rows], mix, put), read, (alpha, gain, bias), dt), n,
+            rows * W * (8 * ns + 4))
+        report(f"add_rmsnorm ({name}, like)", lambda i: ops.add_rmsnorm(
+            resid[i][:rows], ys[i][:rows], gain, 1e-6, dt), n, rows * W * 12)
+    er, dest = rnd(T * topk, W).to(dt), torch.randperm(T * topk, device=dev).to(torch.int32)
+    tw, lg = torch.rand(T, topk, device=dev), rnd(T)
+    pend = ops.CombinePending(er, dest, tw, ys[0], lg)
+    report("stream_step with a mixture's rows (prompt)", lambda i: ops.stream_step(
+        xs[i], StreamUpdate(pend, mix, put), read, (alpha, gain, bias), dt), n,
+        T * W * (8 * ns + 2 * topk + 4))
+    report("combine + add_rmsnorm (prompt, like)", lambda i: ops.add_rmsnorm(
+        resid[i], pend, gain, 1e-6, dt), n, T * W * (8 + 2 * topk + 4))
+    table = rnd(8192, W).to(dt)
+    ids = torch.randint(0, 8192, (T,), device=dev, dtype=torch.int32)
+    report("embed_streams", lambda i: ops.embed_streams(table, ids, ns), 1, T * W * (2 + 4 * ns))
+    report("embed (like)", lambda i: ops.embed(table, ids), 1, T * W * 6)
+    del xs, er, pend
+
+    # the memory beside gated linear attention with a state of the same size
+    mh, K, V = W // 128, 64, 128
+    fw = mh * (2 * K + 2 * V)
+    nf = max(2, min(8, _copies(T * fw * 2)))
+    fr = [rnd(T, fw).to(dt) * 0.3 for _ in range(nf)]
+    gw, gb = (rnd(2 * mh, W) * 0.02).to(dt), torch.cat([torch.zeros(mh), torch.full((mh,), 3.0)]).to(dev)
+    gnorm = torch.ones(mh * V, device=dev)
+    x16 = [rnd(T, W).to(dt) for _ in range(2)]
+    decay = [torch.rand(T, mh * K, device=dev) * 0.1 + 0.9 for _ in range(2)]
+    low, w2, b2 = rnd(T, 64), rnd(64, mh * K) * 0.1, torch.zeros(mh * K, device=dev)
+    cut = lambda f, r: (f[:r, :mh * K], f[:r, mh * K:2 * mh * K], f[:r, 2 * mh * K:2 * mh * K + mh * V])
+    for name, rows, st in (("prompt", T, prompt), ("single tokens", B, single)):
+        S = st.num_seqs
+        ms = torch.zeros(S, mh, device=dev)
+        nst = max(2, min(8, _copies(S * mh * K * V * 4)))
+        state = [torch.zeros(S, mh, K, V, device=dev) for _ in range(nst)]
+        nrm = [torch.zeros(S, mh, K, device=dev) for _ in range(nst)]
+        gates = ops.memory_gates(x16[0][:rows].contiguous(), gw, gb, 15.0, ms, st)
+        xg = [x[:rows].contiguous() for x in x16]
+        report(f"memory_gates with their products ({name})", lambda i: ops.memory_gates(
+            xg[i], gw, gb, 15.0, ms, st), 2, rows * W * 2 + 4 * mh * W)
+        lr = low[:rows].contiguous()
+        report(f"lowrank_decay ({name}, like, without its products)", lambda i: ops.lowrank_decay(
+            lr, w2, b2, "sigmoid_root", tau=8.0), 1, 4 * rows * (64 + mh * K))
+        nv = min(nf, nst)
+        fin = lambda f: (gnorm, f[:rows, 2 * mh * K + mh * V:], 1e-6, 1e-6)
+        nbytes = rows * mh * (4 * K + 6 * V) + 2 * S * mh * K * V * 4
+        flops = rows * mh * 6.0 * K * V
+        report(f"matrix_memory with norm and gate ({name})", lambda i: ops.matrix_memory(
+            *cut(fr[i], rows), gates, state[i], nrm[i], st, mh, K, V, 0.125, finish=fin(fr[i])), nv,
+            nbytes, flops)
+
+        def like(i):
+            o = ops.linear_recurrence(*cut(fr[i], rows), decay[i % 2][:rows], None, state[i], st, mh,
+                                      K, V, 0.125, False)
+            return ops.head_norm_gate(o, gnorm, fr[i][:rows, 2 * mh * K + mh * V:], 1e-6, dt)
+        report(f"linear_recurrence + head_norm_gate ({name}, like)", like, nv,
+               nbytes + rows * mh * K * 4, flops)
+        if rows == T:
+            report("matrix_memory token by token (prompt)", lambda i: ops.matrix_memory(
+                *cut(fr[i], rows), gates, state[i], nrm[i], st, mh, K, V, 0.125, form="walk",
+                finish=fin(fr[i])), nv, nbytes, flops, 5)
+    del fr
+
+    # attention: sinks and gates beside the same kernels without
+    dq, dk = H * D, G * D
+    width = dq + 2 * dk
+    pages = -(-T // page)
+    kp, vp = (rnd(pages, G, page, D) * 0.3).to(dt), rnd(pages, G, page, D).to(dt)
+    bt, scale = torch.arange(pages, dtype=torch.int32, device=dev).view(1, pages), D ** -0.5
+    q3, sink, gate = rnd(T, H, D).to(dt), rnd(H), rnd(T, H).to(dt)
+    keys = sum(min(p + 1, win) if win else p + 1 for p in range(T))
+    flops = 4.0 * H * D * keys
+    for form in ("tc", "mma"):
+        for name, opt in (("with sinks and gates", dict(sink=sink, gate=gate)), ("plain, like", {})):
+            report(f"prompt attention, 16-bit weights, {form} ({name})", lambda i:
+                   ops.paged_attention_prefill_exact(q3, kp, vp, bt, prompt.cu_q, prompt.q_pos0, win,
+                                                     scale, kernel=form, **opt), 1, 0, flops)
+    per = -(-C // page)
+    nc = min(_copies(B * C * G * D * 4), 4)
+    kcs = [(rnd(B * per, G, page, D) * 0.3).to(dt) for _ in range(nc)]
+    vcs = [rnd(B * per, G, page, D).to(dt) for _ in range(nc)]
+    btd = torch.randperm(B * per, device=dev).to(torch.int32).view(B, per)
+    span = min(C, win) if win else C
+    for name, opt in (("with sinks and gates", dict(sink=sink, gate=gate[:B])), ("plain, like", {})):
+        report(f"single-token attention, 16-bit weights ({name})", lambda i:
+               ops.paged_attention_decode_exact(q3[:B], kcs[i], vcs[i], btd, single.kv_len, C, win,
+                                                scale, **opt), nc, B * span * G * D * 4)
+    del kcs, vcs
+    rows16 = [rnd(T, width + 16).to(dt) for _ in range(2)]
+    cw, cb, cst = rnd(width, 4), rnd(width), torch.zeros(1, 3, width, device=dev)
+    report("causal_conv with an input bias (prompt)", lambda i: ops.causal_conv(
+        rows16[i][:, :width], cw, None, cst, prompt, silu=False, in_bias=cb), 2, T * width * 4)
+    report("causal_conv (prompt, like)", lambda i: ops.causal_conv(
+        rows16[i][:, :width], cw, None, cst, prompt, silu=False), 2, T * width * 4)
+    freq = torch.rand(32, device=dev)
+    slots = torch.arange(T, dtype=torch.int32, device=dev)
+    prep = lambda i, g, kc, vc, sl: ops.attention_prepare(
+        rows16[i][:, :dq + 2 * g * D], prompt.positions, freq, 1.0, 64, True, H, g, D, D, None, None,
+        1e-6, False, None, None, kc, vc, sl)
+    report("attention_prepare of queries alone (prompt)", lambda i: prep(i, 0, None, None, None), 2,
+           T * dq * 4)
+    report("attention_prepare (prompt, like)", lambda i: prep(i, G, kp, vp, slots), 2, T * width * 4)
+
+    # router and experts
+    wr, corr, ex = rnd(E, W) * 0.02, rnd(E), rnd(W)
+    rule = dict(correction=corr, group_count=4, group_keep=2, renorm_eps=1e-20, extra_w=ex)
+    for name, opt in (("sigmoid scores, groups by pair sums", dict(score="sigmoid",
+                                                                   group_value="pair_sum")),
+                      ("softmax scores, groups by maxima, like", {})):
+        report(f"router (prompt, {name})", lambda i: ops.router_topk(
+            x16[i], wr, topk, True, 1.5, **rule, **opt), 2, T * W * 2 + E * W * 4)
+    idx = torch.stack([torch.randperm(E, device=dev)[:topk] for _ in range(T)]).to(torch.int32)
+    offsets, rows, _ = ops.moe_dispatch(idx, E)
+    up = [(rnd(E, I, W) * 0.02).to(dt) for _ in range(2)]
+    gu = [(rnd(E, 2 * I, W) * 0.02).to(dt) for _ in range(2)]
+    report("experts' up product with gelu (prompt)", lambda i: ops.grouped_up(
+        x16[i], rows, offsets, up[i], "gelu"), 2, 0, 2.0 * T * topk * I * W)
+    report("experts' gate/up product with silu (prompt, like)", lambda i: ops.grouped_gate_up_swiglu(
+        x16[i], rows, offsets, gu[i]), 2, 0, 4.0 * T * topk * I * W)
+    few = idx[:B].contiguous()
+    offs, rws, _ = ops.moe_dispatch(few, E)
+    touched = int(torch.unique(few).numel())
+    xb = x16[0][:B].contiguous()
+    report("experts' up product with gelu (single tokens)", lambda i: ops.grouped_up(
+        xb, rws, offs, up[i], "gelu"), 2, touched * I * W * 2)
+    report("experts' gate/up product with silu (single tokens, like)", lambda i:
+           ops.grouped_gate_up_swiglu(xb, rws, offs, gu[i]), 2, touched * 2 * I * W * 2)
+    ff = [rnd(T, 4 * I).to(dt) for _ in range(3)]
+    for act in ("gelu", "relu_squared"):
+        report(f"activate: {act} (prompt)", lambda i: ops.activate(ff[i], act, out=ff[i]), 3,
+               T * 4 * I * 4)
+    report("silu_mul (prompt, like)", lambda i: ops.silu_mul(ff[i]), 3, T * 4 * I * 3)
+    return out
+
+
 def main(argv=None):
     ap = argparse.ArgumentParser(description=__doc__.split("\n\n")[0])
     ap.add_argument("case", choices=["attn_decode", "grouped", "dense", "attn_prefill", "router",
                                      "qkv", "latent_attn", "rowwise", "recurrent", "delta",
-                                     "prepared", "paired"])
+                                     "prepared", "paired", "streams"])
     ap.add_argument("--softcap", type=float, default=0.0,
                     help="attn_decode, attn_prefill: squash scores to softcap * tanh(s / softcap)")
     ap.add_argument("--rank", type=int, default=512, help="latent_attn: entries of the latent")

@@ -1880,7 +1880,8 @@ _GATE_FORMS = {"silu": 0, "sigmoid": 1}
 
 
 def head_norm_gate(o: torch.Tensor, gain: torch.Tensor, gate: torch.Tensor, eps: float,
-                   out_dtype: torch.dtype, gate_form: str = "silu", den=None):
+                   out_dtype: torch.dtype, gate_form: str = "silu", den=None,
+                   out: Optional[torch.Tensor] = None):
     """out[t, h] = o[t, h] / sqrt(mean(o[t, h]^2) + eps) * gain * act(gate[t, h]) (act:
     silu, or sigmoid with ``gate_form`` "sigmoid") for
     o fp32 [T, heads, vdim]; ``gain`` fp32 [vdim] (shared by the heads) or [heads * vdim];
@@ -1893,7 +1894,9 @@ def head_norm_gate(o: torch.Tensor, gain: torch.Tensor, gate: torch.Tensor, eps:
     ldg = _row_view("head_norm_gate: gate", gate, H * V)
     if gain.numel() not in (V, H * V) or gate.dtype != out_dtype or gate.shape[0] != T:
         raise KernelError("head_norm_gate: gain or gate do not fit the heads")
-    out = torch.empty((T, H * V), dtype=out_dtype, device=o.device)
+    if out is None:
+        out = torch.empty((T, H * V), dtype=out_dtype, device=o.device)
+    _chk("out", out, out_dtype)
     nq, floor, den_eps = den if den is not None else (None, None, 0.0)
     _chk("nq", nq, torch.float32, optional=True)
     _chk("floor", floor, torch.float32, optional=True)
@@ -2633,61 +2636,94 @@ def memory_gates(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, cap: floa
 MEMORY_CHUNK_MIN_TOKENS = 32
 
 
+# Value entries a head may have for the memory's kernels to finish the head's row themselves.
+MEMORY_FINISH_MAX_VDIM = 128
+
+
 def matrix_memory(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: torch.Tensor,
                   state: torch.Tensor, normaliser: torch.Tensor, step, heads: int, dim: int,
-                  vdim: int, q_scale: float, form: Optional[str] = None):
+                  vdim: int, q_scale: float, form: Optional[str] = None, finish=None):
     """S_t = keep S_(t-1) + put k v^T and n_t = keep n_(t-1) + put k along each sequence, from
     and back to ``state`` [slots, heads, dim, vdim] and ``normaliser`` [slots, heads, dim]
     (fp32); ``gates`` as ``memory_gates`` leaves them; q, k [T, heads * dim] and v [T, heads *
     vdim] are views with unit inner stride, q counts times ``q_scale``.  ``form`` of sequences
     that bring several tokens: "walk" (token by token), "chunks" (bfloat16 on the tensor cores)
     or None (chunks from MEMORY_CHUNK_MIN_TOKENS tokens a sequence on, where they apply).
-    Returns S_t^T q fp32 [T, heads, vdim] and n_t . q fp32 [T, heads]."""
+    Returns num = S_t^T q fp32 [T, heads, vdim] and nq = n_t . q fp32 [T, heads]; with ``finish``
+    = (gain fp32 [heads * vdim], gate view [T, heads * vdim], eps, den_eps) the rows
+    [T, heads * vdim] in q's type: y = num / (max(|nq|, floor) + den_eps), y / sqrt(mean(y^2) +
+    eps) * gain * sigmoid(gate) per head."""
     ldq = _row_view("matrix_memory: q", q, heads * dim)
     ldk = _row_view("matrix_memory: k", k, heads * dim)
     ldv = _row_view("matrix_memory: v", v, heads * vdim)
     _chk("gates", gates, torch.float32)
     _chk("state", state, torch.float32)
     _chk("normaliser", normaliser, torch.float32)
-    T = q.shape[0]
+    T, S, dev = q.shape[0], step.num_seqs, q.device
     if not (q.dtype == k.dtype == v.dtype) or k.shape[0] != T or v.shape[0] != T \
             or tuple(gates.shape) != (4, T, heads) \
             or tuple(state.shape[1:]) != (heads, dim, vdim) \
             or tuple(normaliser.shape[1:]) != (heads, dim):
         raise KernelError("matrix_memory: q, k, v, gates and state do not fit together")
-    num = torch.empty((T, heads, vdim), dtype=torch.float32, device=q.device)
-    nq = torch.empty((T, heads), dtype=torch.float32, device=q.device)
-    views = (_ptr(q), ctypes.c_longlong(ldq), _ptr(k), ctypes.c_longlong(ldk), _ptr(v),
-             ctypes.c_longlong(ldv), _dtype_code(q), _ptr(gates), _ptr(state), _ptr(normaliser))
-    S = step.num_seqs
     singles = S if step.all_decode else int(getattr(step, "num_decode_seqs", 0))
+    applies = q.dtype == torch.bfloat16 and bool(_lib().ix_mm_chunks_applies(dim, vdim))
+    if form is None:
+        form = ("chunks" if applies and int(step.max_q_len) >= MEMORY_CHUNK_MIN_TOKENS else "walk")
+    if form not in ("walk", "chunks") or (form == "chunks" and not applies):
+        raise KernelError(f"matrix_memory: no form {form!r} for {q.dtype}, heads of {dim} / {vdim}")
+    gain = gate = y = None
+    eps = den_eps = 0.0
+    ldg = 0
+    if finish is not None:
+        gain, gate, eps, den_eps = finish
+        _chk("gain", gain, torch.float32)
+        ldg = _row_view("matrix_memory: gate", gate, heads * vdim)
+        if gain.numel() != heads * vdim or gate.dtype != q.dtype or gate.shape[0] != T:
+            raise KernelError("matrix_memory: gain or gate do not fit the heads")
+        y = torch.empty((T, heads * vdim), dtype=q.dtype, device=dev)
+    small = finish is not None and vdim <= MEMORY_FINISH_MAX_VDIM
+    fin = (_ptr(gain), _ptr(gate), ctypes.c_longlong(ldg), ctypes.c_float(eps),
+           ctypes.c_float(den_eps), _ptr(y))
+    off = (_ptr(None), _ptr(None), ctypes.c_longlong(0), ctypes.c_float(0.0), ctypes.c_float(0.0),
+           _ptr(None))
+    num = nq = None
+    if not small or (singles < S and form == "walk"):     # something leaves its rows unfinished
+        num = torch.empty((T, heads, vdim), dtype=torch.float32, device=dev)
+        nq = torch.empty((T, heads), dtype=torch.float32, device=dev)
+    views = (_ptr(q), ctypes.c_longlong(ldq), _ptr(k), ctypes.c_longlong(ldk), _ptr(v),
+             ctypes.c_longlong(ldv))
+    held = (_ptr(gates), _ptr(state), _ptr(normaliser))
+    first, last = 0, T                    # rows that still have to be finished
     if singles:
-        _check(_lib().ix_mm_single(*views, _ptr(step.state_slot), _ptr(num), _ptr(nq), T, singles,
-                                   heads, dim, vdim, ctypes.c_float(q_scale), _stream()),
-               "mm_single")
+        _check(_lib().ix_mm_single(
+            *views, _dtype_code(q), *held, _ptr(step.state_slot), _ptr(num), _ptr(nq), T, singles,
+            heads, dim, vdim, ctypes.c_float(q_scale), *(fin if small else off), _stream()),
+            "mm_single")
         _count()
-    if singles < S:
-        applies = q.dtype == torch.bfloat16 and bool(_lib().ix_mm_chunks_applies(dim, vdim))
-        if form is None:
-            form = ("chunks" if applies and int(step.max_q_len) >= MEMORY_CHUNK_MIN_TOKENS
-                    else "walk")
-        if form not in ("walk", "chunks") or (form == "chunks" and not applies):
-            raise KernelError(f"matrix_memory: no form {form!r} for {q.dtype}, heads of {dim} / "
-                              f"{vdim}")
-        if form == "chunks":
-            tokens = T - singles         # single tokens come first, one each
-            size = _lib().ix_mm_chunks_scratch_floats
-            size.restype = ctypes.c_longlong
-            scratch = torch.empty((size(tokens, S - singles, heads, dim, vdim),),
-                                  dtype=torch.float32, device=q.device)
-            _check(_lib().ix_mm_chunks(
-                *views[:6], *views[7:], _ptr(step.cu_q), _ptr(step.state_slot), _ptr(num),
-                _ptr(nq), T, tokens, S, singles, int(step.max_q_len), heads, dim, vdim,
-                ctypes.c_float(q_scale), _ptr(scratch), _stream()), "mm_chunks")
-            _count(3)
-            return num, nq
-        _check(_lib().ix_mm_walk(*views, _ptr(step.cu_q), _ptr(step.state_slot), _ptr(num),
-                                 _ptr(nq), T, S, singles, heads, dim, vdim,
-                                 ctypes.c_float(q_scale), _stream()), "mm_walk")
+        if small:
+            first = singles
+    if singles < S and form == "chunks":
+        tokens = T - singles             # single tokens come first, one each
+        size = _lib().ix_mm_chunks_scratch_floats
+        size.restype = ctypes.c_longlong
+        scratch = torch.empty((size(tokens, S - singles, heads, dim, vdim),),
+                              dtype=torch.float32, device=dev)
+        _check(_lib().ix_mm_chunks(
+            *views, *held, _ptr(step.cu_q), _ptr(step.state_slot), _ptr(num), _ptr(nq), T, tokens,
+            S, singles, int(step.max_q_len), heads, dim, vdim, ctypes.c_float(q_scale),
+            _ptr(scratch), *(fin if small else off), _stream()), "mm_chunks")
+        _count(3)
+        if small:
+            last = first
+    elif singles < S:
+        _check(_lib().ix_mm_walk(
+            *views, _dtype_code(q), *held, _ptr(step.cu_q), _ptr(step.state_slot), _ptr(num),
+            _ptr(nq), T, S, singles, heads, dim, vdim, ctypes.c_float(q_scale), _stream()),
+            "mm_walk")
         _count()
-    return num, nq
+    if finish is None:
+        return num, nq
+    if last > first:
+        head_norm_gate(num[first:last], gain, gate[first:last], eps, q.dtype, gate_form="sigmoid",
+                       den=(nq[first:last], gates[2, first:last], den_eps), out=y[first:last])
+    return y

@@ -76,13 +76,10 @@ class MatrixMemoryMixer:
         gates = ops.memory_gates(x, self.gate_w, self.gate_b, s.gate_cap, cache.state[MAXIMUM],
                                  step)                       # fp32 [4, T, heads]
         front = ops.linear(x, self.front_w)                  # [T, q | k | v | g]
-        num, nq = ops.matrix_memory(front[:, :hk], front[:, hk:2 * hk],
-                                    front[:, 2 * hk:2 * hk + hv], gates, cache.state[MEMORY],
-                                    cache.state[NORMALISER], step, s.heads, s.dim, s.vdim,
-                                    s.q_scale)
-        y = ops.head_norm_gate(num, self.norm_w, front[:, 2 * hk + hv:2 * hk + 2 * hv],
-                               s.norm_eps, self.ctx.dtype, gate_form="sigmoid",
-                               den=(nq, gates[2], s.den_eps))
+        y = ops.matrix_memory(
+            front[:, :hk], front[:, hk:2 * hk], front[:, 2 * hk:2 * hk + hv], gates,
+            cache.state[MEMORY], cache.state[NORMALISER], step, s.heads, s.dim, s.vdim, s.q_scale,
+            finish=(self.norm_w, front[:, 2 * hk + hv:2 * hk + 2 * hv], s.norm_eps, s.den_eps))
         return ops.linear(y, self.o_w)
 
 

@@ -918,7 +918,8 @@ def memory_gates(x, w, bias, cap, m_state, step):
     return out
 
 
-def matrix_memory(q, k, v, gates, state, normaliser, step, heads, dim, vdim, q_scale):
+def matrix_memory(q, k, v, gates, state, normaliser, step, heads, dim, vdim, q_scale, form=None,
+                  finish=None):
     T = q.shape[0]
     qf = _f(q).reshape(T, heads, dim) * q_scale
     kf, vf = _f(k).reshape(T, heads, dim), _f(v).reshape(T, heads, vdim)
@@ -933,4 +934,7 @@ def matrix_memory(q, k, v, gates, state, normaliser, step, heads, dim, vdim, q_s
             num[t] = torch.einsum("hkv,hk->hv", S, qf[t])
             nq[t] = (n * qf[t]).sum(-1)
         state[slot], normaliser[slot] = S, n
+    if finish is not None:
+        gain, gate, eps, den_eps = finish
+        return head_norm_gate(num, gain, gate, eps, q.dtype, "sigmoid", den=(nq, gates[2], den_eps))
     return num, nq

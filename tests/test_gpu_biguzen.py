@@ -215,6 +215,31 @@ def test_matrix_memory(dtype, H, K, V, q_lens):
         assert torch.equal(gS[-1].cpu(), S[-1]) and torch.equal(gn[-1].cpu(), n[-1])
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,K,V", [(3, 10, 6), (2, 48, 48), (2, 64, 128), (1, 24, 200), (2, 16, 7)])
+@pytest.mark.parametrize("q_lens", [[1, 1, 1], [1, 5, 2], [1, 1, 200, 64, 65], [100]])
+def test_matrix_memory_finishes_the_heads(dtype, H, K, V, q_lens):
+    """Division by the normaliser, norm, gain and gate in the memory's kernels where a block has
+    the whole head, else behind them."""
+    step, rows, gates, S, n = _memory_case(K + V + 1, H, K, V, q_lens, dtype)
+    r = _rand(V)
+    T = step.num_tokens
+    gain, gate = r(H * V), r(T, H * V + 2 * (V % 2) + 4).to(dtype)
+    n = n * 0.02                                     # some denominators are the floor's
+    refS, refn = S.clone(), n.clone()
+    ref = host_ops.matrix_memory(*_views(rows, H, K, V), gates, refS, refn, step, H, K, V, 0.3,
+                                 finish=(gain, gate[:, :H * V], 1e-5, 1e-6)).float()
+    for form in ["walk"] + (["chunks"] if dtype == torch.bfloat16 and max(q_lens) > 1 else []):
+        gS, gn = S.clone().cuda(), n.clone().cuda()
+        y = _ops().matrix_memory(*_views(rows.cuda(), H, K, V), gates.cuda(), gS, gn, _cuda(step),
+                                 H, K, V, 0.3, form=form,
+                                 finish=(gain.cuda(), gate.cuda()[:, :H * V], 1e-5, 1e-6))
+        assert y.dtype == dtype
+        err = (y.cpu().float() - ref).abs().max() / ref.abs().max()
+        assert float(err) < (3e-4 if dtype == torch.float32 else 1e-2), (form, float(err))
+        assert float((gS.cpu() - refS).abs().max() / refS.abs().max()) < 6e-5
+
+
 @pytest.mark.parametrize("form,dtype", [("walk", torch.float32), ("walk", torch.bfloat16),
                                         ("chunks", torch.bfloat16)])
 def test_memory_carries_what_was_written_far_back(form, dtype):
