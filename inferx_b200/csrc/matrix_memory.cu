@@ -26,7 +26,7 @@ __device__ __forceinline__ float mm_log_sigmoid(float z) {
 // ---------------------------------------------------------------------------
 // Steps of single tokens: one warp per (token, head) forms both dot products and moves the
 // running maximum on.  x [T, W] and w [2 H, W] (input gates' rows, then forget gates') of one
-// type; gates [4, T, H]: keep, put, floor and
+// type; gates [4, H, T]: keep, put, floor and
 // the logarithm of keep.
 // ---------------------------------------------------------------------------
 #define MG_WARPS 4
@@ -78,7 +78,7 @@ mm_gates_single_kernel(const TA* __restrict__ x, const TA* __restrict__ w,
     const float before = *mp;
     const float m = fmaxf(f + before, i);
     *mp = m;
-    const size_t at = (size_t)t * H + h, plane = (size_t)T * H;
+    const size_t at = (size_t)h * T + t, plane = (size_t)T * H;
     gates[at] = expf(f + before - m);
     gates[plane + at] = expf(i - m);
     gates[2 * plane + at] = expf(-m);
@@ -106,7 +106,7 @@ IX_API int ix_mm_gates_single(const void* x, const void* w, int dtype, const flo
 }
 
 // ---------------------------------------------------------------------------
-// Any step: z fp32 [T, 2 H] holds the dot products; one block per (head, sequence) walks the
+// Any step: z fp32 [2 H, T] holds the dot products; one block per (head, sequence) walks the
 // sequence in tiles of a token per thread.  A span of tokens is the pair (F, M): m at its
 // end is max(m before it + F, M); spans join as (F1 + F2, max(M1 + F2, M2)).  keep uses the
 // m of the token before as that token's own thread formed it.
@@ -131,8 +131,8 @@ mm_gates_scan_kernel(const float* __restrict__ z, const float* __restrict__ bias
     const bool ok = t < end;
     float i = -INFINITY, f = 0.f;          // past the end: a span that changes nothing
     if (ok) {
-      i = mm_cap(z[(size_t)t * 2 * H + h] + bi, cap);
-      f = mm_log_sigmoid(mm_cap(z[(size_t)t * 2 * H + H + h] + bf, cap));
+      i = mm_cap(z[(size_t)h * T + t] + bi, cap);
+      f = mm_log_sigmoid(mm_cap(z[(size_t)(H + h) * T + t] + bf, cap));
     }
     float F = f, M = i;
 #pragma unroll
@@ -156,7 +156,7 @@ mm_gates_scan_kernel(const float* __restrict__ z, const float* __restrict__ bias
     float before = __shfl_up_sync(0xffffffffu, m, 1);
     if (lane == 0) before = warp == 0 ? carry : last[warp - 1];
     if (ok) {
-      const size_t at = (size_t)t * H + h;
+      const size_t at = (size_t)h * T + t;
       gates[at] = expf(f + before - m);
       gates[plane + at] = expf(i - m);
       gates[2 * plane + at] = expf(-m);
@@ -206,7 +206,8 @@ mm_single_kernel(const TA* __restrict__ q, long long ldq, const TA* __restrict__
   const int t = blockIdx.z, h = blockIdx.y, v0 = blockIdx.x * MD_COLS;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const size_t at = (size_t)t * H + h, plane = (size_t)T * H;
-  const float keep = gates[at], put = gates[plane + at];
+  const size_t gate_at = (size_t)h * T + t;
+  const float keep = gates[gate_at], put = gates[plane + gate_at];
   const size_t slot_head = (size_t)state_slot[t] * H + h;
   for (int i = tid; i < K; i += MD_WARPS * 32) {
     q_s[i] = to_f32(q[t * ldq + (size_t)h * K + i]) * q_scale;
@@ -280,7 +281,7 @@ mm_single_kernel(const TA* __restrict__ q, long long ldq, const TA* __restrict__
     }
     a = block_sum(a, scratch);
     if (fin.gain) {
-      const float y = total / (fmaxf(fabsf(a), gates[2 * plane + at]) + fin.den_eps);
+      const float y = total / (fmaxf(fabsf(a), gates[2 * plane + gate_at]) + fin.den_eps);
       const float ss = block_sum(y * y, scratch);     // 0 beyond V
       if (tid < V) {
         const size_t c = (size_t)h * V + tid;
@@ -295,7 +296,7 @@ mm_single_kernel(const TA* __restrict__ q, long long ldq, const TA* __restrict__
 }
 
 // q, k [T, H K] and v [T, H V] are views with row pitches; sequences 0 .. singles - 1 bring one
-// token each (token s of the step).  gates [4, T, H] as the gate kernels leave them.  num fp32
+// token each (token s of the step).  gates [4, H, T] as the gate kernels leave them.  num fp32
 // [T, H, V], nq fp32 [T, H]; or, with `gain`, the finished rows in `out` (see MmFinish).
 IX_API int ix_mm_single(const void* q, long long ldq, const void* k, long long ldk,
                         const void* v, long long ldv, int dtype, const float* gates, float* S,
@@ -366,7 +367,7 @@ mm_walk_kernel(const TA* __restrict__ q, long long ldq, const TA* __restrict__ k
       const int c = i / K, kk = i - c * K;
       const size_t t = (size_t)(t0 + c);
       q_s[i] = to_f32(q[t * ldq + (size_t)h * K + kk]) * q_scale;
-      k_s[i] = to_f32(k[t * ldk + (size_t)h * K + kk]) * gates[plane + t * H + h];
+      k_s[i] = to_f32(k[t * ldk + (size_t)h * K + kk]) * gates[plane + (size_t)h * T + t];
     }
     for (int i = threadIdx.x; i < n * MW_COLS; i += blockDim.x) {
       const int c = i / MW_COLS, j = i % MW_COLS;
@@ -374,7 +375,7 @@ mm_walk_kernel(const TA* __restrict__ q, long long ldq, const TA* __restrict__ k
                     : (v0 + j < V ? to_f32(v[(size_t)(t0 + c) * ldv + (size_t)h * V + v0 + j])
                                   : 0.f);
     }
-    if (threadIdx.x < n) keep_s[threadIdx.x] = gates[(size_t)(t0 + threadIdx.x) * H + h];
+    if (threadIdx.x < n) keep_s[threadIdx.x] = gates[(size_t)h * T + t0 + threadIdx.x];
     __syncthreads();
     for (int c = 0; c < n; ++c) {
       const float vj = v_s[c * MW_COLS + lane], keep = keep_s[c];

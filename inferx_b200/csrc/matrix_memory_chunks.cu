@@ -87,13 +87,13 @@ __device__ __forceinline__ void mc_load(bf16* dst, int pitch, const bf16* src, l
 
 // G of the chunk's tokens and put by one warp; tokens past the end: G of the last, put 0.
 __device__ __forceinline__ void mc_gates(float* G, float* put, const float* gates, size_t plane,
-                                         size_t first, int H, int n) {
+                                         size_t first, int n) {
   const int lane = threadIdx.x & 31;
   float carry = 0.f;
 #pragma unroll
   for (int half = 0; half < 2; ++half) {
     const int t = half * 32 + lane;
-    float g = t < n ? gates[3 * plane + first + (size_t)t * H] : 0.f;
+    float g = t < n ? gates[3 * plane + first + t] : 0.f;
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
       const float p = __shfl_up_sync(0xffffffffu, g, o);
@@ -102,7 +102,7 @@ __device__ __forceinline__ void mc_gates(float* G, float* put, const float* gate
     g += carry;
     carry = __shfl_sync(0xffffffffu, g, 31);
     G[t] = g;
-    put[t] = t < n ? gates[plane + first + (size_t)t * H] : 0.f;
+    put[t] = t < n ? gates[plane + first + t] : 0.f;
   }
 }
 
@@ -142,7 +142,7 @@ mm_chunk_own_kernel(const bf16* __restrict__ k, long long ldk, const bf16* __res
   mc_load(k_hi, pk, k + (size_t)at.t0 * ldk + (size_t)h * K, ldk, at.n, K, Kp, vec_k);
   mc_load(v_s, pv, v + (size_t)at.t0 * ldv + (size_t)h * V + v0, ldv, at.n, min(VT, V - v0), VT,
           vec_v);
-  if (warp == 0) mc_gates(G, put, gates, plane, (size_t)at.t0 * H + h, H, at.n);
+  if (warp == 0) mc_gates(G, put, gates, plane, (size_t)h * T + at.t0, at.n);
   mc_async_wait();
   __syncthreads();
   const float g_end = G[MC_L - 1];
@@ -315,7 +315,7 @@ mm_chunk_out_kernel(const bf16* __restrict__ q, long long ldq, const bf16* __res
     mc_async8(s_lo + r * pv + c, reinterpret_cast<const uint2*>(w) + 1, ok ? 8 : 0);
   }
   for (int i = tid; i < Kp; i += MC_THREADS) n_s[i] = i < K ? scr_n[cell * K + i] : 0.f;
-  if (warp == 0) mc_gates(G, put, gates, plane, (size_t)at.t0 * H + h, H, at.n);
+  if (warp == 0) mc_gates(G, put, gates, plane, (size_t)h * T + at.t0, at.n);
   mc_async_wait();
   __syncthreads();
   if (warp * 16 >= at.n) return;                        // (no barrier follows)
@@ -423,9 +423,9 @@ mm_chunk_out_kernel(const bf16* __restrict__ q, long long ldq, const bf16* __res
   }
   if (fin.gain) {        // one tile holds the head's whole output
     const size_t fa = (size_t)(at.t0 + min(ra, at.n - 1)), fb = (size_t)(at.t0 + min(rb, at.n - 1));
-    const float da = q_scale / (fmaxf(fabsf(sum_a * q_scale), gates[2 * plane + fa * H + h]) +
+    const float da = q_scale / (fmaxf(fabsf(sum_a * q_scale), gates[2 * plane + (size_t)h * T + fa]) +
                                 fin.den_eps);
-    const float db = q_scale / (fmaxf(fabsf(sum_b * q_scale), gates[2 * plane + fb * H + h]) +
+    const float db = q_scale / (fmaxf(fabsf(sum_b * q_scale), gates[2 * plane + (size_t)h * T + fb]) +
                                 fin.den_eps);
     float qa = 0.f, qb = 0.f;
 #pragma unroll

@@ -548,7 +548,8 @@ IX_API int ix_linear_recurrence(const void* q, long long ldq, const void* k, lon
 // ---------------------------------------------------------------------------
 // head norm + gate.  One warp per (token, head).  `gain` covers all heads
 // (gain_per_head) or is shared by them.  gate_form 0: silu(gate); 1: sigmoid(gate).  With
-// `nq` ([T, H]; null: o as it is) a head's row is first divided by max(|nq|, floor) + den_eps.
+// `nq` ([T, H]; null: o as it is) a head's row is first divided by max(|nq|, floor) + den_eps,
+// floor of (token t, head h) at t + h * floor_ld.
 // ---------------------------------------------------------------------------
 #define HNG_WARPS 4
 
@@ -557,7 +558,8 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, const float* 
                                       int gain_per_head, const TG* __restrict__ gate,
                                       long long ldg, TA* __restrict__ out, int H, int V,
                                       float eps, int gate_form, const float* __restrict__ nq,
-                                      const float* __restrict__ floor_, float den_eps) {
+                                      const float* __restrict__ floor_,
+                                               long long floor_ld, float den_eps) {
   IX_PDL_WAIT();
   const int t = blockIdx.x;
   const int h = blockIdx.y * HNG_WARPS + (threadIdx.x >> 5);
@@ -568,7 +570,7 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, const float* 
   float den = 1.f;
   if (nq) {
     const size_t at = (size_t)t * H + h;
-    den = 1.0f / (fmaxf(fabsf(nq[at]), floor_[at]) + den_eps);
+    den = 1.0f / (fmaxf(fabsf(nq[at]), floor_[t + h * floor_ld]) + den_eps);
   }
   for (int c = lane; c < V; c += 32) {
     const float x = row[c] * den;
@@ -595,7 +597,8 @@ __global__ void head_norm_gate_bf16_vec_kernel(const float* __restrict__ o,
                                                const bf16* __restrict__ gate, long long ldg,
                                                bf16* __restrict__ out, int H, int V, float eps,
                                                const float* __restrict__ nq,
-                                               const float* __restrict__ floor_, float den_eps) {
+                                               const float* __restrict__ floor_,
+                                               long long floor_ld, float den_eps) {
   IX_PDL_WAIT();
   const int t = blockIdx.x;
   const int lane = threadIdx.x & 31;
@@ -607,7 +610,7 @@ __global__ void head_norm_gate_bf16_vec_kernel(const float* __restrict__ o,
   if (ok) x = reinterpret_cast<const float4*>(o + ((size_t)t * H + h) * V)[sub];
   if (nq && ok) {
     const size_t at = (size_t)t * H + h;
-    const float den = 1.0f / (fmaxf(fabsf(nq[at]), floor_[at]) + den_eps);
+    const float den = 1.0f / (fmaxf(fabsf(nq[at]), floor_[t + h * floor_ld]) + den_eps);
     x.x *= den; x.y *= den; x.z *= den; x.w *= den;
   }
   float ss = x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
@@ -632,7 +635,7 @@ __global__ void head_norm_gate_bf16_vec_kernel(const float* __restrict__ o,
 IX_API int ix_head_norm_gate(const float* o, const float* gain, int gain_per_head,
                              const void* gate, int gate_dtype, long long ldg, void* out,
                              int out_dtype, int T, int H, int V, float eps, int gate_form,
-                             const float* nq, const float* floor_, float den_eps,
+                             const float* nq, const float* floor_, long long floor_ld, float den_eps,
                              cudaStream_t stream) {
   if (T <= 0) return IX_OK;
   if ((nq == nullptr) != (floor_ == nullptr)) return IX_ERR_SIZE;
@@ -651,7 +654,7 @@ IX_API int ix_head_norm_gate(const float* o, const float* gain, int gain_per_hea
                           : head_norm_gate_bf16_vec_kernel<GL, false>;                        \
     ix_launch(kern, dim3(T, vgroups), dim3(32 * HNG_WARPS), 0, stream, o, gain,               \
               gain_per_head, (const bf16*)gate, ldg, (bf16*)out, H, V, eps, nq, floor_,       \
-              den_eps);                                                                       \
+              floor_ld, den_eps);                                                                      \
   } while (0)
     if (gl == 32) IX_HNG(32);
     else if (gl == 16) IX_HNG(16);
@@ -666,6 +669,6 @@ IX_API int ix_head_norm_gate(const float* o, const float* gain, int gain_per_hea
                     ix_launch(head_norm_gate_kernel<TA, TA>, dim3(T, groups),
                               dim3(32 * HNG_WARPS), 0, stream, o, gain, gain_per_head,
                               (const TA*)gate, ldg, (TA*)out, H, V, eps, gate_form, nq, floor_,
-                              den_eps));
+                              floor_ld, den_eps));
   return ix_launch_status();
 }

@@ -74,9 +74,10 @@ __device__ __forceinline__ void st_store(bf16* p, const StVec<VW>& r) {
   }
 }
 
-// FIXED: n == NS, the constants live in registers; otherwise n <= NS and they are read from
-// shared memory.
-template <int NS, bool FIXED, int VW, typename TY, typename TO>
+// FIXED: n == NS; otherwise n <= NS.  With FIXED and a plain y the constants live in registers;
+// they are read from shared memory otherwise: combining a mixture's rows is a chain of
+// dependent reads (row numbers, then rows), for which more threads in flight are worth more.
+template <int NS, bool FIXED, bool COMBINE, int VW, typename TY, typename TO>
 __global__ void __launch_bounds__(ST_THREADS)
 stream_step_kernel(float* __restrict__ streams, const TY* __restrict__ y, StCombine cmb,
                    const float* __restrict__ mix, const float* __restrict__ put,
@@ -96,12 +97,13 @@ stream_step_kernel(float* __restrict__ streams, const TY* __restrict__ y, StComb
   __syncthreads();
   const int c = (blockIdx.x * ST_THREADS + threadIdx.x) * VW;
   if (c >= W) return;
-  float mr[FIXED ? NS * NS : 1], pr[FIXED ? NS : 1], rr[FIXED ? NS : 1];
-  if (FIXED) {
+  constexpr bool REGS = FIXED && !COMBINE;
+  float mr[REGS ? NS * NS : 1], pr[REGS ? NS : 1], rr[REGS ? NS : 1];
+  if (REGS) {
 #pragma unroll
-    for (int i = 0; i < (FIXED ? NS * NS : 1); ++i) mr[i] = mix_s[i];
+    for (int i = 0; i < (REGS ? NS * NS : 1); ++i) mr[i] = mix_s[i];
 #pragma unroll
-    for (int i = 0; i < (FIXED ? NS : 1); ++i) {
+    for (int i = 0; i < (REGS ? NS : 1); ++i) {
       pr[i] = put_s[i];
       rr[i] = read_s[i];
     }
@@ -118,30 +120,49 @@ stream_step_kernel(float* __restrict__ streams, const TY* __restrict__ y, StComb
     float* x = streams + t * n * W + c;
     StVec<VW> old[NS], d;
 #pragma unroll
-    for (int s = 0; s < NS; ++s)
-      if (FIXED || s < n) old[s] = st_load<VW>(x + (size_t)s * W);
-#pragma unroll
     for (int e = 0; e < VW; ++e) d.v[e] = 0.f;
-    if (updates) {
-      if (cmb.rows) {
-        const TY* er = reinterpret_cast<const TY*>(cmb.rows);
-#pragma unroll 4
-        for (int j = 0; j < cmb.k; ++j) {
-          const float w = cmb.weight ? cmb.weight[t * cmb.k + j] : 1.0f;
-          const StVec<VW> f = st_load<VW>(er + (size_t)cmb.dest[t * cmb.k + j] * W + c);
+    if (COMBINE) {
+      // four assignments at a time, without a branch between their reads: row numbers and
+      // weights, then the rows
+      const TY* er = reinterpret_cast<const TY*>(cmb.rows);
+      const int* dest = cmb.dest + t * cmb.k;
+      const float* weight = cmb.weight ? cmb.weight + t * cmb.k : read;
+      const float sg = cmb.shared && cmb.shared_logit
+                           ? 1.0f / (1.0f + expf(-cmb.shared_logit[t])) : 1.0f;
+      for (int j0 = 0; j0 < cmb.k; j0 += 4) {
+        int row[4];
+        float w[4];
+        StVec<VW> f[4];
 #pragma unroll
-          for (int e = 0; e < VW; ++e) d.v[e] = fmaf(w, f.v[e], d.v[e]);
+        for (int j = 0; j < 4; ++j) {
+          const int a = min(j0 + j, cmb.k - 1);
+          row[j] = dest[a];
+          w[j] = weight[cmb.weight ? a : 0];
         }
-        if (cmb.shared) {
-          const float sg =
-              cmb.shared_logit ? 1.0f / (1.0f + expf(-cmb.shared_logit[t])) : 1.0f;
-          const StVec<VW> f = st_load<VW>(reinterpret_cast<const TY*>(cmb.shared) + t * W + c);
 #pragma unroll
-          for (int e = 0; e < VW; ++e) d.v[e] = fmaf(sg, f.v[e], d.v[e]);
+        for (int j = 0; j < 4; ++j) f[j] = st_load<VW>(er + (size_t)row[j] * W + c);
+        if (j0 == 0) {
+#pragma unroll
+          for (int s = 0; s < NS; ++s)
+            if (FIXED || s < n) old[s] = st_load<VW>(x + (size_t)s * W);
         }
-      } else {
-        d = st_load<VW>(y + t * W + c);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const float wj = j0 + j < cmb.k ? (cmb.weight ? w[j] : 1.0f) : 0.f;
+#pragma unroll
+          for (int e = 0; e < VW; ++e) d.v[e] = fmaf(wj, f[j].v[e], d.v[e]);
+        }
       }
+      if (cmb.shared) {
+        const StVec<VW> f = st_load<VW>(reinterpret_cast<const TY*>(cmb.shared) + t * W + c);
+#pragma unroll
+        for (int e = 0; e < VW; ++e) d.v[e] = fmaf(sg, f.v[e], d.v[e]);
+      }
+    } else {
+#pragma unroll
+      for (int s = 0; s < NS; ++s)
+        if (FIXED || s < n) old[s] = st_load<VW>(x + (size_t)s * W);
+      if (updates) d = st_load<VW>(y + t * W + c);
     }
     StVec<VW> u;
 #pragma unroll
@@ -151,13 +172,13 @@ stream_step_kernel(float* __restrict__ streams, const TY* __restrict__ y, StComb
       if (!FIXED && o >= n) break;
       StVec<VW> v;
       if (updates) {
-        const float po = FIXED ? pr[FIXED ? o : 0] : put_s[o];
+        const float po = REGS ? pr[REGS ? o : 0] : put_s[o];
 #pragma unroll
         for (int e = 0; e < VW; ++e) v.v[e] = po * d.v[e];
 #pragma unroll
         for (int s = 0; s < NS; ++s) {
           if (!FIXED && s >= n) break;
-          const float m = FIXED ? mr[FIXED ? s * NS + o : 0] : mix_s[s * n + o];
+          const float m = REGS ? mr[REGS ? s * NS + o : 0] : mix_s[s * n + o];
 #pragma unroll
           for (int e = 0; e < VW; ++e) v.v[e] = fmaf(m, old[s].v[e], v.v[e]);
         }
@@ -165,7 +186,7 @@ stream_step_kernel(float* __restrict__ streams, const TY* __restrict__ y, StComb
       } else {
         v = old[o];
       }
-      const float ro = FIXED ? rr[FIXED ? o : 0] : read_s[o];
+      const float ro = REGS ? rr[REGS ? o : 0] : read_s[o];
 #pragma unroll
       for (int e = 0; e < VW; ++e) u.v[e] = fmaf(ro, v.v[e], u.v[e]);
     }
@@ -210,9 +231,12 @@ IX_API int ix_stream_step(float* streams, const void* y, int y_dtype, const void
   if (by > 65535) by = 65535;
   const dim3 grid(colsx, by);
 #define ST_GO(NS, FIXED, VW)                                                                    \
-  ix_launch(stream_step_kernel<NS, FIXED, VW, TY, TO>, grid, dim3(ST_THREADS), 0, stream,       \
-            streams, (const TY*)y, cmb, mix, put, read, alpha, gain, bias, rows, (TO*)out, R, W, \
-            n, write_back)
+  do {                                                                                          \
+    auto kern = mix && c_rows ? stream_step_kernel<NS, FIXED, true, VW, TY, TO>                 \
+                              : stream_step_kernel<NS, FIXED, false, VW, TY, TO>;               \
+    ix_launch(kern, grid, dim3(ST_THREADS), 0, stream, streams, (const TY*)y, cmb, mix, put,    \
+              read, alpha, gain, bias, rows, (TO*)out, R, W, n, write_back);                    \
+  } while (0)
 #define ST_N(VW)                                                                                \
   do {                                                                                          \
     if (n == 1) ST_GO(1, true, VW);                                                             \

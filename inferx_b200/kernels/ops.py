@@ -1886,8 +1886,8 @@ def head_norm_gate(o: torch.Tensor, gain: torch.Tensor, gate: torch.Tensor, eps:
     silu, or sigmoid with ``gate_form`` "sigmoid") for
     o fp32 [T, heads, vdim]; ``gain`` fp32 [vdim] (shared by the heads) or [heads * vdim];
     ``gate`` a view [T, heads * vdim] with unit inner stride in ``out_dtype``.  ``den`` (nq,
-    floor, den_eps) with nq and floor fp32 [T, heads]: a head's row is first divided by
-    max(|nq|, floor) + den_eps."""
+    floor, den_eps) with nq fp32 [T, heads] and floor fp32 [heads, T] (a view of columns): a
+    head's row is first divided by max(|nq|, floor) + den_eps."""
     _chk("o", o, torch.float32)
     _chk("gain", gain, torch.float32)
     T, H, V = o.shape
@@ -1899,14 +1899,17 @@ def head_norm_gate(o: torch.Tensor, gain: torch.Tensor, gate: torch.Tensor, eps:
     _chk("out", out, out_dtype)
     nq, floor, den_eps = den if den is not None else (None, None, 0.0)
     _chk("nq", nq, torch.float32, optional=True)
-    _chk("floor", floor, torch.float32, optional=True)
-    if nq is not None and (nq.numel() != T * H or floor is None or floor.numel() != T * H):
-        raise KernelError("head_norm_gate: one denominator per (token, head)")
+    floor_ld = 0
+    if nq is not None:
+        if nq.numel() != T * H or floor is None or tuple(floor.shape) != (H, T) or \
+                floor.dtype != torch.float32:
+            raise KernelError("head_norm_gate: one denominator per (token, head)")
+        floor_ld = _row_view("head_norm_gate: floor", floor, T)
     _check(_lib().ix_head_norm_gate(
         _ptr(o), _ptr(gain), 1 if (gain.numel() == H * V and H > 1) else 0, _ptr(gate),
         _dtype_code(gate), ctypes.c_longlong(ldg), _ptr(out), _dtype_code(out), T, H, V,
         ctypes.c_float(eps), _GATE_FORMS[gate_form], _ptr(nq), _ptr(floor),
-        ctypes.c_float(den_eps), _stream()), "head_norm_gate")
+        ctypes.c_longlong(floor_ld), ctypes.c_float(den_eps), _stream()), "head_norm_gate")
     _count()
     return out
 
@@ -2604,7 +2607,7 @@ MEMORY_GATES_SINGLE_TOKENS = 128
 
 def memory_gates(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, cap: float,
                  m_state: torch.Tensor, step):
-    """fp32 [4, T, H]: exp(f + m_(t-1) - m_t), exp(i - m_t), exp(-m_t) and the first one's
+    """fp32 [4, H, T]: exp(f + m_(t-1) - m_t), exp(i - m_t), exp(-m_t) and the first one's
     logarithm of every token and head, with the log gates i = cap tanh(z_i / cap), f = logsigmoid(cap tanh(z_f / cap)), z =
     x . w^T + bias (``w`` [2 H, W]: the input gates' rows, then the forget gates') and m_t =
     max(f + m_(t-1), i) along each sequence from and back to ``m_state`` fp32 [slots, H]."""
@@ -2616,14 +2619,14 @@ def memory_gates(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, cap: floa
     H = w.shape[0] // 2
     if w.shape[1] != W or bias.numel() != 2 * H or m_state.shape[1] != H:
         raise KernelError("memory_gates: weights, biases and state disagree")
-    gates = torch.empty((4, T, H), dtype=torch.float32, device=x.device)
+    gates = torch.empty((4, H, T), dtype=torch.float32, device=x.device)
     if step.all_decode and T == step.num_seqs and T <= MEMORY_GATES_SINGLE_TOKENS:
         _check(_lib().ix_mm_gates_single(
             _ptr(x), _ptr(w), _dtype_code(x), _ptr(bias), ctypes.c_float(cap), _ptr(m_state),
             _ptr(step.state_slot), _ptr(gates), T, W, H, _stream()), "mm_gates_single")
         _count()
         return gates
-    z = linear(x, w, out_dtype=torch.float32)
+    z = linear(w, x, out_dtype=torch.float32)       # [2 H, T]: a head's numbers side by side
     _check(_lib().ix_mm_gates_scan(
         _ptr(z), _ptr(bias), ctypes.c_float(cap), _ptr(m_state), _ptr(step.state_slot),
         _ptr(step.cu_q), _ptr(gates), T, step.num_seqs, H, _stream()), "mm_gates_scan")
@@ -2661,7 +2664,7 @@ def matrix_memory(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: torc
     _chk("normaliser", normaliser, torch.float32)
     T, S, dev = q.shape[0], step.num_seqs, q.device
     if not (q.dtype == k.dtype == v.dtype) or k.shape[0] != T or v.shape[0] != T \
-            or tuple(gates.shape) != (4, T, heads) \
+            or tuple(gates.shape) != (4, heads, T) \
             or tuple(state.shape[1:]) != (heads, dim, vdim) \
             or tuple(normaliser.shape[1:]) != (heads, dim):
         raise KernelError("matrix_memory: q, k, v, gates and state do not fit together")
@@ -2725,5 +2728,5 @@ def matrix_memory(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: torc
         return num, nq
     if last > first:
         head_norm_gate(num[first:last], gain, gate[first:last], eps, q.dtype, gate_form="sigmoid",
-                       den=(nq[first:last], gates[2, first:last], den_eps), out=y[first:last])
+                       den=(nq[first:last], gates[2, :, first:last], den_eps), out=y[first:last])
     return y

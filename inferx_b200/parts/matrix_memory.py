@@ -74,7 +74,7 @@ class MatrixMemoryMixer:
         s, ops = self.spec, self.ctx.ops
         hk, hv = self.hk, self.hv
         gates = ops.memory_gates(x, self.gate_w, self.gate_b, s.gate_cap, cache.state[MAXIMUM],
-                                 step)                       # fp32 [4, T, heads]
+                                 step)                       # fp32 [4, heads, T]
         front = ops.linear(x, self.front_w)                  # [T, q | k | v | g]
         y = ops.matrix_memory(
             front[:, :hk], front[:, hk:2 * hk], front[:, 2 * hk:2 * hk + hv], gates,

@@ -541,7 +541,7 @@ def head_norm_gate(o, weight, gate, eps, out_dtype, gate_form="silu", den=None):
     T, H, V = o.shape
     if den is not None:
         nq, floor, den_eps = den
-        o = o / (torch.maximum(nq.abs(), floor) + den_eps)[:, :, None]
+        o = o / (torch.maximum(nq.abs(), floor.T) + den_eps)[:, :, None]
     n = o / torch.sqrt((o * o).mean(-1, keepdim=True) + eps)
     n = n * (weight.reshape(H, V) if weight.numel() == H * V else weight)
     g = _f(gate).reshape(T, H, V)
@@ -905,14 +905,14 @@ def memory_gates(x, w, bias, cap, m_state, step):
     z = _f(x) @ _f(w).T + bias
     i = cap * torch.tanh(z[:, :H] / cap)
     f = torch.nn.functional.logsigmoid(cap * torch.tanh(z[:, H:] / cap))
-    out = torch.zeros(4, T, H)
+    out = torch.zeros(4, H, T)
     for s in range(step.num_seqs):
         slot = int(step.state_slot[s])
         m = m_state[slot].clone()
         for t in range(int(step.cu_q[s]), int(step.cu_q[s + 1])):
             new = torch.maximum(f[t] + m, i[t])
-            out[0, t], out[1, t] = torch.exp(f[t] + m - new), torch.exp(i[t] - new)
-            out[2, t], out[3, t] = torch.exp(-new), f[t] + m - new
+            out[0, :, t], out[1, :, t] = torch.exp(f[t] + m - new), torch.exp(i[t] - new)
+            out[2, :, t], out[3, :, t] = torch.exp(-new), f[t] + m - new
             m = new
         m_state[slot] = m
     return out
@@ -928,9 +928,9 @@ def matrix_memory(q, k, v, gates, state, normaliser, step, heads, dim, vdim, q_s
         slot = int(step.state_slot[s])
         S, n = state[slot].clone(), normaliser[slot].clone()
         for t in range(int(step.cu_q[s]), int(step.cu_q[s + 1])):
-            kk = gates[1, t][:, None] * kf[t]
-            S = gates[0, t][:, None, None] * S + kk[:, :, None] * vf[t][:, None, :]
-            n = gates[0, t][:, None] * n + kk
+            kk = gates[1, :, t][:, None] * kf[t]
+            S = gates[0, :, t][:, None, None] * S + kk[:, :, None] * vf[t][:, None, :]
+            n = gates[0, :, t][:, None] * n + kk
             num[t] = torch.einsum("hkv,hk->hv", S, qf[t])
             nq[t] = (n * qf[t]).sum(-1)
         state[slot], normaliser[slot] = S, n

@@ -179,13 +179,13 @@ def _memory_case(seed, H, K, V, q_lens, dtype, forget=2.0):
     rows = r(T, 2 * H * K + H * V + 5).to(dtype)
     z = r(T, 2 * H)
     i, f = z[:, :H] * 2.0, torch.nn.functional.logsigmoid(z[:, H:] * 2.0 + forget)
-    gates = torch.zeros(4, T, H)
+    gates = torch.zeros(4, H, T)
     for s in range(step.num_seqs):
         m = torch.zeros(H)
         for t in range(int(step.cu_q[s]), int(step.cu_q[s + 1])):
             new = torch.maximum(f[t] + m, i[t])
-            gates[0, t], gates[1, t] = torch.exp(f[t] + m - new), torch.exp(i[t] - new)
-            gates[2, t], gates[3, t] = torch.exp(-new), f[t] + m - new
+            gates[0, :, t], gates[1, :, t] = torch.exp(f[t] + m - new), torch.exp(i[t] - new)
+            gates[2, :, t], gates[3, :, t] = torch.exp(-new), f[t] + m - new
             m = new
     S, n = r(len(q_lens) + 1, H, K, V), r(len(q_lens) + 1, H, K)
     return step, rows, gates, S, n
@@ -252,16 +252,16 @@ def test_memory_carries_what_was_written_far_back(form, dtype):
         rows = torch.zeros(401, 2 * K + V)
         rows[0, K:2 * K], rows[0, 2 * K:] = 1.0, 3.0       # key of ones, value of threes
         rows[400, :K] = 1.0                                # the query
-        gates = torch.zeros(4, 401, H)
+        gates = torch.zeros(4, H, 401)
         gates[0], gates[1], gates[2], gates[3] = 1.0, 0.0, 1.0, 0.0
-        gates[1, 0] = 0.5
+        gates[1, :, 0] = 0.5
         at, last = 0, None
         for c in cuts:
             step = _cuda(_step([c], [at]))
             part = rows[at:at + c].to(dtype).cuda()
             f = None if c == 1 else form
             num, nq = _ops().matrix_memory(*_views(part, H, K, V),
-                                           gates[:, at:at + c].contiguous().cuda(), S, n, step, H,
+                                           gates[:, :, at:at + c].contiguous().cuda(), S, n, step, H,
                                            K, V, 1.0, form=f)
             at, last = at + c, (num[-1], nq[-1])
         assert at == 401
@@ -281,7 +281,7 @@ def test_memory_does_not_depend_on_the_cut_or_the_batch():
     at, nums, nqs = 0, [], []
     for c in (33, 2, 64, 100, 31):
         rs = torch.cat([other[1][:1], other[1][1:91], rows[at:at + c]])
-        gs = torch.cat([other[2][:, :91], gates[:, at:at + c]], dim=1).contiguous()
+        gs = torch.cat([other[2][:, :, :91], gates[:, :, at:at + c]], dim=2).contiguous()
         st = _cuda(_step([1, 90, c], [0, 0, at], slots=[3, 4, 0]))
         a, b = _ops().matrix_memory(*_views(rs.cuda(), H, K, V), gs.cuda(), pS, pn, st, H, K, V, 0.2)
         nums.append(a[91:])
@@ -297,8 +297,8 @@ def test_memory_does_not_depend_on_the_cut_or_the_batch():
 def test_head_norm_with_denominator(dtype, V, form):
     T, H, r = 11, 3, _rand(V)
     o, gain, gate = r(T, H, V), r(H * V), r(T, H * V + 3).to(dtype)
-    nq, floor = r(T, H), torch.rand(T, H)
-    nq[0], floor[0] = 0.0, 0.0                  # the added constant alone divides
+    nq, floor = r(T, H), torch.rand(H, T)
+    nq[0], floor[:, 0] = 0.0, 0.0                  # the added constant alone divides
     for den in (None, (nq, floor, 1e-6)):
         ref = host_ops.head_norm_gate(o, gain, gate[:, :H * V], 1e-5, dtype, form, den=den)
         got = _ops().head_norm_gate(o.cuda(), gain.cuda(), gate.cuda()[:, :H * V], 1e-5, dtype, form,
