@@ -204,7 +204,9 @@ IX_API int ix_stream_concat(const float* resid, const void* delta, int delta_dty
 // causal convolution over time per channel.  x [T, C] is a view with row pitch ldx;
 // w [C, taps] (the last column multiplies the current token); state [slots, taps-1, C]
 // holds a request's last taps-1 inputs (oldest first).  A thread owns one channel of one
-// token; the sum runs from the oldest tap to the newest whatever the step's cut.
+// token; the sum runs from the oldest tap to the newest whatever the step's cut.  In a step
+// whose sequences all bring one token (`singles`) the thread is its channel's only reader of the
+// state and moves it on as well; otherwise a second kernel does.
 // ---------------------------------------------------------------------------
 #define CONV_THREADS 128
 #define CONV_MAX_TAPS 16
@@ -213,18 +215,18 @@ template <typename TA>
 __global__ void causal_conv_kernel(const TA* __restrict__ x, long long ldx,
                                    const float* __restrict__ in_bias,
                                    const float* __restrict__ w, const float* __restrict__ bias,
-                                   const float* __restrict__ state,
+                                   float* __restrict__ state,
                                    const int* __restrict__ cu_q,
                                    const int* __restrict__ seq_of_token,
                                    const int* __restrict__ state_slot, TA* __restrict__ out,
-                                   int C, int taps, int act) {
+                                   int C, int taps, int act, int singles) {
   IX_PDL_WAIT();
   const int t = blockIdx.x;
   const int c = blockIdx.y * CONV_THREADS + threadIdx.x;
   if (c >= C) return;
   const int s = seq_of_token[t];
   const int begin = cu_q[s];
-  const float* st = state + (size_t)state_slot[s] * (taps - 1) * C;
+  float* st = state + (size_t)state_slot[s] * (taps - 1) * C;
   float acc = bias ? bias[c] : 0.f;
   const float ib = in_bias ? in_bias[c] : 0.f;
   for (int j = 0; j < taps; ++j) {
@@ -238,6 +240,7 @@ __global__ void causal_conv_kernel(const TA* __restrict__ x, long long ldx,
       v = st[(size_t)(taps - 1 - back) * C + c];
     }
     acc = fmaf(w[(size_t)c * taps + j], v, acc);
+    if (singles && j > 0) st[(size_t)(j - 1) * C + c] = v;     // read above it already
   }
   if (act) acc = acc / (1.0f + expf(-acc));
   out[(size_t)t * C + c] = from_f32<TA>(acc);
@@ -362,17 +365,18 @@ __global__ void conv_state_update_kernel(const TA* __restrict__ x, long long ldx
 }
 
 // in_bias (fp32 [C], or null) is added to every input of the step before it is used or kept
-// (not to the zeros before a sequence's start).
+// (not to the zeros before a sequence's start).  singles: every sequence brings one token.
 IX_API int ix_causal_conv(const void* x, int dtype, long long ldx, const float* in_bias,
                           const float* w, const float* bias, float* state, const int* cu_q,
                           const int* seq_of_token, const int* state_slot, void* out, int T, int S,
-                          int C, int taps, int act, cudaStream_t stream) {
+                          int C, int taps, int act, int singles, cudaStream_t stream) {
   if (T <= 0 || S <= 0) return IX_OK;
   if (C <= 0 || taps < 1 || taps > CONV_MAX_TAPS || ldx < C) return IX_ERR_SIZE;
   const int cb = (C + CONV_THREADS - 1) / CONV_THREADS;
   if (cb > 65535) return IX_ERR_SIZE;
   const size_t two = dtype == IX_F32 ? 8 : 4;
-  const bool run = T >= CONV_RUN_MIN_TOKENS && taps >= 2 && taps <= 4 && C % 2 == 0 &&
+  if (singles && T != S) return IX_ERR_SIZE;
+  const bool run = !singles && T >= CONV_RUN_MIN_TOKENS && taps >= 2 && taps <= 4 && C % 2 == 0 &&
                    ldx % 2 == 0 && (uintptr_t)x % two == 0 && (uintptr_t)out % two == 0;
   const dim3 rgrid((T + CONV_RUN - 1) / CONV_RUN, (C / 2 + CONV_THREADS - 1) / CONV_THREADS);
 #define CONV_GO(TAPS)                                                                        \
@@ -385,9 +389,9 @@ IX_API int ix_causal_conv(const void* x, int dtype, long long ldx, const float* 
     else if (run && taps == 4) CONV_GO(4);
     else
       ix_launch(causal_conv_kernel<TA>, dim3(T, cb), dim3(CONV_THREADS), 0, stream,
-                (const TA*)x, ldx, in_bias, w, bias, (const float*)state, cu_q, seq_of_token,
-                state_slot, (TA*)out, C, taps, act);
-    if (taps > 1)
+                (const TA*)x, ldx, in_bias, w, bias, state, cu_q, seq_of_token, state_slot,
+                (TA*)out, C, taps, act, singles);
+    if (taps > 1 && !singles)
       ix_launch(conv_state_update_kernel<TA>, dim3(S, cb), dim3(CONV_THREADS), 0, stream,
                 (const TA*)x, ldx, in_bias, state, cu_q, state_slot, C, taps);
   });

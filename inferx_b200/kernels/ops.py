@@ -1993,11 +1993,12 @@ def causal_conv(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor],
             (bias is not None and bias.numel() != C):
         raise KernelError("causal_conv: state or bias do not fit the channels and taps")
     out = torch.empty((T, C), dtype=x.dtype, device=x.device)
+    singles = bool(getattr(step, "all_decode", False)) and T == step.num_seqs
     _check(_lib().ix_causal_conv(
         _ptr(x), _dtype_code(x), ctypes.c_longlong(ldx), _ptr(in_bias), _ptr(w), _ptr(bias),
         _ptr(state), _ptr(step.cu_q), _ptr(step.seq_of_token), _ptr(step.state_slot), _ptr(out), T,
-        step.num_seqs, C, taps, 1 if silu else 0, _stream()), "causal_conv")
-    _count(2 if taps > 1 else 1)
+        step.num_seqs, C, taps, 1 if silu else 0, 1 if singles else 0, _stream()), "causal_conv")
+    _count(2 if taps > 1 and not singles else 1)
     return out
 
 

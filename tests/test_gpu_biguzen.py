@@ -309,7 +309,7 @@ def test_head_norm_with_denominator(dtype, V, form):
 # -- attention's options ----------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("C,taps", [(40, 1), (64, 3), (37, 5), (128, 4)])
-@pytest.mark.parametrize("q_lens", [[1, 1, 7], [2, 1100], [3]])
+@pytest.mark.parametrize("q_lens", [[1, 1, 7], [2, 1100], [3], [1, 1, 1, 1]])
 def test_convolution_adds_its_input_bias_first(dtype, C, taps, q_lens):
     q_lens = sorted(q_lens, key=lambda n: n != 1)
     r = _rand(C + taps)
