@@ -1055,8 +1055,8 @@ def designs(args):
     fudulix = args.design == "fudulix"
     dominex = args.design == "dominex"
     biguzen = args.design == "biguzen"
-    sizes = (BIGUZEN_SIZES if biguzen else DOMINEX_SIZES if dominex else FUDULIX_SIZES if fudulix else MAPOVIK_SIZES if mapovik
-             else TINAPEL_SIZES if tinapel else DESIGN_SIZES)
+    sizes = (BIGUZEN_SIZES if biguzen else DOMINEX_SIZES if dominex else FUDULIX_SIZES
+             if fudulix else MAPOVIK_SIZES if mapovik else TINAPEL_SIZES if tinapel else DESIGN_SIZES)
     first, second = (("fudulix", "qwen2_moe") if fudulix else ("mapovik", "tinapel") if mapovik
                      else ("tinapel", "qwen2_moe") if tinapel else ("zuzisun", "qwen2_dense"))
     names = args.design_sizes.split(",") if args.design_sizes else list(sizes)
@@ -1158,8 +1158,8 @@ def main(argv=None):
                          "beside the closest Qwen2-MoE at equal sizes (random weights); --layers (4), "
                          "--batch, --context (4096), --prefill-tokens (2048) apply")
     ap.add_argument("--design-sizes", default="", help="with --designs: of 1k,2k,4k (all)")
-    ap.add_argument("--design", default="zuzisun", choices=["zuzisun", "tinapel", "mapovik", "fudulix", "dominex",
-                                                              "biguzen"],
+    ap.add_argument("--design", default="zuzisun",
+                    choices=["zuzisun", "tinapel", "mapovik", "fudulix", "dominex", "biguzen"],
                     help="with --designs: which design stands beside its closest model")
     ap.add_argument("--design-pattern", default="wkv,gla,attention,attention",
                     help="with --design tinapel: the mixers of the layers, repeated; with "

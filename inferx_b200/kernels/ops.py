@@ -576,7 +576,8 @@ def router_topk(x: torch.Tensor, w: torch.Tensor, top_k: int, renormalize: bool,
             _ptr(x), _ptr(w), _ptr(extra_w), _dtype_code(x), T, H, E, top_k,
             1 if renormalize else 0, ctypes.c_float(scale), _ptr(correction), int(group_count),
             int(group_keep), ctypes.c_float(-1.0 if renorm_eps is None else renorm_eps),
-            1 if score == "sigmoid" else 0, 1 if group_value == "pair_sum" else 0, _ptr(tw), _ptr(ti), _ptr(ex), _ptr(scratch), _stream())
+            1 if score == "sigmoid" else 0, 1 if group_value == "pair_sum" else 0, _ptr(tw),
+            _ptr(ti), _ptr(ex), _ptr(scratch), _stream())
     else:
         code = _lib().ix_router_topk(
             _ptr(x), _ptr(w), _ptr(extra_w), _dtype_code(x), T, H, E, top_k,
@@ -2609,9 +2610,9 @@ MEMORY_GATES_SINGLE_TOKENS = 128
 def memory_gates(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, cap: float,
                  m_state: torch.Tensor, step):
     """fp32 [4, H, T]: exp(f + m_(t-1) - m_t), exp(i - m_t), exp(-m_t) and the first one's
-    logarithm of every token and head, with the log gates i = cap tanh(z_i / cap), f = logsigmoid(cap tanh(z_f / cap)), z =
-    x . w^T + bias (``w`` [2 H, W]: the input gates' rows, then the forget gates') and m_t =
-    max(f + m_(t-1), i) along each sequence from and back to ``m_state`` fp32 [slots, H]."""
+    logarithm of every token and head, with the log gates i = cap tanh(z_i / cap), f =
+    logsigmoid(cap tanh(z_f / cap)), z = x . w^T + bias (``w`` [2 H, W]: the input gates' rows,
+    then the forget gates') and m_t = max(f + m_(t-1), i) along each sequence from and back to ``m_state`` fp32 [slots, H]."""
     _chk("x", x)
     _chk("w", w, x.dtype)
     _chk("bias", bias, torch.float32)

@@ -211,9 +211,9 @@ class PreparedAttentionMixer:
     for it; the projections may have biases.  The window may keep a request's first tokens visible,
     the softmax may have one (or a learned number per head, exponentiated) added to its
     denominator, and a head's result may be multiplied by a gate of its own.  A layer may
-    project queries alone and read another layer's keys and values.  Keys and values live in the framework's pages (the
-    value pages as wide as the value heads); the convolutions' last inputs in the state
-    slots.  Norms, angles, scores and weights are fp32 in every element type."""
+    project queries alone and read another layer's keys and values.  Keys and values live in
+    the framework's pages (the value pages as wide as the value heads); the convolutions' last
+    inputs in the state slots.  Norms, angles, scores and weights are fp32 in every element type."""
 
     def __init__(self, spec, ctx, prefix: str):
         self.spec, self.ctx, self.prefix = spec, ctx, prefix
@@ -343,8 +343,8 @@ class PreparedAttentionMixer:
             freq, magnitude, rot, interleaved = self.position.pair_table()
         q = ops.attention_prepare(
             qkv, step.positions, freq, magnitude, rot, interleaved, s.heads,
-            s.kv_heads if self.own_kv else 0, s.head_dim, self.vdim, self.q_gain, self.k_gain, s.norm_eps, s.head_unit_norm,
-            earlier, self.lam, cache.k if cache.writes else None,
+            s.kv_heads if self.own_kv else 0, s.head_dim, self.vdim, self.q_gain, self.k_gain,
+            s.norm_eps, s.head_unit_norm, earlier, self.lam, cache.k if cache.writes else None,
             cache.v if cache.writes else None, group.slots if cache.writes else None)
         if s.value_mix == "source":
             # this layer's values as projected (and convolved): a view of its own rows

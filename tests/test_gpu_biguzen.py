@@ -196,7 +196,7 @@ def _views(rows, H, K, V):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("H,K,V", [(3, 10, 6), (2, 48, 48), (2, 64, 128), (1, 130, 36), (1, 24, 200),
+@pytest.mark.parametrize("H,K,V", [(3, 10, 6), (3, 40, 48), (2, 64, 128), (1, 130, 36), (1, 24, 200),
                                    (2, 16, 7)])
 @pytest.mark.parametrize("q_lens", [[1, 1, 1], [1, 5, 2], [1, 1, 200, 64, 65], [31], [321]])
 def test_matrix_memory(dtype, H, K, V, q_lens):
@@ -216,7 +216,7 @@ def test_matrix_memory(dtype, H, K, V, q_lens):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("H,K,V", [(3, 10, 6), (2, 48, 48), (2, 64, 128), (1, 24, 200), (2, 16, 7)])
+@pytest.mark.parametrize("H,K,V", [(3, 10, 6), (3, 40, 48), (2, 64, 128), (1, 24, 200), (2, 16, 7)])
 @pytest.mark.parametrize("q_lens", [[1, 1, 1], [1, 5, 2], [1, 1, 200, 64, 65], [100]])
 def test_matrix_memory_finishes_the_heads(dtype, H, K, V, q_lens):
     """Division by the normaliser, norm, gain and gate in the memory's kernels where a block has
@@ -361,7 +361,7 @@ def _kv_case(seed, H, G, D, VD, page, q_lens, starts, dtype):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("H,G,D,VD", [(5, 1, 6, 10), (6, 2, 24, 40), (8, 2, 64, 64), (4, 4, 64, 128),
-                                      (16, 1, 128, 128), (6, 1, 128, 64)])
+                                      (16, 1, 128, 128), (5, 1, 128, 64)])
 @pytest.mark.parametrize("window", [0, 1, 40])
 @pytest.mark.parametrize("q_lens,starts", [([1, 1, 1], [0, 39, 700]), ([150, 2], [0, 77]),
                                            ([1, 1, 70], [200, 5, 30])])
@@ -439,7 +439,7 @@ def test_each_head_has_a_sink_of_its_own(dtype, decode, D):
 
 # -- experts --------------------------------------------------------------------------------
 @pytest.mark.parametrize("T", [3, 40, 300])
-@pytest.mark.parametrize("E,k,groups,keep", [(12, 3, 3, 2), (8, 2, 8, 5), (40, 4, 4, 1), (6, 6, 2, 2)])
+@pytest.mark.parametrize("E,k,groups,keep", [(15, 4, 3, 2), (8, 2, 8, 5), (40, 4, 4, 1), (6, 6, 2, 2)])
 def test_groups_valued_by_their_two_best(T, E, k, groups, keep):
     r = _rand(T + E)
     x, w, corr = r(T, 64), r(E, 64) * 0.2, r(E) - 3.0         # every choice score is negative
@@ -452,7 +452,8 @@ def test_groups_valued_by_their_two_best(T, E, k, groups, keep):
     assert float(same.float().mean()) > 0.99                  # (a tie in fp32 may fall elsewhere)
     torch.testing.assert_close(gw.cpu()[same], rw[same], rtol=1e-5, atol=1e-6)
     assert torch.allclose(gw.sum(-1).cpu(), torch.full((T,), 1.7), rtol=1e-5)
-    if T == 300 and groups < E and keep < groups:   # the rule matters: the largest score alone chooses otherwise
+    if T == 300 and groups < E and keep < groups:
+        # the rule matters: the largest score alone chooses otherwise
         _, other, _ = host_ops.router_topk(x, w, k, True, 1.7, **dict(
             rule, correction=corr, group_value="max"))
         assert (other != ri).any()
