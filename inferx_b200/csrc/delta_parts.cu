@@ -346,7 +346,8 @@ causal_conv_run_kernel(const TA* __restrict__ x, long long ldx,
 // reads from the old state lies above what it has written.
 template <typename TA>
 __global__ void conv_state_update_kernel(const TA* __restrict__ x, long long ldx,
-                                         const float* __restrict__ in_bias, float* __restrict__ state, const int* __restrict__ cu_q,
+                                         const float* __restrict__ in_bias,
+                                         float* __restrict__ state, const int* __restrict__ cu_q,
                                          const int* __restrict__ state_slot, int C, int taps) {
   IX_PDL_WAIT();
   const int s = blockIdx.x;

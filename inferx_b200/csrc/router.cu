@@ -71,9 +71,9 @@ __device__ __forceinline__ void select_topk(float* p, int E, int k, int renorm, 
 // How the chosen experts are picked and weighted beyond the plain top-k: `correction`
 // ([E] or null) is added to the scores for the choice alone; with `groups` > 0 the E
 // outputs form that many equal groups of neighbours, a group's value is its largest
-// corrected score (`pair_sum`: the sum of its two largest), and only outputs of the `keep` groups with the largest values can be
-// chosen (ties to the lower group); `renorm_eps` >= 0 divides the chosen scores by (their
-// sum + renorm_eps).  `active` 0: the plain rule above.
+// corrected score (`pair_sum`: the sum of its two largest), and only outputs of the `keep`
+// groups with the largest values can be chosen (ties to the lower group); `renorm_eps` >= 0
+// divides the chosen scores by (their sum + renorm_eps).  `active` 0: the plain rule above.
 struct RouteRule {
   const float* correction;
   int groups;
